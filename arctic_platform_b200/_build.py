@@ -72,25 +72,52 @@ def _compile_one(src: Path, verbose: bool) -> Path:
     return obj
 
 
+# what serving a stateful architecture needs (models/registry.py): the GEMMs, the ragged-batch kernels, the status word
+SERVE_STEMS = ("status", "gemm_tcgen05", "gemm_tcgen05_2cta", "gemm_simt", "serve_layers", "serve_attention",
+               "serve_attention_tc", "retention")
+SERVE_LIB = OUT_DIR / "libapb200_serve.so"
+
+
+def build_cuda_subset(stems, lib: Path, verbose: bool = False) -> Path:
+    """Builds ``lib`` from some of the sources only (same objects as the full build, so nothing compiles twice)."""
+    OUT_DIR.mkdir(parents=True, exist_ok=True)
+    OBJ_DIR.mkdir(parents=True, exist_ok=True)
+    srcs = [CSRC / f"{s}.cu" for s in stems]
+    if lib.exists() and lib.stat().st_mtime >= _newest_mtime(srcs + _headers()):
+        return lib
+    with cf.ThreadPoolExecutor(max_workers=min(8, len(srcs))) as ex:
+        objs = list(ex.map(lambda s: _compile_one(s, verbose), srcs))
+    return _link(objs, lib)
+
+
+def cuda_up_to_date() -> bool:
+    return CUDA_LIB.exists() and CUDA_LIB.stat().st_mtime >= _newest_mtime(cuda_sources() + _headers())
+
+
+def _link(objs, lib: Path) -> Path:
+    tmp = lib.with_name(f"{lib.name}.{os.getpid()}")
+    cmd = [_nvcc(), "-shared", "-o", str(tmp), *map(str, objs), "-cudart", "static"]
+    res = subprocess.run(cmd, capture_output=True, text=True)
+    if res.returncode != 0:
+        raise RuntimeError(f"link failed:\n{res.stdout}\n{res.stderr}")
+    os.replace(tmp, lib)
+    return lib
+
+
 def build_cuda(force: bool = False, verbose: bool = False) -> Path:
     OUT_DIR.mkdir(parents=True, exist_ok=True)
     OBJ_DIR.mkdir(parents=True, exist_ok=True)
     srcs = cuda_sources()
     if not srcs:
         raise RuntimeError("no CUDA sources found")
-    if (not force and CUDA_LIB.exists()
-            and CUDA_LIB.stat().st_mtime >= _newest_mtime(srcs + _headers())):
+    if not force and cuda_up_to_date():
         return CUDA_LIB
     if force:
         for o in OBJ_DIR.glob("*.o"):
             o.unlink()
     with cf.ThreadPoolExecutor(max_workers=min(8, len(srcs))) as ex:
         objs = list(ex.map(lambda s: _compile_one(s, verbose), srcs))
-    cmd = [_nvcc(), "-shared", "-o", str(CUDA_LIB), *map(str, objs), "-cudart", "static"]
-    res = subprocess.run(cmd, capture_output=True, text=True)
-    if res.returncode != 0:
-        raise RuntimeError(f"link failed:\n{res.stdout}\n{res.stderr}")
-    return CUDA_LIB
+    return _link(objs, CUDA_LIB)
 
 
 def build_runtime(force: bool = False) -> Path:

@@ -17,6 +17,7 @@ enum GemmEpilogue : int {
   kEpiF32AtomicPeer = 7,   // GEMM -> reduce-scatter: red.add of the partial row into the fp32 buffer of the rank
                            // that owns the row (owner = row / rows_per_rank), over its NVLink peer mapping
   kEpiBf16ScatterPeer = 8, // GEMM -> all-to-all: bf16 row stored to (peer, row) = row_map[m] (MoE combine)
+  kEpiGeGLU = 9,       // as kEpiSwiGLU with the tanh form of GELU as the activation of the gate
 };
 
 struct PeerTensorMaps {
@@ -63,6 +64,10 @@ struct GemmParams {
 };
 
 __device__ __forceinline__ float silu_f(float x) { return x / (1.f + __expf(-x)); }
+// 0.5 x (1 + tanh(u)), u = sqrt(2/pi) (x + 0.044715 x^3), written as x * sigmoid(2 u)
+__device__ __forceinline__ float gelu_tanh_f(float x) {
+  return x / (1.f + expf(-1.5957691216057308f * (x + 0.044715f * x * x * x)));
+}
 
 // One output row, 32 consecutive accumulator columns starting at `col0` (raw fp32 bits in `r`).  Covers every
 // epilogue except the two lm-head ones, which keep running state across the chunks of a tile.
@@ -73,7 +78,7 @@ __device__ __forceinline__ void gemm_store_chunk(const GemmParams& p, int row, i
   float v[32];
 #pragma unroll
   for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(r[j]) * p.alpha;
-  if (p.epi == kEpiBf16 || (p.epi == kEpiSwiGLU && p.C != nullptr)) {
+  if (p.epi == kEpiBf16 || ((p.epi == kEpiSwiGLU || p.epi == kEpiGeGLU) && p.C != nullptr)) {
     if (p.bias) {
 #pragma unroll
       for (int j = 0; j < 32; ++j)
@@ -92,7 +97,7 @@ __device__ __forceinline__ void gemm_store_chunk(const GemmParams& p, int row, i
       }
     }
   }
-  if (p.epi == kEpiSwiGLU) {
+  if (p.epi == kEpiSwiGLU || p.epi == kEpiGeGLU) {
     __nv_bfloat16* dst =
         static_cast<__nv_bfloat16*>(p.C2) + static_cast<long long>(row) * p.ldc2 + (col0 >> 1);
 #pragma unroll
@@ -100,7 +105,10 @@ __device__ __forceinline__ void gemm_store_chunk(const GemmParams& p, int row, i
       if (q * 16 < ncols && col0 + q * 16 < p.N) {
         float a[8];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) a[j] = silu_f(v[q * 16 + 2 * j]) * v[q * 16 + 2 * j + 1];
+        for (int j = 0; j < 8; ++j) {
+          const float g = v[q * 16 + 2 * j];
+          a[j] = (p.epi == kEpiSwiGLU ? silu_f(g) : gelu_tanh_f(g)) * v[q * 16 + 2 * j + 1];
+        }
         uint4 o;
         o.x = pack_bf16x2(a[0], a[1]);
         o.y = pack_bf16x2(a[2], a[3]);

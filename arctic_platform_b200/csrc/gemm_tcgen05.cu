@@ -525,12 +525,13 @@ static int gemm_bf16_impl(const void* A, const void* B, void* C, int M, int N, i
   if ((lda % 8) || (ldb % 8) || (N % 8) || (reinterpret_cast<uintptr_t>(A) & 15) ||
       (reinterpret_cast<uintptr_t>(B) & 15) || (reinterpret_cast<uintptr_t>(C) & 15))
     return kBadArgument;
-  if (epi == kEpiBf16 || epi == kEpiSwiGLU) {
+  const bool glu = epi == kEpiSwiGLU || epi == kEpiGeGLU;
+  if (epi == kEpiBf16 || glu) {
     if (C && (ldc % 8)) return kBadArgument;
   } else if (ldc % 4) {
     return kBadArgument;
   }
-  if (epi == kEpiSwiGLU && (!C2 || (ldc2 % 8) || (N % 16))) return kBadArgument;
+  if (glu && (!C2 || (ldc2 % 8) || (N % 16))) return kBadArgument;
   const int k_blocks = (K + kBK - 1) / kBK;
   if (splits < 1) splits = 1;
   if (splits > k_blocks) splits = k_blocks;
@@ -538,7 +539,7 @@ static int gemm_bf16_impl(const void* A, const void* B, void* C, int M, int N, i
   // Large plain problems go to the CTA-pair kernel (256 x 256 tiles, half of B per SM): at least one full wave
   // of pairs, automatic tile choice, no grid cap.  APB_GEMM_PAIR=0 keeps everything on the one-CTA kernel.
   if (bn == 0 && splits == 1 && !tile_map && max_ctas <= 0 && pair_kernel_enabled() &&
-      (epi == kEpiBf16 || epi == kEpiF32 || epi == kEpiF32Accum || epi == kEpiSwiGLU) &&
+      (epi == kEpiBf16 || epi == kEpiF32 || epi == kEpiF32Accum || glu) &&
       !(epi == kEpiBf16 && !C) && M >= 512 &&
       static_cast<long long>((M + 255) / 256) * ((N + 255) / 256) >= sm_count() / 2)
     return apb_gemm_bf16_pair(A, B, C, M, N, K, lda, ldb, ldc, a_mn, b_mn, epi, alpha, bias, C2, ldc2, stream);

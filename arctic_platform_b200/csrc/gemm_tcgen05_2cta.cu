@@ -316,17 +316,18 @@ int apb_gemm_bf16_pair(const void* A, const void* B, void* C, int M, int N, int 
                        long long ldc2, cudaStream_t stream) {
   using namespace apb;
   if (M <= 0 || N <= 0 || K <= 0) return 0;
-  if (epi != kEpiBf16 && epi != kEpiF32 && epi != kEpiF32Accum && epi != kEpiSwiGLU) return kBadArgument;
+  const bool glu = epi == kEpiSwiGLU || epi == kEpiGeGLU;
+  if (epi != kEpiBf16 && epi != kEpiF32 && epi != kEpiF32Accum && !glu) return kBadArgument;
   if ((lda % 8) || (ldb % 8) || (N % 8) || (reinterpret_cast<uintptr_t>(A) & 15) ||
       (reinterpret_cast<uintptr_t>(B) & 15) || (reinterpret_cast<uintptr_t>(C) & 15))
     return kBadArgument;
-  if (epi == kEpiBf16 || epi == kEpiSwiGLU) {
+  if (epi == kEpiBf16 || glu) {
     if (C && (ldc % 8)) return kBadArgument;
     if (epi == kEpiBf16 && !C) return kBadArgument;
   } else if (!C || (ldc % 4)) {
     return kBadArgument;
   }
-  if (epi == kEpiSwiGLU && (!C2 || (ldc2 % 8) || (N % 16))) return kBadArgument;
+  if (glu && (!C2 || (ldc2 % 8) || (N % 16))) return kBadArgument;
 
   CUtensorMap ta, tb;
   int rc;

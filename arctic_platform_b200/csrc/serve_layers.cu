@@ -1,0 +1,322 @@
+// Small kernels of a serving step over a RAGGED batch: several sequences, each with its own run of new tokens (a
+// portion of a prompt, or one decoded token), share one packed row axis.
+//
+// A batch is described by per-entry arrays: e_start / e_len (rows of the entry), e_slot (state slot of its sequence)
+// and e_pos0 (position of its first row, i.e. tokens of the sequence before this step).  A decode step is the special
+// case "entry i = row i = slot i, e_len 0 or 1", with every array living in device buffers, so that it can be captured
+// in a CUDA graph.
+//
+// Per-sequence state that a step reads at the entry's first rows and replaces at its last rows (the previous token,
+// the convolution history) is double buffered: `parity[slot]` names the half that is read, the other half is written,
+// and serve_commit flips the parity once at the end of the step.  A position-0 entry ignores whatever its slot holds.
+//
+// The kernels take bf16 or fp32 activations (dtype argument: 0 = bf16, 1 = fp32); the residual stream, norms and
+// convolution histories are fp32 in both.
+#include "common.cuh"
+#include "host_utils.cuh"
+#include "serve_common.cuh"
+
+namespace apb {
+
+// ---------------------------------------------------------------------------- embedding
+// x[row] = embed[token] (+ bigram[hash(previous token, token)]), fp32; `x0` (optional) receives the same row in the
+// activation type (the right half of the loop-input operand), `kv_slot` the row's cache slot (page * 16 + offset, -1 for
+// an entry without tokens).
+template <typename T>
+__global__ void __launch_bounds__(128)
+embed_hash_kernel(const int* __restrict__ tokens, const int* __restrict__ row_entry, const ServeEntries e,
+                  const int* __restrict__ prev, const T* __restrict__ embed, const T* __restrict__ bigram,
+                  long long buckets, long long mul_prev, long long mul_cur, int vocab, int W, float* __restrict__ x,
+                  T* __restrict__ x0, long long ld0, const int* __restrict__ page_table, int max_pages,
+                  int* __restrict__ kv_slot) {
+  pdl_entry();
+  const int row = blockIdx.x;
+  const int en = row_entry ? row_entry[row] : row;
+  if (kv_slot && threadIdx.x == 0) {
+    const int r = row - e.start[en], pos = e.pos0[en] + r;
+    const bool live = r >= 0 && r < e.len[en] && pos >= 0 && pos / kServePage < max_pages;
+    kv_slot[row] = live ? page_table[static_cast<long long>(en) * max_pages + pos / kServePage] * kServePage + pos % kServePage : -1;
+  }
+  int tok = tokens[row];
+  tok = tok < 0 ? 0 : (tok >= vocab ? vocab - 1 : tok);
+  const T* big = nullptr;
+  if (bigram) {
+    const int r = row - e.start[en];
+    long long b = buckets;                        // first token of a sequence
+    if (e.pos0[en] + r > 0) {
+      int pt = r > 0 ? tokens[row - 1] : prev[e.slot[en]];
+      pt = pt < 0 ? 0 : (pt >= vocab ? vocab - 1 : pt);
+      b = (static_cast<long long>(pt) * mul_prev + static_cast<long long>(tok) * mul_cur) % buckets;
+      if (b < 0) b += buckets;
+    }
+    big = bigram + b * W;
+  }
+  const T* src = embed + static_cast<long long>(tok) * W;
+  for (int i = threadIdx.x; i < W; i += blockDim.x) {
+    float v = to_f32(src[i]);
+    if (big) v += to_f32(big[i]);
+    x[static_cast<long long>(row) * W + i] = v;
+    if (x0) x0[static_cast<long long>(row) * ld0 + i] = from_f32<T>(v);
+  }
+}
+
+// Start of a pass over looped layers: the left half of the loop-input operand receives the residual stream in the
+// activation type, and the stream itself restarts from `init` (the pass's step vector), onto which the loop-input
+// projection is then accumulated.
+template <typename T>
+__global__ void __launch_bounds__(256)
+loop_begin_kernel(float* __restrict__ x, const T* __restrict__ init, int W, T* __restrict__ out, long long ld,
+                  long long n) {
+  pdl_entry();
+  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < n;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const int c = static_cast<int>(i % W);
+    out[(i / W) * ld + c] = from_f32<T>(x[i]);
+    x[i] = to_f32(init[c]);
+  }
+}
+
+// ---------------------------------------------------------------------------- norm + input convolutions
+// h = x / rms(x) * g  (one gain for the whole row), then up to two causal depth-wise convolutions over time that share
+// h:  out_k[t] = h[t] + sum_j w_k[j] h[t - taps + 1 + j].  w_k is [taps, W]; a null w_k copies h.  The history of h
+// before the entry's first row comes from the slot's state [2][taps - 1][W]; the last taps - 1 rows of h replace it.
+// One block = up to kNormRows consecutive rows of one entry (tiles[2 i] = entry, tiles[2 i + 1] = first row; without a
+// table block i is entry i, which then has at most kNormRows rows).
+constexpr int kNormRows = 8;
+constexpr int kNormThreads = 256;
+
+template <typename T>
+__global__ void __launch_bounds__(kNormThreads)
+norm_conv_kernel(const float* __restrict__ x, const T* __restrict__ gain, const T* __restrict__ w1,
+                 const T* __restrict__ w2, T* __restrict__ out1, T* __restrict__ out2, float* __restrict__ state,
+                 const int* __restrict__ parity, const ServeEntries e, const int* __restrict__ tiles, int W, int taps,
+                 float eps) {
+  pdl_entry();
+  extern __shared__ float rs[];                    // [hist + kNormRows] row factors g / rms, rows r0 - hist ...
+  const int en = tiles ? tiles[2 * blockIdx.x] : blockIdx.x;
+  const int r0 = tiles ? tiles[2 * blockIdx.x + 1] : 0;
+  const int len = e.len[en];
+  if (r0 >= len) return;
+  const int nr = min(kNormRows, len - r0);
+  const int hist = taps - 1;
+  const int start = e.start[en], pos0 = e.pos0[en];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const float g = to_f32(*gain);
+  for (int i = warp; i < hist + nr; i += kNormThreads / 32) {
+    const int r = r0 - hist + i;
+    float ss = 0.f;
+    if (r >= 0) {
+      const float* xr = x + static_cast<long long>(start + r) * W;
+      if ((W & 3) == 0) {
+        for (int c = lane * 4; c < W; c += 128) {
+          const float4 v = *reinterpret_cast<const float4*>(xr + c);
+          ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+        }
+      } else {
+        for (int c = lane; c < W; c += 32) ss += xr[c] * xr[c];
+      }
+      ss = warp_sum(ss);
+    }
+    if (lane == 0) rs[i] = g / sqrtf(ss / W + eps);
+  }
+  __syncthreads();
+  const int slot = e.slot[en];
+  const float* old_h = nullptr;
+  float* new_h = nullptr;
+  if (hist > 0 && slot >= 0) {
+    const int par = parity[slot] & 1;
+    old_h = state + (static_cast<long long>(slot) * 2 + par) * hist * W;
+    new_h = state + (static_cast<long long>(slot) * 2 + (par ^ 1)) * hist * W;
+  }
+  // h of row r (relative to the entry; negative rows come from the state or lie before the sequence)
+  auto h_at = [&](int r, int c) -> float {
+    if (r >= 0) return x[static_cast<long long>(start + r) * W + c] * rs[r - r0 + hist];
+    return (pos0 + r >= 0 && old_h) ? old_h[static_cast<long long>(hist + r) * W + c] : 0.f;
+  };
+  for (int c = threadIdx.x; c < W; c += kNormThreads) {
+    for (int i = 0; i < nr; ++i) {
+      const int r = r0 + i;
+      const float h = h_at(r, c);
+      float a1 = h, a2 = h;
+      if (w1 || w2) {
+#pragma unroll 4
+        for (int j = 0; j < taps; ++j) {
+          const float hv = j == hist ? h : h_at(r - hist + j, c);
+          if (w1) a1 += to_f32(w1[j * W + c]) * hv;
+          if (w2) a2 += to_f32(w2[j * W + c]) * hv;
+        }
+      }
+      const long long o = static_cast<long long>(start + r) * W + c;
+      out1[o] = from_f32<T>(a1);
+      if (out2) out2[o] = from_f32<T>(a2);
+    }
+    if (new_h && r0 + nr == len)
+      for (int i = 0; i < hist; ++i) new_h[static_cast<long long>(i) * W + c] = h_at(len - hist + i, c);
+  }
+}
+
+// Final norm of selected rows: out[i] = x[rows[i]] / rms * g (rows == null: row i).  One block per row.
+template <typename T>
+__global__ void __launch_bounds__(256)
+gain_norm_rows_kernel(const float* __restrict__ x, const int* __restrict__ rows, const T* __restrict__ gain,
+                      T* __restrict__ out, int W, float eps) {
+  pdl_entry();
+  __shared__ float red[8];
+  const float* xr = x + static_cast<long long>(rows ? rows[blockIdx.x] : static_cast<int>(blockIdx.x)) * W;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < W; c += 256) ss += xr[c] * xr[c];
+  ss = warp_sum(ss);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+  __syncthreads();
+  ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) ss += red[i];
+  const float f = to_f32(*gain) / sqrtf(ss / W + eps);
+  for (int c = threadIdx.x; c < W; c += 256) out[static_cast<long long>(blockIdx.x) * W + c] = from_f32<T>(xr[c] * f);
+}
+
+// ---------------------------------------------------------------------------- q/k norm + paged cache write
+// p [rows, ld]: q heads at column q_col, k heads at k_col, v heads at v_col.  q and k heads are divided by their root
+// mean square (no weight); q goes back in place, k and v go to their cache slot (page * 16 + offset, < 0: nothing is
+// written) of kcache [pages, G, 16, D] and vcache [pages, G, 16, E].  One warp per (row, head).
+template <typename T>
+__global__ void __launch_bounds__(256)
+qk_norm_cache_kernel(T* __restrict__ p, long long ld, int q_col, int k_col, int v_col, const int* __restrict__ kv_slot,
+                     T* __restrict__ kcache, T* __restrict__ vcache, int rows, int H, int G, int D, int E, float eps) {
+  pdl_entry();
+  const int lane = threadIdx.x & 31;
+  const long long gw = (blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x) >> 5;
+  const int units = H + 2 * G;
+  if (gw >= static_cast<long long>(rows) * units) return;
+  const int row = static_cast<int>(gw / units), u = static_cast<int>(gw % units);
+  T* pr = p + static_cast<long long>(row) * ld;
+  const bool is_q = u < H, is_v = u >= H + G;
+  const int hk = is_q ? u : (is_v ? u - H - G : u - H);
+  const int n = is_v ? E : D;
+  T* src = pr + (is_q ? q_col : is_v ? v_col : k_col) + static_cast<long long>(hk) * n;
+  T* dst = src;
+  if (!is_q) {
+    const int slot = kv_slot[row];
+    if (slot < 0) return;
+    dst = (is_v ? vcache : kcache) + ((static_cast<long long>(slot / kServePage) * G + hk) * kServePage + slot % kServePage) * n;
+  }
+  const bool vec = sizeof(T) == 2 && (n & 7) == 0 && n <= 256 && (reinterpret_cast<uintptr_t>(src) & 15) == 0;
+  if (vec) {                                       // 8 elements per lane, one 16-byte access each way
+    uint4 raw = make_uint4(0u, 0u, 0u, 0u);
+    const bool mine = lane * 8 < n;
+    if (mine) raw = *reinterpret_cast<const uint4*>(src + lane * 8);
+    if (!is_v) {
+      __nv_bfloat162* h2 = reinterpret_cast<__nv_bfloat162*>(&raw);
+      float f[8], ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float2 t = __bfloat1622float2(h2[i]);
+        f[2 * i] = t.x;
+        f[2 * i + 1] = t.y;
+        ss += t.x * t.x + t.y * t.y;
+      }
+      const float r = 1.f / sqrtf(warp_sum(ss) / n + eps);
+      raw.x = pack_bf16x2(f[0] * r, f[1] * r);
+      raw.y = pack_bf16x2(f[2] * r, f[3] * r);
+      raw.z = pack_bf16x2(f[4] * r, f[5] * r);
+      raw.w = pack_bf16x2(f[6] * r, f[7] * r);
+    }
+    if (mine) *reinterpret_cast<uint4*>(dst + lane * 8) = raw;
+    return;
+  }
+  float r = 1.f;
+  if (!is_v) {
+    float ss = 0.f;
+    for (int i = lane; i < n; i += 32) {
+      const float v = to_f32(src[i]);
+      ss += v * v;
+    }
+    r = 1.f / sqrtf(warp_sum(ss) / n + eps);
+  }
+  for (int i = lane; i < n; i += 32) dst[i] = is_v ? src[i] : from_f32<T>(to_f32(src[i]) * r);
+}
+
+// ---------------------------------------------------------------------------- end of a step
+// Every entry that fed tokens: remember its last token and flip the parity of its double-buffered state.
+__global__ void __launch_bounds__(128)
+serve_commit_kernel(const int* __restrict__ tokens, const ServeEntries e, int n_entries, int* __restrict__ prev,
+                    int* __restrict__ parity) {
+  pdl_entry();
+  const int en = blockIdx.x * blockDim.x + threadIdx.x;
+  if (en >= n_entries) return;
+  const int len = e.len[en], slot = e.slot[en];
+  if (len <= 0 || slot < 0) return;
+  prev[slot] = tokens[e.start[en] + len - 1];
+  parity[slot] ^= 1;
+}
+
+}  // namespace apb
+
+extern "C" {
+using namespace apb;
+
+int apb_embed_hash(const int* tokens, const int* row_entry, const int* e_start, const int* e_len, const int* e_slot,
+                   const int* e_pos0, const int* prev, const void* embed, const void* bigram, long long buckets,
+                   long long mul_prev, long long mul_cur, int vocab, int W, float* x, void* x0, long long ld0,
+                   const int* page_table, int max_pages, int* kv_slot, int rows, int dtype, cudaStream_t s) {
+  if (rows <= 0) return 0;
+  if (!tokens || !embed || !x || (bigram && (buckets <= 0 || !prev)) || (kv_slot && !page_table)) return kBadArgument;
+  const ServeEntries e{e_start, e_len, e_slot, e_pos0};
+  APB_SERVE_DTYPE(dtype, return static_cast<int>(launch_kernel(
+                             embed_hash_kernel<T>, dim3(rows), dim3(128), 0, s, tokens, row_entry, e, prev,
+                             static_cast<const T*>(embed), static_cast<const T*>(bigram), buckets, mul_prev, mul_cur,
+                             vocab, W, x, static_cast<T*>(x0), ld0, page_table, max_pages, kv_slot)));
+}
+
+int apb_loop_begin(float* x, const void* init, int rows, int W, void* out, long long ld, int dtype, cudaStream_t s) {
+  if (rows <= 0) return 0;
+  if (!x || !init || !out) return kBadArgument;
+  const long long n = static_cast<long long>(rows) * W;
+  const int grid = static_cast<int>(n / 256 + 1 < sm_count() * 8 ? n / 256 + 1 : sm_count() * 8);
+  APB_SERVE_DTYPE(dtype, return static_cast<int>(launch_kernel(loop_begin_kernel<T>, dim3(grid), dim3(256), 0, s, x,
+                                                               static_cast<const T*>(init), W, static_cast<T*>(out), ld,
+                                                               n)));
+}
+
+// tiles: device int32 [n_tiles][2] or null (then n_tiles is the number of entries, none longer than 8 rows).
+int apb_norm_conv(const float* x, const void* gain, const void* w1, const void* w2, void* out1, void* out2,
+                  float* state, const int* parity, const int* e_start, const int* e_len, const int* e_slot,
+                  const int* e_pos0, const int* tiles, int n_tiles, int W, int taps, float eps, int dtype,
+                  cudaStream_t s) {
+  if (n_tiles <= 0) return 0;
+  if (taps < 1 || taps > 1024 || !x || !gain || !out1 || (taps > 1 && (!state || !parity))) return kBadArgument;
+  const ServeEntries e{e_start, e_len, e_slot, e_pos0};
+  const size_t smem = (taps - 1 + kNormRows) * sizeof(float);
+  APB_SERVE_DTYPE(dtype, return static_cast<int>(launch_kernel(
+                             norm_conv_kernel<T>, dim3(n_tiles), dim3(kNormThreads), smem, s, x,
+                             static_cast<const T*>(gain), static_cast<const T*>(w1), static_cast<const T*>(w2),
+                             static_cast<T*>(out1), static_cast<T*>(out2), state, parity, e, tiles, W, taps, eps)));
+}
+
+int apb_gain_norm_rows(const float* x, const int* rows, const void* gain, void* out, int n, int W, float eps, int dtype,
+                       cudaStream_t s) {
+  if (n <= 0) return 0;
+  APB_SERVE_DTYPE(dtype, return static_cast<int>(launch_kernel(gain_norm_rows_kernel<T>, dim3(n), dim3(256), 0, s, x, rows,
+                                                               static_cast<const T*>(gain), static_cast<T*>(out), W,
+                                                               eps)));
+}
+
+int apb_qk_norm_cache(void* p, long long ld, int q_col, int k_col, int v_col, const int* kv_slot, void* kcache,
+                      void* vcache, int rows, int H, int G, int D, int E, float eps, int dtype, cudaStream_t s) {
+  if (rows <= 0) return 0;
+  if (H <= 0 || G <= 0 || D <= 0 || E <= 0 || H % G) return kBadArgument;
+  const long long warps = static_cast<long long>(rows) * (H + 2 * G);
+  const int grid = static_cast<int>((warps * 32 + 255) / 256);
+  APB_SERVE_DTYPE(dtype, return static_cast<int>(launch_kernel(
+                             qk_norm_cache_kernel<T>, dim3(grid), dim3(256), 0, s, static_cast<T*>(p), ld, q_col, k_col,
+                             v_col, kv_slot, static_cast<T*>(kcache), static_cast<T*>(vcache), rows, H, G, D, E, eps)));
+}
+
+int apb_serve_commit(const int* tokens, const int* e_start, const int* e_len, const int* e_slot, const int* e_pos0,
+                     int n_entries, int* prev, int* parity, cudaStream_t s) {
+  if (n_entries <= 0) return 0;
+  const ServeEntries e{e_start, e_len, e_slot, e_pos0};
+  return static_cast<int>(launch_kernel(serve_commit_kernel, dim3((n_entries + 127) / 128), dim3(128), 0, s, tokens, e,
+                                        n_entries, prev, parity));
+}
+}

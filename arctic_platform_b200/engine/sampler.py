@@ -225,6 +225,8 @@ class _TPDecode:
 
 
 class SamplerEngine:
+    MIN_PAGES = 64
+
     def __init__(self, cfg: DecoderConfig, device="cuda", model: Optional[DecoderLM] = None,
                  kv_cache_tokens: int = 1 << 20, max_batch: int = 256, max_seq_len: int = 8192,
                  cascade: bool = True, sync_interval: int = 16, use_cuda_graph: bool = True, seed: int = 0,
@@ -275,7 +277,7 @@ class SamplerEngine:
         self.fp8 = quantization == "fp8" and not cfg.is_moe
         self._fp8_stale = True
         self._fp8_w: List[dict] = []
-        self.num_pages = max(64, kv_cache_tokens // PAGE)
+        self.num_pages = max(self.MIN_PAGES, kv_cache_tokens // PAGE)
         self.max_pages = (max_seq_len + PAGE - 1) // PAGE + 1
         self._alloc_cache()
         self.pages = PageAllocator(self.num_pages)
@@ -284,6 +286,7 @@ class SamplerEngine:
         self._step_count = 0
         self._asleep = False
         self._alloc_state()
+        self._alloc_layer_buffers()
         self._tpd = _TPDecode(self.device, tp_group, max_batch, cfg.hidden_size) if self.tp > 1 else None
         self._sync_plan = None           # table of the one-kernel weight hand-over (parallel/weight_sync.py)
 
@@ -303,6 +306,7 @@ class SamplerEngine:
         return 2 * c.num_layers * self.num_pages * c.num_kv_heads * PAGE * c.head_dim * 2
 
     def _alloc_state(self) -> None:
+        """Device state of the slots and of a decode step that does not depend on the kind of layers."""
         B, dev, c = self.max_batch, self.device, self.cfg
         i32 = dict(device=dev, dtype=torch.int32)
         self.d_tokens = torch.zeros(B, **i32)
@@ -341,19 +345,24 @@ class SamplerEngine:
         self._filter_on = False
         self.splits = 4
         self.n_groups = B            # rows in use in the node tables (a power-of-two bucket bounds the prefix grid)
-        Hq, D = c.num_heads, c.head_dim
         f32 = dict(device=dev, dtype=torch.float32)
+        self.d_logits = torch.empty((B, c.vocab_size), **f32)
+        self.d_new_tok = torch.zeros(B, **i32)
+        self.d_new_lp = torch.zeros(B, **f32)
+
+    def _alloc_layer_buffers(self) -> None:
+        """Scratch of the layers' decode step."""
+        B, dev, c = self.max_batch, self.device, self.cfg
+        i32, f32 = dict(device=dev, dtype=torch.int32), dict(device=dev, dtype=torch.float32)
+        Hq, D = c.num_heads, c.head_dim
         # partial results per source: header level, prompt level, private pass
         self.part_o = [torch.empty((B, Hq, self.splits, D), **f32) for _ in range(3)]
         self.part_ml = [torch.empty((B, Hq, self.splits, 2), **f32) for _ in range(3)]
-        self.d_logits = torch.empty((B, c.vocab_size), **f32)
         # fp32 split-K accumulators of the two skinny projections (kept zero between uses by the norm kernel)
         self.acc_o = torch.zeros((B, c.hidden_size), **f32)
         self.acc_d = torch.zeros((B, c.hidden_size), **f32)
         self.acc_qkv = torch.zeros((B, c.qkv_size), **f32)
         self.acc_gu = torch.zeros((B, 2 * c.intermediate_size), **f32) if not c.is_moe else None   # split-K gate/up sums
-        self.d_new_tok = torch.zeros(B, **i32)
-        self.d_new_lp = torch.zeros(B, **f32)
         self.d_slots = torch.full((B,), -1, **i32)                              # cache slot of the token being fed
         self.d_x = torch.empty((B, c.hidden_size), device=dev, dtype=torch.bfloat16)   # its embedding row
 
@@ -480,6 +489,33 @@ class SamplerEngine:
         n = max(1, int(self.n_groups))
         return min(self.n_node_rows, 1 << (n - 1).bit_length())
 
+    def _decode_logits(self, B: int) -> torch.Tensor:
+        """Feeds the pending token of slots [0, B) through the model; logits ``[B, V]`` fp32 in ``d_logits``."""
+        c = self.cfg
+        positions = self.d_pos[:B]
+        slots = self.d_slots[:B]
+        x = self.d_x[:B]
+        # one kernel: cache slot of the fed token (page-table look-up) + its embedding row
+        _lib.check(_fn("begin")(_lib.ptr(self.d_tokens), _lib.ptr(self.d_pos), _lib.ptr(self.d_active),
+                                _lib.ptr(self.d_page_table), self.max_pages, _lib.ptr(self.model.embed),
+                                self.model.embed.stride(0), c.hidden_size, c.vocab_size, _lib.ptr(slots), _lib.ptr(x), B,
+                                _lib.stream_ptr()), "decode_begin")
+        stream = None
+        attn = lambda li, q, k, v: self._decode_attention(li, q, B)
+        if self.tp > 1 and not self.fp8:
+            h = self._decode_layers_tp(x, positions, slots, B)
+        elif self.split_k and not c.is_moe and not self.fp8:
+            h = self._decode_layers_splitk(x, positions, slots, B)
+        else:
+            for li in range(c.num_layers):
+                x, stream = self._block(li, x, stream, positions, slots, attn)
+            h, _ = norm.rmsnorm(x, self.model.final_norm, c.rms_norm_eps, stream)
+        return self._output_logits(h, self.d_logits[:B])
+
+    def _output_logits(self, h: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """fp32 logits of final-norm hidden rows."""
+        return gemm.matmul_nt(h, self.model.output_weight, out=out, out_dtype=torch.float32)
+
     @torch.no_grad()
     def _decode_step(self, B: int) -> None:
         """One token for slots [0, B).  Reads and updates device state only, so the whole step can be
@@ -489,26 +525,7 @@ class SamplerEngine:
         # still running; valid here because no kernel of a decode step writes the weights
         prev_chain = _fn("chain")(1)
         try:
-            positions = self.d_pos[:B]
-            slots = self.d_slots[:B]
-            x = self.d_x[:B]
-            # one kernel: cache slot of the fed token (page-table look-up) + its embedding row
-            _lib.check(_fn("begin")(_lib.ptr(self.d_tokens), _lib.ptr(self.d_pos), _lib.ptr(self.d_active),
-                                    _lib.ptr(self.d_page_table), self.max_pages, _lib.ptr(self.model.embed),
-                                    self.model.embed.stride(0), c.hidden_size, c.vocab_size, _lib.ptr(slots), _lib.ptr(x), B,
-                                    _lib.stream_ptr()), "decode_begin")
-            stream = None
-            attn = lambda li, q, k, v: self._decode_attention(li, q, B)
-            if self.tp > 1 and not self.fp8:
-                h = self._decode_layers_tp(x, positions, slots, B)
-            elif self.split_k and not c.is_moe and not self.fp8:
-                h = self._decode_layers_splitk(x, positions, slots, B)
-            else:
-                for li in range(c.num_layers):
-                    x, stream = self._block(li, x, stream, positions, slots, attn)
-                h, _ = norm.rmsnorm(x, self.model.final_norm, c.rms_norm_eps, stream)
-            logits = self.d_logits[:B]
-            gemm.matmul_nt(h, self.model.output_weight, out=logits)
+            logits = self._decode_logits(B)
             if self._filter_on:
                 _lib.check(_fn("sample_f")(_lib.ptr(logits), logits.stride(0), _lib.ptr(self.d_temp), B, c.vocab_size,
                                            ctypes.c_uint(self.seed & 0xFFFFFFFF), _lib.ptr(self.d_step),
@@ -948,15 +965,13 @@ class SamplerEngine:
                         src.append(int(s0.private_pages[0]))
                         dst.append(int(live[slot].private_pages[0]))
             if src:
-                si = torch.tensor(src, device=self.device)
-                di = torch.tensor(dst, device=self.device)
-                self.kcache[:, di] = self.kcache[:, si]
-                self.vcache[:, di] = self.vcache[:, si]
+                self._copy_pages(torch.tensor(src, device=self.device), torch.tensor(dst, device=self.device))
+            self._fork_slots([(mem[0], mem[1:]) for _, mem in batch if len(mem) > 1])
             # first token of every rollout
             rows = [gi for gi, (_, mem) in enumerate(batch) for _ in mem]
             slots = [slot for _, mem in batch for slot in mem]
             hrep = h.index_select(0, torch.tensor(rows, device=self.device))
-            logits = gemm.matmul_nt(hrep.contiguous(), self.model.output_weight, out_dtype=torch.float32)
+            logits = self._output_logits(hrep.contiguous())
             n = len(slots)
             temp = torch.full((n,), float(sp.temperature), device=self.device, dtype=torch.float32)
             tok0 = torch.empty(n, device=self.device, dtype=torch.int32)
@@ -1006,6 +1021,15 @@ class SamplerEngine:
             self.d_priv_table[st] = to_device(torch.from_numpy(pv), self.device)
             self.d_priv_len[st] = to_device(torch.from_numpy(plen), self.device)
             self.d_shared_tokens[st] = to_device(torch.from_numpy(sh), self.device)
+
+    def _copy_pages(self, src: torch.Tensor, dst: torch.Tensor) -> None:
+        """Copies KV pages (a prompt's partial last page to every rollout) in all layers."""
+        self.kcache[:, dst] = self.kcache[:, src]
+        self.vcache[:, dst] = self.vcache[:, src]
+
+    def _fork_slots(self, forks: List[Tuple[int, List[int]]]) -> None:
+        """``(slot, other slots)``: the others continue from the state the first one's prompt left.  Nothing to do
+        for models whose only state is the K/V cache."""
 
     def _set_groups(self, group_members: Dict[int, List[int]], root_members: Dict[int, List[int]],
                     live: Dict[int, _Seq]) -> None:

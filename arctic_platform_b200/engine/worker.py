@@ -20,6 +20,7 @@ import torch
 from ..common.utils.batch import log_dp_shard_tokens
 from ..common.utils.metrics import combine_metric_microbatches
 from ..utils import sft_profile
+from ..models import registry
 from ..models.config import DecoderConfig, resolve_config
 from ..models.decoder import DecoderLM
 from ..rl.processors.pipeline import run_pipeline
@@ -118,8 +119,12 @@ class EngineWorker:
                                  "master weights and fp32 accumulation")
             if self.device.type != "cuda":
                 dtype = getattr(torch, lo.optimization_dtype)
+        stateful = registry.is_stateful(self.model_cfg)
+        if stateful and self.job_type != "sampling":
+            raise ValueError(f"{self.model_cfg.architecture} models are served (job_type 'sampling'); there is no "
+                             f"{self.job_type!r} engine for them")
         if lo.debug is not None and model is None:
-            if lo.debug.num_layers is not None:
+            if lo.debug.num_layers is not None and not stateful:
                 import dataclasses
                 n = int(lo.debug.num_layers)
                 lt = self.model_cfg.layer_types
@@ -131,6 +136,9 @@ class EngineWorker:
             if self.job_type == "sampling" else 1
         if self.job_type != "sampling" or tp > 1:
             self._ensure_process_group(job_config)
+        if stateful and tp > 1:
+            raise ValueError(f"{self.model_cfg.architecture} is served on one GPU per replica "
+                             f"(tensor_parallel_size={tp})")
         if self.job_type == "sampling" and tp > 1:
             return self._initialize_tp_sampler(job_config, model, tp, dtype, seed)
         scorer = (self.job_type == "log_prob" and job_config.get("log_prob_engine") == "vllm"
@@ -139,7 +147,10 @@ class EngineWorker:
             from .sampler import SamplerEngine
             vc = dict(job_config.get("vllm_config") or {})
             m = model if model is not None else self._load_model(job_config, dtype, seed)
-            if self.model_cfg.layer_types is not None:
+            if stateful:
+                # paged K/V plus state slots, layers supplied by the model (raises without a CUDA device)
+                from .stateful_sampler import StatefulSampler as SamplerEngine  # noqa: F811
+            elif self.model_cfg.layer_types is not None:
                 # hybrid family: recurrent state + sparse K/V layers, served by the stateful tensor-op engine
                 from .hybrid_sampler import HybridSampler as SamplerEngine      # noqa: F811
             elif vc.get("enable_return_routed_experts") and self.model_cfg.is_moe:
@@ -298,7 +309,7 @@ class EngineWorker:
         if not name:
             return None
         tensor_op = self.device.type != "cuda" or vc.get("speculative_engine") == "tensor_op"
-        if not tensor_op or self.model_cfg.layer_types is not None:
+        if not tensor_op or self.model_cfg.layer_types is not None or registry.is_stateful(self.model_cfg):
             logger.warning("speculative decoding (%s) is not available on this sampler engine; decoding without it", name)
             return None
         from pathlib import Path
@@ -317,7 +328,7 @@ class EngineWorker:
     def _load_model(self, job_config, dtype, seed) -> DecoderLM:
         from pathlib import Path
         from ..models.conversion_cache import load_through_cache
-        m = DecoderLM(self.model_cfg, self.device, dtype)
+        m = registry.new_model(self.model_cfg, self.device, dtype)
         path = Path(str(job_config["model_name"]))
         lo = getattr(self, "loader_options", None)
         random_init = bool(lo is not None and lo.debug is not None and lo.debug.random_init)

@@ -272,10 +272,17 @@ PRESETS: Dict[str, DecoderConfig] = {
 def resolve_config(model_name_or_path: str) -> DecoderConfig:
     """Preset name (case-insensitive, with or without an ``org/`` prefix) or a directory with ``config.json``."""
     p = Path(model_name_or_path)
+    from . import registry
     if p.is_dir() and (p / "config.json").exists():
-        return DecoderConfig.from_hf_dict(json.loads((p / "config.json").read_text()), name=p.name)
+        d = json.loads((p / "config.json").read_text())
+        if "architecture" in d:                  # a design with a configuration class of its own
+            return registry.config_class(d["architecture"]).from_dict(d, name=p.name)
+        return DecoderConfig.from_hf_dict(d, name=p.name)
     key = model_name_or_path.split("/")[-1].lower()
     if key in PRESETS:
         return PRESETS[key]
-    raise ValueError(f"unknown model {model_name_or_path!r}: give a preset ({sorted(PRESETS)}) or a directory "
-                     "containing config.json")
+    others = registry.presets()
+    if key in others:
+        return others[key]
+    raise ValueError(f"unknown model {model_name_or_path!r}: give a preset ({sorted([*PRESETS, *others])}) or a "
+                     "directory containing config.json")

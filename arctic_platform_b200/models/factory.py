@@ -15,6 +15,7 @@ from typing import Any, Callable, Dict, List, Optional, Tuple
 
 import torch
 
+from . import registry
 from .config import DecoderConfig, resolve_config
 from .decoder import DecoderLM
 
@@ -196,6 +197,14 @@ def _load_moe(ctx: LoaderContext, device, seed: int) -> DecoderLM:
     return model
 
 
+@register_loader("stateful", matches=lambda c: registry.is_stateful(c.hf_config), options=_options_schema())
+def _load_stateful(ctx: LoaderContext, device, seed: int):
+    """Architectures of ``models/registry.py``: served by the stateful paged engine on a GPU."""
+    if ctx.spec.parallelism.expert_parallel > 1 or ctx.spec.parallelism.sequence_parallel > 1:
+        raise ValueError(f"{ctx.hf_config.architecture} is served on one GPU per replica")
+    return _instantiate(ctx, device, seed)
+
+
 def _instantiate(ctx: LoaderContext, device, seed: int) -> DecoderLM:
     from pathlib import Path
     from .conversion_cache import load_through_cache
@@ -203,11 +212,11 @@ def _instantiate(ctx: LoaderContext, device, seed: int) -> DecoderLM:
     dtype = _torch_dtype(ctx.spec.dtype) if dev.type == "cuda" else torch.float32
     cfg = ctx.hf_config
     debug = ctx.spec.loader_options.get("debug") or {}
-    if debug.get("num_layers") is not None:                    # test-only: a shallower model of the same family
+    if debug.get("num_layers") is not None and not registry.is_stateful(cfg):   # test-only: a shallower model of the same family
         import dataclasses
         n, lt = int(debug["num_layers"]), cfg.layer_types
         cfg = dataclasses.replace(cfg, num_layers=n, layer_types=None if lt is None else tuple(lt[:n]))
-    model = DecoderLM(cfg, dev, dtype)
+    model = registry.new_model(cfg, dev, dtype)
     p = Path(ctx.spec.model_path_or_name)
     if p.is_dir() and any(p.glob("*.safetensors")) and not debug.get("random_init"):
         load_through_cache(model, p, cache_dir=ctx.spec.loader_options.get("weight_conversion_cache_dir"))

@@ -38,6 +38,8 @@ _LINEAR_ATTN_ATTR = {"in_proj_qkv.weight": "in_qkv", "in_proj_z.weight": "in_z",
 
 def hf_param_names(cfg: DecoderConfig) -> List[str]:
     """Every Hugging Face tensor name of the architecture, in layer order."""
+    if hasattr(cfg, "tensor_names"):             # an architecture with names of its own (models/registry.py)
+        return cfg.tensor_names()
     names = ["model.embed_tokens.weight"]
     for i in range(cfg.num_layers):
         p = f"model.layers.{i}."
@@ -104,6 +106,9 @@ def _local_expert(moe, e: int) -> Optional[int]:
 def iter_hf_tensors(model) -> Iterator[Tuple[str, torch.Tensor]]:
     """Yields ``(hf_name, tensor)`` views/slices of the fused parameters (no copies except the
     de-interleave of gate/up)."""
+    if hasattr(model, "iter_named_tensors"):
+        yield from model.iter_named_tensors()
+        return
     cfg: DecoderConfig = model.cfg
     yield "model.embed_tokens.weight", model.embed.data
     qs, ks = cfg.q_size, cfg.kv_size
@@ -171,6 +176,8 @@ def iter_hf_tensors(model) -> Iterator[Tuple[str, torch.Tensor]]:
 @torch.no_grad()
 def load_hf_tensor(model, name: str, tensor: torch.Tensor) -> None:
     """Copies one Hugging Face tensor into its place inside the fused parameters."""
+    if hasattr(model, "load_named_tensor"):
+        return model.load_named_tensor(name, tensor)
     cfg: DecoderConfig = model.cfg
     qs, ks = cfg.q_size, cfg.kv_size
 
@@ -442,7 +449,7 @@ def load_hf_checkpoint(model, ckpt_dir, strict: bool = True) -> int:
     seen = set()
     for f in files:
         for raw, t in read_safetensors(f):
-            name = text_name(raw)
+            name = raw if raw in expected else text_name(raw)
             if name is None:                  # vision tower / extra heads of a composite checkpoint: kept, not trained
                 if getattr(model, "passthrough", None) is None:
                     model.passthrough = PassthroughTensors()

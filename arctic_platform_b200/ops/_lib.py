@@ -55,12 +55,30 @@ def _load(path: Path, builder):
         raise NativeLibraryError(f"cannot load {path}: {exc}") from exc
 
 
+_serve_only = False
+
+
+def serve_only() -> None:
+    """For processes that only serve a stateful architecture: unless the full kernel library is built and current,
+    compile and load just the kernels such a model needs.  Call it before the first kernel."""
+    global _serve_only
+    _serve_only = not _build.cuda_up_to_date()
+    if _serve_only:
+        try:
+            _build.build_cuda_subset(_build.SERVE_STEMS, _build.SERVE_LIB)
+        except Exception as exc:
+            raise NativeLibraryError(f"{_build.SERVE_LIB.name} could not be built: {exc}") from exc
+
+
 def cuda_lib() -> ctypes.CDLL:
     global _cuda
     if _cuda is None:
         with _lock:
             if _cuda is None:
-                lib = _load(_build.CUDA_LIB, _build.build_cuda)
+                if _serve_only:
+                    lib = _load(_build.SERVE_LIB, lambda: _build.build_cuda_subset(_build.SERVE_STEMS, _build.SERVE_LIB))
+                else:
+                    lib = _load(_build.CUDA_LIB, _build.build_cuda)
                 _declare_cuda(lib)
                 _cuda = lib
     return _cuda

@@ -19,6 +19,7 @@ EPI_F32 = 1
 EPI_F32_ATOMIC = 2
 EPI_F32_ACCUM = 3
 EPI_SWIGLU = 4
+EPI_GEGLU = 9
 
 
 def _check2d(t: torch.Tensor, name: str) -> None:

@@ -1,0 +1,260 @@
+"""Operations of a serving step over a ragged batch (CUDA only).
+
+A step advances several sequences at once, each by its own run of new tokens: a portion of a prompt of any length, or
+one decoded token.  :class:`StepBatch` is the device-side description of such a step; the functions below launch the
+kernels of ``serve_layers.cu``, ``serve_attention.cu``, ``serve_attention_tc.cu``, ``retention.cu`` and
+``gemm_simt.cu`` on it.  They take bf16 or fp32 activations; the residual stream and all carried state are fp32.
+"""
+from __future__ import annotations
+
+import ctypes
+from dataclasses import dataclass
+from typing import Dict, List, Optional, Sequence, Tuple
+
+import numpy as np
+import torch
+
+from . import _lib, gemm
+from ..utils.transfer_stats import to_device
+
+PAGE = 16               # tokens per KV page
+NORM_ROWS = 8           # rows per block of the norm + convolution kernel
+
+_FN: Dict[str, object] = {}
+
+
+def _fn(name: str):
+    if name not in _FN:
+        c = ctypes
+        vp, i, ll, f = c.c_void_p, c.c_int, c.c_longlong, c.c_float
+        sigs = {
+            "apb_embed_hash": [vp] * 9 + [ll, ll, ll, i, i, vp, vp, ll, vp, i, vp, i, i, vp],
+            "apb_loop_begin": [vp, vp, i, i, vp, ll, i, vp],
+            "apb_norm_conv": [vp] * 13 + [i, i, i, f, i, vp],
+            "apb_gain_norm_rows": [vp, vp, vp, vp, i, i, f, i, vp],
+            "apb_qk_norm_cache": [vp, ll, i, i, i, vp, vp, vp, i, i, i, i, i, f, i, vp],
+            "apb_serve_commit": [vp] * 5 + [i, vp, vp, vp],
+            "apb_sigmoid_attn": [vp, ll, vp, vp, vp, vp, vp, vp, i, vp, vp, vp, vp, ll, i, i, i, i, i, f, f, i, vp],
+            "apb_retention": [vp, ll, i, i, i, i, vp, vp, i, vp, f, vp, vp, vp, ll, f, f, vp, vp, vp, vp, vp] + [i] * 8 + [vp],
+            "apb_gemm_simt": [vp, vp, vp, i, i, i, ll, ll, ll, i, vp, vp, ll, i, vp],
+        }
+        _FN[name] = _lib.declare(name, sigs[name])
+    return _FN[name]
+
+
+def _call(name: str, *args) -> None:
+    _lib.check(_fn(name)(*args, _lib.stream_ptr()), name)
+
+
+def dtype_code(dtype: torch.dtype) -> int:
+    if dtype == torch.bfloat16:
+        return 0
+    if dtype == torch.float32:
+        return 1
+    raise ValueError(f"the serving kernels take bfloat16 or float32, got {dtype}")
+
+
+# --------------------------------------------------------------------------------------------- the batch
+@dataclass
+class StepEntry:
+    """One sequence's part of a step: ``tokens`` continue the sequence in state slot ``slot`` at position ``pos0``;
+    ``pages`` are its KV pages, in order, enough for ``pos0 + len(tokens)`` tokens."""
+    slot: int
+    tokens: np.ndarray
+    pos0: int
+    pages: np.ndarray
+
+
+@dataclass
+class StepBatch:
+    rows: int
+    n_entries: int
+    tokens: torch.Tensor                   # [rows] int32
+    row_entry: Optional[torch.Tensor]      # [rows], None: row i belongs to entry i
+    start: torch.Tensor                    # [entries] first row, rows, state slot, position of the first row
+    len: torch.Tensor
+    slot: torch.Tensor
+    pos0: torch.Tensor
+    page_table: torch.Tensor               # [entries, max_pages]
+    kv_slot: torch.Tensor                  # [rows] cache slot of every row (written by ``embed``)
+    tiles: Optional[torch.Tensor] = None   # [n, 2] (entry, first row) of the norm + convolution blocks
+    one_token: bool = True                 # some entry has exactly one row
+    longer: bool = False                   # some entry has more than one row
+    host: Optional[np.ndarray] = None      # [entries, 4] start, len, slot, pos0 (None for a captured decode step)
+
+    @staticmethod
+    def plan(entries: Sequence[StepEntry]) -> Dict[str, np.ndarray]:
+        """Host tables of a step: pure bookkeeping, no device involved."""
+        lens = np.array([len(e.tokens) for e in entries], dtype=np.int32)
+        if len(entries) == 0 or (lens <= 0).any():
+            raise ValueError("every entry of a step brings at least one token")
+        slots = np.array([e.slot for e in entries], dtype=np.int32)
+        if len(set(slots.tolist())) != len(entries):
+            raise ValueError("a sequence can take part in a step only once")
+        start = np.concatenate([[0], np.cumsum(lens)[:-1]]).astype(np.int32)
+        pos0 = np.array([e.pos0 for e in entries], dtype=np.int32)
+        n_pages = [(e.pos0 + len(e.tokens) + PAGE - 1) // PAGE for e in entries]
+        for e, n in zip(entries, n_pages):
+            if len(e.pages) < n:
+                raise ValueError(f"slot {e.slot}: {len(e.pages)} pages do not hold {e.pos0 + len(e.tokens)} tokens")
+        table = np.zeros((len(entries), max(n_pages)), dtype=np.int32)
+        for i, (e, n) in enumerate(zip(entries, n_pages)):
+            table[i, :n] = e.pages[:n]
+        tiles = np.array([(i, r) for i, n in enumerate(lens) for r in range(0, n, NORM_ROWS)], dtype=np.int32)
+        return {"tokens": np.concatenate([np.asarray(e.tokens) for e in entries]).astype(np.int32),
+                "row_entry": np.repeat(np.arange(len(entries), dtype=np.int32), lens), "start": start, "len": lens,
+                "slot": slots, "pos0": pos0, "table": table, "tiles": tiles}
+
+    @staticmethod
+    def build(entries: Sequence[StepEntry], device) -> "StepBatch":
+        p = StepBatch.plan(entries)
+        names = ("tokens", "row_entry", "start", "len", "slot", "pos0", "table", "tiles")
+        flat = torch.from_numpy(np.concatenate([p[n].reshape(-1) for n in names]))
+        dev = to_device(flat.pin_memory(), device)                   # all tables of the step in one copy
+        t, o = {}, 0
+        for n in names:
+            t[n] = dev[o:o + p[n].size].view(p[n].shape)
+            o += p[n].size
+        lens = p["len"]
+        rows = int(lens.sum())
+        return StepBatch(rows, len(entries), t["tokens"], t["row_entry"], t["start"], t["len"], t["slot"], t["pos0"],
+                         t["table"], torch.empty(rows, device=device, dtype=torch.int32), t["tiles"],
+                         bool((lens == 1).any()), bool((lens > 1).any()),
+                         np.stack([p["start"], lens, p["slot"], p["pos0"]], 1))
+
+    def entry_ptrs(self):
+        return _lib.ptr(self.start), _lib.ptr(self.len), _lib.ptr(self.slot), _lib.ptr(self.pos0)
+
+
+# --------------------------------------------------------------------------------------------- embedding and loop input
+def embed(b: StepBatch, table: torch.Tensor, bigram: Optional[torch.Tensor], hash_spec: Optional[Tuple[int, int, int]],
+          prev: torch.Tensor, x: torch.Tensor, x0: Optional[torch.Tensor] = None) -> None:
+    """``x [rows, W]`` fp32 = token rows + hashed bigram rows (``hash_spec`` = buckets, multiplier of the previous and
+    of the current token); ``x0`` receives them in the activation type.  Also fills ``b.kv_slot``."""
+    V, W = table.shape
+    buckets, mp, mc = hash_spec or (0, 0, 0)
+    _call("apb_embed_hash", _lib.ptr(b.tokens), _lib.ptr(b.row_entry), *b.entry_ptrs(), _lib.ptr(prev), _lib.ptr(table),
+          _lib.ptr(bigram), buckets, mp, mc, V, W, _lib.ptr(x), _lib.ptr(x0), 0 if x0 is None else x0.stride(0),
+          _lib.ptr(b.page_table), b.page_table.stride(0), _lib.ptr(b.kv_slot), b.rows, dtype_code(table.dtype))
+
+
+def loop_begin(x: torch.Tensor, init: torch.Tensor, out: torch.Tensor) -> None:
+    """``out [rows, W]`` (a column slice) = ``x`` in the activation type; ``x`` = ``init [W]`` in every row."""
+    _call("apb_loop_begin", _lib.ptr(x), _lib.ptr(init), x.shape[0], x.shape[1], _lib.ptr(out), out.stride(0),
+          dtype_code(out.dtype))
+
+
+# --------------------------------------------------------------------------------------------- norms and convolutions
+def norm_conv(b: StepBatch, x: torch.Tensor, gain: torch.Tensor, w1: Optional[torch.Tensor],
+              w2: Optional[torch.Tensor], two: bool, state: Optional[torch.Tensor], parity: torch.Tensor, taps: int,
+              eps: float) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
+    """``h = x / rms(x) * gain`` and up to two causal depth-wise input convolutions of it: ``h + conv(h, w_k)`` with
+    ``w_k [taps, W]`` (None: ``h``).  ``state [slots, 2, taps - 1, W]`` fp32 is the double-buffered history of ``h``."""
+    T, W = x.shape
+    o1 = torch.empty((T, W), device=x.device, dtype=gain.dtype)
+    o2 = torch.empty_like(o1) if two else None
+    n = b.n_entries if b.tiles is None else b.tiles.shape[0]
+    _call("apb_norm_conv", _lib.ptr(x), _lib.ptr(gain), _lib.ptr(w1), _lib.ptr(w2), _lib.ptr(o1), _lib.ptr(o2),
+          _lib.ptr(state), _lib.ptr(parity), *b.entry_ptrs(), _lib.ptr(b.tiles), n, W, taps, float(eps),
+          dtype_code(gain.dtype))
+    return o1, o2
+
+
+def gain_norm_rows(x: torch.Tensor, rows: Optional[torch.Tensor], gain: torch.Tensor, eps: float) -> torch.Tensor:
+    n = x.shape[0] if rows is None else rows.shape[0]
+    out = torch.empty((n, x.shape[1]), device=x.device, dtype=gain.dtype)
+    _call("apb_gain_norm_rows", _lib.ptr(x), _lib.ptr(rows), _lib.ptr(gain), _lib.ptr(out), n, x.shape[1], float(eps),
+          dtype_code(gain.dtype))
+    return out
+
+
+def qk_norm_cache(b: StepBatch, p: torch.Tensor, cols: Tuple[int, int, int], kcache: torch.Tensor, vcache: torch.Tensor,
+                  heads: int, eps: float) -> None:
+    """q and k columns of ``p`` divided by their root mean square per head (q in place), k and v into the page cache
+    (``[pages, G, PAGE, D]`` and ``[pages, G, PAGE, E]``)."""
+    G, D, E = kcache.shape[1], kcache.shape[3], vcache.shape[3]
+    _call("apb_qk_norm_cache", _lib.ptr(p), p.stride(0), *cols, _lib.ptr(b.kv_slot), _lib.ptr(kcache), _lib.ptr(vcache),
+          b.rows, heads, G, D, E, float(eps), dtype_code(p.dtype))
+
+
+def commit(b: StepBatch, prev: torch.Tensor, parity: torch.Tensor) -> None:
+    """End of a step: last tokens of the entries, parity of the double-buffered states."""
+    _call("apb_serve_commit", _lib.ptr(b.tokens), *b.entry_ptrs(), b.n_entries, _lib.ptr(prev), _lib.ptr(parity))
+
+
+# --------------------------------------------------------------------------------------------- products
+def linear(a: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, *, accumulate: bool = False,
+           out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+    """``a [M, K] @ w [N, K]^T``.  ``accumulate``: added onto fp32 ``out`` (few rows: cut along K over the SMs)."""
+    M, K = a.shape
+    N = w.shape[0]
+    if out is None:
+        out = torch.empty((M, N), device=a.device, dtype=out_dtype or a.dtype)
+    f32_out = out.dtype == torch.float32
+    if _simt(a, w, out):
+        epi = gemm.EPI_F32_ACCUM if accumulate else (gemm.EPI_F32 if f32_out else gemm.EPI_BF16)
+        _gemm_simt(a, w, out, epi)
+        return out
+    if accumulate:
+        tiles = ((M + 127) // 128) * ((N + 127) // 128)
+        splits = max(1, min(_sm_count(a.device) // tiles, (K + 63) // 64))
+        gemm.gemm_raw(a, w, out, M=M, N=N, K=K, epi=gemm.EPI_F32_ATOMIC if splits > 1 else gemm.EPI_F32_ACCUM,
+                      splits=splits, bn=128 if splits > 1 else 0)
+    else:
+        gemm.gemm_raw(a, w, out, M=M, N=N, K=K, epi=gemm.EPI_F32 if f32_out else gemm.EPI_BF16)
+    return out
+
+
+def gate_up_gelu(x: torch.Tensor, w_gu: torch.Tensor, out: torch.Tensor) -> None:
+    """``out [M, ff]`` (may be a column slice) = gelu_tanh(gate) * up; gate and up rows interleaved in ``w_gu``."""
+    M, K = x.shape
+    N = w_gu.shape[0]
+    if _simt(x, w_gu, out) or N % 16:
+        _gemm_simt(x, w_gu, None, gemm.EPI_GEGLU, out2=out)
+    else:
+        gemm.gemm_raw(x, w_gu, None, M=M, N=N, K=K, epi=gemm.EPI_GEGLU, out2=out)
+
+
+_SMS: Dict[int, int] = {}
+
+
+def _sm_count(device) -> int:
+    i = torch.device(device).index or 0
+    if i not in _SMS:
+        _SMS[i] = torch.cuda.get_device_properties(i).multi_processor_count
+    return _SMS[i]
+
+
+def _simt(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> bool:
+    """fp32 operands, or rows the TMA-fed kernels cannot address (not a multiple of 16 bytes)."""
+    return (a.dtype == torch.float32 or bool(a.stride(0) % 8 or w.stride(0) % 8 or w.shape[0] % 8 or out.stride(0) % 8)
+            or bool((a.data_ptr() | w.data_ptr() | out.data_ptr()) & 15))
+
+
+def _gemm_simt(a, w, out, epi, out2=None) -> None:
+    _call("apb_gemm_simt", _lib.ptr(a), _lib.ptr(w), _lib.ptr(out), a.shape[0], w.shape[0], a.shape[1], a.stride(0),
+          w.stride(0), 0 if out is None else out.stride(0), epi, None, _lib.ptr(out2),
+          0 if out2 is None else out2.stride(0), dtype_code(a.dtype))
+
+
+# --------------------------------------------------------------------------------------------- sequence mixers
+def sigmoid_attention(b: StepBatch, q: torch.Tensor, heads: int, kcache: torch.Tensor, vcache: torch.Tensor,
+                      bias: torch.Tensor, scale: float, out: torch.Tensor, out_scale: float = 1.0) -> None:
+    """``q [rows, heads * D]`` (column slice) over the entries' pages -> ``out [rows, heads * E]`` (column slice)."""
+    G, D, E = kcache.shape[1], kcache.shape[3], vcache.shape[3]
+    _call("apb_sigmoid_attn", _lib.ptr(q), q.stride(0), _lib.ptr(b.row_entry), *b.entry_ptrs(), _lib.ptr(b.page_table),
+          b.page_table.stride(0), _lib.ptr(kcache), _lib.ptr(vcache), _lib.ptr(bias), _lib.ptr(out), out.stride(0),
+          b.rows, heads, G, D, E, float(scale), float(out_scale), dtype_code(q.dtype))
+
+
+def retention(b: StepBatch, p: torch.Tensor, cols: Tuple[int, int, int, int], rope: Tuple[torch.Tensor, torch.Tensor],
+              rot_dims: int, log2_decay: torch.Tensor, state: torch.Tensor, out: torch.Tensor, eps: float,
+              k_scale: float, out_scale: float = 1.0) -> None:
+    """Retention of the q, k, v columns of ``p`` with the carried ``state [slots, H, D, E]`` (fp32), per-head norm, the
+    silu gate of the g columns; ``out [rows, H * E]`` (column slice)."""
+    _, H, D, E = state.shape
+    scratch = torch.empty((b.rows, H, E), device=p.device, dtype=torch.float32) if b.longer else None
+    _call("apb_retention", _lib.ptr(p), p.stride(0), *cols, _lib.ptr(rope[0]), _lib.ptr(rope[1]), rot_dims,
+          _lib.ptr(log2_decay), float(k_scale), _lib.ptr(state), _lib.ptr(scratch), _lib.ptr(out), out.stride(0),
+          float(out_scale), float(eps), _lib.ptr(b.row_entry), *b.entry_ptrs(), b.n_entries, b.rows, H, D, E,
+          int(b.one_token), int(b.longer), dtype_code(p.dtype))
