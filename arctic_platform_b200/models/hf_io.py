@@ -307,7 +307,7 @@ def write_safetensors(path, tensors: Dict[str, torch.Tensor], metadata: Optional
         f.write(hb)
         for t in items:
             if t.numel():
-                f.write(t.view(torch.uint8).reshape(-1).numpy().tobytes())
+                f.write(t.reshape(-1).view(torch.uint8).numpy().tobytes())
 
 
 def _composite_stream(model, source):
