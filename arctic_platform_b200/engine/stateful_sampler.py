@@ -109,6 +109,9 @@ class StatefulSampler(SamplerEngine):
     def kv_bytes(self) -> int:
         return self.cache.num_bytes() if self.cache is not None else 0
 
+    def _cascade_on(self) -> bool:
+        return False
+
     def _copy_pages(self, src, dst) -> None:
         self.cache.copy_pages(src, dst)
 

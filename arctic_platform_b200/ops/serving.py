@@ -8,7 +8,7 @@ kernels of ``serve_layers.cu``, ``serve_attention.cu``, ``serve_attention_tc.cu`
 from __future__ import annotations
 
 import ctypes
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 from typing import Dict, List, Optional, Sequence, Tuple
 
 import numpy as np
@@ -35,6 +35,8 @@ def _fn(name: str):
             "apb_qk_norm_cache": [vp, ll, i, i, i, vp, vp, vp, i, i, i, i, i, f, i, vp],
             "apb_serve_commit": [vp] * 5 + [i, vp, vp, vp],
             "apb_sigmoid_attn": [vp, ll, vp, vp, vp, vp, vp, vp, i, vp, vp, vp, vp, ll, i, i, i, i, i, f, f, i, vp],
+            "apb_sigmoid_attn_mma": [vp, ll, vp, vp, vp, vp, i, vp, i, vp, vp, vp, vp, ll, vp] + [i] * 7 + [f, f, vp],
+            "apb_sigmoid_attn_tc": [vp, ll, i, vp, i, vp, i, vp, vp, i, vp, vp, ll, i, i, i, i, f, f, vp],
             "apb_retention": [vp, ll, i, i, i, i, vp, vp, i, vp, f, vp, vp, vp, ll, f, f, vp, vp, vp, vp, vp] + [i] * 8 + [vp],
             "apb_gemm_simt": [vp, vp, vp, i, i, i, ll, ll, ll, i, vp, vp, ll, i, vp],
         }
@@ -80,6 +82,7 @@ class StepBatch:
     tiles: Optional[torch.Tensor] = None   # [n, 2] (entry, first row) of the norm + convolution blocks
     one_token: bool = True                 # some entry has exactly one row
     longer: bool = False                   # some entry has more than one row
+    tables: Dict[tuple, torch.Tensor] = field(default_factory=dict)
     host: Optional[np.ndarray] = None      # [entries, 4] start, len, slot, pos0 (None for a captured decode step)
 
     @staticmethod
@@ -119,8 +122,13 @@ class StepBatch:
         rows = int(lens.sum())
         return StepBatch(rows, len(entries), t["tokens"], t["row_entry"], t["start"], t["len"], t["slot"], t["pos0"],
                          t["table"], torch.empty(rows, device=device, dtype=torch.int32), t["tiles"],
-                         bool((lens == 1).any()), bool((lens > 1).any()),
-                         np.stack([p["start"], lens, p["slot"], p["pos0"]], 1))
+                         bool((lens == 1).any()), bool((lens > 1).any()), host=np.stack([p["start"], lens, p["slot"], p["pos0"]], 1))
+
+    def table(self, key, make) -> torch.Tensor:
+        """Device copy of a host table derived from the batch, made once and shared by its layers."""
+        if key not in self.tables:
+            self.tables[key] = to_device(torch.from_numpy(make()).pin_memory(), self.tokens.device)
+        return self.tables[key]
 
     def entry_ptrs(self):
         return _lib.ptr(self.start), _lib.ptr(self.len), _lib.ptr(self.slot), _lib.ptr(self.pos0)
@@ -238,13 +246,74 @@ def _gemm_simt(a, w, out, epi, out2=None) -> None:
 
 
 # --------------------------------------------------------------------------------------------- sequence mixers
+SHORT_ROWS = 16         # entries up to this length take the few-query tiles, longer ones the tcgen05 kernel
+MAX_SPLITS = 8
+
+
+def tile_work(host: np.ndarray, heads: int, kv_heads: int, min_len: int, tile: int = 128) -> np.ndarray:
+    """Work items of the tcgen05 attention kernel for the entries of at least ``min_len`` rows, longest key range
+    first: ``[n, 12]`` int32 = entry, key blocks, KV head, 0, then for each of two groups (first row, valid rows, head,
+    keys visible to the first row).  The groups are two query heads of the KV head on the same row tile; a head left over
+    pairs two consecutive row tiles (``valid = 0``: no second group)."""
+    R = heads // kv_heads
+    parts = []
+    for en, (start, n, _slot, pos0) in enumerate(host.tolist()):
+        if n < min_len:
+            continue
+        t = np.arange(0, n, tile)
+        rows, valid, keys = start + t, np.minimum(tile, n - t), pos0 + t + 1
+        last = keys + valid - 1                                              # keys visible to a tile's last row
+
+        def items(rows0, valid0, keys0, h0, rows1, valid1, keys1, h1, seen):
+            m = len(rows0)
+            it = np.zeros((kv_heads, m, 12), dtype=np.int64)
+            g = np.arange(kv_heads)[:, None]
+            it[..., 0], it[..., 1], it[..., 2] = en, (seen + tile - 1) // tile, g
+            for o, (r, v, h, k) in ((4, (rows0, valid0, h0, keys0)), (8, (rows1, valid1, h1, keys1))):
+                it[..., o], it[..., o + 1], it[..., o + 2], it[..., o + 3] = r, v, g * R + h, k
+            parts.append(it.reshape(-1, 12))
+
+        for h in range(0, R - 1, 2):
+            items(rows, valid, keys, h, rows, valid, keys, h + 1, last)
+        if R % 2:
+            a, b = slice(0, None, 2), slice(1, None, 2)
+            odd = len(t) % 2
+            second = [np.concatenate([x[b], x[-1:] * 0]) if odd else x[b] for x in (rows, valid, keys, last)]
+            items(rows[a], valid[a], keys[a], R - 1, second[0], second[1], second[2], R - 1, np.maximum(last[a], second[3]))
+    if not parts:
+        return np.zeros((0, 12), dtype=np.int32)
+    work = np.concatenate(parts)
+    return np.ascontiguousarray(work[np.argsort(-work[:, 1], kind="stable")], dtype=np.int32)
+
+
 def sigmoid_attention(b: StepBatch, q: torch.Tensor, heads: int, kcache: torch.Tensor, vcache: torch.Tensor,
                       bias: torch.Tensor, scale: float, out: torch.Tensor, out_scale: float = 1.0) -> None:
-    """``q [rows, heads * D]`` (column slice) over the entries' pages -> ``out [rows, heads * E]`` (column slice)."""
+    """``q [rows, heads * D]`` (column slice) over the entries' pages -> ``out [rows, heads * E]`` (column slice).
+    bf16 with head sizes that are multiples of 8 runs on tensor cores; fp32 and odd sizes on CUDA cores."""
     G, D, E = kcache.shape[1], kcache.shape[3], vcache.shape[3]
-    _call("apb_sigmoid_attn", _lib.ptr(q), q.stride(0), _lib.ptr(b.row_entry), *b.entry_ptrs(), _lib.ptr(b.page_table),
-          b.page_table.stride(0), _lib.ptr(kcache), _lib.ptr(vcache), _lib.ptr(bias), _lib.ptr(out), out.stride(0),
-          b.rows, heads, G, D, E, float(scale), float(out_scale), dtype_code(q.dtype))
+    aligned = not (D % 8 or E % 8 or q.stride(0) % 8 or out.stride(0) % 8 or (q.data_ptr() | out.data_ptr()) & 15)
+    if q.dtype != torch.bfloat16 or not aligned or max(D, E) > 256:
+        _call("apb_sigmoid_attn", _lib.ptr(q), q.stride(0), _lib.ptr(b.row_entry), *b.entry_ptrs(),
+              _lib.ptr(b.page_table), b.page_table.stride(0), _lib.ptr(kcache), _lib.ptr(vcache), _lib.ptr(bias),
+              _lib.ptr(out), out.stride(0), b.rows, heads, G, D, E, float(scale), float(out_scale), dtype_code(q.dtype))
+        return
+    lens = np.ones(1, dtype=np.int64) if b.host is None else b.host[:, 1]
+    limit = SHORT_ROWS if max(D, E) <= 128 else int(lens.max())
+    short = lens[lens <= limit]
+    if len(short):
+        longest = int(short.max())
+        passes = min(256, (longest * (heads // G) + 15) // 16)
+        splits = max(1, min(MAX_SPLITS, 2 * _sm_count(q.device) // (b.n_entries * G * passes)))
+        part = torch.empty((b.n_entries, longest, heads, splits, E), device=q.device, dtype=torch.float32) \
+            if splits > 1 else None
+        _call("apb_sigmoid_attn_mma", _lib.ptr(q), q.stride(0), *b.entry_ptrs(), b.n_entries, _lib.ptr(b.page_table),
+              b.page_table.stride(0), _lib.ptr(kcache), _lib.ptr(vcache), _lib.ptr(bias), _lib.ptr(out), out.stride(0),
+              _lib.ptr(part), heads, G, D, E, 1, longest, splits, float(scale), float(out_scale))
+    if len(short) < len(lens):
+        work = b.table(("sigmoid", heads, G), lambda: tile_work(b.host, heads, G, limit + 1))
+        _call("apb_sigmoid_attn_tc", _lib.ptr(q), q.stride(0), b.rows, _lib.ptr(work), work.shape[0],
+              _lib.ptr(b.page_table), b.page_table.stride(0), _lib.ptr(kcache), _lib.ptr(vcache), kcache.shape[0],
+              _lib.ptr(bias), _lib.ptr(out), out.stride(0), heads, G, D, E, float(scale), float(out_scale))
 
 
 def retention(b: StepBatch, p: torch.Tensor, cols: Tuple[int, int, int, int], rope: Tuple[torch.Tensor, torch.Tensor],

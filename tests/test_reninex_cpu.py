@@ -151,3 +151,25 @@ def test_oracle_retention_equals_the_quadratic_form():
     for h in range(2):
         w = torch.where(j <= i, decay[h] ** (i - j).clamp(min=0).double(), torch.zeros(()).double())
         assert torch.allclose(((q[:, h] @ k[:, h].t()) * w) @ v[:, h], o[:, h])
+
+
+@pytest.mark.parametrize("heads,kv", [(4, 2), (3, 1), (5, 5), (6, 2), (1, 1)])
+def test_attention_work_items_cover_every_row_and_head_once(heads, kv):
+    from arctic_platform_b200.ops.serving import tile_work
+    host = np.array([[0, 300, 1, 40], [300, 5, 0, 1000], [305, 129, 2, 0], [434, 128, 3, 7]])
+    work = tile_work(host, heads, kv, 17)
+    seen = {}
+    for en, blocks, g, _, *groups in work.tolist():
+        last = 0
+        for row, valid, head, keys in (groups[:4], groups[4:]):
+            if valid == 0:
+                continue
+            start, n, _, pos0 = host[en]
+            assert head // (heads // kv) == g and keys == pos0 + (row - start) + 1 and row + valid <= start + n
+            last = max(last, keys + valid - 1)
+            for r in range(row, row + valid):
+                seen[r, head] = seen.get((r, head), 0) + 1
+        assert blocks == -(-last // 128)
+    rows = [r for s, n, _, _ in host.tolist() if n > 16 for r in range(s, s + n)]
+    assert seen == {(r, h): 1 for r in rows for h in range(heads)}
+    assert (np.diff(work[:, 1]) <= 0).all()
