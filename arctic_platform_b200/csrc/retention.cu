@@ -10,41 +10,13 @@
 //  * retention_chunk_kernel   longer entries, chunk by chunk: inside a chunk of C tokens the masked products
 //                             (q_i . k_j) decay^(i-j), across chunks the carried state.  One CTA per (entry, head,
 //                             32-column slice of E), fp32 CUDA-core arithmetic; followed by retention_out_kernel.
+//
+// bf16 engines run longer entries on tensor cores (retention_mma.cu).
 #include "common.cuh"
 #include "host_utils.cuh"
-#include "serve_common.cuh"
+#include "retention.cuh"
 
 namespace apb {
-
-struct RetentionParams {
-  ServeEntries e;
-  const void* p;          // projection buffer [rows, ld]
-  long long ld;
-  int q_col, k_col, v_col, g_col;
-  const float* cos_t;     // [positions, rot_dims / 2]
-  const float* sin_t;
-  int rot_dims;
-  const float* log2_decay;  // [H] log2 of the decay (-inf for 0)
-  float k_scale;
-  float* state;           // [slots, H, D, E]
-  float* o;               // [rows, H, E] fp32, un-normalised (chunk kernels)
-  void* out;              // [rows, ldo] (activation type), already offset to its first column
-  long long ldo;
-  float out_scale, eps;
-  int H, D, E;
-};
-
-__device__ __forceinline__ float decay_pow(float log2_decay, int n) { return n == 0 ? 1.f : exp2f(log2_decay * n); }
-
-// Element d of a rotated head whose raw values start at `src`.
-template <typename T>
-__device__ __forceinline__ float rotated(const T* src, int d, int rot, const float* c, const float* s) {
-  const int half = rot >> 1;
-  const float a = to_f32(src[d]);
-  if (d >= rot) return a;
-  if (d < half) return a * c[d] - to_f32(src[d + half]) * s[d];
-  return a * c[d - half] + to_f32(src[d - half]) * s[d - half];
-}
 
 // ---------------------------------------------------------------------------- one token
 constexpr int kRetThreads = 256;
@@ -245,6 +217,29 @@ retention_out_kernel(const RetentionParams p, const int* __restrict__ row_entry,
   const T* g = static_cast<const T*>(p.p) + static_cast<long long>(row) * p.ld + p.g_col + static_cast<long long>(h) * E;
   T* out = static_cast<T*>(p.out) + static_cast<long long>(row) * p.ldo + static_cast<long long>(h) * E;
   float ss = 0.f;
+  if (sizeof(T) == 2 && (E & 3) == 0 && E <= 512 && ((reinterpret_cast<uintptr_t>(g) | reinterpret_cast<uintptr_t>(out)) & 7) == 0) {
+    float4 v[4];                                    // four elements per lane and 128-column step
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int i = k * 128 + lane * 4;
+      v[k] = i < E ? __ldcs(reinterpret_cast<const float4*>(o + i)) : make_float4(0.f, 0.f, 0.f, 0.f);
+      ss += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+    }
+    const float f = p.out_scale / sqrtf(warp_sum(ss) / E + p.eps);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int i = k * 128 + lane * 4;
+      if (i >= E) continue;
+      const uint2 gr = *reinterpret_cast<const uint2*>(g + i);
+      const float2 g0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gr.x));
+      const float2 g1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gr.y));
+      uint2 r;
+      r.x = pack_bf16x2(v[k].x * f * (g0.x / (1.f + expf(-g0.x))), v[k].y * f * (g0.y / (1.f + expf(-g0.y))));
+      r.y = pack_bf16x2(v[k].z * f * (g1.x / (1.f + expf(-g1.x))), v[k].w * f * (g1.y / (1.f + expf(-g1.y))));
+      *reinterpret_cast<uint2*>(out + i) = r;
+    }
+    return;
+  }
   for (int i = lane; i < E; i += 32) ss += o[i] * o[i];
   const float f = p.out_scale / sqrtf(warp_sum(ss) / E + p.eps);
   for (int i = lane; i < E; i += 32) {
@@ -328,5 +323,27 @@ int apb_retention(const void* p, long long ld, int q_col, int k_col, int v_col, 
     return kBadArgument;
   }
   return 0;
+}
+
+// The output stage alone, for o written by apb_retention_mma: out [rows, ldo] = o / rms(o) * silu(g) * out_scale for the
+// rows of entries longer than one token.
+int apb_retention_out(const void* p, long long ld, int g_col, float* o, void* out, long long ldo, float out_scale, float eps,
+                      const int* row_entry, const int* e_start, const int* e_len, const int* e_slot, const int* e_pos0,
+                      int rows, int H, int E, int dtype, cudaStream_t s) {
+  if (rows <= 0) return 0;
+  RetentionParams a{};
+  a.e = ServeEntries{e_start, e_len, e_slot, e_pos0};
+  a.p = p;
+  a.ld = ld;
+  a.g_col = g_col;
+  a.o = o;
+  a.out = out;
+  a.ldo = ldo;
+  a.out_scale = out_scale;
+  a.eps = eps;
+  a.H = H;
+  a.E = E;
+  const int grid = static_cast<int>((static_cast<long long>(rows) * H * 32 + 255) / 256);
+  APB_SERVE_DTYPE(dtype, return static_cast<int>(launch_kernel(retention_out_kernel<T>, dim3(grid), dim3(256), 0, s, a, row_entry, rows)));
 }
 }

@@ -38,6 +38,8 @@ def _fn(name: str):
             "apb_sigmoid_attn_mma": [vp, ll, vp, vp, vp, vp, i, vp, i, vp, vp, vp, vp, ll, vp] + [i] * 7 + [f, f, vp],
             "apb_sigmoid_attn_tc": [vp, ll, i, vp, i, vp, i, vp, vp, i, vp, vp, ll, i, i, i, i, f, f, vp],
             "apb_retention": [vp, ll, i, i, i, i, vp, vp, i, vp, f, vp, vp, vp, ll, f, f, vp, vp, vp, vp, vp] + [i] * 8 + [vp],
+            "apb_retention_mma": [vp, ll, i, i, i, vp, vp, i, vp, f] + [vp] * 7 + [i, vp, vp, i, i, i, i, vp],
+            "apb_retention_out": [vp, ll, i, vp, vp, ll, f, f, vp, vp, vp, vp, vp, i, i, i, i, vp],
             "apb_gemm_simt": [vp, vp, vp, i, i, i, ll, ll, ll, i, vp, vp, ll, i, vp],
         }
         _FN[name] = _lib.declare(name, sigs[name])
@@ -82,7 +84,8 @@ class StepBatch:
     tiles: Optional[torch.Tensor] = None   # [n, 2] (entry, first row) of the norm + convolution blocks
     one_token: bool = True                 # some entry has exactly one row
     longer: bool = False                   # some entry has more than one row
-    tables: Dict[tuple, torch.Tensor] = field(default_factory=dict)
+    tables: Dict[tuple, torch.Tensor] = field(default_factory=dict)       # derived tables, on the device / host
+    host_tables: Dict[tuple, dict] = field(default_factory=dict)
     host: Optional[np.ndarray] = None      # [entries, 4] start, len, slot, pos0 (None for a captured decode step)
 
     @staticmethod
@@ -316,6 +319,35 @@ def sigmoid_attention(b: StepBatch, q: torch.Tensor, heads: int, kcache: torch.T
               _lib.ptr(bias), _lib.ptr(out), out.stride(0), heads, G, D, E, float(scale), float(out_scale))
 
 
+MIN_SEGMENT = 256       # tokens; a multiple of the kernel's chunk
+
+
+def segment_plan(host: np.ndarray, slices: int, slots: int) -> Dict[str, object]:
+    """Cuts entries longer than one row into segments so that about ``slots`` blocks (``slices`` per segment) run at
+    once.  ``seg [n, 6]``: entry, first token, tokens, scratch state before the segment (-1: none), scratch state for its
+    contribution (-1: none), last of its entry.  ``chains [m, 4]``: entry, first scratch state, segments, first segment --
+    for the entries of more than one segment."""
+    work = [(en, int(n)) for en, n in enumerate(host[:, 1]) if n > 1]
+    total = sum(n for _, n in work)
+    want = max(1, slots // slices)
+    size = max(n for _, n in work) if len(work) * 2 >= want else max(MIN_SEGMENT, -(-total // want))
+    size = -(-size // 32) * 32
+    seg, chains, states = [], [], 0
+    for en, n in work:
+        k = max(1, -(-n // size))
+        step = -(-(-(-n // k)) // 32) * 32 if k > 1 else n
+        k = -(-n // step)
+        if k > 1:
+            chains.append((en, states, k, len(seg)))
+        for i in range(k):
+            last = i + 1 == k
+            seg.append((en, i * step, min(step, n - i * step), states + i if k > 1 else -1,
+                        -1 if last else states + i + 1, int(last)))
+        states += k if k > 1 else 0
+    return {"seg": np.array(seg, dtype=np.int32).reshape(-1, 6), "states": states,
+            "chains": np.array(chains, dtype=np.int32).reshape(-1, 4)}
+
+
 def retention(b: StepBatch, p: torch.Tensor, cols: Tuple[int, int, int, int], rope: Tuple[torch.Tensor, torch.Tensor],
               rot_dims: int, log2_decay: torch.Tensor, state: torch.Tensor, out: torch.Tensor, eps: float,
               k_scale: float, out_scale: float = 1.0) -> None:
@@ -323,7 +355,24 @@ def retention(b: StepBatch, p: torch.Tensor, cols: Tuple[int, int, int, int], ro
     silu gate of the g columns; ``out [rows, H * E]`` (column slice)."""
     _, H, D, E = state.shape
     scratch = torch.empty((b.rows, H, E), device=p.device, dtype=torch.float32) if b.longer else None
-    _call("apb_retention", _lib.ptr(p), p.stride(0), *cols, _lib.ptr(rope[0]), _lib.ptr(rope[1]), rot_dims,
-          _lib.ptr(log2_decay), float(k_scale), _lib.ptr(state), _lib.ptr(scratch), _lib.ptr(out), out.stride(0),
-          float(out_scale), float(eps), _lib.ptr(b.row_entry), *b.entry_ptrs(), b.n_entries, b.rows, H, D, E,
-          int(b.one_token), int(b.longer), dtype_code(p.dtype))
+    aligned = not (D % 8 or E % 8 or p.stride(0) % 8 or p.data_ptr() & 15 or any(c % 8 for c in cols))
+    mma = b.longer and p.dtype == torch.bfloat16 and aligned and D <= 128
+    if b.one_token or not mma:
+        _call("apb_retention", _lib.ptr(p), p.stride(0), *cols, _lib.ptr(rope[0]), _lib.ptr(rope[1]), rot_dims,
+              _lib.ptr(log2_decay), float(k_scale), _lib.ptr(state), _lib.ptr(scratch), _lib.ptr(out), out.stride(0),
+              float(out_scale), float(eps), _lib.ptr(b.row_entry), *b.entry_ptrs(), b.n_entries, b.rows, H, D, E,
+              int(b.one_token), int(b.longer and not mma), dtype_code(p.dtype))
+    if mma:
+        slices = H * ((E + 63) // 64)
+        key = ("retention", slices)
+        if key not in b.host_tables:
+            b.host_tables[key] = segment_plan(b.host, slices, 2 * _sm_count(p.device))
+        plan = b.host_tables[key]
+        seg = b.table(key + ("seg",), lambda: plan["seg"])
+        chains = b.table(key + ("chains",), lambda: plan["chains"]) if len(plan["chains"]) else None
+        carry = torch.empty((plan["states"], H, D, E), device=p.device, dtype=torch.float32) if plan["states"] else None
+        _call("apb_retention_mma", _lib.ptr(p), p.stride(0), *cols[:3], _lib.ptr(rope[0]), _lib.ptr(rope[1]), rot_dims,
+              _lib.ptr(log2_decay), float(k_scale), _lib.ptr(state), _lib.ptr(scratch), *b.entry_ptrs(), _lib.ptr(seg),
+              len(plan["seg"]), _lib.ptr(carry), _lib.ptr(chains), len(plan["chains"]), H, D, E)
+        _call("apb_retention_out", _lib.ptr(p), p.stride(0), cols[3], _lib.ptr(scratch), _lib.ptr(out), out.stride(0),
+              float(out_scale), float(eps), _lib.ptr(b.row_entry), *b.entry_ptrs(), b.rows, H, E, dtype_code(p.dtype))

@@ -227,24 +227,18 @@ def test_sigmoid_attention_inputs_show_a_lost_key():
 
 
 # ---------------------------------------------------------------------------- retention
-@pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("H,D,E,rot,base", [(4, 32, 64, 32, 1e6), (3, 22, 10, 6, 100.0), (2, 128, 128, 64, 1e4),
-                                            (1, 64, 200, 0, 1e4), (2, 48, 256, 48, 500.0), (2, 192, 96, 128, 1e4)])
-def test_retention_in_portions(dtype, H, D, E, rot, base):
+def _run_retention(dtype, H, D, E, rot, base, decay, lens, schedules, tol):
     from arctic_platform_b200.ops import _lib, norm, serving
-    decay = [1.0, 0.97, 0.5, 0.0][:H] if H > 1 else [0.995]
     l2 = torch.tensor([math.log2(x) if x else float("-inf") for x in decay], device="cuda")
-    eps, ks, out_scale, lens = 1e-5, D ** -0.5, 0.6, [200, 41, 90]
-    rope = norm.rope_tables(256, max(2, rot), base, "cuda")
+    eps, ks, out_scale = 1e-5, D ** -0.5, 0.6
+    rope = norm.rope_tables(max(lens), max(2, rot), base, "cuda")
     pad8 = lambda n: (n + 7) // 8 * 8
     cols, o = [], 8
     for n in (H * D, H * D, H * E, H * E):
         cols.append(o)
         o += pad8(n)
-    state = torch.full((3, H, D, E), 7.0, device="cuda")
-    prev, parity = (torch.zeros(3, dtype=torch.int32, device="cuda") for _ in range(2))
-    tol = {torch.float32: 2e-4, torch.bfloat16: 0.06}[dtype]
-    for rnd, cuts in enumerate(([1000], [2, 1, 31, 64, 5, 33], [100, 1, 1, 1, 1, 1, 1, 1, 1, 1, 1, 1], [65, 3])):
+    state = torch.full((len(lens), H, D, E), 7.0, device="cuda")
+    for rnd, cuts in enumerate(schedules):
         g = torch.Generator().manual_seed(rnd)
         P, want, pages = [], [], _pages(lens)[0]
         for n in lens:
@@ -269,3 +263,19 @@ def test_retention_in_portions(dtype, H, D, E, rot, base):
         for i, w in enumerate(want):
             assert _rel(torch.cat(got[i]), w) < tol, (rnd, i, _rel(torch.cat(got[i]), w))
     _lib.check_status("retention")
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,D,E,rot,base", [(4, 32, 64, 32, 1e6), (3, 22, 10, 6, 100.0), (2, 128, 128, 64, 1e4),
+                                            (1, 64, 200, 0, 1e4), (2, 48, 256, 48, 500.0), (2, 192, 96, 128, 1e4),
+                                            (2, 40, 24, 8, 50.0), (1, 8, 8, 2, 10.0)])
+def test_retention_in_portions(dtype, H, D, E, rot, base):
+    decay = [1.0, 0.97, 0.5, 0.0][:H] if H > 1 else [0.995]
+    cuts = ([1000], [2, 1, 31, 64, 5, 33], [100, 1, 1, 1, 1, 1, 1, 1, 1, 1, 1, 1], [65, 3])
+    _run_retention(dtype, H, D, E, rot, base, decay, [200, 41, 90], cuts, {torch.float32: 2e-4, torch.bfloat16: 0.06}[dtype])
+
+
+@pytest.mark.parametrize("D,E", [(64, 64), (128, 192)])
+def test_retention_over_segments(D, E):
+    """Long entries are cut into segments whose states are chained; slow decays make a lost segment visible."""
+    _run_retention(torch.bfloat16, 2, D, E, D, 1e4, [0.9995, 0.97], [1500, 700, 333], ([5000], [900, 1, 450, 2]), 0.06)

@@ -173,3 +173,25 @@ def test_attention_work_items_cover_every_row_and_head_once(heads, kv):
     rows = [r for s, n, _, _ in host.tolist() if n > 16 for r in range(s, s + n)]
     assert seen == {(r, h): 1 for r in rows for h in range(heads)}
     assert (np.diff(work[:, 1]) <= 0).all()
+
+
+@pytest.mark.parametrize("lens,slices,slots", [([2100, 700, 1, 64], 8, 296), ([500] * 200, 32, 296), ([2], 1, 296),
+                                               ([8192], 32, 296), ([257, 31], 4, 40)])
+def test_retention_segments_cover_every_long_entry_in_order(lens, slices, slots):
+    from arctic_platform_b200.ops.serving import segment_plan
+    host = np.array([[0, n, i, 0] for i, n in enumerate(lens)])
+    plan = segment_plan(host, slices, slots)
+    at, used = {}, set()
+    for i, (en, t, n, before, out, last) in enumerate(plan["seg"].tolist()):
+        assert t == at.get(en, 0) and n > 0
+        at[en] = t + n
+        assert last == (at[en] == lens[en]) and (out >= 0) == (before >= 0 and not last)
+        assert last or n % 32 == 0
+        if before >= 0:
+            assert before not in used and (last or out == before + 1)
+            used.add(before)
+    assert at == {i: n for i, n in enumerate(lens) if n > 1}
+    assert used == set(range(plan["states"]))
+    for en, base, k, first in plan["chains"].tolist():
+        assert k > 1 and plan["seg"][first:first + k, 0].tolist() == [en] * k
+        assert plan["seg"][first:first + k, 3].tolist() == list(range(base, base + k))
