@@ -151,24 +151,55 @@ retention_mma_kernel(const RetentionParams p, const RetentionSegments sg, int st
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();                               // raw rows have landed; everybody is done with the last chunk
     // ---- rotate, scale, split
-    const int pairs = dp >> 1;
+    auto put = [&](__nv_bfloat16* hi_t, __nv_bfloat16* lo_t, int o, float x, float y) {
+      uint32_t hi, lo;
+      rm_split2(x, y, hi, lo);
+      *reinterpret_cast<uint32_t*>(hi_t + o) = hi;
+      *reinterpret_cast<uint32_t*>(lo_t + o) = lo;
+    };
+    const int half = p.rot_dims >> 1;
+    int d_done = 0;                                // dimensions covered by the paired loop
+    if ((half & 1) == 0) {                         // two neighbouring rotation pairs (d, d + half), (d + 1, d + 1 + half)
+      d_done = p.rot_dims;
+      const int q2 = half >> 1;
+#pragma unroll 4
+      for (int i = threadIdx.x; i < kRmC * q2; i += kRmThreads) {
+        const int r = i / q2, d = (i - r * q2) * 2, o = r * ds + d;
+        float2 qu = make_float2(0.f, 0.f), qv = qu, ku = qu, kv = qu, c = qu, sn = qu;
+        if (r < n) {
+          const long long tr = static_cast<long long>(pos0 + t0 + r) * half + d;
+          c = *reinterpret_cast<const float2*>(p.cos_t + tr);
+          sn = *reinterpret_cast<const float2*>(p.sin_t + tr);
+          const __nv_bfloat16* rq = raw + r * dp + d;
+          const __nv_bfloat16* rk = rq + kRmC * dp;
+          qu = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(rq));
+          qv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(rq + half));
+          ku = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(rk));
+          kv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(rk + half));
+        }
+        if (!state_only) {
+          put(Qh, Ql, o, qu.x * c.x - qv.x * sn.x, qu.y * c.y - qv.y * sn.y);
+          put(Qh, Ql, o + half, qv.x * c.x + qu.x * sn.x, qv.y * c.y + qu.y * sn.y);
+        }
+        put(Kh, Kl, o, (ku.x * c.x - kv.x * sn.x) * p.k_scale, (ku.y * c.y - kv.y * sn.y) * p.k_scale);
+        put(Kh, Kl, o + half, (kv.x * c.x + ku.x * sn.x) * p.k_scale, (kv.y * c.y + ku.y * sn.y) * p.k_scale);
+      }
+    }
+    const int pairs = (dp - d_done) >> 1;          // unrotated dimensions (and the padding), or odd rotations
     for (int i = threadIdx.x; i < kRmC * pairs; i += kRmThreads) {
-      const int r = i / pairs, d = (i % pairs) * 2;
-      uint32_t qh = 0, ql = 0, kh = 0, kl = 0;
+      const int r = i / pairs, d = d_done + (i % pairs) * 2, o = r * ds + d;
+      float2 qv = make_float2(0.f, 0.f), kv = qv;
       if (r < n && d < D) {
-        const long long tr = static_cast<long long>(pos0 + t0 + r) * (p.rot_dims >> 1);
+        const long long tr = static_cast<long long>(pos0 + t0 + r) * half;
         const float* c = p.cos_t + tr;
         const float* sn = p.sin_t + tr;
         const __nv_bfloat16* rq = raw + r * dp;
         const __nv_bfloat16* rk = raw + (kRmC + r) * dp;
-        if (!state_only) rm_split2(rotated(rq, d, p.rot_dims, c, sn), rotated(rq, d + 1, p.rot_dims, c, sn), qh, ql);
-        rm_split2(rotated(rk, d, p.rot_dims, c, sn) * p.k_scale, rotated(rk, d + 1, p.rot_dims, c, sn) * p.k_scale, kh, kl);
+        qv = make_float2(rotated(rq, d, p.rot_dims, c, sn), rotated(rq, d + 1, p.rot_dims, c, sn));
+        kv = make_float2(rotated(rk, d, p.rot_dims, c, sn) * p.k_scale, rotated(rk, d + 1, p.rot_dims, c, sn) * p.k_scale);
       }
-      const int o = r * ds + d;
-      *reinterpret_cast<uint32_t*>(Qh + o) = qh;
-      *reinterpret_cast<uint32_t*>(Ql + o) = ql;
-      *reinterpret_cast<uint32_t*>(Kh + o) = kh;
-      *reinterpret_cast<uint32_t*>(Kl + o) = kl;
+      if (!state_only) put(Qh, Ql, o, qv.x, qv.y);
+      put(Kh, Kl, o, kv.x, kv.y);
     }
     for (int i = threadIdx.x; i < kRmC * (kRmBE / 2); i += kRmThreads) {
       const int r = i / (kRmBE / 2), c = (i % (kRmBE / 2)) * 2;

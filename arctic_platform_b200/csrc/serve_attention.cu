@@ -118,8 +118,8 @@ __device__ __forceinline__ void sm_mma(float (&c)[4], const uint32_t (&a)[4], ui
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-// N16: upper bound of D / 16 and E / 16.
-template <int N16>
+// N16: upper bound of D / 16 and E / 16; FULL: both are equal to it (the index arithmetic is then constant).
+template <int N16, bool FULL>
 __global__ void __launch_bounds__(kSigThreads)
 sigmoid_attn_mma_kernel(const SigmoidMmaParams p) {
   pdl_entry();
@@ -127,7 +127,7 @@ sigmoid_attn_mma_kernel(const SigmoidMmaParams p) {
   const int en = blockIdx.x / p.G, g = blockIdx.x % p.G;
   const int len = p.e.len[en];
   if (len < p.min_len || len > p.max_len) return;
-  const int D = p.D, E = p.E, R = p.H / p.G;
+  const int D = FULL ? N16 * 16 : p.D, E = FULL ? N16 * 16 : p.E, R = p.H / p.G;
   const int d16 = (D + 15) >> 4, e16 = (E + 15) >> 4;
   const int k_row = d16 * 32 + 16, v_row = e16 * 32 + 16;            // ring row bytes
   const int stage_bytes = kServePage * (k_row + v_row);
@@ -179,7 +179,9 @@ sigmoid_attn_mma_kernel(const SigmoidMmaParams p) {
         const uint32_t dst = ring + (j % kSmStages) * stage_bytes;
         const __nv_bfloat16* kp = p.kcache + base * D;
         const __nv_bfloat16* vp = p.vcache + base * E;
+#pragma unroll
         for (int i = lane; i < kServePage * kc; i += 32) sm_cp_async16(dst + (i / kc) * k_row + (i % kc) * 16, kp + i * 8);
+#pragma unroll
         for (int i = lane; i < kServePage * vc; i += 32)
           sm_cp_async16(dst + kServePage * k_row + (i / vc) * v_row + (i % vc) * 16, vp + i * 8);
       }
@@ -328,8 +330,12 @@ int apb_sigmoid_attn_mma(const void* q, long long ldq, const int* e_start, const
     return static_cast<int>(launch_kernel(fn, grid, dim3(kSigThreads), smem, s, p));
   };
   const int n16 = d16 > e16 ? d16 : e16;
-  const int rc = n16 <= 4 ? run(sigmoid_attn_mma_kernel<4>) : n16 <= 8 ? run(sigmoid_attn_mma_kernel<8>)
-                                                                      : run(sigmoid_attn_mma_kernel<16>);
+  const bool same = D == E;
+  const int rc = same && D == 128 ? run(sigmoid_attn_mma_kernel<8, true>)
+                 : same && D == 64 ? run(sigmoid_attn_mma_kernel<4, true>)
+                 : n16 <= 4        ? run(sigmoid_attn_mma_kernel<4, false>)
+                 : n16 <= 8        ? run(sigmoid_attn_mma_kernel<8, false>)
+                                   : run(sigmoid_attn_mma_kernel<16, false>);
   if (rc || splits == 1) return rc;
   const int mg = static_cast<int>((static_cast<long long>(n_entries) * max_len * H * 32 + 255) / 256);
   return static_cast<int>(launch_kernel(sigmoid_merge_kernel, dim3(mg), dim3(256), 0, s, p, n_entries, splits));

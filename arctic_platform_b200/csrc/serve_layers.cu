@@ -155,6 +155,140 @@ norm_conv_kernel(const float* __restrict__ x, const T* __restrict__ gain, const 
   }
 }
 
+template <typename T>
+__device__ __forceinline__ float4 load4(const T* p) {
+  if constexpr (sizeof(T) == 2) {
+    const uint2 r = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+  } else {
+    return *reinterpret_cast<const float4*>(p);
+  }
+}
+template <typename T>
+__device__ __forceinline__ void store4(T* p, float4 v) {
+  if constexpr (sizeof(T) == 2) {
+    uint2 r;
+    r.x = pack_bf16x2(v.x, v.y);
+    r.y = pack_bf16x2(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = r;
+  } else {
+    *reinterpret_cast<float4*>(p) = v;
+  }
+}
+__device__ __forceinline__ void fma4(float4& a, const float4& w, const float4& h) {
+  a.x += w.x * h.x;
+  a.y += w.y * h.y;
+  a.z += w.z * h.z;
+  a.w += w.w * h.w;
+}
+
+// The same for a compile-time number of taps and W a multiple of 4: four channels per thread, the rows of the tile
+// loaded at once, the window in registers.
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(kNormThreads)
+norm_conv_vec_kernel(const float* __restrict__ x, const T* __restrict__ gain, const T* __restrict__ w1,
+                     const T* __restrict__ w2, T* __restrict__ out1, T* __restrict__ out2, float* __restrict__ state,
+                     const int* __restrict__ parity, const ServeEntries e, const int* __restrict__ tiles, int W,
+                     float eps) {
+  pdl_entry();
+  constexpr int kHist = TAPS - 1;
+  __shared__ float rs[kHist + kNormRows];
+  __shared__ float red[kNormThreads / 32];
+  const int en = tiles ? tiles[2 * blockIdx.x] : blockIdx.x;
+  const int r0 = tiles ? tiles[2 * blockIdx.x + 1] : 0;
+  const int len = e.len[en];
+  if (r0 >= len) return;
+  const int nr = min(kNormRows, len - r0);
+  const int start = e.start[en], pos0 = e.pos0[en];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const float g = to_f32(*gain);
+  if (len == 1) {                                  // a decoded token: the whole block sums its row
+    const float* xr = x + static_cast<long long>(start) * W;
+    float ss = 0.f;
+#pragma unroll 4
+    for (int c = threadIdx.x * 4; c < W; c += kNormThreads * 4) {
+      const float4 v = *reinterpret_cast<const float4*>(xr + c);
+      ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
+    ss = warp_sum(ss);
+    if (lane == 0) red[warp] = ss;
+    __syncthreads();
+    if (threadIdx.x == 0) {
+      ss = 0.f;
+      for (int i = 0; i < kNormThreads / 32; ++i) ss += red[i];
+      rs[kHist] = g / sqrtf(ss / W + eps);
+    }
+  } else {
+    for (int i = warp; i < kHist + nr; i += kNormThreads / 32) {
+      const int r = r0 - kHist + i;
+      if (r < 0) continue;
+      const float* xr = x + static_cast<long long>(start + r) * W;
+      float ss = 0.f;
+#pragma unroll 8
+      for (int c = lane * 4; c < W; c += 128) {
+        const float4 v = *reinterpret_cast<const float4*>(xr + c);
+        ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+      }
+      ss = warp_sum(ss);
+      if (lane == 0) rs[i] = g / sqrtf(ss / W + eps);
+    }
+  }
+  __syncthreads();
+  const int slot = e.slot[en];
+  const float* old_h = nullptr;
+  float* new_h = nullptr;
+  if (kHist > 0 && slot >= 0) {
+    const int par = parity[slot] & 1;
+    old_h = state + (static_cast<long long>(slot) * 2 + par) * kHist * W;
+    new_h = state + (static_cast<long long>(slot) * 2 + (par ^ 1)) * kHist * W;
+  }
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int c = threadIdx.x * 4; c < W; c += kNormThreads * 4) {
+    float4 h[kHist + kNormRows];                   // rows r0 - hist .. r0 + 7
+#pragma unroll
+    for (int i = 0; i < kHist + kNormRows; ++i) {
+      const int r = r0 - kHist + i;
+      h[i] = zero;
+      if (r >= 0 && i < kHist + nr)
+        h[i] = *reinterpret_cast<const float4*>(x + static_cast<long long>(start + r) * W + c);
+      else if (r < 0 && pos0 + r >= 0 && old_h)
+        h[i] = *reinterpret_cast<const float4*>(old_h + static_cast<long long>(kHist + r) * W + c);
+    }
+    float4 a[TAPS], b[TAPS];
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) {
+      a[j] = w1 ? load4(w1 + static_cast<long long>(j) * W + c) : zero;
+      b[j] = w2 ? load4(w2 + static_cast<long long>(j) * W + c) : zero;
+    }
+#pragma unroll
+    for (int i = 0; i < kHist + kNormRows; ++i)
+      if (r0 - kHist + i >= 0 && i < kHist + nr) {
+        const float f = rs[i];
+        h[i] = make_float4(h[i].x * f, h[i].y * f, h[i].z * f, h[i].w * f);
+      }
+#pragma unroll
+    for (int i = 0; i < kNormRows; ++i)
+      if (i < nr) {
+        float4 y1 = h[i + kHist], y2 = y1;
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) {
+          fma4(y1, a[j], h[i + j]);
+          fma4(y2, b[j], h[i + j]);
+        }
+        const long long o = static_cast<long long>(start + r0 + i) * W + c;
+        store4(out1 + o, y1);
+        if (out2) store4(out2 + o, y2);
+      }
+    if (new_h && r0 + nr == len) {
+#pragma unroll
+      for (int i = 0; i < kHist + kNormRows; ++i)  // rows len - hist .. len - 1
+        if (i >= nr && i < nr + kHist) *reinterpret_cast<float4*>(new_h + static_cast<long long>(i - nr) * W + c) = h[i];
+    }
+  }
+}
+
 // Final norm of selected rows: out[i] = x[rows[i]] / rms * g (rows == null: row i).  One block per row.
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -286,6 +420,16 @@ int apb_norm_conv(const float* x, const void* gain, const void* w1, const void* 
   if (n_tiles <= 0) return 0;
   if (taps < 1 || taps > 1024 || !x || !gain || !out1 || (taps > 1 && (!state || !parity))) return kBadArgument;
   const ServeEntries e{e_start, e_len, e_slot, e_pos0};
+  if ((W & 3) == 0 && taps <= 5) {
+#define APB_NORM_CONV(TT)                                                                                             \
+  return static_cast<int>(launch_kernel(norm_conv_vec_kernel<T, TT>, dim3(n_tiles), dim3(kNormThreads), 0, s, x,      \
+                                        static_cast<const T*>(gain), static_cast<const T*>(w1),                       \
+                                        static_cast<const T*>(w2), static_cast<T*>(out1), static_cast<T*>(out2),      \
+                                        state, parity, e, tiles, W, eps))
+    APB_SERVE_DTYPE(dtype, if (taps == 1) APB_NORM_CONV(1); if (taps == 2) APB_NORM_CONV(2); if (taps == 3) APB_NORM_CONV(3);
+                    if (taps == 4) APB_NORM_CONV(4); APB_NORM_CONV(5));
+#undef APB_NORM_CONV
+  }
   const size_t smem = (taps - 1 + kNormRows) * sizeof(float);
   APB_SERVE_DTYPE(dtype, return static_cast<int>(launch_kernel(
                              norm_conv_kernel<T>, dim3(n_tiles), dim3(kNormThreads), smem, s, x,

@@ -328,13 +328,19 @@ def segment_plan(host: np.ndarray, slices: int, slots: int) -> Dict[str, object]
     contribution (-1: none), last of its entry.  ``chains [m, 4]``: entry, first scratch state, segments, first segment --
     for the entries of more than one segment."""
     work = [(en, int(n)) for en, n in enumerate(host[:, 1]) if n > 1]
-    total = sum(n for _, n in work)
-    want = max(1, slots // slices)
-    size = max(n for _, n in work) if len(work) * 2 >= want else max(MIN_SEGMENT, -(-total // want))
-    size = -(-size // 32) * 32
+    want, size = slots // slices, max(n for _, n in work)
+    if want >= 3 * len(work):            # fewer: the extra pass over the states costs more than it frees
+        lo, hi = 1, -(-size // 32)       # the smallest segment (in chunks of 32) that needs no second wave of blocks
+        while lo < hi:
+            mid = (lo + hi) // 2
+            if sum(-(-n // (mid * 32)) for _, n in work) <= want:
+                hi = mid
+            else:
+                lo = mid + 1
+        size = max(MIN_SEGMENT, lo * 32)
     seg, chains, states = [], [], 0
     for en, n in work:
-        k = max(1, -(-n // size))
+        k = -(-n // size)
         step = -(-(-(-n // k)) // 32) * 32 if k > 1 else n
         k = -(-n // step)
         if k > 1:

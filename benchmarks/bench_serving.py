@@ -1,0 +1,316 @@
+"""Serving speed of a stateful architecture beside the dense decoder of equal layer size.
+
+    python bench.py --workload serving [--serving-models reninex-2048,reninex-4096]
+    python benchmarks/bench_serving.py [--models ...] [--kernels-only] [--only prefill|decode] [--iters 20]
+
+For every model (random weights, synthetic prompts) two parts are measured on one GPU:
+
+* kernels: each step of ONE layer on a prefill batch (4 prompts x 2048 tokens) and on a decode batch (128 sequences after
+  2048 tokens), next to the like kernel of a Qwen3-style layer of the same width, heads and feed-forward (for retention:
+  the gated delta rule of the hybrid family at the same heads and sizes).  ``floor_ms`` is the slower of algorithmic bytes
+  over the measured copy bandwidth and FLOPs over the measured bf16 GEMM peak, ``frac`` = floor / time.  CUDA events
+  around every launch, L2 overwritten before it, median over the iterations.
+* engine: prefill and decode tokens/s through ``generate`` of both engines, the dense model with as many layers as the
+  stateful one has layer runs.
+
+Prints one JSON line per measurement.
+"""
+from __future__ import annotations
+
+import argparse
+import json
+import statistics
+import sys
+import time
+from pathlib import Path
+
+import numpy as np
+import torch
+
+ROOT = Path(__file__).resolve().parents[1]
+if str(ROOT) not in sys.path:
+    sys.path.insert(0, str(ROOT))
+
+SEQ, PREFILL_SEQS, DECODE_SEQS = 2048, 4, 128
+
+
+def peaks():
+    f = ROOT / "MEASURED_PEAKS.json"
+    if f.is_file():
+        d = json.loads(f.read_text())
+        return d["hbm_gbs"] * 1e9, d["bf16_tflops"] * 1e12, "measured"
+    return 6.65e12, 1.59e15, "fallback"
+
+
+class Timer:
+    def __init__(self, iters: int):
+        from arctic_platform_b200.ops import _lib
+        self.iters, self.lib = iters, _lib
+        self.flush = torch.empty(256 << 20, device="cuda", dtype=torch.uint8)
+
+    def __call__(self, fn) -> float:
+        """Median milliseconds of ``fn`` with a cold L2."""
+        for _ in range(3):
+            fn()
+        marks = []
+        for _ in range(self.iters):
+            self.lib.cuda_lib().apb_fill_u32(self.lib.ptr(self.flush), self.flush.numel(), 1, self.lib.stream_ptr())
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record()
+            fn()
+            e1.record()
+            marks.append((e0, e1))
+        torch.cuda.synchronize()
+        return statistics.median(a.elapsed_time(b) for a, b in marks)
+
+
+def _bf(*shape, std=1.0):
+    return (torch.randn(*shape, device="cuda") * std).to(torch.bfloat16)
+
+
+def stateful_ops(cfg, phase):
+    """``(name, fn, bytes, flops)`` of the steps of layer 0 on the phase's batch."""
+    from arctic_platform_b200.engine.stateful_sampler import StateCache
+    from arctic_platform_b200.models.reninex import ReninexLM
+    from arctic_platform_b200.ops import serving
+    import dataclasses
+    one = dataclasses.replace(cfg, layers=cfg.layers[:1], loop=None, vocab_size=1024, bigram=None)
+    model = ReninexLM(one, "cuda", torch.bfloat16).init_weights(0)
+    model.prepare_serving(SEQ + 8)
+    blk, s, W = model.blocks[0], one.layers[0], cfg.hidden_size
+    L, R = s.left, s.right
+    n = PREFILL_SEQS if phase == "prefill" else DECODE_SEQS
+    per = SEQ // 16 + 1
+    cache = StateCache(model.cache_layout(), n * per, n, "cuda", torch.bfloat16)
+    for t in (cache.k[0], cache.v[0]):
+        t.normal_()
+    pages = np.random.default_rng(0).permutation(n * per).astype(np.int32).reshape(n, per)
+    if phase == "prefill":
+        b = serving.StepBatch.build([serving.StepEntry(i, np.arange(SEQ) % 1000, 0, pages[i]) for i in range(n)], "cuda")
+        keys = SEQ * (SEQ + 1) // 2 * n
+    else:
+        i32 = dict(device="cuda", dtype=torch.int32)
+        one_ = torch.arange(n, **i32)
+        b = serving.StepBatch(n, n, one_.clone(), None, one_, torch.ones(n, **i32), one_, torch.full((n,), SEQ, **i32),
+                              torch.from_numpy(pages).cuda(), torch.empty(n, **i32))
+        keys = (SEQ + 1) * n
+    T = b.rows
+    x = torch.randn(T, W, device="cuda")
+    serving.embed(b, model.embed, None, None, cache.prev, torch.empty_like(x))
+    h = _bf(T, W)
+    p = serving.linear(h, blk.w_in)
+    a = _bf(T, blk.w_out.shape[1])
+    c, o = blk.in_cols, blk.out_cols
+    Nin, K = blk.w_in.shape[0], blk.w_out.shape[1]
+    ctx = T if phase == "prefill" else keys                  # K/V rows that have to be read once
+    kv_row = L.kv_heads * (L.dim + L.vdim) * 2
+    state = n * R.heads * R.dim * R.vdim * 4
+    cols = tuple(c["right." + m][0] for m in "qkvg")
+    rope = model._rope[R.rot_dims, R.rot_base]
+    ret_flops = T * R.heads * (2 * 64 * (R.dim + R.vdim) / 2 + 4 * R.dim * R.vdim)
+    return [
+        ("norm + 2 input convolutions", lambda: serving.norm_conv(b, x, blk.norm1, blk.canon1, blk.canon2, True, cache.conv[0],
+                                                                 cache.parity, cfg.conv_taps, cfg.norm_eps),
+         T * W * 8 + (2 * n * (cfg.conv_taps - 1) * W * 4), 0),
+        ("input projections (GEMM)", lambda: serving.linear(h, blk.w_in, p), 2 * (T * W + Nin * W + T * Nin), 2 * T * W * Nin),
+        ("gate/up + GELU (GEMM)", lambda: serving.gate_up_gelu(h, blk.w_gu, a[:, o["down"][0]:]),
+         2 * (T * W + 2 * s.ff * W + T * s.ff), 4 * T * W * s.ff),
+        ("q/k norm + cache write", lambda: serving.qk_norm_cache(b, p, (c["left.q"][0], c["left.k"][0], c["left.v"][0]),
+                                                               cache.k[0], cache.v[0], L.heads, cfg.norm_eps),
+         2 * T * (2 * L.heads * L.dim) + 2 * T * kv_row, 0),
+        ("attention", lambda: serving.sigmoid_attention(b, p[:, c["left.q"][0]:], L.heads, cache.k[0], cache.v[0], blk.pb,
+                                                        L.scale, a[:, o["left.o"][0]:], s.left_scale),
+         ctx * kv_row + 2 * T * L.heads * (L.dim + L.vdim), 2 * keys * L.heads * (L.dim + L.vdim)),
+        ("recurrent mixer", lambda: serving.retention(b, p, cols, rope, R.rot_dims, blk.log2_decay, cache.state[0],
+                                                      a[:, o["right.o"][0]:], cfg.norm_eps, R.dim ** -0.5, s.right_scale),
+         2 * T * R.heads * (2 * R.dim + 3 * R.vdim) + state * (2 if phase == "decode" else 1), ret_flops),
+        ("output projections (GEMM, += fp32)", lambda: serving.linear(a, blk.w_out, x, accumulate=True),
+         2 * (T * K + K * W) + 8 * T * W, 2 * T * K * W),
+    ]
+
+
+def dense_config(cfg):
+    """The Qwen3-style decoder with the width, heads and feed-forward of the model's first layer, one layer per run."""
+    from arctic_platform_b200.models.config import DecoderConfig
+    s = cfg.layers[0]
+    return DecoderConfig(vocab_size=cfg.vocab_size, hidden_size=cfg.hidden_size, intermediate_size=s.ff,
+                         num_layers=len(cfg.layer_runs()), num_heads=s.left.heads, num_kv_heads=s.left.kv_heads,
+                         head_dim=s.left.dim, tie_word_embeddings=False, name=f"dense-{cfg.hidden_size}")
+
+
+def dense_ops(cfg, phase):
+    """The like steps of the dense layer (and of the gated delta rule), keyed by the names of ``stateful_ops``."""
+    import dataclasses
+    from arctic_platform_b200.engine.sampler import SamplerEngine, _fn
+    from arctic_platform_b200.models.decoder import DecoderLM
+    from arctic_platform_b200.models.linear_attention import gated_delta_rule_chunked
+    from arctic_platform_b200.ops import _lib, gemm, norm
+    from arctic_platform_b200.ops.attention import AttnLayout, attention_fwd_cuda
+    d = dataclasses.replace(dense_config(cfg), num_layers=1, vocab_size=1024)
+    R = cfg.layers[0].right
+    n = PREFILL_SEQS if phase == "prefill" else DECODE_SEQS
+    T = SEQ * n if phase == "prefill" else n
+    keys = SEQ * (SEQ + 1) // 2 * n if phase == "prefill" else (SEQ + 1) * n
+    W, D, Hq, G, ff = d.hidden_size, d.head_dim, d.num_heads, d.num_kv_heads, d.intermediate_size
+    model = DecoderLM(d, "cuda", torch.bfloat16).init_weights(0)
+    blk = model.blocks[0]
+    eng = SamplerEngine(d, "cuda", model=model, kv_cache_tokens=(SEQ + 32) * n, max_batch=max(8, n), max_seq_len=SEQ + 32,
+                        cascade=False, use_cuda_graph=False)
+    x, res = _bf(T, W), _bf(T, W)
+    qkv = _bf(T, d.qkv_size)
+    act = _bf(T, ff)
+    pos = torch.arange(T, device="cuda", dtype=torch.int32) % SEQ
+    slots = torch.arange(T, device="cuda", dtype=torch.int32)
+    rope = model.rope("cuda")
+    q, k, v = norm.qknorm_rope(qkv, blk.q_norm, blk.k_norm, *rope, pos, Hq, G, D, 1e-6)
+    kv_row = 2 * G * D * 2
+    acc, accq = torch.zeros(T, W, device="cuda"), torch.zeros(T, d.qkv_size, device="cuda")
+    tiles = lambda m: (m + 127) // 128
+
+    def qk_and_cache():
+        qq, kk, vv = norm.qknorm_rope(qkv, blk.q_norm, blk.k_norm, *rope, pos, Hq, G, D, 1e-6)
+        _lib.check(_fn("kvw")(_lib.ptr(kk), kk.stride(0), _lib.ptr(vv), vv.stride(0), _lib.ptr(slots),
+                              _lib.ptr(eng.kcache[0]), _lib.ptr(eng.vcache[0]), T, G, D, _lib.stream_ptr()), "kvw")
+
+    ops = {}
+    if phase == "prefill":
+        layout = AttnLayout.from_cu_seqlens(np.arange(n + 1) * SEQ)
+        ops["attention"] = (lambda: attention_fwd_cuda(q, k, v.contiguous(), layout, D ** -0.5, need_lse=False),
+                            T * kv_row + 4 * T * Hq * D, 4 * keys * Hq * D)
+        ops["output projections (GEMM, += fp32)"] = (lambda: gemm.matmul_nt(act, blk.wdown),
+                                                     2 * (T * ff + ff * W + T * W), 2 * T * ff * W)
+        ops["q/k norm + cache write"] = (qk_and_cache, 2 * T * 2 * Hq * D + 2 * T * kv_row, 0)
+        ops["norm + 2 input convolutions"] = (lambda: norm.rmsnorm(x, blk.ln1, 1e-6, res), T * W * 8, 0)
+        qr, kr, vr = (torch.randn(SEQ, R.heads, m, device="cuda") for m in (R.dim, R.dim, R.vdim))
+        gr, br = -torch.rand(SEQ, R.heads, device="cuda") * 0.1, torch.rand(SEQ, R.heads, device="cuda")
+
+        def delta():
+            with torch.no_grad():
+                for _ in range(n):
+                    gated_delta_rule_chunked(qr, kr, vr, gr, br)
+        ops["recurrent mixer"] = (delta, 2 * T * R.heads * (2 * R.dim + 3 * R.vdim) + n * R.heads * R.dim * R.vdim * 4,
+                                  T * R.heads * (2 * 64 * (R.dim + R.vdim) / 2 + 4 * R.dim * R.vdim))
+        ops["input projections (GEMM)"] = (lambda: gemm.matmul_nt(x, blk.wqkv), 2 * (T * W + d.qkv_size * (W + T)),
+                                           2 * T * W * d.qkv_size)
+        ops["gate/up + GELU (GEMM)"] = (lambda: gemm.gate_up_swiglu(x, blk.wgu, keep_gu=False),
+                                        2 * (T * W + 2 * ff * W + T * ff), 4 * T * W * ff)
+    else:
+        per = SEQ // 16 + 1
+        eng.d_page_table[:n, :per] = torch.from_numpy(np.random.default_rng(0).permutation(n * per).astype(np.int32).reshape(n, per)).cuda()
+        eng.d_len[:n], eng.d_active[:n] = SEQ + 1, 1
+        eng.kcache.normal_()
+        eng.vcache.normal_()
+        sd, sq = max(1, min(148 // tiles(W), (ff + 63) // 64)), max(1, min(148 // tiles(d.qkv_size), (W + 63) // 64))
+        qb = torch.empty(T, Hq, D, device="cuda", dtype=torch.bfloat16)
+        ops["attention"] = (lambda: eng._decode_attention(0, q, n), keys * kv_row + 4 * T * Hq * D, 4 * keys * Hq * D)
+        ops["output projections (GEMM, += fp32)"] = (
+            lambda: gemm.gemm_raw(act, blk.wdown, acc, M=T, N=W, K=ff, epi=gemm.EPI_F32_ATOMIC, splits=sd, bn=128),
+            2 * (T * ff + ff * W) + 8 * T * W, 2 * T * ff * W)
+        ops["q/k norm + cache write"] = (lambda: _lib.check(_fn("qkv_post")(
+            _lib.ptr(accq), accq.stride(0), _lib.ptr(blk.q_norm), _lib.ptr(blk.k_norm), _lib.ptr(rope[0]), _lib.ptr(rope[1]),
+            _lib.ptr(pos), _lib.ptr(slots), _lib.ptr(qb), _lib.ptr(eng.kcache[0]), _lib.ptr(eng.vcache[0]), T, Hq, G, D, 1e-6,
+            _lib.stream_ptr()), "qkv_post"), 8 * T * d.qkv_size + 2 * T * Hq * D + T * kv_row, 0)
+        ops["norm + 2 input convolutions"] = (lambda: eng._norm_f32(acc, blk.ln1, res), T * W * 14, 0)
+        ops["input projections (GEMM)"] = (
+            lambda: gemm.gemm_raw(x, blk.wqkv, accq, M=T, N=d.qkv_size, K=W, epi=gemm.EPI_F32_ATOMIC, splits=sq, bn=128),
+            2 * (T * W + d.qkv_size * W) + 8 * T * d.qkv_size, 2 * T * W * d.qkv_size)
+        ops["gate/up + GELU (GEMM)"] = (lambda: gemm.gemm_raw(x, blk.wgu, None, M=T, N=2 * ff, K=W, epi=gemm.EPI_SWIGLU,
+                                                              out2=act, bn=0), 2 * (T * W + 2 * ff * W + T * ff), 4 * T * W * ff)
+        S = torch.randn(n, R.heads, R.dim, R.vdim, device="cuda")
+        ks, qs, vs = (torch.randn(n, R.heads, m, device="cuda") for m in (R.dim, R.dim, R.vdim))
+        al = torch.rand(n, R.heads, device="cuda")
+
+        def delta_step():                                 # the state part of GatedDeltaNet.step
+            s2 = S * al[:, :, None, None]
+            pred = torch.einsum("bhkv,bhk->bhv", s2, ks)
+            s2 = s2 + torch.einsum("bhk,bhv->bhkv", ks, vs - pred)
+            torch.einsum("bhkv,bhk->bhv", s2, qs)
+        ops["recurrent mixer"] = (delta_step, 2 * T * R.heads * (2 * R.dim + 3 * R.vdim) + 2 * S.numel() * 4,
+                                  T * R.heads * 4 * R.dim * R.vdim)
+    ops["_keep"] = eng
+    return ops
+
+
+def bench_kernels(name, cfg, phase, iters):
+    bw, peak, of = peaks()
+    timer = Timer(iters)
+
+    def measured(fn, nbytes, flops):
+        ms = timer(fn)
+        floor = max(nbytes / bw, flops / peak) * 1e3
+        return ms, floor, floor / ms
+
+    like = {k: measured(*v) for k, v in dense_ops(cfg, phase).items() if k != "_keep"}
+    torch.cuda.empty_cache()
+    for op, fn, nbytes, flops in stateful_ops(cfg, phase):
+        ms, floor, frac = measured(fn, nbytes, flops)
+        row = {"model": name, "phase": phase, "step": op, "ms": round(ms, 4), "floor_ms": round(floor, 4),
+               "frac": round(frac, 3), "of": of}
+        if op in like:
+            row.update(like_ms=round(like[op][0], 4), like_frac=round(like[op][2], 3), ratio=round(frac / like[op][2], 2))
+        print(json.dumps(row), flush=True)
+
+
+def bench_engine(name, cfg, seqs, new_tokens):
+    from arctic_platform_b200.engine.sampler import SamplerEngine
+    from arctic_platform_b200.engine.stateful_sampler import StatefulSampler
+    from arctic_platform_b200.models.decoder import DecoderLM
+    from arctic_platform_b200.models.reninex import ReninexLM
+    prompts = [np.random.default_rng(i).integers(1, cfg.vocab_size, SEQ).tolist() for i in range(seqs)]
+    limits = dict(kv_cache_tokens=seqs * (SEQ + new_tokens + 32), max_batch=seqs, max_seq_len=SEQ + new_tokens + 16)
+    d = dense_config(cfg)
+    for label, make in (
+            (name, lambda: StatefulSampler(cfg, "cuda", model=ReninexLM(cfg, "cuda", torch.bfloat16).init_weights(0), **limits)),
+            (d.name, lambda: SamplerEngine(d, "cuda", model=DecoderLM(d, "cuda", torch.bfloat16).init_weights(0), cascade=False,
+                                           **limits))):
+        eng = make()
+
+        def run(n):
+            torch.cuda.synchronize()
+            t = time.perf_counter()
+            eng.generate(prompts, {"temperature": 1.0, "max_tokens": n, "ignore_eos": True})
+            torch.cuda.synchronize()
+            return time.perf_counter() - t
+
+        for n in (1, new_tokens):
+            run(n)
+        pre = statistics.median(run(1) for _ in range(3))
+        full = statistics.median(run(new_tokens) for _ in range(3))
+        params = sum(p.numel() for p in eng.model.parameters())
+        fl = cfg if label == name else d
+        print(json.dumps({
+            "model": label, "engine": type(eng).__name__, "sequences": seqs, "prompt_len": SEQ, "new_tokens": new_tokens,
+            "parameters": params, "layer_runs": len(cfg.layer_runs()),
+            "prefill_tokens_per_s": round(seqs * SEQ / pre), "decode_tokens_per_s": round(seqs * (new_tokens - 1) / (full - pre)),
+            "decode_ms_per_step": round((full - pre) * 1e3 / (new_tokens - 1), 3),
+            "gflop_per_token": round(fl.flops_per_token(SEQ, backward=False) / 1e9, 3),
+            "prefill_tflops": round(seqs * SEQ / pre * (fl.flops_per_token(SEQ, backward=False) - 2.0 * cfg.vocab_size * cfg.hidden_size) / 1e12, 1)}),
+            flush=True)
+        del eng
+        torch.cuda.empty_cache()
+
+
+def main(models, kernels_only=False, only=None, iters=20, seqs=64, new_tokens=129) -> None:
+    from arctic_platform_b200.models.config import resolve_config
+    from arctic_platform_b200.ops import _lib
+    for name in models:
+        cfg = resolve_config(name)
+        for phase in ("prefill", "decode"):
+            if only in (None, phase):
+                bench_kernels(name, cfg, phase, iters)
+                torch.cuda.empty_cache()
+        if not kernels_only:
+            bench_engine(name, cfg, seqs, new_tokens)
+    _lib.check_status("serving benchmark")
+
+
+if __name__ == "__main__":
+    ap = argparse.ArgumentParser()
+    ap.add_argument("--models", default="reninex-2048,reninex-4096")
+    ap.add_argument("--kernels-only", action="store_true")
+    ap.add_argument("--only", choices=["prefill", "decode"])
+    ap.add_argument("--iters", type=int, default=20)
+    ap.add_argument("--seqs", type=int, default=64)
+    ap.add_argument("--new-tokens", type=int, default=129)
+    a = ap.parse_args()
+    main(a.models.split(","), a.kernels_only, a.only, a.iters, a.seqs, a.new_tokens)
