@@ -19,10 +19,10 @@
 namespace apb {
 
 // ---------------------------------------------------------------------------- one token
-constexpr int kRetThreads = 256;
+constexpr int kRetDecThreads = 128;
 
 template <typename T, int VEC>
-__global__ void __launch_bounds__(kRetThreads)
+__global__ void __launch_bounds__(kRetDecThreads)
 retention_decode_kernel(const RetentionParams p) {
   pdl_entry();
   extern __shared__ float ret_smem[];
@@ -33,21 +33,21 @@ retention_decode_kernel(const RetentionParams p) {
   float* ks = qs + D;              // [D]
   float* vs = ks + D;              // [E]
   float* red = vs + E;             // [ny][E]
-  __shared__ float wsum[kRetThreads / 32];
+  __shared__ float wsum[kRetDecThreads / 32];
   const int row = p.e.start[en], slot = p.e.slot[en], pos = p.e.pos0[en];
   const T* pr = static_cast<const T*>(p.p) + static_cast<long long>(row) * p.ld;
   const float* c = p.cos_t + static_cast<long long>(pos) * (p.rot_dims / 2);
   const float* sn = p.sin_t + static_cast<long long>(pos) * (p.rot_dims / 2);
-  for (int d = threadIdx.x; d < D; d += kRetThreads) {
+  for (int d = threadIdx.x; d < D; d += kRetDecThreads) {
     qs[d] = rotated(pr + p.q_col + static_cast<long long>(h) * D, d, p.rot_dims, c, sn);
     ks[d] = rotated(pr + p.k_col + static_cast<long long>(h) * D, d, p.rot_dims, c, sn) * p.k_scale;
   }
-  for (int i = threadIdx.x; i < E; i += kRetThreads)
+  for (int i = threadIdx.x; i < E; i += kRetDecThreads)
     vs[i] = to_f32(pr[p.v_col + static_cast<long long>(h) * E + i]);
   __syncthreads();
   const float dec = pos == 0 ? 0.f : exp2f(p.log2_decay[h]);
   float* S = p.state + (static_cast<long long>(slot) * p.H + h) * D * E;
-  const int nx = min(E / VEC, kRetThreads), ny = kRetThreads / nx;
+  const int nx = min(E / VEC, kRetDecThreads), ny = kRetDecThreads / nx;
   const int tx = threadIdx.x % nx, ty = threadIdx.x / nx;
   if (ty < ny) {
     for (int cx = tx; cx < E / VEC; cx += nx) {
@@ -102,7 +102,7 @@ retention_decode_kernel(const RetentionParams p) {
   }
   __syncthreads();
   float ss = 0.f;
-  for (int i = threadIdx.x; i < E; i += kRetThreads) {
+  for (int i = threadIdx.x; i < E; i += kRetDecThreads) {
     float o = 0.f;
     for (int y = 0; y < ny; ++y) o += red[y * E + i];
     red[i] = o;
@@ -113,16 +113,17 @@ retention_decode_kernel(const RetentionParams p) {
   __syncthreads();
   ss = 0.f;
 #pragma unroll
-  for (int i = 0; i < kRetThreads / 32; ++i) ss += wsum[i];
+  for (int i = 0; i < kRetDecThreads / 32; ++i) ss += wsum[i];
   const float f = p.out_scale / sqrtf(ss / E + p.eps);
   T* out = static_cast<T*>(p.out) + static_cast<long long>(row) * p.ldo + static_cast<long long>(h) * E;
-  for (int i = threadIdx.x; i < E; i += kRetThreads) {
+  for (int i = threadIdx.x; i < E; i += kRetDecThreads) {
     const float g = to_f32(pr[p.g_col + static_cast<long long>(h) * E + i]);
     out[i] = from_f32<T>(red[i] * f * (g / (1.f + expf(-g))));
   }
 }
 
 // ---------------------------------------------------------------------------- chunks, fp32 arithmetic
+constexpr int kRetThreads = 256;
 constexpr int kRetC = 32;      // tokens per chunk
 constexpr int kRetBE = 32;     // E columns per CTA
 
@@ -290,17 +291,17 @@ int apb_retention(const void* p, long long ld, int q_col, int k_col, int v_col, 
   if (decode) {
     const bool v4 = (E & 3) == 0;
     const int cols = v4 ? E / 4 : E;
-    const int nx = cols < kRetThreads ? cols : kRetThreads;
-    const size_t smem = (2 * D + E + static_cast<size_t>(kRetThreads / nx) * E) * sizeof(float);
+    const int nx = cols < kRetDecThreads ? cols : kRetDecThreads;
+    const size_t smem = (2 * D + E + static_cast<size_t>(kRetDecThreads / nx) * E) * sizeof(float);
     int rc = 0;
     if (dtype == 0) {
       auto fn = v4 ? retention_decode_kernel<__nv_bfloat16, 4> : retention_decode_kernel<__nv_bfloat16, 1>;
       rc = retention_smem_limit(reinterpret_cast<const void*>(fn), smem);
-      if (!rc) rc = static_cast<int>(launch_kernel(fn, dim3(n_entries, H), dim3(kRetThreads), smem, s, a));
+      if (!rc) rc = static_cast<int>(launch_kernel(fn, dim3(n_entries, H), dim3(kRetDecThreads), smem, s, a));
     } else if (dtype == 1) {
       auto fn = v4 ? retention_decode_kernel<float, 4> : retention_decode_kernel<float, 1>;
       rc = retention_smem_limit(reinterpret_cast<const void*>(fn), smem);
-      if (!rc) rc = static_cast<int>(launch_kernel(fn, dim3(n_entries, H), dim3(kRetThreads), smem, s, a));
+      if (!rc) rc = static_cast<int>(launch_kernel(fn, dim3(n_entries, H), dim3(kRetDecThreads), smem, s, a));
     } else {
       rc = kBadArgument;
     }

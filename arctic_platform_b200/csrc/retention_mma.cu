@@ -6,6 +6,9 @@
 // begin with.  The state itself stays in fp32 registers (the accumulator fragments of the update product), its hi / lo
 // copy in shared memory is only the operand of the next chunk's q S product.
 //
+// q and k are rotated, scaled and split once per (row, head) by retention_split_kernel; the chunk kernel copies the
+// halves to shared memory while the previous chunk is being computed.
+//
 // One CTA = (segment of an entry, head, 64-column slice of E), two CTAs per SM.  An entry is one segment when there are
 // enough entries to fill the GPU.  Otherwise it is cut into several: a first launch (state_only) computes what each
 // segment adds to the state, retention_carry_kernel chains them into the state before each segment, and the second
@@ -29,8 +32,9 @@ struct RetentionSegments {
   float* carry;           // [scratch states][H][D][E]
 };
 
-__device__ __forceinline__ void rm_cp_async16(uint32_t dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+// 16 bytes, or zeros when `bytes` is 0
+__device__ __forceinline__ void rm_cp_async16(uint32_t dst, const void* src, int bytes) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(bytes) : "memory");
 }
 __device__ __forceinline__ void rm_ldsm4(const __nv_bfloat16* a, uint32_t (&r)[4]) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
@@ -57,35 +61,87 @@ __device__ __forceinline__ void rm_split2(float x, float y, uint32_t& hi, uint32
   lo = pack_bf16x2(x - h.x, y - h.y);
 }
 
-__host__ __device__ inline int rm_smem_bytes(int D) {
-  const int dp = (D + 15) / 16 * 16, ds = dp + 8;
-  return 2 * (4 * kRmC * ds + 3 * kRmC * kRmVS + 2 * kRmC * kRmAS + 2 * dp * kRmVS + kRmC * (2 * dp + kRmBE)) + 256;
+// qk [rows][H][4][dp]: hi and lo of the rotated q, hi and lo of the rotated and scaled k; dp = D rounded up to 16, the
+// padding zero.  Rows of one-token entries are skipped.  One warp per (row, head).
+__global__ void __launch_bounds__(256)
+retention_split_kernel(const RetentionParams p, const int* __restrict__ row_entry, int rows, __nv_bfloat16* __restrict__ qk) {
+  pdl_entry();
+  const int lane = threadIdx.x & 31;
+  const long long gw = (blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x) >> 5;
+  if (gw >= static_cast<long long>(rows) * p.H) return;
+  const int row = static_cast<int>(gw / p.H), h = static_cast<int>(gw % p.H);
+  const int en = row_entry ? row_entry[row] : row;
+  if (p.e.len[en] <= 1) return;
+  const int D = p.D, dp = (D + 15) & ~15, half = p.rot_dims >> 1;
+  const long long tr = static_cast<long long>(p.e.pos0[en] + row - p.e.start[en]) * half;
+  const __nv_bfloat16* pr = static_cast<const __nv_bfloat16*>(p.p) + static_cast<long long>(row) * p.ld;
+  const __nv_bfloat16* q = pr + p.q_col + h * D;
+  const __nv_bfloat16* k = pr + p.k_col + h * D;
+  __nv_bfloat16* out = qk + gw * 4 * dp;
+  auto put = [&](int part, int d, float x, float y) {
+    uint32_t hi, lo;
+    rm_split2(x, y, hi, lo);
+    *reinterpret_cast<uint32_t*>(out + part * dp + d) = hi;
+    *reinterpret_cast<uint32_t*>(out + (part + 1) * dp + d) = lo;
+  };
+  int d_done = 0;                                  // dimensions covered by the paired loop
+  if ((half & 1) == 0) {                           // two neighbouring rotation pairs (d, d + half), (d + 1, d + 1 + half)
+    d_done = p.rot_dims;
+    for (int d = lane * 2; d < half; d += 64) {
+      const float2 c = *reinterpret_cast<const float2*>(p.cos_t + tr + d);
+      const float2 sn = *reinterpret_cast<const float2*>(p.sin_t + tr + d);
+      const float2 qu = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(q + d));
+      const float2 qv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(q + d + half));
+      const float2 ku = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(k + d));
+      const float2 kv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(k + d + half));
+      put(0, d, qu.x * c.x - qv.x * sn.x, qu.y * c.y - qv.y * sn.y);
+      put(0, d + half, qv.x * c.x + qu.x * sn.x, qv.y * c.y + qu.y * sn.y);
+      put(2, d, (ku.x * c.x - kv.x * sn.x) * p.k_scale, (ku.y * c.y - kv.y * sn.y) * p.k_scale);
+      put(2, d + half, (kv.x * c.x + ku.x * sn.x) * p.k_scale, (kv.y * c.y + ku.y * sn.y) * p.k_scale);
+    }
+  }
+  for (int d = d_done + lane * 2; d < dp; d += 64) {     // unrotated dimensions and padding, or odd rotations
+    float2 a = make_float2(0.f, 0.f), b = a;
+    if (d < D) {
+      a = make_float2(rotated(q, d, p.rot_dims, p.cos_t + tr, p.sin_t + tr), rotated(q, d + 1, p.rot_dims, p.cos_t + tr, p.sin_t + tr));
+      b = make_float2(rotated(k, d, p.rot_dims, p.cos_t + tr, p.sin_t + tr) * p.k_scale,
+                      rotated(k, d + 1, p.rot_dims, p.cos_t + tr, p.sin_t + tr) * p.k_scale);
+    }
+    put(0, d, a.x, a.y);
+    put(2, d, b.x, b.y);
+  }
 }
 
+__host__ __device__ inline int rm_smem_bytes(int D) {
+  const int dp = (D + 15) / 16 * 16, ds = dp + 8;
+  return 2 * (6 * kRmC * ds + 4 * kRmC * kRmVS + 2 * kRmC * kRmAS + 2 * dp * kRmVS) + 256;
+}
+
+// DP: D rounded up to 16 when known at compile time, else 0.
+template <int DP>
 __global__ void __launch_bounds__(kRmThreads, 2)
-retention_mma_kernel(const RetentionParams p, const RetentionSegments sg, int state_only) {
+retention_mma_kernel(const RetentionParams p, const RetentionSegments sg, const __nv_bfloat16* __restrict__ qk,
+                     int state_only) {
   pdl_entry();
   extern __shared__ __align__(128) uint8_t rm_smem[];
   const int* w = sg.seg + blockIdx.x * 6;
   const int en = w[0], t_begin = w[1], n_tok = w[2], carry_in = w[3], carry_out = w[4], is_last = w[5];
   if (state_only && carry_out < 0) return;
   const int h = blockIdx.y, e0 = blockIdx.z * kRmBE;
-  const int D = p.D, E = p.E, dp = (D + 15) & ~15, ds = dp + 8, d16 = dp >> 4;
+  const int D = p.D, E = p.E, dp = DP ? DP : (D + 15) & ~15, ds = dp + 8, d16 = dp >> 4;
   const int be = min(kRmBE, E - e0);
   const int start = p.e.start[en] + t_begin, pos0 = p.e.pos0[en] + t_begin, slot = p.e.slot[en];
   __nv_bfloat16* Qh = reinterpret_cast<__nv_bfloat16*>(rm_smem);
   __nv_bfloat16* Ql = Qh + kRmC * ds;
-  __nv_bfloat16* Kh = Ql + kRmC * ds;
-  __nv_bfloat16* Kl = Kh + kRmC * ds;
-  __nv_bfloat16* V = Kl + kRmC * ds;             // [32][72] values
-  __nv_bfloat16* Wh = V + kRmC * kRmVS;          // values times decay^(n - 1 - j), hi / lo
+  __nv_bfloat16* K2 = Ql + kRmC * ds;            // two buffers of (hi, lo) [32][ds]
+  __nv_bfloat16* V2 = K2 + 4 * kRmC * ds;        // two buffers of values [32][72]
+  __nv_bfloat16* Wh = V2 + 2 * kRmC * kRmVS;     // values times decay^(n - 1 - j), hi / lo
   __nv_bfloat16* Wl = Wh + kRmC * kRmVS;
   __nv_bfloat16* Ah = Wl + kRmC * kRmVS;         // [32][40] decayed scores
   __nv_bfloat16* Al = Ah + kRmC * kRmAS;
   __nv_bfloat16* Sh = Al + kRmC * kRmAS;         // [dp][72] carried state
   __nv_bfloat16* Sl = Sh + dp * kRmVS;
-  __nv_bfloat16* raw = Sl + dp * kRmVS;          // [32][dp] q, [32][dp] k, [32][64] v as they come from memory
-  float* pw = reinterpret_cast<float*>(raw + kRmC * (2 * dp + kRmBE));   // decay powers 0 .. 32
+  float* pw = reinterpret_cast<float*>(Sl + dp * kRmVS);     // decay powers 0 .. 32
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int quad_row = lane >> 2, quad_col = (lane & 3) * 2;
   const int mat = lane >> 3, rowin = lane & 7;
@@ -93,21 +149,26 @@ retention_mma_kernel(const RetentionParams p, const RetentionSegments sg, int st
 
   if (threadIdx.x <= kRmC) pw[threadIdx.x] = decay_pow(p.log2_decay[h], threadIdx.x);
 
-  auto fetch = [&](int t0) {
-    const int n = min(kRmC, n_tok - t0), dc = D >> 3, vc = be >> 3;
-    for (int i = threadIdx.x; i < n * (2 * dc + vc); i += kRmThreads) {
-      const int r = i / (2 * dc + vc), c = i % (2 * dc + vc);
-      const __nv_bfloat16* row = pb + static_cast<long long>(start + t0 + r) * p.ld;
-      if (c < dc)
-        rm_cp_async16(smem_u32(raw + r * dp + c * 8), row + p.q_col + h * D + c * 8);
-      else if (c < 2 * dc)
-        rm_cp_async16(smem_u32(raw + (kRmC + r) * dp + (c - dc) * 8), row + p.k_col + h * D + (c - dc) * 8);
-      else
-        rm_cp_async16(smem_u32(raw + 2 * kRmC * dp + r * kRmBE + (c - 2 * dc) * 8), row + p.v_col + h * E + e0 + (c - 2 * dc) * 8);
+  // rows beyond the segment are filled with zeros
+  const int pc = dp >> 3;                        // 16-byte chunks of one part
+  auto fetch_part = [&](int t0, int part, __nv_bfloat16* dst) {         // hi and lo of q (part 0) or k (part 2)
+#pragma unroll
+    for (int i = threadIdx.x; i < kRmC * 2 * pc; i += kRmThreads) {
+      const int r = i / (2 * pc), c = i % (2 * pc), ok = t0 + r < n_tok;
+      const __nv_bfloat16* src = qk + ((static_cast<long long>(start + (ok ? t0 + r : 0)) * p.H + h) * 4 + part) * dp + c * 8;
+      rm_cp_async16(smem_u32(dst + (c / pc) * (kRmC * ds) + r * ds + (c % pc) * 8), src, ok ? 16 : 0);
     }
-    asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  fetch(0);
+  auto fetch_kv = [&](int t0, int buf) {
+    fetch_part(t0, 2, K2 + buf * 2 * kRmC * ds);
+    const int r = threadIdx.x >> 3, c = threadIdx.x & 7, ok = t0 + r < n_tok && c * 8 < be;
+    const __nv_bfloat16* src = pb + static_cast<long long>(start + (ok ? t0 + r : 0)) * p.ld + p.v_col + h * E + e0 + (ok ? c * 8 : 0);
+    rm_cp_async16(smem_u32(V2 + buf * kRmC * kRmVS + r * kRmVS + c * 8), src, ok ? 16 : 0);
+  };
+  static_assert(kRmThreads == kRmC * kRmBE / 8, "one 16-byte chunk of the values per thread");
+  if (!state_only) fetch_part(0, 0, Qh);
+  fetch_kv(0, 0);
+  asm volatile("cp.async.commit_group;" ::: "memory");
 
   // the warp's 16 state rows, fp32: accumulator fragments over eight 8-column tiles
   float s[8][4];
@@ -146,77 +207,24 @@ retention_mma_kernel(const RetentionParams p, const RetentionSegments sg, int st
   bool have_state = s_in != nullptr;
   if (have_state) store_state_operand();
 
-  for (int t0 = 0; t0 < n_tok; t0 += kRmC) {
+  for (int t0 = 0, buf = 0; t0 < n_tok; t0 += kRmC, buf ^= 1) {
     const int n = min(kRmC, n_tok - t0);
+    const bool more = t0 + kRmC < n_tok;
+    const __nv_bfloat16* Kh = K2 + buf * 2 * kRmC * ds;
+    const __nv_bfloat16* Kl = Kh + kRmC * ds;
+    const __nv_bfloat16* V = V2 + buf * kRmC * kRmVS;
     asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();                               // raw rows have landed; everybody is done with the last chunk
-    // ---- rotate, scale, split
-    auto put = [&](__nv_bfloat16* hi_t, __nv_bfloat16* lo_t, int o, float x, float y) {
-      uint32_t hi, lo;
-      rm_split2(x, y, hi, lo);
-      *reinterpret_cast<uint32_t*>(hi_t + o) = hi;
-      *reinterpret_cast<uint32_t*>(lo_t + o) = lo;
-    };
-    const int half = p.rot_dims >> 1;
-    int d_done = 0;                                // dimensions covered by the paired loop
-    if ((half & 1) == 0) {                         // two neighbouring rotation pairs (d, d + half), (d + 1, d + 1 + half)
-      d_done = p.rot_dims;
-      const int q2 = half >> 1;
-#pragma unroll 4
-      for (int i = threadIdx.x; i < kRmC * q2; i += kRmThreads) {
-        const int r = i / q2, d = (i - r * q2) * 2, o = r * ds + d;
-        float2 qu = make_float2(0.f, 0.f), qv = qu, ku = qu, kv = qu, c = qu, sn = qu;
-        if (r < n) {
-          const long long tr = static_cast<long long>(pos0 + t0 + r) * half + d;
-          c = *reinterpret_cast<const float2*>(p.cos_t + tr);
-          sn = *reinterpret_cast<const float2*>(p.sin_t + tr);
-          const __nv_bfloat16* rq = raw + r * dp + d;
-          const __nv_bfloat16* rk = rq + kRmC * dp;
-          qu = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(rq));
-          qv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(rq + half));
-          ku = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(rk));
-          kv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(rk + half));
-        }
-        if (!state_only) {
-          put(Qh, Ql, o, qu.x * c.x - qv.x * sn.x, qu.y * c.y - qv.y * sn.y);
-          put(Qh, Ql, o + half, qv.x * c.x + qu.x * sn.x, qv.y * c.y + qu.y * sn.y);
-        }
-        put(Kh, Kl, o, (ku.x * c.x - kv.x * sn.x) * p.k_scale, (ku.y * c.y - kv.y * sn.y) * p.k_scale);
-        put(Kh, Kl, o + half, (kv.x * c.x + ku.x * sn.x) * p.k_scale, (kv.y * c.y + ku.y * sn.y) * p.k_scale);
-      }
-    }
-    const int pairs = (dp - d_done) >> 1;          // unrotated dimensions (and the padding), or odd rotations
-    for (int i = threadIdx.x; i < kRmC * pairs; i += kRmThreads) {
-      const int r = i / pairs, d = d_done + (i % pairs) * 2, o = r * ds + d;
-      float2 qv = make_float2(0.f, 0.f), kv = qv;
-      if (r < n && d < D) {
-        const long long tr = static_cast<long long>(pos0 + t0 + r) * half;
-        const float* c = p.cos_t + tr;
-        const float* sn = p.sin_t + tr;
-        const __nv_bfloat16* rq = raw + r * dp;
-        const __nv_bfloat16* rk = raw + (kRmC + r) * dp;
-        qv = make_float2(rotated(rq, d, p.rot_dims, c, sn), rotated(rq, d + 1, p.rot_dims, c, sn));
-        kv = make_float2(rotated(rk, d, p.rot_dims, c, sn) * p.k_scale, rotated(rk, d + 1, p.rot_dims, c, sn) * p.k_scale);
-      }
-      if (!state_only) put(Qh, Ql, o, qv.x, qv.y);
-      put(Kh, Kl, o, kv.x, kv.y);
-    }
+    __syncthreads();                               // this chunk has landed; everybody is done with the last one
+    if (more) fetch_kv(t0 + kRmC, buf ^ 1);
     for (int i = threadIdx.x; i < kRmC * (kRmBE / 2); i += kRmThreads) {
-      const int r = i / (kRmBE / 2), c = (i % (kRmBE / 2)) * 2;
-      uint32_t v = 0, wh = 0, wl = 0;
-      if (r < n && c < be) {
-        v = *reinterpret_cast<const uint32_t*>(raw + 2 * kRmC * dp + r * kRmBE + c);
-        const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v));
-        const float g = pw[n - 1 - r];
-        rm_split2(f.x * g, f.y * g, wh, wl);
-      }
-      const int o = r * kRmVS + c;
-      *reinterpret_cast<uint32_t*>(V + o) = v;
+      const int r = i / (kRmBE / 2), o = r * kRmVS + (i % (kRmBE / 2)) * 2;
+      const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(V + o));
+      const float g = r < n ? pw[n - 1 - r] : 0.f;
+      uint32_t wh, wl;
+      rm_split2(f.x * g, f.y * g, wh, wl);
       *reinterpret_cast<uint32_t*>(Wh + o) = wh;
       *reinterpret_cast<uint32_t*>(Wl + o) = wl;
     }
-    __syncthreads();
-    if (t0 + kRmC < n_tok) fetch(t0 + kRmC);        // the raw rows are free again: overlap the next chunk's loads
     const int r0 = (warp & 1) * 16, c0 = (warp >> 1) * 16;     // this warp's tile of the output
     float o[2][4];
 #pragma unroll
@@ -226,6 +234,7 @@ retention_mma_kernel(const RetentionParams p, const RetentionSegments sg, int st
       const int k0 = (warp >> 1) * 8;
       float a[4] = {0.f, 0.f, 0.f, 0.f};
       const bool live = k0 <= r0 + 15;
+#pragma unroll 4
       for (int ks = 0; ks < d16; ++ks) {
         uint32_t qh[4], ql[4];
         const int ao = (r0 + rowin + (mat & 1) * 8) * ds + ks * 16 + (mat >> 1) * 8;
@@ -268,7 +277,9 @@ retention_mma_kernel(const RetentionParams p, const RetentionSegments sg, int st
         }
       }
     }
-    __syncthreads();                               // scores visible; nobody reads the state operand any more
+    __syncthreads();                               // scores and W visible; nobody reads q or the state operand any more
+    if (more && !state_only) fetch_part(t0 + kRmC, 0, Qh);
+    asm volatile("cp.async.commit_group;" ::: "memory");
     if (!state_only) {
       for (int ks = 0; ks < (r0 + 16) / 16; ++ks) {
         uint32_t ah[4], al[4], v[4];
@@ -323,7 +334,7 @@ retention_mma_kernel(const RetentionParams p, const RetentionSegments sg, int st
         }
       }
     }
-    if (!state_only && t0 + kRmC < n_tok) store_state_operand();
+    if (!state_only && more) store_state_operand();
     have_state = true;
   }
   // ---- the state after the segment
@@ -368,14 +379,15 @@ using namespace apb;
 
 // bf16; D a multiple of 8 up to 128, E a multiple of 8; every column offset and ld a multiple of 8.  Writes o [rows, H, E]
 // (fp32) for the segments' rows and the entries' states.  n_chains > 0: some entries have several segments (carry is
-// scratch for their states).
+// scratch for their states).  qk: bf16 scratch [rows, H, 4, D rounded up to 16].
 int apb_retention_mma(const void* p, long long ld, int q_col, int k_col, int v_col, const float* cos_t, const float* sin_t,
                       int rot_dims, const float* log2_decay, float k_scale, float* state, float* o, const int* e_start,
                       const int* e_len, const int* e_slot, const int* e_pos0, const int* seg, int n_seg, float* carry,
-                      const int* chains, int n_chains, int H, int D, int E, cudaStream_t s) {
+                      const int* chains, int n_chains, const int* row_entry, void* qk, int rows, int H, int D, int E,
+                      cudaStream_t s) {
   if (n_seg <= 0) return 0;
   if (H <= 0 || D <= 0 || E <= 0 || (D % 8) || (E % 8) || D > kRmMaxD || (ld % 8) || (q_col % 8) || (k_col % 8) || (v_col % 8) ||
-      (reinterpret_cast<uintptr_t>(p) & 15) || (rot_dims & 1) || rot_dims > D || rot_dims < 0 || !seg || !o ||
+      (reinterpret_cast<uintptr_t>(p) & 15) || (rot_dims & 1) || rot_dims > D || rot_dims < 0 || !seg || !o || !qk ||
       (n_chains > 0 && (!carry || !chains)))
     return kBadArgument;
   RetentionParams a{};
@@ -396,16 +408,23 @@ int apb_retention_mma(const void* p, long long ld, int q_col, int k_col, int v_c
   a.D = D;
   a.E = E;
   const RetentionSegments sg{seg, carry};
-  const int smem = rm_smem_bytes(D);
-  cudaError_t e = cudaFuncSetAttribute(retention_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-  if (e != cudaSuccess) return static_cast<int>(e);
+  const int smem = rm_smem_bytes(D), dp = (D + 15) / 16 * 16;
   const dim3 grid(n_seg, H, (E + kRmBE - 1) / kRmBE);
-  if (n_chains > 0) {
-    e = launch_kernel(retention_mma_kernel, grid, dim3(kRmThreads), smem, s, a, sg, 1);
-    if (e != cudaSuccess) return static_cast<int>(e);
-    e = launch_kernel(retention_carry_kernel, dim3(n_chains, H, (D * E + 255) / 256), dim3(256), 0, s, a, sg, chains);
-    if (e != cudaSuccess) return static_cast<int>(e);
-  }
-  return static_cast<int>(launch_kernel(retention_mma_kernel, grid, dim3(kRmThreads), smem, s, a, sg, 0));
+  const int sgrid = static_cast<int>((static_cast<long long>(rows) * H * 32 + 255) / 256);
+  __nv_bfloat16* qkp = static_cast<__nv_bfloat16*>(qk);
+  cudaError_t e = launch_kernel(retention_split_kernel, dim3(sgrid), dim3(256), 0, s, a, row_entry, rows, qkp);
+  if (e != cudaSuccess) return static_cast<int>(e);
+  auto run = [&](auto fn) -> cudaError_t {
+    cudaError_t r = cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (r != cudaSuccess) return r;
+    if (n_chains > 0) {
+      r = launch_kernel(fn, grid, dim3(kRmThreads), smem, s, a, sg, qkp, 1);
+      if (r != cudaSuccess) return r;
+      r = launch_kernel(retention_carry_kernel, dim3(n_chains, H, (D * E + 255) / 256), dim3(256), 0, s, a, sg, chains);
+      if (r != cudaSuccess) return r;
+    }
+    return launch_kernel(fn, grid, dim3(kRmThreads), smem, s, a, sg, qkp, 0);
+  };
+  return static_cast<int>(dp == 128 ? run(retention_mma_kernel<128>) : dp == 64 ? run(retention_mma_kernel<64>) : run(retention_mma_kernel<0>));
 }
 }

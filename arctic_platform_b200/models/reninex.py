@@ -400,7 +400,7 @@ PRESETS: Dict[str, ReninexConfig] = {
                                   (1, 2, 2), "reninex-tiny"),
     # layers of the size of a 1.7B / 8B dense decoder's
     "reninex-2048": ReninexConfig(151936, 2048, _uniform(8, (16, 8, 128, 128), (8, 128, 256, 128), 6144), 1e-6, 4,
-                                  (65521, 127, 7), (2, 6, 2), "reninex-2048"),
+                                  (65521, 1009, 37), (2, 6, 2), "reninex-2048"),
     "reninex-4096": ReninexConfig(151936, 4096, _uniform(8, (32, 8, 128, 128), (16, 128, 256, 128), 12288), 1e-6, 4,
-                                  (65521, 127, 7), (2, 6, 2), "reninex-4096"),
+                                  (65521, 1009, 37), (2, 6, 2), "reninex-4096"),
 }

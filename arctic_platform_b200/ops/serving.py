@@ -38,7 +38,7 @@ def _fn(name: str):
             "apb_sigmoid_attn_mma": [vp, ll, vp, vp, vp, vp, i, vp, i, vp, vp, vp, vp, ll, vp] + [i] * 7 + [f, f, vp],
             "apb_sigmoid_attn_tc": [vp, ll, i, vp, i, vp, i, vp, vp, i, vp, vp, ll, i, i, i, i, f, f, vp],
             "apb_retention": [vp, ll, i, i, i, i, vp, vp, i, vp, f, vp, vp, vp, ll, f, f, vp, vp, vp, vp, vp] + [i] * 8 + [vp],
-            "apb_retention_mma": [vp, ll, i, i, i, vp, vp, i, vp, f] + [vp] * 7 + [i, vp, vp, i, i, i, i, vp],
+            "apb_retention_mma": [vp, ll, i, i, i, vp, vp, i, vp, f] + [vp] * 7 + [i, vp, vp, i, vp, vp, i, i, i, i, vp],
             "apb_retention_out": [vp, ll, i, vp, vp, ll, f, f, vp, vp, vp, vp, vp, i, i, i, i, vp],
             "apb_gemm_simt": [vp, vp, vp, i, i, i, ll, ll, ll, i, vp, vp, ll, i, vp],
         }
@@ -376,9 +376,11 @@ def retention(b: StepBatch, p: torch.Tensor, cols: Tuple[int, int, int, int], ro
         plan = b.host_tables[key]
         seg = b.table(key + ("seg",), lambda: plan["seg"])
         chains = b.table(key + ("chains",), lambda: plan["chains"]) if len(plan["chains"]) else None
+        qk = torch.empty((b.rows, H, 4, (D + 15) // 16 * 16), device=p.device, dtype=torch.bfloat16)
         carry = torch.empty((plan["states"], H, D, E), device=p.device, dtype=torch.float32) if plan["states"] else None
         _call("apb_retention_mma", _lib.ptr(p), p.stride(0), *cols[:3], _lib.ptr(rope[0]), _lib.ptr(rope[1]), rot_dims,
               _lib.ptr(log2_decay), float(k_scale), _lib.ptr(state), _lib.ptr(scratch), *b.entry_ptrs(), _lib.ptr(seg),
-              len(plan["seg"]), _lib.ptr(carry), _lib.ptr(chains), len(plan["chains"]), H, D, E)
+              len(plan["seg"]), _lib.ptr(carry), _lib.ptr(chains), len(plan["chains"]), _lib.ptr(b.row_entry), _lib.ptr(qk),
+              b.rows, H, D, E)
         _call("apb_retention_out", _lib.ptr(p), p.stride(0), cols[3], _lib.ptr(scratch), _lib.ptr(out), out.stride(0),
               float(out_scale), float(eps), _lib.ptr(b.row_entry), *b.entry_ptrs(), b.rows, H, E, dtype_code(p.dtype))

@@ -1,7 +1,7 @@
 """Serving speed of a stateful architecture beside the dense decoder of equal layer size.
 
     python bench.py --workload serving [--serving-models reninex-2048,reninex-4096]
-    python benchmarks/bench_serving.py [--models ...] [--kernels-only] [--only prefill|decode] [--iters 20]
+    python benchmarks/bench_serving.py [--models ...] [--kernels-only] [--only prefill|decode] [--step NAME] [--iters 20]
 
 For every model (random weights, synthetic prompts) two parts are measured on one GPU:
 
@@ -231,7 +231,7 @@ def dense_ops(cfg, phase):
     return ops
 
 
-def bench_kernels(name, cfg, phase, iters):
+def bench_kernels(name, cfg, phase, iters, step=None, compare=True):
     bw, peak, of = peaks()
     timer = Timer(iters)
 
@@ -240,9 +240,12 @@ def bench_kernels(name, cfg, phase, iters):
         floor = max(nbytes / bw, flops / peak) * 1e3
         return ms, floor, floor / ms
 
-    like = {k: measured(*v) for k, v in dense_ops(cfg, phase).items() if k != "_keep"}
+    like = {k: measured(*v) for k, v in dense_ops(cfg, phase).items() if k != "_keep" and (step is None or step in k)} \
+        if compare else {}
     torch.cuda.empty_cache()
     for op, fn, nbytes, flops in stateful_ops(cfg, phase):
+        if step is not None and step not in op:
+            continue
         ms, floor, frac = measured(fn, nbytes, flops)
         row = {"model": name, "phase": phase, "step": op, "ms": round(ms, 4), "floor_ms": round(floor, 4),
                "frac": round(frac, 3), "of": of}
@@ -290,14 +293,14 @@ def bench_engine(name, cfg, seqs, new_tokens):
         torch.cuda.empty_cache()
 
 
-def main(models, kernels_only=False, only=None, iters=20, seqs=64, new_tokens=129) -> None:
+def main(models, kernels_only=False, only=None, iters=20, seqs=64, new_tokens=129, step=None, compare=True) -> None:
     from arctic_platform_b200.models.config import resolve_config
     from arctic_platform_b200.ops import _lib
     for name in models:
         cfg = resolve_config(name)
         for phase in ("prefill", "decode"):
             if only in (None, phase):
-                bench_kernels(name, cfg, phase, iters)
+                bench_kernels(name, cfg, phase, iters, step, compare)
                 torch.cuda.empty_cache()
         if not kernels_only:
             bench_engine(name, cfg, seqs, new_tokens)
@@ -309,8 +312,10 @@ if __name__ == "__main__":
     ap.add_argument("--models", default="reninex-2048,reninex-4096")
     ap.add_argument("--kernels-only", action="store_true")
     ap.add_argument("--only", choices=["prefill", "decode"])
+    ap.add_argument("--step", help="only the steps whose name contains this")
+    ap.add_argument("--no-compare", action="store_true", help="leave the dense kernels out")
     ap.add_argument("--iters", type=int, default=20)
     ap.add_argument("--seqs", type=int, default=64)
     ap.add_argument("--new-tokens", type=int, default=129)
     a = ap.parse_args()
-    main(a.models.split(","), a.kernels_only, a.only, a.iters, a.seqs, a.new_tokens)
+    main(a.models.split(","), a.kernels_only, a.only, a.iters, a.seqs, a.new_tokens, a.step, not a.no_compare)

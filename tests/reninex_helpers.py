@@ -43,9 +43,9 @@ CONFIGS = {
     "bare": config([layer(heads=8, kv=1, dim=16, vdim=16, r_heads=4, r_dim=16, r_vdim=32, rot=0,
                           decay=[1.0, 0.9, 0.0, 0.5], ls=1.0, rs=1.0)], width=64, vocab=96, taps=0, bigram=None, loop=None),
     # wide heads, two taps, a loop that starts with the first layer and leaves one after it
-    "wide-heads": config([layer(heads=4, kv=2, dim=96, vdim=96, r_heads=2, r_dim=128, r_vdim=128, rot=96, base=1e6),
+    "wide-heads": config([layer(heads=4, kv=2, dim=96, vdim=96, r_heads=2, r_dim=128, r_vdim=128, rot=96, base=2e5),
                           layer(heads=2, kv=1, dim=192, vdim=160, r_heads=2, r_dim=48, r_vdim=80, rot=48)],
-                         width=256, vocab=512, taps=2, loop=(0, 1, 2)),
+                         width=256, vocab=456, taps=2, loop=(0, 1, 2)),
 }
 
 
