@@ -224,6 +224,36 @@ class StatefulSampler(SamplerEngine):
             return torch.empty((0, self.cfg.vocab_size), device=self.device, dtype=torch.float32)
         return self._output_logits(self.model.output_rows(x, self._rows_of(rows)))
 
+    @torch.no_grad()
+    def score(self, prompts: Sequence[Sequence[int]], completions: Sequence[Sequence[int]], top_k: int = 1,
+              portion: int = 1024):
+        """Log-probabilities of given completions (teacher forcing), one list per sequence; ``top_k`` > 1 also returns the
+        ``top_k`` most likely tokens per position, as ``{"log_probs": rows, "top_log_probs": [[{token: lp}]]}``."""
+        rows, tops = [], []
+        for prompt, comp in zip(prompts, completions):
+            if len(prompt) == 0:
+                raise ValueError("empty prompt")
+            seq = [*prompt, *comp]
+            slot, lp, top = self.open_sequence(), [], []
+            try:
+                for at in range(0, len(seq) - 1, portion):
+                    part = seq[at:min(at + portion, len(seq) - 1)]
+                    want = list(range(max(0, len(prompt) - 1 - at), len(part)))
+                    z = self.step([(slot, part, want)])
+                    if not want:
+                        continue
+                    z = torch.log_softmax(z, -1)
+                    nxt = torch.tensor([seq[at + w + 1] for w in want], device=z.device)
+                    lp += z.gather(1, nxt[:, None])[:, 0].tolist()
+                    if top_k > 1:
+                        v, i = torch.topk(z, int(top_k), dim=-1)
+                        top += [dict(zip(ii, vv)) for ii, vv in zip(i.tolist(), v.tolist())]
+            finally:
+                self.close_sequence(slot)
+            rows.append(lp)
+            tops.append(top)
+        return {"log_probs": rows, "top_log_probs": tops} if top_k > 1 else rows
+
     # ------------------------------------------------------------------ sleep / wake
     def sleep(self, level: int = 1) -> None:
         """Level 1 frees caches and states, level 2 the weights too (they come back with the next weight sync)."""

@@ -542,6 +542,8 @@ class EngineWorker:
         model = self._target_model()
         if self.sampler is not None and getattr(self.sampler, "_asleep", False):
             raise RuntimeError("sampler is asleep; call wake() first")
+        if registry.is_stateful(self.model_cfg):
+            return self.sampler.score(prompts, completions, top_k)
         P = max(len(p) for p in prompts)
         R = max(len(c) for c in completions)
         ids = torch.zeros((len(prompts), P + R), dtype=torch.int64)

@@ -20,6 +20,7 @@ wall time: when the next timed step would end past it, all ranks stop together (
 line reports the steps actually timed in ``steps`` with the request in ``steps_requested``.
 
     python bench.py [--gpus N --steps K --warmup W]          # N > 1 under torch.distributed.run
+    python bench.py --workload serving                        # stateful architectures beside the dense decoder
     python bench.py --impl reference                          # the reference's own stack, if installable
 """
 from __future__ import annotations
@@ -44,6 +45,10 @@ def parse_args():
     ap.add_argument("--steps", type=int, default=2)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
+    ap.add_argument("--workload", default="grpo", choices=["grpo", "serving"],
+                    help="grpo: the benchmark step (default); serving: prefill / decode speed and per-kernel roofline "
+                         "fractions of the stateful architectures beside the dense decoder (benchmarks/bench_serving.py)")
+    ap.add_argument("--serving-models", default="reninex-2048,reninex-4096")
     ap.add_argument("--model", default="qwen3-4b")
     ap.add_argument("--prompts-per-gpu", type=int, default=8)
     ap.add_argument("--samples", type=int, default=16)
@@ -139,6 +144,10 @@ def main():
     args = parse_args()
     if args.impl == "reference":
         reference_arm(args)
+        return
+    if args.workload == "serving":
+        from benchmarks import bench_serving
+        bench_serving.main(args.serving_models.split(","))
         return
     import torch
     import torch.distributed as dist

@@ -192,6 +192,10 @@ def test_worker_serves_a_checkpoint_directory(tmp_path):
     first = worker.sampler.generate(prompts, sp)
     for o in first:
         _follow(cfg, w, prompts[o["prompt_index"]], o, 0.25)
+    scored = worker.score_completions(prompts, [o["token_ids"] for o in first], top_k=3)
+    for o, lp, top in zip(first, scored["log_probs"], scored["top_log_probs"]):
+        assert np.abs(np.array(lp) - np.array(o["logprobs"])).max() < 0.2
+        assert all(len(t) == 3 and abs(max(t.values()) - v) < 0.2 for t, v in zip(top, lp))
     worker.sampler.sleep(1)
     with pytest.raises(RuntimeError, match="asleep"):
         worker.sampler.generate(prompts, sp)
