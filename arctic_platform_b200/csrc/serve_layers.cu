@@ -81,7 +81,7 @@ loop_begin_kernel(float* __restrict__ x, const T* __restrict__ init, int W, T* _
 // h:  out_k[t] = h[t] + sum_j w_k[j] h[t - taps + 1 + j].  w_k is [taps, W]; a null w_k copies h.  The history of h
 // before the entry's first row comes from the slot's state [2][taps - 1][W]; the last taps - 1 rows of h replace it.
 // One block = up to kNormRows consecutive rows of one entry (tiles[2 i] = entry, tiles[2 i + 1] = first row; without a
-// table block i is entry i, which then has at most kNormRows rows).
+// table block i is entry i, which then has at most one row).
 constexpr int kNormRows = 8;
 constexpr int kNormThreads = 256;
 
@@ -156,51 +156,41 @@ norm_conv_kernel(const float* __restrict__ x, const T* __restrict__ gain, const 
 }
 
 template <typename T>
-__device__ __forceinline__ float4 load4(const T* p) {
-  if constexpr (sizeof(T) == 2) {
-    const uint2 r = *reinterpret_cast<const uint2*>(p);
-    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x));
-    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
-    return make_float4(a.x, a.y, b.x, b.y);
-  } else {
-    return *reinterpret_cast<const float4*>(p);
-  }
+__device__ __forceinline__ float2 load2(const T* p) {
+  if constexpr (sizeof(T) == 2)
+    return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
+  else
+    return *reinterpret_cast<const float2*>(p);
 }
 template <typename T>
-__device__ __forceinline__ void store4(T* p, float4 v) {
-  if constexpr (sizeof(T) == 2) {
-    uint2 r;
-    r.x = pack_bf16x2(v.x, v.y);
-    r.y = pack_bf16x2(v.z, v.w);
-    *reinterpret_cast<uint2*>(p) = r;
-  } else {
-    *reinterpret_cast<float4*>(p) = v;
-  }
+__device__ __forceinline__ void store2(T* p, float2 v) {
+  if constexpr (sizeof(T) == 2)
+    *reinterpret_cast<uint32_t*>(p) = pack_bf16x2(v.x, v.y);
+  else
+    *reinterpret_cast<float2*>(p) = v;
 }
-__device__ __forceinline__ void fma4(float4& a, const float4& w, const float4& h) {
+__device__ __forceinline__ void fma2(float2& a, const float2& w, const float2& h) {
   a.x += w.x * h.x;
   a.y += w.y * h.y;
-  a.z += w.z * h.z;
-  a.w += w.w * h.w;
 }
 
-// The same for a compile-time number of taps and W a multiple of 4: four channels per thread, the rows of the tile
-// loaded at once, the window in registers.
-template <typename T, int TAPS>
-__global__ void __launch_bounds__(kNormThreads)
+// The same for a compile-time number of taps and W a multiple of 4: two channels per thread, the rows of the tile
+// loaded at once, the window in registers.  ROWS = 1 (decoded tokens) is for launches without a tile table.
+template <typename T, int TAPS, int ROWS>
+__global__ void __launch_bounds__(kNormThreads, ROWS == 1 ? 4 : 2)
 norm_conv_vec_kernel(const float* __restrict__ x, const T* __restrict__ gain, const T* __restrict__ w1,
                      const T* __restrict__ w2, T* __restrict__ out1, T* __restrict__ out2, float* __restrict__ state,
                      const int* __restrict__ parity, const ServeEntries e, const int* __restrict__ tiles, int W,
                      float eps) {
   pdl_entry();
   constexpr int kHist = TAPS - 1;
-  __shared__ float rs[kHist + kNormRows];
+  __shared__ float rs[kHist + ROWS];
   __shared__ float red[kNormThreads / 32];
   const int en = tiles ? tiles[2 * blockIdx.x] : blockIdx.x;
   const int r0 = tiles ? tiles[2 * blockIdx.x + 1] : 0;
   const int len = e.len[en];
   if (r0 >= len) return;
-  const int nr = min(kNormRows, len - r0);
+  const int nr = min(ROWS, len - r0);
   const int start = e.start[en], pos0 = e.pos0[en];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const float g = to_f32(*gain);
@@ -244,47 +234,49 @@ norm_conv_vec_kernel(const float* __restrict__ x, const T* __restrict__ gain, co
     old_h = state + (static_cast<long long>(slot) * 2 + par) * kHist * W;
     new_h = state + (static_cast<long long>(slot) * 2 + (par ^ 1)) * kHist * W;
   }
-  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-  for (int c = threadIdx.x * 4; c < W; c += kNormThreads * 4) {
-    float4 h[kHist + kNormRows];                   // rows r0 - hist .. r0 + 7
+  const float2 zero = make_float2(0.f, 0.f);
+#pragma unroll (ROWS == 1 ? 2 : 1)
+  for (int c = threadIdx.x * 2; c < W; c += kNormThreads * 2) {
+    float2 h[kHist + ROWS];                   // rows r0 - hist .. r0 + ROWS - 1
+    const float* xp = x + static_cast<long long>(start + r0 - kHist) * W + c;
 #pragma unroll
-    for (int i = 0; i < kHist + kNormRows; ++i) {
+    for (int i = 0; i < kHist + ROWS; ++i, xp += W) {
       const int r = r0 - kHist + i;
       h[i] = zero;
       if (r >= 0 && i < kHist + nr)
-        h[i] = *reinterpret_cast<const float4*>(x + static_cast<long long>(start + r) * W + c);
+        h[i] = *reinterpret_cast<const float2*>(xp);
       else if (r < 0 && pos0 + r >= 0 && old_h)
-        h[i] = *reinterpret_cast<const float4*>(old_h + static_cast<long long>(kHist + r) * W + c);
+        h[i] = *reinterpret_cast<const float2*>(old_h + static_cast<long long>(kHist + r) * W + c);
     }
-    float4 a[TAPS], b[TAPS];
+    float2 a[TAPS], b[TAPS];
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) {
-      a[j] = w1 ? load4(w1 + static_cast<long long>(j) * W + c) : zero;
-      b[j] = w2 ? load4(w2 + static_cast<long long>(j) * W + c) : zero;
+      a[j] = w1 ? load2(w1 + static_cast<long long>(j) * W + c) : zero;
+      b[j] = w2 ? load2(w2 + static_cast<long long>(j) * W + c) : zero;
     }
 #pragma unroll
-    for (int i = 0; i < kHist + kNormRows; ++i)
+    for (int i = 0; i < kHist + ROWS; ++i)
       if (r0 - kHist + i >= 0 && i < kHist + nr) {
         const float f = rs[i];
-        h[i] = make_float4(h[i].x * f, h[i].y * f, h[i].z * f, h[i].w * f);
+        h[i] = make_float2(h[i].x * f, h[i].y * f);
       }
+    long long o = static_cast<long long>(start + r0) * W + c;
 #pragma unroll
-    for (int i = 0; i < kNormRows; ++i)
+    for (int i = 0; i < ROWS; ++i, o += W)
       if (i < nr) {
-        float4 y1 = h[i + kHist], y2 = y1;
+        float2 y1 = h[i + kHist], y2 = y1;
 #pragma unroll
         for (int j = 0; j < TAPS; ++j) {
-          fma4(y1, a[j], h[i + j]);
-          fma4(y2, b[j], h[i + j]);
+          fma2(y1, a[j], h[i + j]);
+          fma2(y2, b[j], h[i + j]);
         }
-        const long long o = static_cast<long long>(start + r0 + i) * W + c;
-        store4(out1 + o, y1);
-        if (out2) store4(out2 + o, y2);
+        store2(out1 + o, y1);
+        if (out2) store2(out2 + o, y2);
       }
     if (new_h && r0 + nr == len) {
 #pragma unroll
-      for (int i = 0; i < kHist + kNormRows; ++i)  // rows len - hist .. len - 1
-        if (i >= nr && i < nr + kHist) *reinterpret_cast<float4*>(new_h + static_cast<long long>(i - nr) * W + c) = h[i];
+      for (int i = 0; i < kHist + ROWS; ++i)  // rows len - hist .. len - 1
+        if (i >= nr && i < nr + kHist) *reinterpret_cast<float2*>(new_h + static_cast<long long>(i - nr) * W + c) = h[i];
     }
   }
 }
@@ -412,7 +404,7 @@ int apb_loop_begin(float* x, const void* init, int rows, int W, void* out, long 
                                                                n)));
 }
 
-// tiles: device int32 [n_tiles][2] or null (then n_tiles is the number of entries, none longer than 8 rows).
+// tiles: device int32 [n_tiles][2] or null (then n_tiles is the number of entries, none longer than one row).
 int apb_norm_conv(const float* x, const void* gain, const void* w1, const void* w2, void* out1, void* out2,
                   float* state, const int* parity, const int* e_start, const int* e_len, const int* e_slot,
                   const int* e_pos0, const int* tiles, int n_tiles, int W, int taps, float eps, int dtype,
@@ -422,7 +414,8 @@ int apb_norm_conv(const float* x, const void* gain, const void* w1, const void* 
   const ServeEntries e{e_start, e_len, e_slot, e_pos0};
   if ((W & 3) == 0 && taps <= 5) {
 #define APB_NORM_CONV(TT)                                                                                             \
-  return static_cast<int>(launch_kernel(norm_conv_vec_kernel<T, TT>, dim3(n_tiles), dim3(kNormThreads), 0, s, x,      \
+  return static_cast<int>(launch_kernel(tiles ? norm_conv_vec_kernel<T, TT, kNormRows> : norm_conv_vec_kernel<T, TT, 1>, \
+                                        dim3(n_tiles), dim3(kNormThreads), 0, s, x,                                   \
                                         static_cast<const T*>(gain), static_cast<const T*>(w1),                       \
                                         static_cast<const T*>(w2), static_cast<T*>(out1), static_cast<T*>(out2),      \
                                         state, parity, e, tiles, W, eps))
