@@ -76,6 +76,7 @@ def _compile_one(src: Path, verbose: bool) -> Path:
 SERVE_STEMS = ("status", "gemm_tcgen05", "gemm_tcgen05_2cta", "gemm_simt", "serve_layers", "serve_attention",
                "serve_attention_tc", "retention", "retention_mma")
 SERVE_LIB = OUT_DIR / "libapb200_serve.so"
+RT_SERVE_LIB = OUT_DIR / "libapb200_rt_serve.so"       # the page allocator (runtime.cpp)
 
 
 def build_cuda_subset(stems, lib: Path, verbose: bool = False) -> Path:
@@ -120,21 +121,21 @@ def build_cuda(force: bool = False, verbose: bool = False) -> Path:
     return _link(objs, CUDA_LIB)
 
 
-def build_runtime(force: bool = False) -> Path:
+def build_runtime(force: bool = False, stems=None, lib: Path = RT_LIB) -> Path:
+    """The host runtime, or (``stems``, ``lib``) a library of some of its sources only."""
     OUT_DIR.mkdir(parents=True, exist_ok=True)
-    srcs = sorted(CSRC.glob("*.cpp"))
+    srcs = sorted(CSRC.glob("*.cpp")) if stems is None else [CSRC / f"{s}.cpp" for s in stems]
     if not srcs:
         raise RuntimeError("no C++ runtime sources found")
-    if (not force and RT_LIB.exists()
-            and RT_LIB.stat().st_mtime >= _newest_mtime(srcs + _headers())):
-        return RT_LIB
+    if not force and lib.exists() and lib.stat().st_mtime >= _newest_mtime(srcs + _headers()):
+        return lib
     cxx = os.environ.get("CXX") or shutil.which("g++") or "g++"
     cmd = [cxx, "-O3", "-std=c++17", "-fPIC", "-shared", "-pthread", "-I", str(CSRC),
-           "-o", str(RT_LIB), *map(str, srcs)]
+           "-o", str(lib), *map(str, srcs)]
     res = subprocess.run(cmd, capture_output=True, text=True)
     if res.returncode != 0:
         raise RuntimeError(f"g++ failed:\n{res.stdout}\n{res.stderr}")
-    return RT_LIB
+    return lib
 
 
 def build_all(force: bool = False, verbose: bool = False) -> None:

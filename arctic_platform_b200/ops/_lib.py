@@ -89,7 +89,11 @@ def rt_lib() -> ctypes.CDLL:
     if _rt is None:
         with _lock:
             if _rt is None:
-                lib = _load(_build.RT_LIB, _build.build_runtime)
+                if _serve_only and not _build.RT_LIB.exists():
+                    lib = _load(_build.RT_SERVE_LIB,
+                                lambda: _build.build_runtime(stems=("runtime",), lib=_build.RT_SERVE_LIB))
+                else:
+                    lib = _load(_build.RT_LIB, _build.build_runtime)
                 _declare_rt(lib)
                 _rt = lib
     return _rt
