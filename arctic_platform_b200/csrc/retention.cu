@@ -19,7 +19,7 @@
 namespace apb {
 
 // ---------------------------------------------------------------------------- one token
-constexpr int kRetDecThreads = 128;
+constexpr int kRetDecThreads = 256;
 
 template <typename T, int VEC>
 __global__ void __launch_bounds__(kRetDecThreads)
