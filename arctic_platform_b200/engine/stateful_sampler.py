@@ -29,7 +29,6 @@ import numpy as np
 import torch
 
 from ..models import registry
-from ..ops import serving
 from ..ops.serving import PAGE, StepBatch, StepEntry
 from ..utils.transfer_stats import to_device
 from .sampler import SamplerEngine, _Seq

@@ -28,7 +28,6 @@ import torch
 from torch import nn
 
 from ..ops import norm, serving
-from .hf_io import interleave_gate_up, split_gate_up
 
 
 @dataclass(frozen=True)
