@@ -18,7 +18,12 @@ enum GemmEpilogue : int {
                            // that owns the row (owner = row / rows_per_rank), over its NVLink peer mapping
   kEpiBf16ScatterPeer = 8, // GEMM -> all-to-all: bf16 row stored to (peer, row) = row_map[m] (MoE combine)
   kEpiGeGLU = 9,       // as kEpiSwiGLU with the tanh form of GELU as the activation of the gate
+  kEpiClampGLU = 10,   // as kEpiSwiGLU: g = min(gate, limit), u = clamp(up, -limit, limit), g sigmoid(1.702 g) (u + 1)
 };
+
+__host__ __device__ inline bool is_glu_epilogue(int epi) {
+  return epi == kEpiSwiGLU || epi == kEpiGeGLU || epi == kEpiClampGLU;
+}
 
 struct PeerTensorMaps {
   CUtensorMap m[8];
@@ -35,6 +40,7 @@ struct GemmParams {
   long long ldc2;
   const __nv_bfloat16* bias;
   float alpha;
+  float glu_limit;           // kEpiClampGLU
   // Optional tile table for grouped problems: {m0, m_end, b_row_offset, n_tile}.
   const int4* tile_map;
   int num_map_tiles;         // entries of tile_map (an upper bound when num_tiles_dev is set)
@@ -69,6 +75,12 @@ __device__ __forceinline__ float gelu_tanh_f(float x) {
   return x / (1.f + expf(-1.5957691216057308f * (x + 0.044715f * x * x * x)));
 }
 
+__device__ __forceinline__ float clamped_glu_f(float g, float u, float limit) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g / (1.f + __expf(-1.702f * g)) * (u + 1.f);
+}
+
 // One output row, 32 consecutive accumulator columns starting at `col0` (raw fp32 bits in `r`).  Covers every
 // epilogue except the two lm-head ones, which keep running state across the chunks of a tile.
 // `ncols` (32, or 16 for the last chunk of a tile width that is not a multiple of 32) clips the chunk at the tile
@@ -78,7 +90,7 @@ __device__ __forceinline__ void gemm_store_chunk(const GemmParams& p, int row, i
   float v[32];
 #pragma unroll
   for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(r[j]) * p.alpha;
-  if (p.epi == kEpiBf16 || ((p.epi == kEpiSwiGLU || p.epi == kEpiGeGLU) && p.C != nullptr)) {
+  if (p.epi == kEpiBf16 || (is_glu_epilogue(p.epi) && p.C != nullptr)) {
     if (p.bias) {
 #pragma unroll
       for (int j = 0; j < 32; ++j)
@@ -97,7 +109,7 @@ __device__ __forceinline__ void gemm_store_chunk(const GemmParams& p, int row, i
       }
     }
   }
-  if (p.epi == kEpiSwiGLU || p.epi == kEpiGeGLU) {
+  if (is_glu_epilogue(p.epi)) {
     __nv_bfloat16* dst =
         static_cast<__nv_bfloat16*>(p.C2) + static_cast<long long>(row) * p.ldc2 + (col0 >> 1);
 #pragma unroll
@@ -106,8 +118,8 @@ __device__ __forceinline__ void gemm_store_chunk(const GemmParams& p, int row, i
         float a[8];
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
-          const float g = v[q * 16 + 2 * j];
-          a[j] = (p.epi == kEpiSwiGLU ? silu_f(g) : gelu_tanh_f(g)) * v[q * 16 + 2 * j + 1];
+          const float g = v[q * 16 + 2 * j], u = v[q * 16 + 2 * j + 1];
+          a[j] = p.epi == kEpiSwiGLU ? silu_f(g) * u : p.epi == kEpiGeGLU ? gelu_tanh_f(g) * u : clamped_glu_f(g, u, p.glu_limit);
         }
         uint4 o;
         o.x = pack_bf16x2(a[0], a[1]);

@@ -10,11 +10,17 @@ namespace apb {
 
 constexpr int kSgTile = 64, kSgK = 16;
 
+__device__ __forceinline__ float clamped_glu(float g, float u, float limit) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g / (1.f + expf(-1.702f * g)) * (u + 1.f);
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256)
 gemm_simt_kernel(const T* __restrict__ A, const T* __restrict__ B, void* __restrict__ C, long long lda, long long ldb,
                  long long ldc, int M, int N, int K, int epi, const T* __restrict__ bias, void* __restrict__ C2,
-                 long long ldc2) {
+                 long long ldc2, float glu_limit) {
   pdl_entry();
   __shared__ float as[kSgK][kSgTile + 4], bs[kSgK][kSgTile + 4];
   const int m0 = blockIdx.y * kSgTile, n0 = blockIdx.x * kSgTile;
@@ -54,8 +60,11 @@ gemm_simt_kernel(const T* __restrict__ A, const T* __restrict__ B, void* __restr
         static_cast<float*>(C)[m * ldc + n] = v;
       else if (epi == kEpiF32Accum || epi == kEpiF32Atomic)
         static_cast<float*>(C)[m * ldc + n] += v;
-      else if (epi == kEpiGeGLU && !(j & 1) && n + 1 < N)
-        static_cast<T*>(C2)[m * ldc2 + (n >> 1)] = from_f32<T>(gelu_tanh_f(v) * (acc[i][j | 1] + (bias ? to_f32(bias[n + 1]) : 0.f)));
+      else if (is_glu_epilogue(epi) && !(j & 1) && n + 1 < N) {
+        const float u = acc[i][j | 1] + (bias ? to_f32(bias[n + 1]) : 0.f);
+        const float y = epi == kEpiGeGLU ? gelu_tanh_f(v) * u : clamped_glu(v, u, glu_limit);
+        static_cast<T*>(C2)[m * ldc2 + (n >> 1)] = from_f32<T>(y);
+      }
     }
   }
 }
@@ -66,16 +75,18 @@ extern "C" {
 using namespace apb;
 
 // epi: 0 C in the operand type, 1 C fp32, 2 / 3 C fp32 += (one writer per element), 9 columns interleaved (gate, up):
-// C2[m, n/2] = gelu_tanh(gate) * up in the operand type.  bias [N] (operand type) or null.
+// C2[m, n/2] = gelu_tanh(gate) * up in the operand type, 10 the same with the clamped GLU (glu_limit > 0).  bias [N] (operand type) or null.
 int apb_gemm_simt(const void* A, const void* B, void* C, int M, int N, int K, long long lda, long long ldb,
-                  long long ldc, int epi, const void* bias, void* C2, long long ldc2, int dtype, cudaStream_t s) {
+                  long long ldc, int epi, const void* bias, void* C2, long long ldc2, float glu_limit, int dtype, cudaStream_t s) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
-  if (epi == kEpiGeGLU ? !C2 : !C) return kBadArgument;
-  if (epi != kEpiBf16 && epi != kEpiF32 && epi != kEpiF32Accum && epi != kEpiF32Atomic && epi != kEpiGeGLU) return kBadArgument;
+  if (epi == kEpiGeGLU || epi == kEpiClampGLU ? !C2 : !C) return kBadArgument;
+  if (epi == kEpiClampGLU && !(glu_limit > 0.f)) return kBadArgument;
+  if (epi != kEpiBf16 && epi != kEpiF32 && epi != kEpiF32Accum && epi != kEpiF32Atomic && epi != kEpiGeGLU && epi != kEpiClampGLU)
+    return kBadArgument;
   const dim3 grid((N + kSgTile - 1) / kSgTile, (M + kSgTile - 1) / kSgTile);
   APB_SERVE_DTYPE(dtype, return static_cast<int>(launch_kernel(
                              gemm_simt_kernel<T>, grid, dim3(256), 0, s, static_cast<const T*>(A),
                              static_cast<const T*>(B), C, lda, ldb, ldc, M, N, K, epi, static_cast<const T*>(bias), C2,
-                             ldc2)));
+                             ldc2, glu_limit)));
 }
 }

@@ -488,9 +488,9 @@ static int launch_gemm_x2(const CUtensorMap& ta, const CUtensorMap& tb, const Ge
 
 }  // namespace apb
 
-extern "C" int apb_gemm_bf16_pair(const void* A, const void* B, void* C, int M, int N, int K, long long lda,
+extern "C" int apb_gemm_bf16_pair_glu(const void* A, const void* B, void* C, int M, int N, int K, long long lda,
                                   long long ldb, long long ldc, int a_mn, int b_mn, int epi, float alpha,
-                                  const void* bias, void* C2, long long ldc2, cudaStream_t stream);
+                                  const void* bias, void* C2, long long ldc2, float glu_limit, cudaStream_t stream);
 
 namespace apb {
 static bool pair_kernel_enabled() {
@@ -518,14 +518,15 @@ static int gemm_bf16_impl(const void* A, const void* B, void* C, int M, int N, i
                          long long ldc, int a_mn, int b_mn, int epi, int splits, float alpha, const void* bias,
                          void* C2, long long ldc2, const void* tile_map, int num_map_tiles, const int* num_tiles_dev,
                          long long b_rows, int bn, int max_ctas, cudaStream_t stream, const void* tile_ext = nullptr,
-                         long long b_k_rows = 0) {
+                         long long b_k_rows = 0, float glu_limit = 0.f) {
   using namespace apb;
   if (M <= 0 || N <= 0 || K <= 0) return 0;
+  if (epi == kEpiClampGLU && !(glu_limit > 0.f)) return kBadArgument;
   if (tile_ext && (!tile_map || splits > 1)) return kBadArgument;
   if ((lda % 8) || (ldb % 8) || (N % 8) || (reinterpret_cast<uintptr_t>(A) & 15) ||
       (reinterpret_cast<uintptr_t>(B) & 15) || (reinterpret_cast<uintptr_t>(C) & 15))
     return kBadArgument;
-  const bool glu = epi == kEpiSwiGLU || epi == kEpiGeGLU;
+  const bool glu = is_glu_epilogue(epi);
   if (epi == kEpiBf16 || glu) {
     if (C && (ldc % 8)) return kBadArgument;
   } else if (ldc % 4) {
@@ -542,7 +543,7 @@ static int gemm_bf16_impl(const void* A, const void* B, void* C, int M, int N, i
       (epi == kEpiBf16 || epi == kEpiF32 || epi == kEpiF32Accum || glu) &&
       !(epi == kEpiBf16 && !C) && M >= 512 &&
       static_cast<long long>((M + 255) / 256) * ((N + 255) / 256) >= sm_count() / 2)
-    return apb_gemm_bf16_pair(A, B, C, M, N, K, lda, ldb, ldc, a_mn, b_mn, epi, alpha, bias, C2, ldc2, stream);
+    return apb_gemm_bf16_pair_glu(A, B, C, M, N, K, lda, ldb, ldc, a_mn, b_mn, epi, alpha, bias, C2, ldc2, glu_limit, stream);
   if (bn == 0) {
     const long long tm = (M + kBM - 1) / kBM;
     const long long t256 = tm * ((N + 255) / 256) * splits;
@@ -604,6 +605,7 @@ static int gemm_bf16_impl(const void* A, const void* B, void* C, int M, int N, i
   p.ldc2 = ldc2;
   p.bias = static_cast<const __nv_bfloat16*>(bias);
   p.alpha = alpha;
+  p.glu_limit = glu_limit;
   p.tile_map = static_cast<const int4*>(tile_map);
   p.num_map_tiles = num_map_tiles;
   p.num_tiles_dev = tile_map ? num_tiles_dev : nullptr;
@@ -627,6 +629,15 @@ int apb_gemm_bf16(const void* A, const void* B, void* C, int M, int N, int K, lo
                   int max_ctas, cudaStream_t stream) {
   return gemm_bf16_impl(A, B, C, M, N, K, lda, ldb, ldc, a_mn, b_mn, epi, splits, alpha, bias, C2, ldc2, tile_map,
                         num_map_tiles, nullptr, b_rows, bn, max_ctas, stream);
+}
+
+// C2 [M, N / 2] = GLU of op(A) op(B)^T (columns interleaved: gate, up) with the activation `epi` (kEpiSwiGLU, kEpiGeGLU or
+// kEpiClampGLU with its limit).
+int apb_gemm_bf16_glu(const void* A, const void* B, int M, int N, int K, long long lda, long long ldb, int epi, float limit,
+                      void* C2, long long ldc2, cudaStream_t stream) {
+  if (!apb::is_glu_epilogue(epi)) return apb::kBadArgument;
+  return gemm_bf16_impl(A, B, nullptr, M, N, K, lda, ldb, 0, 0, 0, epi, 1, 1.f, nullptr, C2, ldc2, nullptr, 0, nullptr, 0, 0,
+                        0, stream, nullptr, 0, limit);
 }
 
 // Grouped GEMM whose tile table was written by a kernel: `tile_map` has room for `max_tiles` entries, the number in

@@ -309,14 +309,15 @@ extern "C" {
 
 // D[M,N] = alpha * op(A) * op(B)^T with the CTA-pair kernel.  Same operand conventions as apb_gemm_bf16
 // (a_mn / b_mn, leading dimensions multiples of 8, 16-byte aligned bases).  Epilogues: bf16 (+bias), f32,
-// f32 accumulate (split along K by the kernel's own choice when that fills the last wave), SwiGLU.  No tile table.  Returns kBadArgument for anything else so that the caller
-// can fall back to the one-CTA kernel.
-int apb_gemm_bf16_pair(const void* A, const void* B, void* C, int M, int N, int K, long long lda, long long ldb,
-                       long long ldc, int a_mn, int b_mn, int epi, float alpha, const void* bias, void* C2,
-                       long long ldc2, cudaStream_t stream) {
+// f32 accumulate (split along K by the kernel's own choice when that fills the last wave), the GLU kinds (glu_limit:
+// kEpiClampGLU).  No tile table.  Returns kBadArgument for anything else so that the caller can fall back to the one-CTA
+// kernel.
+int apb_gemm_bf16_pair_glu(const void* A, const void* B, void* C, int M, int N, int K, long long lda, long long ldb,
+                           long long ldc, int a_mn, int b_mn, int epi, float alpha, const void* bias, void* C2,
+                           long long ldc2, float glu_limit, cudaStream_t stream) {
   using namespace apb;
   if (M <= 0 || N <= 0 || K <= 0) return 0;
-  const bool glu = epi == kEpiSwiGLU || epi == kEpiGeGLU;
+  const bool glu = is_glu_epilogue(epi);
   if (epi != kEpiBf16 && epi != kEpiF32 && epi != kEpiF32Accum && !glu) return kBadArgument;
   if ((lda % 8) || (ldb % 8) || (N % 8) || (reinterpret_cast<uintptr_t>(A) & 15) ||
       (reinterpret_cast<uintptr_t>(B) & 15) || (reinterpret_cast<uintptr_t>(C) & 15))
@@ -382,6 +383,7 @@ int apb_gemm_bf16_pair(const void* A, const void* B, void* C, int M, int N, int 
   p.ldc2 = ldc2;
   p.bias = static_cast<const __nv_bfloat16*>(bias);
   p.alpha = alpha;
+  p.glu_limit = glu_limit;
   p.status = status_device_ptr();
 
   // How many pairs can be resident at once (SMs of a pair must sit in one cluster-capable group, so this can be
@@ -420,5 +422,12 @@ int apb_gemm_bf16_pair(const void* A, const void* B, void* C, int M, int N, int 
   cudaError_t e = cudaLaunchKernelEx(&cfg, gemm_bf16_pair_kernel, ta, tb, p);
   if (e != cudaSuccess) return static_cast<int>(e);
   return static_cast<int>(cudaGetLastError());
+}
+
+int apb_gemm_bf16_pair(const void* A, const void* B, void* C, int M, int N, int K, long long lda, long long ldb,
+                       long long ldc, int a_mn, int b_mn, int epi, float alpha, const void* bias, void* C2,
+                       long long ldc2, cudaStream_t stream) {
+  if (epi == apb::kEpiClampGLU) return apb::kBadArgument;      // needs its limit
+  return apb_gemm_bf16_pair_glu(A, B, C, M, N, K, lda, ldb, ldc, a_mn, b_mn, epi, alpha, bias, C2, ldc2, 0.f, stream);
 }
 }

@@ -19,15 +19,15 @@
 namespace apb {
 
 // ---------------------------------------------------------------------------- embedding
-// x[row] = embed[token] (+ bigram[hash(previous token, token)]), fp32; `x0` (optional) receives the same row in the
-// activation type (the right half of the loop-input operand), `kv_slot` the row's cache slot (page * 16 + offset, -1 for
-// an entry without tokens).
+// x[row] = (embed[token] (+ bigram[hash(previous token, token)])) * scale, fp32, written `copies` times (parallel residual
+// streams start equal); `x0` (optional) receives the same row in the activation type (the right half of the loop-input
+// operand), `kv_slot` the row's cache slot (page * 16 + offset, -1 for an entry without tokens).
 template <typename T>
 __global__ void __launch_bounds__(128)
 embed_hash_kernel(const int* __restrict__ tokens, const int* __restrict__ row_entry, const ServeEntries e,
                   const int* __restrict__ prev, const T* __restrict__ embed, const T* __restrict__ bigram,
-                  long long buckets, long long mul_prev, long long mul_cur, int vocab, int W, float* __restrict__ x,
-                  T* __restrict__ x0, long long ld0, const int* __restrict__ page_table, int max_pages,
+                  long long buckets, long long mul_prev, long long mul_cur, int vocab, int W, float scale, int copies,
+                  float* __restrict__ x, T* __restrict__ x0, long long ld0, const int* __restrict__ page_table, int max_pages,
                   int* __restrict__ kv_slot) {
   pdl_entry();
   const int row = blockIdx.x;
@@ -55,7 +55,8 @@ embed_hash_kernel(const int* __restrict__ tokens, const int* __restrict__ row_en
   for (int i = threadIdx.x; i < W; i += blockDim.x) {
     float v = to_f32(src[i]);
     if (big) v += to_f32(big[i]);
-    x[static_cast<long long>(row) * W + i] = v;
+    v *= scale;
+    for (int c = 0; c < copies; ++c) x[(static_cast<long long>(row) * copies + c) * W + i] = v;
     if (x0) x0[static_cast<long long>(row) * ld0 + i] = from_f32<T>(v);
   }
 }
@@ -281,11 +282,12 @@ norm_conv_vec_kernel(const float* __restrict__ x, const T* __restrict__ gain, co
   }
 }
 
-// Final norm of selected rows: out[i] = x[rows[i]] / rms * g (rows == null: row i).  One block per row.
+// Final norm of selected rows: out[i] = x[rows[i]] / rms * g (rows == null: row i), with one gain (gain_step 0) or one per
+// channel (gain_step 1).  One block per row.
 template <typename T>
 __global__ void __launch_bounds__(256)
 gain_norm_rows_kernel(const float* __restrict__ x, const int* __restrict__ rows, const T* __restrict__ gain,
-                      T* __restrict__ out, int W, float eps) {
+                      int gain_step, T* __restrict__ out, int W, float eps) {
   pdl_entry();
   __shared__ float red[8];
   const float* xr = x + static_cast<long long>(rows ? rows[blockIdx.x] : static_cast<int>(blockIdx.x)) * W;
@@ -297,8 +299,9 @@ gain_norm_rows_kernel(const float* __restrict__ x, const int* __restrict__ rows,
   ss = 0.f;
 #pragma unroll
   for (int i = 0; i < 8; ++i) ss += red[i];
-  const float f = to_f32(*gain) / sqrtf(ss / W + eps);
-  for (int c = threadIdx.x; c < W; c += 256) out[static_cast<long long>(blockIdx.x) * W + c] = from_f32<T>(xr[c] * f);
+  const float f = 1.f / sqrtf(ss / W + eps);
+  for (int c = threadIdx.x; c < W; c += 256)
+    out[static_cast<long long>(blockIdx.x) * W + c] = from_f32<T>(xr[c] * f * to_f32(gain[c * gain_step]));
 }
 
 // ---------------------------------------------------------------------------- q/k norm + paged cache write
@@ -362,6 +365,69 @@ qk_norm_cache_kernel(T* __restrict__ p, long long ld, int q_col, int k_col, int 
   for (int i = lane; i < n; i += 32) dst[i] = is_v ? src[i] : from_f32<T>(to_f32(src[i]) * r);
 }
 
+// ---------------------------------------------------------------------------- rotation + paged cache write
+// Rotary positions on neighbouring pairs: of every head of D columns the first `rot` are rotated, dimension 2i with 2i + 1,
+// by the angles of the row's position (tables [positions, rot / 2]).  q (HQ heads at q_col) is rotated in place; k (HK
+// heads at k_col) goes to kcache [pages, G, 16, HK / G * D], v (G heads of E at v_col) to vcache [pages, G, 16, E].  HK = 0:
+// q only.  One thread handles V neighbouring columns (8 bf16, or one pair).
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+rope_cache_kernel(T* __restrict__ p, long long ld, int q_col, int k_col, int v_col, const int* __restrict__ row_entry,
+                  const ServeEntries e, const int* __restrict__ kv_slot, const float* __restrict__ cos_t,
+                  const float* __restrict__ sin_t, int rot, T* __restrict__ kcache, T* __restrict__ vcache, int rows,
+                  int HQ, int HK, int G, int D, int E) {
+  pdl_entry();
+  const int du = (D + V - 1) / V, eu = (E + V - 1) / V;             // units of a head
+  const int nq = HQ * du, nk = HK * du, units = nq + nk + (HK ? G * eu : 0);
+  const long long idx = blockIdx.x * 256LL + threadIdx.x;
+  if (idx >= static_cast<long long>(rows) * units) return;
+  const int row = static_cast<int>(idx / units);
+  int u = static_cast<int>(idx % units);
+  const int en = row_entry ? row_entry[row] : row;
+  const int r = row - e.start[en];
+  if (r < 0 || r >= e.len[en]) return;
+  const bool is_q = u < nq, is_v = u >= nq + nk;
+  u -= is_q ? 0 : (is_v ? nq + nk : nq);
+  const int w = is_v ? E : D, per = is_v ? eu : du;
+  const int head = u / per, c0 = (u % per) * V;
+  const int n = V == 8 ? 8 : min(V, w - c0);
+  T* src = p + static_cast<long long>(row) * ld + (is_q ? q_col : is_v ? v_col : k_col) + static_cast<long long>(head) * w + c0;
+  T* dst = src;
+  if (!is_q) {
+    const int slot = kv_slot[row];
+    if (slot < 0) return;
+    const int maps = HK / G;                                         // key heads side by side in one cache row
+    const int g = is_v ? head : head / maps;
+    const long long tok = (static_cast<long long>(slot / kServePage) * G + g) * kServePage + slot % kServePage;
+    dst = is_v ? vcache + tok * E + c0 : kcache + (tok * maps + head % maps) * D + c0;
+  }
+  const long long tr = static_cast<long long>(e.pos0[en] + r) * (rot >> 1);
+  if constexpr (V == 8) {
+    uint4 raw = *reinterpret_cast<const uint4*>(src);
+    if (!is_v && c0 < rot) {
+      uint32_t* w2 = reinterpret_cast<uint32_t*>(&raw);
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (c0 + 2 * i < rot) {
+          const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w2[i]));
+          const float c = cos_t[tr + (c0 >> 1) + i], s = sin_t[tr + (c0 >> 1) + i];
+          w2[i] = pack_bf16x2(f.x * c - f.y * s, f.y * c + f.x * s);
+        }
+    }
+    *reinterpret_cast<uint4*>(dst) = raw;
+  } else {
+    T a = src[0], b = n > 1 ? src[1] : src[0];
+    if (!is_v && c0 + 1 < rot) {
+      const float c = cos_t[tr + (c0 >> 1)], s = sin_t[tr + (c0 >> 1)];
+      const float x = to_f32(a), y = to_f32(b);
+      a = from_f32<T>(x * c - y * s);
+      b = from_f32<T>(y * c + x * s);
+    }
+    dst[0] = a;
+    if (n > 1) dst[1] = b;
+  }
+}
+
 // ---------------------------------------------------------------------------- end of a step
 // Every entry that fed tokens: remember its last token and flip the parity of its double-buffered state.
 __global__ void __launch_bounds__(128)
@@ -383,15 +449,16 @@ using namespace apb;
 
 int apb_embed_hash(const int* tokens, const int* row_entry, const int* e_start, const int* e_len, const int* e_slot,
                    const int* e_pos0, const int* prev, const void* embed, const void* bigram, long long buckets,
-                   long long mul_prev, long long mul_cur, int vocab, int W, float* x, void* x0, long long ld0,
-                   const int* page_table, int max_pages, int* kv_slot, int rows, int dtype, cudaStream_t s) {
+                   long long mul_prev, long long mul_cur, int vocab, int W, float scale, int copies, float* x, void* x0,
+                   long long ld0, const int* page_table, int max_pages, int* kv_slot, int rows, int dtype,
+                   cudaStream_t s) {
   if (rows <= 0) return 0;
-  if (!tokens || !embed || !x || (bigram && (buckets <= 0 || !prev)) || (kv_slot && !page_table)) return kBadArgument;
+  if (!tokens || !embed || !x || copies < 1 || (bigram && (buckets <= 0 || !prev)) || (kv_slot && !page_table)) return kBadArgument;
   const ServeEntries e{e_start, e_len, e_slot, e_pos0};
   APB_SERVE_DTYPE(dtype, return static_cast<int>(launch_kernel(
                              embed_hash_kernel<T>, dim3(rows), dim3(128), 0, s, tokens, row_entry, e, prev,
                              static_cast<const T*>(embed), static_cast<const T*>(bigram), buckets, mul_prev, mul_cur,
-                             vocab, W, x, static_cast<T*>(x0), ld0, page_table, max_pages, kv_slot)));
+                             vocab, W, scale, copies, x, static_cast<T*>(x0), ld0, page_table, max_pages, kv_slot)));
 }
 
 int apb_loop_begin(float* x, const void* init, int rows, int W, void* out, long long ld, int dtype, cudaStream_t s) {
@@ -430,12 +497,12 @@ int apb_norm_conv(const float* x, const void* gain, const void* w1, const void* 
                              static_cast<T*>(out1), static_cast<T*>(out2), state, parity, e, tiles, W, taps, eps)));
 }
 
-int apb_gain_norm_rows(const float* x, const int* rows, const void* gain, void* out, int n, int W, float eps, int dtype,
-                       cudaStream_t s) {
+int apb_gain_norm_rows(const float* x, const int* rows, const void* gain, int gain_step, void* out, int n, int W, float eps,
+                       int dtype, cudaStream_t s) {
   if (n <= 0) return 0;
   APB_SERVE_DTYPE(dtype, return static_cast<int>(launch_kernel(gain_norm_rows_kernel<T>, dim3(n), dim3(256), 0, s, x, rows,
-                                                               static_cast<const T*>(gain), static_cast<T*>(out), W,
-                                                               eps)));
+                                                               static_cast<const T*>(gain), gain_step,
+                                                               static_cast<T*>(out), W, eps)));
 }
 
 int apb_qk_norm_cache(void* p, long long ld, int q_col, int k_col, int v_col, const int* kv_slot, void* kcache,
@@ -447,6 +514,31 @@ int apb_qk_norm_cache(void* p, long long ld, int q_col, int k_col, int v_col, co
   APB_SERVE_DTYPE(dtype, return static_cast<int>(launch_kernel(
                              qk_norm_cache_kernel<T>, dim3(grid), dim3(256), 0, s, static_cast<T*>(p), ld, q_col, k_col,
                              v_col, kv_slot, static_cast<T*>(kcache), static_cast<T*>(vcache), rows, H, G, D, E, eps)));
+}
+
+// row_entry [rows] or null (row i belongs to entry i).  HK = 0: only q is rotated (a layer that reads another layer's cache).
+int apb_rope_cache(void* p, long long ld, int q_col, int k_col, int v_col, const int* row_entry, const int* e_start,
+                   const int* e_len, const int* e_slot, const int* e_pos0, const int* kv_slot, const float* cos_t,
+                   const float* sin_t, int rot, void* kcache, void* vcache, int rows, int HQ, int HK, int G, int D, int E,
+                   int dtype, cudaStream_t s) {
+  if (rows <= 0) return 0;
+  if (HQ <= 0 || HK < 0 || G <= 0 || HK % G || D <= 0 || E <= 0 || rot < 0 || (rot & 1) || rot > D ||
+      (rot && (!cos_t || !sin_t)) || (HK && (!kcache || !vcache || !kv_slot)))
+    return kBadArgument;
+  const ServeEntries e{e_start, e_len, e_slot, e_pos0};
+  const bool vec = dtype == 0 && !((D | E | q_col | (HK ? k_col | v_col : 0)) & 7) && !(ld & 7) &&
+                   !((reinterpret_cast<uintptr_t>(p) | reinterpret_cast<uintptr_t>(kcache) | reinterpret_cast<uintptr_t>(vcache)) & 15);
+  const int V = vec ? 8 : 2;
+  const int du = (D + V - 1) / V, eu = (E + V - 1) / V;
+  const long long n = static_cast<long long>(rows) * (static_cast<long long>(HQ + HK) * du + (HK ? G * eu : 0));
+  const int grid = static_cast<int>((n + 255) / 256);
+#define APB_ROPE(TT, VV)                                                                                              \
+  return static_cast<int>(launch_kernel(rope_cache_kernel<TT, VV>, dim3(grid), dim3(256), 0, s, static_cast<TT*>(p), ld, \
+                                        q_col, k_col, v_col, row_entry, e, kv_slot, cos_t, sin_t, rot,                \
+                                        static_cast<TT*>(kcache), static_cast<TT*>(vcache), rows, HQ, HK, G, D, E))
+  if (vec) APB_ROPE(__nv_bfloat16, 8);
+  APB_SERVE_DTYPE(dtype, APB_ROPE(T, 2));
+#undef APB_ROPE
 }
 
 int apb_serve_commit(const int* tokens, const int* e_start, const int* e_len, const int* e_slot, const int* e_pos0,

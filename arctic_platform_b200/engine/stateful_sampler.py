@@ -4,8 +4,9 @@
 allocator, slots, sampling kernels, CUDA-graph decode loop, ``generate`` -- with the layers and their memory supplied by
 the model through a small protocol (``models/registry.py`` lists the architectures):
 
-* ``model.cache_layout()``       what each layer run keeps per sequence: paged K/V with its own head sizes, an fp32
-                                 recurrent state, the history of a short convolution (any of them may be absent);
+* ``model.cache_layout()``       what each layer run keeps per sequence: paged K/V with its own head sizes (or the run
+                                 whose pages it reads), an fp32 recurrent state, the history of a short convolution (any
+                                 of them may be absent);
 * ``model.prepare_serving(n)``   tables for ``n`` positions;
 * ``model.serve_rows(batch, cache)``   one pass over a ragged :class:`~arctic_platform_b200.ops.serving.StepBatch`,
                                  reading and advancing caches and states; the same code for prompts, portions, decoded
@@ -45,6 +46,12 @@ class StateCache:
         f32 = dict(device=device, dtype=torch.float32)
         for run in layout:
             kv, st, cv = run.get("kv"), run.get("state"), run.get("conv")
+            if "kv_from" in run:                              # reads the pages an earlier run writes
+                self.k.append(self.k[run["kv_from"]])
+                self.v.append(self.v[run["kv_from"]])
+                self.state.append(None)
+                self.conv.append(None)
+                continue
             # zero-filled: the unwritten tail of a last page is multiplied by weight 0 and must be finite
             self.k.append(torch.zeros((pages, kv[0], PAGE, kv[1]), device=device, dtype=dtype) if kv else None)
             self.v.append(torch.zeros((pages, kv[0], PAGE, kv[2]), device=device, dtype=dtype) if kv else None)
@@ -54,7 +61,7 @@ class StateCache:
         self.parity = torch.zeros(slots, device=device, dtype=torch.int32)    # valid half of double-buffered state
 
     def _paged(self):
-        return [t for t in self.k + self.v if t is not None]
+        return list({id(t): t for t in self.k + self.v if t is not None}.values())
 
     def _slotted(self):
         return [t for t in self.state + self.conv if t is not None] + [self.prev, self.parity]

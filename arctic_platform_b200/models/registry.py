@@ -17,6 +17,7 @@ def register_architecture(name: str, module: str, config_class: str, model_class
 
 
 register_architecture("Reninex", "arctic_platform_b200.models.reninex", "ReninexConfig", "ReninexLM")
+register_architecture("Rigulorn", "arctic_platform_b200.models.rigulorn", "RigulornConfig", "RigulornLM")
 
 
 def architectures() -> Tuple[str, ...]:

@@ -2,8 +2,8 @@
 
 A step advances several sequences at once, each by its own run of new tokens: a portion of a prompt of any length, or
 one decoded token.  :class:`StepBatch` is the device-side description of such a step; the functions below launch the
-kernels of ``serve_layers.cu``, ``serve_attention.cu``, ``serve_attention_tc.cu``, ``retention.cu`` and
-``gemm_simt.cu`` on it.  They take bf16 or fp32 activations; the residual stream and all carried state are fp32.
+kernels of ``serve_*.cu``, ``retention*.cu``, ``ssm*.cu`` and ``gemm_simt.cu`` on it.  They take bf16 or fp32 activations;
+the residual streams and all carried state are fp32.
 """
 from __future__ import annotations
 
@@ -28,11 +28,19 @@ def _fn(name: str):
         c = ctypes
         vp, i, ll, f = c.c_void_p, c.c_int, c.c_longlong, c.c_float
         sigs = {
-            "apb_embed_hash": [vp] * 9 + [ll, ll, ll, i, i, vp, vp, ll, vp, i, vp, i, i, vp],
+            "apb_embed_hash": [vp] * 9 + [ll, ll, ll, i, i, f, i, vp, vp, ll, vp, i, vp, i, i, vp],
             "apb_loop_begin": [vp, vp, i, i, vp, ll, i, vp],
             "apb_norm_conv": [vp] * 13 + [i, i, i, f, i, vp],
-            "apb_gain_norm_rows": [vp, vp, vp, vp, i, i, f, i, vp],
+            "apb_gain_norm_rows": [vp, vp, vp, i, vp, i, i, f, i, vp],
             "apb_qk_norm_cache": [vp, ll, i, i, i, vp, vp, vp, i, i, i, i, i, f, i, vp],
+            "apb_rope_cache": [vp, ll, i, i, i] + [vp] * 8 + [i, vp, vp] + [i] * 7 + [vp],
+            "apb_stream_step": [vp] * 7 + [i] * 5 + [f, i, vp],
+            "apb_softmax_attn": [vp, ll] + [vp] * 6 + [i, vp, vp, vp, ll] + [i] * 5 + [f, f, i, i, vp, f, f, i, vp],
+            "apb_softmax_attn_mma": [vp, ll] + [vp] * 4 + [i, vp, i, vp, vp, vp, ll, vp] + [i] * 7 + [f, f, i, i, vp, f, f, vp],
+            "apb_softmax_attn_tc": [vp, ll, i, vp, i, vp, i, vp, vp, i, vp, ll, i, i, i, i, f, f, vp, f, f, vp],
+            "apb_ssm": [vp, ll, i, i, vp, vp, i] + [vp] * 6 + [ll] + [vp] * 7 + [i, vp] + [i] * 8 + [vp],
+            "apb_ssm_mma": [vp, ll] + [vp] * 9 + [i, vp, vp, vp] + [i] * 5 + [vp],
+            "apb_ssm_out": [vp, vp, ll, vp, vp, ll, i, i, i, f, i, vp],
             "apb_serve_commit": [vp] * 5 + [i, vp, vp, vp],
             "apb_sigmoid_attn": [vp, ll, vp, vp, vp, vp, vp, vp, i, vp, vp, vp, vp, ll, i, i, i, i, i, f, f, i, vp],
             "apb_sigmoid_attn_mma": [vp, ll, vp, vp, vp, vp, i, vp, i, vp, vp, vp, vp, ll, vp] + [i] * 7 + [f, f, vp],
@@ -40,7 +48,8 @@ def _fn(name: str):
             "apb_retention": [vp, ll, i, i, i, i, vp, vp, i, vp, f, vp, vp, vp, ll, f, f, vp, vp, vp, vp, vp] + [i] * 8 + [vp],
             "apb_retention_mma": [vp, ll, i, i, i, vp, vp, i, vp, f] + [vp] * 7 + [i, vp, vp, i, vp, vp, i, i, i, i, vp],
             "apb_retention_out": [vp, ll, i, vp, vp, ll, f, f, vp, vp, vp, vp, vp, i, i, i, i, vp],
-            "apb_gemm_simt": [vp, vp, vp, i, i, i, ll, ll, ll, i, vp, vp, ll, i, vp],
+            "apb_gemm_simt": [vp, vp, vp, i, i, i, ll, ll, ll, i, vp, vp, ll, f, i, vp],
+            "apb_gemm_bf16_glu": [vp, vp, i, i, i, ll, ll, i, f, vp, ll, vp],
         }
         _FN[name] = _lib.declare(name, sigs[name])
     return _FN[name]
@@ -139,13 +148,14 @@ class StepBatch:
 
 # --------------------------------------------------------------------------------------------- embedding and loop input
 def embed(b: StepBatch, table: torch.Tensor, bigram: Optional[torch.Tensor], hash_spec: Optional[Tuple[int, int, int]],
-          prev: torch.Tensor, x: torch.Tensor, x0: Optional[torch.Tensor] = None) -> None:
-    """``x [rows, W]`` fp32 = token rows + hashed bigram rows (``hash_spec`` = buckets, multiplier of the previous and
-    of the current token); ``x0`` receives them in the activation type.  Also fills ``b.kv_slot``."""
+          prev: torch.Tensor, x: torch.Tensor, x0: Optional[torch.Tensor] = None, scale: float = 1.0) -> None:
+    """``x [rows, W]`` fp32 = (token rows + hashed bigram rows) * ``scale`` (``hash_spec`` = buckets, multiplier of the
+    previous and of the current token); ``x [rows, streams, W]`` receives them once per stream, ``x0`` in the activation
+    type.  Also fills ``b.kv_slot``."""
     V, W = table.shape
     buckets, mp, mc = hash_spec or (0, 0, 0)
     _call("apb_embed_hash", _lib.ptr(b.tokens), _lib.ptr(b.row_entry), *b.entry_ptrs(), _lib.ptr(prev), _lib.ptr(table),
-          _lib.ptr(bigram), buckets, mp, mc, V, W, _lib.ptr(x), _lib.ptr(x0), 0 if x0 is None else x0.stride(0),
+          _lib.ptr(bigram), buckets, mp, mc, V, W, float(scale), x.shape[1] if x.dim() == 3 else 1, _lib.ptr(x), _lib.ptr(x0), 0 if x0 is None else x0.stride(0),
           _lib.ptr(b.page_table), b.page_table.stride(0), _lib.ptr(b.kv_slot), b.rows, dtype_code(table.dtype))
 
 
@@ -174,7 +184,7 @@ def norm_conv(b: StepBatch, x: torch.Tensor, gain: torch.Tensor, w1: Optional[to
 def gain_norm_rows(x: torch.Tensor, rows: Optional[torch.Tensor], gain: torch.Tensor, eps: float) -> torch.Tensor:
     n = x.shape[0] if rows is None else rows.shape[0]
     out = torch.empty((n, x.shape[1]), device=x.device, dtype=gain.dtype)
-    _call("apb_gain_norm_rows", _lib.ptr(x), _lib.ptr(rows), _lib.ptr(gain), _lib.ptr(out), n, x.shape[1], float(eps),
+    _call("apb_gain_norm_rows", _lib.ptr(x), _lib.ptr(rows), _lib.ptr(gain), int(gain.numel() > 1), _lib.ptr(out), n, x.shape[1], float(eps),
           dtype_code(gain.dtype))
     return out
 
@@ -186,6 +196,32 @@ def qk_norm_cache(b: StepBatch, p: torch.Tensor, cols: Tuple[int, int, int], kca
     G, D, E = kcache.shape[1], kcache.shape[3], vcache.shape[3]
     _call("apb_qk_norm_cache", _lib.ptr(p), p.stride(0), *cols, _lib.ptr(b.kv_slot), _lib.ptr(kcache), _lib.ptr(vcache),
           b.rows, heads, G, D, E, float(eps), dtype_code(p.dtype))
+
+
+def rope_cache(b: StepBatch, p: torch.Tensor, cols: Tuple[int, ...], rope: Tuple[torch.Tensor, torch.Tensor], rot_dims: int,
+               q_heads: int, dim: int, kcache: torch.Tensor, vcache: torch.Tensor, write: bool = True) -> None:
+    """Rotates the first ``rot_dims`` of every ``dim`` columns of the q and k columns of ``p`` (neighbouring pairs); q in
+    place, k and v into the page cache (``[pages, G, PAGE, maps * dim]`` and ``[pages, G, PAGE, E]``).  ``write`` False: q only."""
+    G, E = kcache.shape[1], vcache.shape[3]
+    q_col, k_col, v_col = (*cols, 0, 0)[:3]
+    _call("apb_rope_cache", _lib.ptr(p), p.stride(0), q_col, k_col, v_col, _lib.ptr(b.row_entry), *b.entry_ptrs(),
+          _lib.ptr(b.kv_slot), _lib.ptr(rope[0]), _lib.ptr(rope[1]), rot_dims, _lib.ptr(kcache), _lib.ptr(vcache), b.rows,
+          q_heads, G * (kcache.shape[3] // dim) if write else 0, G, dim, E, dtype_code(p.dtype))
+
+
+# --------------------------------------------------------------------------------------------- parallel residual streams
+def stream_step(x: torch.Tensor, y: Optional[torch.Tensor], mix: Optional[torch.Tensor], out_w: Optional[torch.Tensor],
+                in_w: Optional[torch.Tensor], gain: Optional[torch.Tensor], eps: float, *, write: bool = True,
+                clear: bool = False, dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+    """One pass over the streams ``x [rows, S, W]`` (fp32): ``x_t <- sum_s mix[s, t] x_s + out_w[t] y`` (``y`` None: left
+    alone), then ``u = sum_t in_w[t] x_t`` (None: the plain sum) and ``u / rms(u) * gain`` in the activation type -- without
+    ``gain`` the fp32 ``u``.  ``write`` False leaves ``x`` as it was; ``clear`` zeroes ``y`` after reading it."""
+    T, S, W = x.shape
+    dt = gain.dtype if gain is not None else (dtype or (in_w if in_w is not None else mix).dtype)
+    h = torch.empty((T, W), device=x.device, dtype=dt if gain is not None else torch.float32)
+    _call("apb_stream_step", _lib.ptr(x), _lib.ptr(y), _lib.ptr(mix), _lib.ptr(out_w), _lib.ptr(in_w), _lib.ptr(gain),
+          _lib.ptr(h), T, W, S, int(write), int(clear), float(eps), dtype_code(dt))
+    return h
 
 
 def commit(b: StepBatch, prev: torch.Tensor, parity: torch.Tensor) -> None:
@@ -216,14 +252,35 @@ def linear(a: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None,
     return out
 
 
-def gate_up_gelu(x: torch.Tensor, w_gu: torch.Tensor, out: torch.Tensor) -> None:
-    """``out [M, ff]`` (may be a column slice) = gelu_tanh(gate) * up; gate and up rows interleaved in ``w_gu``."""
+def accumulates(rows: int, width: int, device) -> bool:
+    """Whether :func:`project` may add parts of its products into the output, which then has to start as zeros."""
+    return 2 * ((rows + 127) // 128) * ((width + 127) // 128) <= _sm_count(device)
+
+
+def project(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
+    """``out [M, N]`` fp32 = ``a @ w^T``; few rows: cut along K over the SMs and added onto ``out``, which holds zeros."""
+    linear(a, w, out, accumulate=accumulates(a.shape[0], w.shape[0], a.device) and not _simt(a, w, out))
+
+
+def gate_up(x: torch.Tensor, w_gu: torch.Tensor, out: torch.Tensor, epi: int, limit: float = 0.0) -> None:
+    """``out [M, ff]`` (may be a column slice) = the GLU ``epi`` of the products; gate and up rows interleaved in ``w_gu``."""
     M, K = x.shape
     N = w_gu.shape[0]
     if _simt(x, w_gu, out) or N % 16:
-        _gemm_simt(x, w_gu, None, gemm.EPI_GEGLU, out2=out)
+        _gemm_simt(x, w_gu, None, epi, out2=out, limit=limit)
     else:
-        gemm.gemm_raw(x, w_gu, None, M=M, N=N, K=K, epi=gemm.EPI_GEGLU, out2=out)
+        _call("apb_gemm_bf16_glu", _lib.ptr(x), _lib.ptr(w_gu), M, N, K, x.stride(0), w_gu.stride(0), epi, float(limit),
+              _lib.ptr(out), out.stride(0))
+
+
+def gate_up_gelu(x: torch.Tensor, w_gu: torch.Tensor, out: torch.Tensor) -> None:
+    """gelu_tanh(gate) * up."""
+    gate_up(x, w_gu, out, gemm.EPI_GEGLU)
+
+
+def gate_up_clamped(x: torch.Tensor, w_gu: torch.Tensor, out: torch.Tensor, limit: float) -> None:
+    """g sigmoid(1.702 g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit)."""
+    gate_up(x, w_gu, out, gemm.EPI_CLAMP_GLU, limit)
 
 
 _SMS: Dict[int, int] = {}
@@ -242,10 +299,10 @@ def _simt(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> bool:
             or bool((a.data_ptr() | w.data_ptr() | out.data_ptr()) & 15))
 
 
-def _gemm_simt(a, w, out, epi, out2=None) -> None:
+def _gemm_simt(a, w, out, epi, out2=None, limit=0.0) -> None:
     _call("apb_gemm_simt", _lib.ptr(a), _lib.ptr(w), _lib.ptr(out), a.shape[0], w.shape[0], a.shape[1], a.stride(0),
           w.stride(0), 0 if out is None else out.stride(0), epi, None, _lib.ptr(out2),
-          0 if out2 is None else out2.stride(0), dtype_code(a.dtype))
+          0 if out2 is None else out2.stride(0), float(limit), dtype_code(a.dtype))
 
 
 # --------------------------------------------------------------------------------------------- sequence mixers
@@ -319,6 +376,85 @@ def sigmoid_attention(b: StepBatch, q: torch.Tensor, heads: int, kcache: torch.T
               _lib.ptr(bias), _lib.ptr(out), out.stride(0), heads, G, D, E, float(scale), float(out_scale))
 
 
+@dataclass(frozen=True)
+class SoftmaxSpec:
+    """Softmax attention over the page cache: ``score = scale q.k``, capped to ``cap tanh(score / cap)`` (0: no cap), chunks of
+    ``chunk`` positions (0: none).  ``maps`` 2: differential attention, ``out = o / rms(o) * post_scale`` with
+    ``o = a1 - lambda a2``."""
+    scale: float
+    cap: float = 0.0
+    chunk: int = 0
+    maps: int = 1
+    post_scale: float = 1.0
+    eps: float = 1e-5
+
+
+MAX_FIXED_CAP = 64.0    # the tcgen05 kernel's bound on the score cap
+
+
+def chunk_tiles(host: np.ndarray, heads: int, kv_heads: int, min_len: int, chunk: int, tile: int = 128) -> np.ndarray:
+    """Work items of the tcgen05 softmax kernel for the entries of at least ``min_len`` rows, longest key range first:
+    ``[n, 8]`` int32 = entry, KV head, head, first row, valid rows, position of the first row, first key of the walk (a
+    multiple of ``PAGE``), first visible key.  No tile leaves its first row's chunk."""
+    parts = []
+    for en, (start, n, _slot, pos0) in enumerate(host.tolist()):
+        if n < min_len:
+            continue
+        at, end = [pos0], pos0 + n
+        if chunk:
+            at += range((pos0 // chunk + 1) * chunk, end, chunk)
+        at = np.array(at, dtype=np.int64)                                       # first positions of the runs
+        runs = np.diff(np.append(at, end))
+        per = -(-runs // tile)
+        base = np.repeat(at, per)
+        pos = base + (np.arange(per.sum()) - np.repeat(np.cumsum(per) - per, per)) * tile
+        valid = np.minimum(tile, np.repeat(at + runs, per) - pos)
+        first = pos // chunk * chunk if chunk else np.zeros_like(pos)
+        it = np.empty((heads, len(pos), 8), dtype=np.int64)
+        h = np.arange(heads)[:, None]
+        it[..., 0], it[..., 1], it[..., 2] = en, h // (heads // kv_heads), h
+        it[..., 3], it[..., 4], it[..., 5] = start + pos - pos0, valid, pos
+        it[..., 6], it[..., 7] = first // PAGE * PAGE, first
+        parts.append(it.reshape(-1, 8))
+    if not parts:
+        return np.zeros((0, 8), dtype=np.int32)
+    work = np.concatenate(parts)
+    return np.ascontiguousarray(work[np.argsort(work[:, 6] - work[:, 5] - work[:, 4], kind="stable")], dtype=np.int32)
+
+
+def softmax_attention(b: StepBatch, q: torch.Tensor, heads: int, kcache: torch.Tensor, vcache: torch.Tensor,
+                      spec: SoftmaxSpec, lam: Optional[torch.Tensor], out: torch.Tensor) -> None:
+    """``q [rows, heads * maps * D]`` (column slice, rotated) over the entries' pages -> ``out [rows, heads * E]`` (column
+    slice).  bf16 with head sizes that are multiples of 8 runs on tensor cores; fp32 and odd sizes on CUDA cores."""
+    G, DK, E = kcache.shape[1], kcache.shape[3], vcache.shape[3]
+    D = DK // spec.maps
+    tail = (float(spec.scale), float(spec.cap), spec.chunk, spec.maps, _lib.ptr(lam), float(spec.post_scale), float(spec.eps))
+    aligned = not (D % 8 or E % 8 or q.stride(0) % 8 or out.stride(0) % 8 or (q.data_ptr() | out.data_ptr()) & 15)
+    if q.dtype != torch.bfloat16 or not aligned or max(DK, E) > 256:
+        _call("apb_softmax_attn", _lib.ptr(q), q.stride(0), _lib.ptr(b.row_entry), *b.entry_ptrs(), _lib.ptr(b.page_table),
+              b.page_table.stride(0), _lib.ptr(kcache), _lib.ptr(vcache), _lib.ptr(out), out.stride(0), b.rows, heads, G, D, E,
+              *tail, dtype_code(q.dtype))
+        return
+    tc = spec.maps == 2 and D % 16 == 0 and D <= 64 and E <= 128 and 0 < spec.cap <= MAX_FIXED_CAP
+    lens = np.ones(1, dtype=np.int64) if b.host is None else b.host[:, 1]
+    limit = SHORT_ROWS if tc else int(lens.max())
+    short = lens[lens <= limit]
+    if len(short):
+        longest = int(short.max())
+        passes = min(256, (longest * (heads // G) * spec.maps + 15) // 16)
+        splits = max(1, min(MAX_SPLITS, 2 * _sm_count(q.device) // (b.n_entries * G * passes)))
+        part = torch.empty((b.n_entries, longest, heads, spec.maps, splits, E + 2), device=q.device, dtype=torch.float32) \
+            if splits > 1 else None
+        _call("apb_softmax_attn_mma", _lib.ptr(q), q.stride(0), *b.entry_ptrs(), b.n_entries, _lib.ptr(b.page_table),
+              b.page_table.stride(0), _lib.ptr(kcache), _lib.ptr(vcache), _lib.ptr(out), out.stride(0), _lib.ptr(part), heads, G,
+              D, E, 1, longest, splits, *tail)
+    if len(short) < len(lens):
+        work = b.table(("softmax", heads, G, spec.chunk), lambda: chunk_tiles(b.host, heads, G, limit + 1, spec.chunk))
+        _call("apb_softmax_attn_tc", _lib.ptr(q), q.stride(0), b.rows, _lib.ptr(work), work.shape[0], _lib.ptr(b.page_table),
+              b.page_table.stride(0), _lib.ptr(kcache), _lib.ptr(vcache), kcache.shape[0], _lib.ptr(out), out.stride(0), heads,
+              G, D, E, *tail[:2], *tail[4:])
+
+
 MIN_SEGMENT = 256       # tokens; a multiple of the kernel's chunk
 
 
@@ -384,3 +520,54 @@ def retention(b: StepBatch, p: torch.Tensor, cols: Tuple[int, int, int, int], ro
               b.rows, H, D, E)
         _call("apb_retention_out", _lib.ptr(p), p.stride(0), cols[3], _lib.ptr(scratch), _lib.ptr(out), out.stride(0),
               float(out_scale), float(eps), _lib.ptr(b.row_entry), *b.entry_ptrs(), b.rows, H, E, dtype_code(p.dtype))
+
+
+@dataclass(frozen=True)
+class SsmWeights:
+    """Parameters of a state-space mixer besides its projections: ``conv [taps, channels]``, ``conv_bias [channels]``, and per
+    head ``dt_bias``, ``a_log``, ``skip``."""
+    conv: torch.Tensor
+    conv_bias: torch.Tensor
+    dt_bias: torch.Tensor
+    a_log: torch.Tensor
+    skip: torch.Tensor
+
+
+def state_space(b: StepBatch, p: torch.Tensor, xbc_col: int, dt_col: int, w: SsmWeights, groups: int, hist: Optional[torch.Tensor],
+                parity: torch.Tensor, state: torch.Tensor) -> torch.Tensor:
+    """Convolution, step sizes and recurrence over the columns ``[x | B | C]`` and ``dt`` of ``p`` with the carried
+    ``state [slots, H, N, E]`` and convolution history ``hist [slots, 2, taps - 1, channels]`` (fp32); ``y [rows, H * E]`` fp32,
+    before the gate."""
+    _, H, N, E = state.shape
+    taps, channels = w.conv.shape
+    y = torch.empty((b.rows, H * E), device=p.device, dtype=torch.float32)
+    ldx = (channels + 7) // 8 * 8
+    xbc = torch.empty((b.rows, ldx), device=p.device, dtype=p.dtype) if b.longer else None
+    steps = torch.empty((b.rows, H, 2), device=p.device, dtype=torch.float32) if b.longer else None
+    mma = b.longer and p.dtype == torch.bfloat16 and N % 8 == 0 and E % 8 == 0 and N <= 128
+    _call("apb_ssm", _lib.ptr(p), p.stride(0), xbc_col, dt_col, _lib.ptr(w.conv), _lib.ptr(w.conv_bias), taps, _lib.ptr(hist),
+          _lib.ptr(parity), _lib.ptr(w.dt_bias), _lib.ptr(w.a_log), _lib.ptr(w.skip), _lib.ptr(xbc), ldx, _lib.ptr(steps),
+          _lib.ptr(state), _lib.ptr(y), *b.entry_ptrs(), b.n_entries, _lib.ptr(b.tiles) if b.longer else None,
+          b.tiles.shape[0] if b.longer else 0, H, E, groups, N, int(b.one_token), int(b.longer and not mma), dtype_code(p.dtype))
+    if mma:
+        slices = H * ((E + 63) // 64)
+        key = ("segments", slices)
+        if key not in b.host_tables:
+            b.host_tables[key] = segment_plan(b.host, slices, 2 * _sm_count(p.device))
+        plan = b.host_tables[key]
+        seg = b.table(key + ("seg",), lambda: plan["seg"])
+        chains = b.table(key + ("chains",), lambda: plan["chains"]) if len(plan["chains"]) else None
+        f32 = dict(device=p.device, dtype=torch.float32)
+        carry = torch.empty((plan["states"], H, N, E), **f32) if plan["states"] else None
+        decay = torch.empty((len(plan["seg"]), H), **f32) if plan["states"] else None
+        _call("apb_ssm_mma", _lib.ptr(xbc), ldx, _lib.ptr(steps), _lib.ptr(w.skip), _lib.ptr(state), _lib.ptr(y),
+              *b.entry_ptrs(), _lib.ptr(seg), len(plan["seg"]), _lib.ptr(carry), _lib.ptr(decay), _lib.ptr(chains),
+              len(plan["chains"]), H, E, groups, N)
+    return y
+
+
+def gated_group_norm(y: torch.Tensor, z: torch.Tensor, gain: torch.Tensor, parts: int, eps: float, out: torch.Tensor) -> None:
+    """``out [rows, n]`` (column slice) = ``v / rms(v) * gain`` in ``parts`` equal parts of every row, ``v = y silu(z)``;
+    ``y`` fp32, ``z`` a column slice in the activation type."""
+    _call("apb_ssm_out", _lib.ptr(y), _lib.ptr(z), z.stride(0), _lib.ptr(gain), _lib.ptr(out), out.stride(0), y.shape[0],
+          y.shape[1], parts, float(eps), dtype_code(out.dtype))
