@@ -504,7 +504,7 @@ int apb_softmax_attn_mma(const void* q, long long ldq, const int* e_start, const
   const int passes = static_cast<int>((static_cast<long long>(max_len) * (H / G) * maps + 15) / 16);
   const dim3 grid(n_entries * G, splits, passes < 256 ? passes : 256);
   auto run = [&](auto fn) -> int {
-    if (smem > 48 * 1024) {
+    if (smem > 46 * 1024) {                  // the default limit counts the static arrays too
       const cudaError_t e = cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
       if (e != cudaSuccess) return static_cast<int>(e);
     }

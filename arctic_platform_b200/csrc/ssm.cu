@@ -311,7 +311,7 @@ ssm_out_kernel(const float* __restrict__ y, const T* __restrict__ z, long long l
 template <typename F>
 static int ssm_smem_limit(F fn, size_t bytes) {
   if (bytes > 220 * 1024) return kBadArgument;
-  return bytes <= 48 * 1024 ? 0 : static_cast<int>(cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes)));
+  return bytes <= 46 * 1024 ? 0 : static_cast<int>(cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes)));
 }
 
 }  // namespace apb
