@@ -20,7 +20,7 @@ wall time: when the next timed step would end past it, all ranks stop together (
 line reports the steps actually timed in ``steps`` with the request in ``steps_requested``.
 
     python bench.py [--gpus N --steps K --warmup W]          # N > 1 under torch.distributed.run
-    python bench.py --workload serving                        # stateful architectures beside the dense decoder
+    python bench.py --workload serving                        # stateful architectures beside the closest older model
     python bench.py --impl reference                          # the reference's own stack, if installable
 """
 from __future__ import annotations
@@ -47,8 +47,8 @@ def parse_args():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--workload", default="grpo", choices=["grpo", "serving"],
                     help="grpo: the benchmark step (default); serving: prefill / decode speed and per-kernel roofline "
-                         "fractions of the stateful architectures beside the dense decoder (benchmarks/bench_serving.py)")
-    ap.add_argument("--serving-models", default="reninex-2048,reninex-4096")
+                         "fractions of the stateful architectures beside the closest older model (benchmarks/bench_serving.py)")
+    ap.add_argument("--serving-models", default="reninex-2048,reninex-4096,rigulorn-2048,rigulorn-4096")
     ap.add_argument("--model", default="qwen3-4b")
     ap.add_argument("--prompts-per-gpu", type=int, default=8)
     ap.add_argument("--samples", type=int, default=16)

@@ -1,17 +1,18 @@
-"""Serving speed of a stateful architecture beside the dense decoder of equal layer size.
+"""Serving speed of the stateful architectures beside the closest older model of equal layer size.
 
-    python bench.py --workload serving [--serving-models reninex-2048,reninex-4096]
+    python bench.py --workload serving [--serving-models reninex-2048,rigulorn-2048,...]
     python benchmarks/bench_serving.py [--models ...] [--kernels-only] [--only prefill|decode] [--step NAME] [--iters 20]
 
 For every model (random weights, synthetic prompts) two parts are measured on one GPU:
 
-* kernels: each step of ONE layer on a prefill batch (4 prompts x 2048 tokens) and on a decode batch (128 sequences after
-  2048 tokens), next to the like kernel of a Qwen3-style layer of the same width, heads and feed-forward (for retention:
-  the gated delta rule of the hybrid family at the same heads and sizes).  ``floor_ms`` is the slower of algorithmic bytes
-  over the measured copy bandwidth and FLOPs over the measured bf16 GEMM peak, ``frac`` = floor / time.  CUDA events
-  around every launch, L2 overwritten before it, median over the iterations.
-* engine: prefill and decode tokens/s through ``generate`` of both engines, the dense model with as many layers as the
-  stateful one has layer runs.
+* kernels: each step of ONE layer of every kind on a prefill batch (4 prompts x 2048 tokens) and on a decode batch (128
+  sequences after 2048 tokens), next to the like kernel of the closest model: for Reninex a Qwen3-style layer of the same
+  width, heads and feed-forward (for retention the gated delta rule of the hybrid family at the same heads and sizes); for
+  Rigulorn a Reninex layer whose K/V rows, state and feed-forward have the same size.  ``floor_ms`` is the slower of
+  algorithmic bytes over the measured copy bandwidth and FLOPs over the measured bf16 GEMM peak, ``frac`` = floor / time.
+  CUDA events around every launch, L2 overwritten before it, median over the iterations.
+* engine: prefill and decode tokens/s through ``generate`` of the model, of the dense decoder with as many layers as the
+  model has layer runs and, for Rigulorn, of the Reninex preset of the same width.
 
 Prints one JSON line per measurement.
 """
@@ -68,8 +69,28 @@ def _bf(*shape, std=1.0):
     return (torch.randn(*shape, device="cuda") * std).to(torch.bfloat16)
 
 
+def phase_batch(phase):
+    """``(batch, page tables, sequences, sum over the rows of the keys they see)``."""
+    from arctic_platform_b200.ops import serving
+    n = PREFILL_SEQS if phase == "prefill" else DECODE_SEQS
+    per = SEQ // 16 + 1
+    pages = np.random.default_rng(0).permutation(n * per).astype(np.int32).reshape(n, per)
+    if phase == "prefill":
+        b = serving.StepBatch.build([serving.StepEntry(i, np.arange(SEQ) % 1000, 0, pages[i]) for i in range(n)], "cuda")
+        return b, n, n * per, SEQ * (SEQ + 1) // 2 * n
+    i32 = dict(device="cuda", dtype=torch.int32)
+    one = torch.arange(n, **i32)
+    b = serving.StepBatch(n, n, one.clone(), None, one, torch.ones(n, **i32), one, torch.full((n,), SEQ, **i32),
+                          torch.from_numpy(pages).cuda(), torch.empty(n, **i32))
+    return b, n, n * per, (SEQ + 1) * n
+
+
 def stateful_ops(cfg, phase):
-    """``(name, fn, bytes, flops)`` of the steps of layer 0 on the phase's batch."""
+    """``(name, fn, bytes, flops)`` of the steps of the model's layers on the phase's batch."""
+    return {"Reninex": reninex_ops, "Rigulorn": rigulorn_ops}[cfg.architecture](cfg, phase)
+
+
+def reninex_ops(cfg, phase):
     from arctic_platform_b200.engine.stateful_sampler import StateCache
     from arctic_platform_b200.models.reninex import ReninexLM
     from arctic_platform_b200.ops import serving
@@ -79,21 +100,10 @@ def stateful_ops(cfg, phase):
     model.prepare_serving(SEQ + 8)
     blk, s, W = model.blocks[0], one.layers[0], cfg.hidden_size
     L, R = s.left, s.right
-    n = PREFILL_SEQS if phase == "prefill" else DECODE_SEQS
-    per = SEQ // 16 + 1
-    cache = StateCache(model.cache_layout(), n * per, n, "cuda", torch.bfloat16)
+    b, n, n_pages, keys = phase_batch(phase)
+    cache = StateCache(model.cache_layout(), n_pages, n, "cuda", torch.bfloat16)
     for t in (cache.k[0], cache.v[0]):
         t.normal_()
-    pages = np.random.default_rng(0).permutation(n * per).astype(np.int32).reshape(n, per)
-    if phase == "prefill":
-        b = serving.StepBatch.build([serving.StepEntry(i, np.arange(SEQ) % 1000, 0, pages[i]) for i in range(n)], "cuda")
-        keys = SEQ * (SEQ + 1) // 2 * n
-    else:
-        i32 = dict(device="cuda", dtype=torch.int32)
-        one_ = torch.arange(n, **i32)
-        b = serving.StepBatch(n, n, one_.clone(), None, one_, torch.ones(n, **i32), one_, torch.full((n,), SEQ, **i32),
-                              torch.from_numpy(pages).cuda(), torch.empty(n, **i32))
-        keys = (SEQ + 1) * n
     T = b.rows
     x = torch.randn(T, W, device="cuda")
     serving.embed(b, model.embed, None, None, cache.prev, torch.empty_like(x))
@@ -129,13 +139,103 @@ def stateful_ops(cfg, phase):
     ]
 
 
+def rigulorn_ops(cfg, phase):
+    import dataclasses
+    from arctic_platform_b200.engine.stateful_sampler import StateCache
+    from arctic_platform_b200.models.rigulorn import RigulornLM
+    from arctic_platform_b200.ops import serving
+    attn = next(s for s in cfg.layers if s.attention and s.ff)
+    ssm = next(s for s in cfg.layers if not s.attention)
+    one = dataclasses.replace(cfg, layers=(attn, ssm), vocab_size=1024)
+    model = RigulornLM(one, "cuda", torch.bfloat16).init_weights(0)
+    model.prepare_serving(SEQ + 8)
+    b, n, n_pages, keys = phase_batch(phase)
+    cache = StateCache(model.cache_layout(), n_pages, n, "cuda", torch.bfloat16)
+    for t in (cache.k[0], cache.v[0]):
+        t.normal_()
+    T, W, S, A, M = b.rows, cfg.hidden_size, cfg.streams, attn.mixer, ssm.mixer
+    blk, mam = model.blocks
+    x = torch.empty(T, S, W, device="cuda")
+    serving.embed(b, model.embed, None, None, cache.prev, x)
+    clear = serving.accumulates(T, W, x.device)
+    y, h = torch.zeros(T, W, device="cuda"), _bf(T, W)
+    p, pm = serving.linear(h, blk.mixer.w_in), serving.linear(h, mam.mixer.w_in)
+    rope = model._rope[A.rot_dims, A.rot_base]
+    ao, mo, fo = _bf(T, A.heads * A.vdim), _bf(T, M.inner), _bf(T, attn.ff)
+    c, cm, mx = blk.mixer.in_cols, mam.mixer.in_cols, mam.mixer
+    w = serving.SsmWeights(mx.conv, mx.conv_bias, mx.dt_bias, mx.a_log, mx.skip)
+    kv_row = A.kv_heads * (2 * A.dim + A.vdim) * 2
+    ctx = T if phase == "prefill" else keys
+    state = n * M.inner * M.state * 4
+    gemm = lambda N, K: (2 * (T * K + N * K + T * N), 2 * T * N * K)
+    out = lambda K: (2 * (T * K + K * W) + (8 if clear else 4) * T * W, 2 * T * W * K)
+
+    def recurrent():
+        s = serving.state_space(b, pm, cm["xbc"][0], cm["dt"][0], w, M.groups, cache.conv[1], cache.parity, cache.state[1])
+        serving.gated_group_norm(s, pm, mx.gain, M.norm_groups, cfg.norm_eps, mo)
+
+    s1 = blk.sub1
+    return [
+        ("stream update + norm", lambda: serving.stream_step(x, y, s1.hc_mix, s1.hc_out, s1.hc_in, s1.norm, cfg.norm_eps, clear=clear),
+         T * W * (8 * S + 4 + 2 + (4 if clear else 0)), 0),
+        ("attention input projections (GEMM)", lambda: serving.linear(h, blk.mixer.w_in, p), *gemm(p.shape[1], W)),
+        ("rotation + cache write", lambda: serving.rope_cache(b, p, tuple(c[m][0] for m in c), rope, A.rot_dims, 2 * A.heads, A.dim,
+                                                             cache.k[0], cache.v[0]),
+         2 * T * (2 * A.heads * 2 * A.dim) + 2 * T * kv_row, 0),
+        ("attention", lambda: serving.softmax_attention(b, p, A.heads, cache.k[0], cache.v[0], blk.mixer.spec, blk.mixer.lam, ao),
+         ctx * kv_row + 2 * T * A.heads * (2 * A.dim + A.vdim), 2 * keys * A.heads * (2 * A.dim + 2 * A.vdim)),
+        ("attention output projection (GEMM)", lambda: serving.project(ao, blk.mixer.w_out, y), *out(ao.shape[1])),
+        ("gate/up + clamped GLU (GEMM)", lambda: serving.gate_up_clamped(h, blk.mlp.w_gu, fo, attn.limit),
+         2 * (T * W + 2 * attn.ff * W + T * attn.ff), 4 * T * W * attn.ff),
+        ("down projection (GEMM)", lambda: serving.project(fo, blk.mlp.w_down, y), *out(attn.ff)),
+        ("state-space input projections (GEMM)", lambda: serving.linear(h, mx.w_in, pm), *gemm(pm.shape[1], W)),
+        ("recurrent mixer", recurrent,
+         2 * T * (2 * M.inner + 2 * M.groups * M.state + M.heads + M.inner) + state * (2 if phase == "decode" else 1),
+         T * M.heads * (2 * 64 * (M.state + M.vdim) / 2 + 4 * M.state * M.vdim)),
+        ("state-space output projection (GEMM)", lambda: serving.project(mo, mx.w_out, y), *out(M.inner)),
+    ]
+
+
+# step of a Rigulorn layer -> the like step of the Reninex layer
+RIGULORN_LIKE = {
+    "stream update + norm": "norm + 2 input convolutions", "attention input projections (GEMM)": "input projections (GEMM)",
+    "rotation + cache write": "q/k norm + cache write", "attention": "attention",
+    "attention output projection (GEMM)": "output projections (GEMM, += fp32)",
+    "gate/up + clamped GLU (GEMM)": "gate/up + GELU (GEMM)", "down projection (GEMM)": "output projections (GEMM, += fp32)",
+    "state-space input projections (GEMM)": "input projections (GEMM)", "recurrent mixer": "recurrent mixer",
+    "state-space output projection (GEMM)": "output projections (GEMM, += fp32)",
+}
+
+
+def reninex_like(cfg):
+    """The Reninex model whose layer has the K/V rows, state and feed-forward of the Rigulorn model's layers."""
+    from arctic_platform_b200.models.reninex import ReninexConfig, _uniform
+    a = next(s for s in cfg.layers if s.attention and s.ff)
+    A, M = a.mixer, next(s for s in cfg.layers if not s.attention).mixer
+    layers = _uniform(1, (A.heads, A.kv_heads, 2 * A.dim, A.vdim), (M.heads, M.state, M.vdim, M.state), a.ff)
+    return ReninexConfig(cfg.vocab_size, cfg.hidden_size, layers, cfg.norm_eps, 4, None, None, f"reninex-like-{cfg.hidden_size}")
+
+
+def like_ops(cfg, phase):
+    """Steps of the closest older model, keyed by the names of ``stateful_ops``: ``name -> (fn, bytes, flops)``."""
+    if cfg.architecture != "Rigulorn":
+        return dense_ops(cfg, phase)
+    ops = {name: rest for name, *rest in reninex_ops(reninex_like(cfg), phase)}
+    return {mine: ops[theirs] for mine, theirs in RIGULORN_LIKE.items()}
+
+
 def dense_config(cfg):
-    """The Qwen3-style decoder with the width, heads and feed-forward of the model's first layer, one layer per run."""
+    """The Qwen3-style decoder with the width, heads and feed-forward of the model's attention layers, one layer per run."""
     from arctic_platform_b200.models.config import DecoderConfig
-    s = cfg.layers[0]
+    if cfg.architecture == "Rigulorn":
+        s = next(s for s in cfg.layers if s.attention and s.ff)
+        heads, kv_heads, dim = s.mixer.heads, s.mixer.kv_heads, 2 * s.mixer.dim
+    else:
+        s = cfg.layers[0]
+        heads, kv_heads, dim = s.left.heads, s.left.kv_heads, s.left.dim
     return DecoderConfig(vocab_size=cfg.vocab_size, hidden_size=cfg.hidden_size, intermediate_size=s.ff,
-                         num_layers=len(cfg.layer_runs()), num_heads=s.left.heads, num_kv_heads=s.left.kv_heads,
-                         head_dim=s.left.dim, tie_word_embeddings=False, name=f"dense-{cfg.hidden_size}")
+                         num_layers=len(cfg.layer_runs()), num_heads=heads, num_kv_heads=kv_heads, head_dim=dim,
+                         tie_word_embeddings=False, name=f"dense-{cfg.hidden_size}")
 
 
 def dense_ops(cfg, phase):
@@ -240,7 +340,7 @@ def bench_kernels(name, cfg, phase, iters, step=None, compare=True):
         floor = max(nbytes / bw, flops / peak) * 1e3
         return ms, floor, floor / ms
 
-    like = {k: measured(*v) for k, v in dense_ops(cfg, phase).items() if k != "_keep" and (step is None or step in k)} \
+    like = {k: measured(*v) for k, v in like_ops(cfg, phase).items() if k != "_keep" and (step is None or step in k)} \
         if compare else {}
     torch.cuda.empty_cache()
     for op, fn, nbytes, flops in stateful_ops(cfg, phase):
@@ -257,16 +357,20 @@ def bench_kernels(name, cfg, phase, iters, step=None, compare=True):
 def bench_engine(name, cfg, seqs, new_tokens):
     from arctic_platform_b200.engine.sampler import SamplerEngine
     from arctic_platform_b200.engine.stateful_sampler import StatefulSampler
-    from arctic_platform_b200.models.decoder import DecoderLM
-    from arctic_platform_b200.models.reninex import ReninexLM
+    from arctic_platform_b200.models import registry
+    from arctic_platform_b200.models.config import resolve_config
     prompts = [np.random.default_rng(i).integers(1, cfg.vocab_size, SEQ).tolist() for i in range(seqs)]
     limits = dict(kv_cache_tokens=seqs * (SEQ + new_tokens + 32), max_batch=seqs, max_seq_len=SEQ + new_tokens + 16)
     d = dense_config(cfg)
-    for label, make in (
-            (name, lambda: StatefulSampler(cfg, "cuda", model=ReninexLM(cfg, "cuda", torch.bfloat16).init_weights(0), **limits)),
-            (d.name, lambda: SamplerEngine(d, "cuda", model=DecoderLM(d, "cuda", torch.bfloat16).init_weights(0), cascade=False,
-                                           **limits))):
-        eng = make()
+    models = [cfg, d]
+    if cfg.architecture == "Rigulorn" and f"reninex-{cfg.hidden_size}" in registry.presets():
+        models.append(resolve_config(f"reninex-{cfg.hidden_size}"))
+    for m in models:
+        model = registry.new_model(m, "cuda", torch.bfloat16).init_weights(0)
+        if registry.is_stateful(m):
+            eng = StatefulSampler(m, "cuda", model=model, **limits)
+        else:
+            eng = SamplerEngine(m, "cuda", model=model, cascade=False, **limits)
 
         def run(n):
             torch.cuda.synchronize()
@@ -280,16 +384,15 @@ def bench_engine(name, cfg, seqs, new_tokens):
         pre = statistics.median(run(1) for _ in range(3))
         full = statistics.median(run(new_tokens) for _ in range(3))
         params = sum(p.numel() for p in eng.model.parameters())
-        fl = cfg if label == name else d
         print(json.dumps({
-            "model": label, "engine": type(eng).__name__, "sequences": seqs, "prompt_len": SEQ, "new_tokens": new_tokens,
-            "parameters": params, "layer_runs": len(cfg.layer_runs()),
+            "model": m.name, "engine": type(eng).__name__, "sequences": seqs, "prompt_len": SEQ, "new_tokens": new_tokens,
+            "parameters": params, "layer_runs": len(m.layer_runs()) if registry.is_stateful(m) else m.num_layers,
             "prefill_tokens_per_s": round(seqs * SEQ / pre), "decode_tokens_per_s": round(seqs * (new_tokens - 1) / (full - pre)),
             "decode_ms_per_step": round((full - pre) * 1e3 / (new_tokens - 1), 3),
-            "gflop_per_token": round(fl.flops_per_token(SEQ, backward=False) / 1e9, 3),
-            "prefill_tflops": round(seqs * SEQ / pre * (fl.flops_per_token(SEQ, backward=False) - 2.0 * cfg.vocab_size * cfg.hidden_size) / 1e12, 1)}),
+            "gflop_per_token": round(m.flops_per_token(SEQ, backward=False) / 1e9, 3),
+            "prefill_tflops": round(seqs * SEQ / pre * (m.flops_per_token(SEQ, backward=False) - 2.0 * cfg.vocab_size * cfg.hidden_size) / 1e12, 1)}),
             flush=True)
-        del eng
+        del eng, model
         torch.cuda.empty_cache()
 
 
@@ -309,9 +412,9 @@ def main(models, kernels_only=False, only=None, iters=20, seqs=64, new_tokens=12
 
 if __name__ == "__main__":
     ap = argparse.ArgumentParser()
-    ap.add_argument("--models", default="reninex-2048,reninex-4096")
+    ap.add_argument("--models", default="reninex-2048,reninex-4096,rigulorn-2048,rigulorn-4096")
     ap.add_argument("--kernels-only", action="store_true")
-    ap.add_argument("--only", choices=["prefill", "decode"])
+    ap.add_argument("--only", choices=["prefill", "decode", "none"], help="which kernels are timed")
     ap.add_argument("--step", help="only the steps whose name contains this")
     ap.add_argument("--no-compare", action="store_true", help="leave the dense kernels out")
     ap.add_argument("--iters", type=int, default=20)
