@@ -44,6 +44,42 @@ __device__ __forceinline__ float xtc_ex2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+// Pairs of fp32 values in one 64-bit register: half the issue slots of the scalar forms.
+__device__ __forceinline__ uint64_t xtc_pair(float lo, float hi) {
+  uint64_t v;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(v) : "f"(lo), "f"(hi));
+  return v;
+}
+__device__ __forceinline__ float2 xtc_unpair(uint64_t v) {
+  float2 f;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(f.x), "=f"(f.y) : "l"(v));
+  return f;
+}
+__device__ __forceinline__ uint64_t xtc_mul2(uint64_t a, uint64_t b) {
+  uint64_t v;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(v) : "l"(a), "l"(b));
+  return v;
+}
+__device__ __forceinline__ uint64_t xtc_fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t v;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(v) : "l"(a), "l"(b), "l"(c));
+  return v;
+}
+__device__ __forceinline__ uint64_t xtc_add2(uint64_t a, uint64_t b) {
+  uint64_t v;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(v) : "l"(a), "l"(b));
+  return v;
+}
+// Waits for a tensor-memory load into r; nothing that reads r can move in front of it.
+__device__ __forceinline__ void xtc_wait_load(uint32_t (&r)[32]) {
+  asm volatile("tcgen05.wait::ld.sync.aligned;"
+               : "+r"(r[0]), "+r"(r[1]), "+r"(r[2]), "+r"(r[3]), "+r"(r[4]), "+r"(r[5]), "+r"(r[6]), "+r"(r[7]),
+               "+r"(r[8]), "+r"(r[9]), "+r"(r[10]), "+r"(r[11]), "+r"(r[12]), "+r"(r[13]), "+r"(r[14]),
+               "+r"(r[15]), "+r"(r[16]), "+r"(r[17]), "+r"(r[18]), "+r"(r[19]), "+r"(r[20]), "+r"(r[21]),
+               "+r"(r[22]), "+r"(r[23]), "+r"(r[24]), "+r"(r[25]), "+r"(r[26]), "+r"(r[27]), "+r"(r[28]),
+               "+r"(r[29]), "+r"(r[30]), "+r"(r[31])
+               :: "memory");
+}
 __device__ __forceinline__ void xtc_group_barrier() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
 
 __global__ void __launch_bounds__(kXtcThreads, 1)
@@ -187,7 +223,13 @@ softmax_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
     const uint32_t t_s = tmem_base + lane_off + g * 128;
     const float zs = p.sp.scale / p.sp.cap, gain = p.sp.cap * 1.4426950408889634f;
     const float ref = score_reference(p.sp.cap) * 1.4426950408889634f;
-    float sum = 0.f;
+    // gain tanh(zs s) = s P(s^2) near zero: the series of tanh_series with the scale and the gain folded in
+    const float z2 = zs * zs, c0 = gain * zs, c1 = c0 * z2 * (-1.f / 3.f), c2 = c0 * z2 * z2 * (2.f / 15.f),
+                c3 = c0 * z2 * z2 * z2 * (-17.f / 315.f), c4 = c0 * z2 * z2 * z2 * z2 * (62.f / 2835.f);
+    const uint64_t p0 = xtc_pair(c0, c0), p1 = xtc_pair(c1, c1), p2 = xtc_pair(c2, c2), p3 = xtc_pair(c3, c3),
+                   p4 = xtc_pair(c4, c4), off = xtc_pair(-ref, -ref);
+    const float small = (kSmallTanh / zs) * (kSmallTanh / zs);
+    uint64_t sum2 = xtc_pair(0.f, 0.f);
     bool ok = true;
     for (int j = 0; j < n_blocks; ++j) {
       if (!mbar_wait(&s_full[g], j & 1, p.status, kTimeoutTmemFull)) {
@@ -199,33 +241,45 @@ softmax_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
       const int limit = pos0 + min(row, valid - 1) + 1 - base;           // visible keys: [skip, limit) of the block
       const int skip = first - base;
       const bool full = pos0 + 1 - base >= kXtcKeys && skip <= 0;        // ... all 128 for every row
-#pragma unroll 1
-      for (int c = 0; c < kXtcKeys / 32; ++c) {
-        uint32_t r[32], pk[16];
-        tmem_ld_32x32(t_s + c * 32, r);
-        tmem_ld_wait();
+      uint32_t ring[2][32];
+      tmem_ld_32x32(t_s, ring[0]);
+#pragma unroll
+      for (int c = 0; c < kXtcKeys / 32; ++c) {        // the next 32 scores are on their way while these are worked on
+        uint32_t(&r)[32] = ring[c & 1];
+        uint32_t pk[16];
+        xtc_wait_load(r);
+        if (c + 1 < kXtcKeys / 32) tmem_ld_32x32(t_s + (c + 1) * 32, ring[(c + 1) & 1]);
+        uint64_t v[16];                                // log2 weights of neighbouring keys
         float top = 0.f;
 #pragma unroll
-        for (int i = 0; i < 32; ++i) top = fmaxf(top, fabsf(__uint_as_float(r[i])));
-        if (__all_sync(0xffffffffu, top * fabsf(zs) <= kSmallTanh)) {
+        for (int i = 0; i < 16; ++i) {
+          const uint64_t x = xtc_pair(__uint_as_float(r[2 * i]), __uint_as_float(r[2 * i + 1]));
+          const uint64_t a = xtc_mul2(x, x);
+          const float2 f = xtc_unpair(a);
+          top = fmaxf(fmaxf(top, f.x), f.y);
+          uint64_t y = xtc_fma2(a, p4, p3);
+          y = xtc_fma2(a, y, p2);
+          y = xtc_fma2(a, y, p1);
+          y = xtc_fma2(a, y, p0);
+          v[i] = xtc_fma2(x, y, off);
+        }
+        if (!__all_sync(0xffffffffu, top <= small)) {  // some score lies beyond the series
 #pragma unroll
-          for (int i = 0; i < 32; ++i)
-            r[i] = __float_as_uint(xtc_ex2(fmaf(tanh_series(__uint_as_float(r[i]) * zs), gain, -ref)));
-        } else {
-#pragma unroll
-          for (int i = 0; i < 32; ++i)
-            r[i] = __float_as_uint(xtc_ex2(fmaf(tanh_any(__uint_as_float(r[i]) * zs), gain, -ref)));
+          for (int i = 0; i < 16; ++i)
+            v[i] = xtc_pair(fmaf(tanh_any(__uint_as_float(r[2 * i]) * zs), gain, -ref),
+                            fmaf(tanh_any(__uint_as_float(r[2 * i + 1]) * zs), gain, -ref));
         }
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
-          float p0 = __uint_as_float(r[2 * i]), p1 = __uint_as_float(r[2 * i + 1]);
+          const float2 f = xtc_unpair(v[i]);
+          float w0 = xtc_ex2(f.x), w1 = xtc_ex2(f.y);
           if (!full) {
             const int a = c * 32 + 2 * i;
-            if (a >= limit || a < skip) p0 = 0.f;
-            if (a + 1 >= limit || a + 1 < skip) p1 = 0.f;
+            if (a >= limit || a < skip) w0 = 0.f;
+            if (a + 1 >= limit || a + 1 < skip) w1 = 0.f;
           }
-          sum += p0 + p1;
-          pk[i] = pack_bf16x2(p0, p1);
+          sum2 = xtc_add2(sum2, xtc_pair(w0, w1));
+          pk[i] = pack_bf16x2(w0, w1);
         }
         tmem_st_32x16(t_s + c * 16, pk);
       }
@@ -233,7 +287,8 @@ softmax_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
       tc_fence_before();
       mbar_arrive(&p_full[g]);
     }
-    s_sum[g][row] = sum;
+    const float2 halves = xtc_unpair(sum2);
+    s_sum[g][row] = halves.x + halves.y;
     xtc_group_barrier();
     if (ok) ok = mbar_wait(o_full, 0, p.status, kTimeoutTmemFull);
     float o[2][32], sq = 0.f;

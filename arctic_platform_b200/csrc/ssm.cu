@@ -5,7 +5,7 @@
 //  * ssm_conv_kernel    longer entries: convolution + silu of every row, step sizes, the new convolution history;
 //  * ssm_scan_kernel    longer entries, token by token in fp32 (the fp32 engine, odd sizes): one CTA per (entry, head,
 //                       32-column slice of E), the slice of the state in shared memory;
-//  * ssm_out_kernel     every row: y silu(z), normalised in equal parts, times a weight.
+//  * gate_norm kernels  every row: y silu(z), normalised in equal parts, times a weight.
 //
 // bf16 engines run the longer entries' recurrence on tensor cores (ssm_mma.cu).
 #include "common.cuh"
@@ -52,7 +52,7 @@ ssm_decode_kernel(const SsmParams p) {
       if (j > 0 && (i < E || group_owner)) new_h[static_cast<long long>(j - 1) * channels + c] = x;
     }
     if (hist > 0 && (i < E || group_owner)) new_h[static_cast<long long>(hist - 1) * channels + c] = cur;
-    xs[i] = to_f32(from_f32<T>(silu_any(v)));                // x, B and C are activations
+    xs[i] = to_f32(from_f32<T>(silu_act<T>(v)));                // x, B and C are activations
   }
   const float2 st = ssm_step_of<T>(p, row, h);
   const float dt = st.x, dec = pos == 0 ? 0.f : exp2f(st.y);
@@ -112,7 +112,7 @@ ssm_decode_kernel(const SsmParams p) {
 // ---------------------------------------------------------------------------- convolution of longer entries
 // One block = up to kSsmRows rows of one entry (tiles[2 i] = entry, tiles[2 i + 1] = first row) x 512 channels, two
 // neighbouring channels per thread.  The first channel block also computes the rows' step sizes.
-constexpr int kSsmRows = 8;
+constexpr int kSsmRows = 16;
 constexpr int kSsmConvThreads = 256;
 
 template <typename T, int TAPS>                              // TAPS 0: any number
@@ -158,7 +158,7 @@ ssm_conv_kernel(const SsmParams p, const int* __restrict__ tiles) {
   };
   T* out = static_cast<T*>(p.xbc) + (start + r0) * p.ldx + c;
   auto put = [&](int i, float2 v) {
-    v = make_float2(silu_any(v.x), silu_any(v.y));
+    v = make_float2(silu_act<T>(v.x), silu_act<T>(v.y));
     if constexpr (sizeof(T) == 2) {
       *reinterpret_cast<uint32_t*>(out + i * p.ldx) = pack_bf16x2(v.x, v.y);     // ldx is even, the pad column exists
     } else {
@@ -174,7 +174,24 @@ ssm_conv_kernel(const SsmParams p, const int* __restrict__ tiles) {
     for (int j = 0; j < TAPS; ++j)
       w[j] = make_float2(to_f32(cw[static_cast<long long>(j) * channels + c]), pair ? to_f32(cw[static_cast<long long>(j) * channels + c + 1]) : 0.f);
 #pragma unroll
-    for (int i = 0; i < kHist + kSsmRows; ++i) x[i] = i < kHist + nr ? at2(r0 - kHist + i) : make_float2(0.f, 0.f);
+    for (int i = 0; i < kHist + kSsmRows; ++i) x[i] = make_float2(0.f, 0.f);
+    bool whole = false;                        // every row of the window is one of the entry's: loads without branches
+    if constexpr (sizeof(T) == 2) {
+      whole = r0 >= kHist && nr == kSsmRows && !((p.ld | p.xbc_col) & 1);
+      if (whole) {
+        const T* src = in + (r0 - kHist) * p.ld + c;
+        uint32_t raw[kHist + kSsmRows];
+#pragma unroll
+        for (int i = 0; i < kHist + kSsmRows; ++i, src += p.ld) raw[i] = *reinterpret_cast<const uint32_t*>(src);
+#pragma unroll
+        for (int i = 0; i < kHist + kSsmRows; ++i) x[i] = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw[i]));
+      }
+    }
+    if (!whole) {
+#pragma unroll
+      for (int i = 0; i < kHist + kSsmRows; ++i)
+        if (i < kHist + nr) x[i] = at2(r0 - kHist + i);
+    }
 #pragma unroll
     for (int i = 0; i < kSsmRows; ++i)
       if (i < nr) {
@@ -255,35 +272,87 @@ ssm_scan_kernel(const SsmParams p) {
 }
 
 // ---------------------------------------------------------------------------- gate and norm
-// out = w * (v / rms(v) per part), v = y silu(z): the gate comes before the norm.  One block per (row, part).
-template <typename T>
+// out = w * (v / rms(v) per part), v = y silu(z): the gate comes before the norm.
+struct GateNormParams {
+  const float* y;           // [rows, inner]
+  const void* z;            // [rows, inner] columns, row stride ldz
+  long long ldz;
+  const void* w;            // [inner]
+  void* out;                // row stride ldo
+  long long ldo;
+  int rows, inner, parts;
+  float eps;
+};
+
+__device__ __forceinline__ float4 gated4(const float* y, const __nv_bfloat16* z) {
+  using T = __nv_bfloat16;
+  const float4 v = __ldcs(reinterpret_cast<const float4*>(y));
+  const uint2 raw = *reinterpret_cast<const uint2*>(z);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+  return make_float4(v.x * silu_act<T>(a.x), v.y * silu_act<T>(a.y), v.z * silu_act<T>(b.x), v.w * silu_act<T>(b.y));
+}
+__device__ __forceinline__ void scaled4(__nv_bfloat16* out, const float4& v, float f, const __nv_bfloat16* w) {
+  const uint2 raw = *reinterpret_cast<const uint2*>(w);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+  *reinterpret_cast<uint2*>(out) = make_uint2(pack_bf16x2(v.x * f * a.x, v.y * f * a.y), pack_bf16x2(v.z * f * b.x, v.w * f * b.y));
+}
+
+// bf16, parts of a multiple of 4 up to 1024 columns, 8-byte aligned: one warp per (row, part).
+constexpr int kGateWarpCols = 1024;
+
 __global__ void __launch_bounds__(256)
-ssm_out_kernel(const float* __restrict__ y, const T* __restrict__ z, long long ldz, const T* __restrict__ w, T* __restrict__ out,
-               long long ldo, int inner, int parts, float eps) {
+gate_norm_warp_kernel(const GateNormParams p) {
+  pdl_entry();
+  const long long gw = (blockIdx.x * 256LL + threadIdx.x) >> 5;
+  if (gw >= static_cast<long long>(p.rows) * p.parts) return;
+  const int lane = threadIdx.x & 31, n = p.inner / p.parts, c0 = static_cast<int>(gw % p.parts) * n;
+  const long long row = gw / p.parts;
+  const float* y = p.y + row * p.inner + c0;
+  const __nv_bfloat16* z = static_cast<const __nv_bfloat16*>(p.z) + row * p.ldz + c0;
+  const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(p.w) + c0;
+  __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + row * p.ldo + c0;
+  float4 v[kGateWarpCols / 128];
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < kGateWarpCols / 128; ++k) {
+    const int i = k * 128 + lane * 4;
+    v[k] = i < n ? gated4(y + i, z + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    ss += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+  }
+  const float f = 1.f / sqrtf(warp_sum(ss) / n + p.eps);
+#pragma unroll
+  for (int k = 0; k < kGateWarpCols / 128; ++k) {
+    const int i = k * 128 + lane * 4;
+    if (i < n) scaled4(out + i, v[k], f, w + i);
+  }
+}
+
+// One block per (row, part), any size.  VEC: bf16 with the alignment of the kernel above.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256)
+gate_norm_kernel(const GateNormParams p) {
   pdl_entry();
   extern __shared__ float ssm_smem[];          // [inner / parts]
   __shared__ float red[8];
-  const int n = inner / parts, c0 = blockIdx.y * n;
+  const int n = p.inner / p.parts, c0 = blockIdx.y * n;
   const long long row = blockIdx.x;
-  const float* yr = y + row * inner + c0;
-  const T* zr = z + row * ldz + c0;
-  T* orow = out + row * ldo + c0;
-  const bool vec = sizeof(T) == 2 && !(n & 3) && !(c0 & 3) && !(inner & 3) &&
-                   !((reinterpret_cast<uintptr_t>(zr) | reinterpret_cast<uintptr_t>(orow) | reinterpret_cast<uintptr_t>(w + c0)) & 7);
+  const float* y = p.y + row * p.inner + c0;
+  const T* z = static_cast<const T*>(p.z) + row * p.ldz + c0;
+  const T* w = static_cast<const T*>(p.w) + c0;
+  T* out = static_cast<T*>(p.out) + row * p.ldo + c0;
   float ss = 0.f;
-  if (vec) {
+  if constexpr (VEC) {
+#pragma unroll 4
     for (int i = threadIdx.x * 4; i < n; i += 1024) {
-      const float4 v = __ldcs(reinterpret_cast<const float4*>(yr + i));
-      const uint2 raw = *reinterpret_cast<const uint2*>(zr + i);
-      const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
-      const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
-      const float4 r = make_float4(v.x * silu_any(a.x), v.y * silu_any(a.y), v.z * silu_any(b.x), v.w * silu_any(b.y));
-      *reinterpret_cast<float4*>(ssm_smem + i) = r;
-      ss += r.x * r.x + r.y * r.y + r.z * r.z + r.w * r.w;
+      const float4 v = gated4(y + i, z + i);
+      *reinterpret_cast<float4*>(ssm_smem + i) = v;
+      ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
     }
   } else {
     for (int i = threadIdx.x; i < n; i += 256) {
-      const float v = yr[i] * silu_any(to_f32(zr[i]));
+      const float v = y[i] * silu_act<T>(to_f32(z[i]));
       ssm_smem[i] = v;
       ss += v * v;
     }
@@ -294,17 +363,11 @@ ssm_out_kernel(const float* __restrict__ y, const T* __restrict__ z, long long l
   ss = 0.f;
 #pragma unroll
   for (int i = 0; i < 8; ++i) ss += red[i];
-  const float f = 1.f / sqrtf(ss / n + eps);
-  if (vec) {
-    for (int i = threadIdx.x * 4; i < n; i += 1024) {
-      const float4 v = *reinterpret_cast<const float4*>(ssm_smem + i);
-      const uint2 raw = *reinterpret_cast<const uint2*>(w + c0 + i);
-      const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
-      const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
-      *reinterpret_cast<uint2*>(orow + i) = make_uint2(pack_bf16x2(v.x * f * a.x, v.y * f * a.y), pack_bf16x2(v.z * f * b.x, v.w * f * b.y));
-    }
+  const float f = 1.f / sqrtf(ss / n + p.eps);
+  if constexpr (VEC) {
+    for (int i = threadIdx.x * 4; i < n; i += 1024) scaled4(out + i, *reinterpret_cast<const float4*>(ssm_smem + i), f, w + i);
   } else {
-    for (int i = threadIdx.x; i < n; i += 256) orow[i] = from_f32<T>(ssm_smem[i] * f * to_f32(w[c0 + i]));
+    for (int i = threadIdx.x; i < n; i += 256) out[i] = from_f32<T>(ssm_smem[i] * f * to_f32(w[i]));
   }
 }
 
@@ -376,15 +439,21 @@ int apb_ssm_out(const float* y, const void* z, long long ldz, const void* w, voi
                 int parts, float eps, int dtype, cudaStream_t s) {
   if (rows <= 0) return 0;
   if (inner <= 0 || parts <= 0 || inner % parts) return kBadArgument;
-  const size_t smem = static_cast<size_t>(inner / parts) * sizeof(float);
-  auto run = [&](auto fn, auto zero) -> int {
-    using T = decltype(zero);
+  const GateNormParams p{y, z, ldz, w, out, ldo, rows, inner, parts, eps};
+  const int n = inner / parts;
+  const bool vec = dtype == 0 && !(n & 3) && !((ldz | ldo) & 3) &&
+                   !((reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out)) & 7);
+  if (vec && n <= kGateWarpCols)
+    return static_cast<int>(launch_kernel(gate_norm_warp_kernel, dim3(static_cast<unsigned>((static_cast<long long>(rows) * parts + 7) / 8)),
+                                          dim3(256), 0, s, p));
+  const size_t smem = static_cast<size_t>(n) * sizeof(float);
+  auto run = [&](auto fn) -> int {
     const int rc = ssm_smem_limit(fn, smem);
-    return rc ? rc : static_cast<int>(launch_kernel(fn, dim3(rows, parts), dim3(256), smem, s, y, static_cast<const T*>(z), ldz,
-                                                    static_cast<const T*>(w), static_cast<T*>(out), ldo, inner, parts, eps));
+    return rc ? rc : static_cast<int>(launch_kernel(fn, dim3(rows, parts), dim3(256), smem, s, p));
   };
-  if (dtype == 0) return run(ssm_out_kernel<__nv_bfloat16>, __nv_bfloat16());
-  if (dtype == 1) return run(ssm_out_kernel<float>, float());
+  if (vec) return run(gate_norm_kernel<__nv_bfloat16, true>);
+  if (dtype == 0) return run(gate_norm_kernel<__nv_bfloat16, false>);
+  if (dtype == 1) return run(gate_norm_kernel<float, false>);
   return kBadArgument;
 }
 }

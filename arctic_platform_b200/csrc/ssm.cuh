@@ -32,7 +32,12 @@ struct SsmParams {
 };
 
 __device__ __forceinline__ float softplus_f(float v) { return v > 20.f ? v : log1pf(expf(v)); }
-__device__ __forceinline__ float silu_any(float v) { return v / (1.f + expf(-v)); }
+// silu of an activation: to fp32 accuracy for fp32 engines, well inside a bf16 rounding step for bf16 ones
+template <typename T>
+__device__ __forceinline__ float silu_act(float v) {
+  if constexpr (sizeof(T) == 2) return __fdividef(v, 1.f + __expf(-v));
+  return v / (1.f + expf(-v));
+}
 
 template <typename T>
 __device__ __forceinline__ float2 ssm_step_of(const SsmParams& p, long long row, int h) {

@@ -522,6 +522,14 @@ def retention(b: StepBatch, p: torch.Tensor, cols: Tuple[int, int, int, int], ro
               float(out_scale), float(eps), _lib.ptr(b.row_entry), *b.entry_ptrs(), b.rows, H, E, dtype_code(p.dtype))
 
 
+SSM_ROWS = 16           # rows per block of the state-space mixer's convolution
+
+
+def row_tiles(host: np.ndarray, rows: int) -> np.ndarray:
+    """``[n, 2]`` int32 (entry, first row) of the blocks of up to ``rows`` rows of the entries longer than one row."""
+    return np.array([(en, r) for en, n in enumerate(host[:, 1].tolist()) if n > 1 for r in range(0, n, rows)], dtype=np.int32)
+
+
 @dataclass(frozen=True)
 class SsmWeights:
     """Parameters of a state-space mixer besides its projections: ``conv [taps, channels]``, ``conv_bias [channels]``, and per
@@ -544,11 +552,12 @@ def state_space(b: StepBatch, p: torch.Tensor, xbc_col: int, dt_col: int, w: Ssm
     ldx = (channels + 7) // 8 * 8
     xbc = torch.empty((b.rows, ldx), device=p.device, dtype=p.dtype) if b.longer else None
     steps = torch.empty((b.rows, H, 2), device=p.device, dtype=torch.float32) if b.longer else None
+    tiles = b.table(("rows", SSM_ROWS), lambda: row_tiles(b.host, SSM_ROWS)) if b.longer else None
     mma = b.longer and p.dtype == torch.bfloat16 and N % 8 == 0 and E % 8 == 0 and N <= 128
     _call("apb_ssm", _lib.ptr(p), p.stride(0), xbc_col, dt_col, _lib.ptr(w.conv), _lib.ptr(w.conv_bias), taps, _lib.ptr(hist),
           _lib.ptr(parity), _lib.ptr(w.dt_bias), _lib.ptr(w.a_log), _lib.ptr(w.skip), _lib.ptr(xbc), ldx, _lib.ptr(steps),
-          _lib.ptr(state), _lib.ptr(y), *b.entry_ptrs(), b.n_entries, _lib.ptr(b.tiles) if b.longer else None,
-          b.tiles.shape[0] if b.longer else 0, H, E, groups, N, int(b.one_token), int(b.longer and not mma), dtype_code(p.dtype))
+          _lib.ptr(state), _lib.ptr(y), *b.entry_ptrs(), b.n_entries, _lib.ptr(tiles),
+          tiles.shape[0] if b.longer else 0, H, E, groups, N, int(b.one_token), int(b.longer and not mma), dtype_code(p.dtype))
     if mma:
         slices = H * ((E + 63) // 64)
         key = ("segments", slices)

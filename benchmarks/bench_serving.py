@@ -196,14 +196,17 @@ def rigulorn_ops(cfg, phase):
     ]
 
 
-# step of a Rigulorn layer -> the like step of the Reninex layer
+# step of a Rigulorn layer -> (model, the like step of its layer); products next to the dense decoder's of the same shape
 RIGULORN_LIKE = {
-    "stream update + norm": "norm + 2 input convolutions", "attention input projections (GEMM)": "input projections (GEMM)",
-    "rotation + cache write": "q/k norm + cache write", "attention": "attention",
-    "attention output projection (GEMM)": "output projections (GEMM, += fp32)",
-    "gate/up + clamped GLU (GEMM)": "gate/up + GELU (GEMM)", "down projection (GEMM)": "output projections (GEMM, += fp32)",
-    "state-space input projections (GEMM)": "input projections (GEMM)", "recurrent mixer": "recurrent mixer",
-    "state-space output projection (GEMM)": "output projections (GEMM, += fp32)",
+    "stream update + norm": ("reninex", "norm + 2 input convolutions"),
+    "attention input projections (GEMM)": ("dense", "input projections (GEMM)"),
+    "rotation + cache write": ("reninex", "q/k norm + cache write"), "attention": ("reninex", "attention"),
+    "attention output projection (GEMM)": ("dense", "attention output projection (GEMM)"),
+    "gate/up + clamped GLU (GEMM)": ("dense", "gate/up + GELU (GEMM)"),
+    "down projection (GEMM)": ("dense", "output projections (GEMM, += fp32)"),
+    "state-space input projections (GEMM)": ("reninex", "input projections (GEMM)"),
+    "recurrent mixer": ("reninex", "recurrent mixer"),
+    "state-space output projection (GEMM)": ("reninex", "output projections (GEMM, += fp32)"),
 }
 
 
@@ -220,8 +223,9 @@ def like_ops(cfg, phase):
     """Steps of the closest older model, keyed by the names of ``stateful_ops``: ``name -> (fn, bytes, flops)``."""
     if cfg.architecture != "Rigulorn":
         return dense_ops(cfg, phase)
-    ops = {name: rest for name, *rest in reninex_ops(reninex_like(cfg), phase)}
-    return {mine: ops[theirs] for mine, theirs in RIGULORN_LIKE.items()}
+    like = reninex_like(cfg)
+    ops = {"reninex": {name: rest for name, *rest in reninex_ops(like, phase)}, "dense": dense_ops(like, phase)}
+    return {mine: ops[model][theirs] for mine, (model, theirs) in RIGULORN_LIKE.items()}
 
 
 def dense_config(cfg):
@@ -258,7 +262,7 @@ def dense_ops(cfg, phase):
                         cascade=False, use_cuda_graph=False)
     x, res = _bf(T, W), _bf(T, W)
     qkv = _bf(T, d.qkv_size)
-    act = _bf(T, ff)
+    act, qo = _bf(T, ff), _bf(T, d.q_size)
     pos = torch.arange(T, device="cuda", dtype=torch.int32) % SEQ
     slots = torch.arange(T, device="cuda", dtype=torch.int32)
     rope = model.rope("cuda")
@@ -279,6 +283,8 @@ def dense_ops(cfg, phase):
                             T * kv_row + 4 * T * Hq * D, 4 * keys * Hq * D)
         ops["output projections (GEMM, += fp32)"] = (lambda: gemm.matmul_nt(act, blk.wdown),
                                                      2 * (T * ff + ff * W + T * W), 2 * T * ff * W)
+        ops["attention output projection (GEMM)"] = (lambda: gemm.matmul_nt(qo, blk.wo), 2 * (T * d.q_size + d.q_size * W + T * W),
+                                                     2 * T * d.q_size * W)
         ops["q/k norm + cache write"] = (qk_and_cache, 2 * T * 2 * Hq * D + 2 * T * kv_row, 0)
         ops["norm + 2 input convolutions"] = (lambda: norm.rmsnorm(x, blk.ln1, 1e-6, res), T * W * 8, 0)
         qr, kr, vr = (torch.randn(SEQ, R.heads, m, device="cuda") for m in (R.dim, R.dim, R.vdim))
@@ -306,6 +312,10 @@ def dense_ops(cfg, phase):
         ops["output projections (GEMM, += fp32)"] = (
             lambda: gemm.gemm_raw(act, blk.wdown, acc, M=T, N=W, K=ff, epi=gemm.EPI_F32_ATOMIC, splits=sd, bn=128),
             2 * (T * ff + ff * W) + 8 * T * W, 2 * T * ff * W)
+        so = max(1, min(148 // tiles(W), (d.q_size + 63) // 64))
+        ops["attention output projection (GEMM)"] = (
+            lambda: gemm.gemm_raw(qo, blk.wo, acc, M=T, N=W, K=d.q_size, epi=gemm.EPI_F32_ATOMIC, splits=so, bn=128),
+            2 * (T * d.q_size + d.q_size * W) + 8 * T * W, 2 * T * d.q_size * W)
         ops["q/k norm + cache write"] = (lambda: _lib.check(_fn("qkv_post")(
             _lib.ptr(accq), accq.stride(0), _lib.ptr(blk.q_norm), _lib.ptr(blk.k_norm), _lib.ptr(rope[0]), _lib.ptr(rope[1]),
             _lib.ptr(pos), _lib.ptr(slots), _lib.ptr(qb), _lib.ptr(eng.kcache[0]), _lib.ptr(eng.vcache[0]), T, Hq, G, D, 1e-6,

@@ -175,3 +175,9 @@ def test_attention_work_items_cover_every_row_once_and_stay_in_a_chunk(heads, kv
     assert seen == {(r, h): 1 for r in rows for h in range(heads)}
     assert (np.diff(keys) <= 0).all()
     assert chunk_tiles(host, heads, kv, 1000, chunk).shape == (0, 8)
+
+
+def test_row_tiles_skip_single_tokens():
+    from arctic_platform_b200.ops.serving import row_tiles
+    host = np.array([[0, 33, 0, 0], [33, 1, 1, 9], [34, 16, 2, 0]])
+    assert row_tiles(host, 16).tolist() == [[0, 0], [0, 16], [0, 32], [2, 0]]
