@@ -72,11 +72,15 @@ def _compile_one(src: Path, verbose: bool) -> Path:
     return obj
 
 
-# what serving a stateful architecture needs (models/registry.py): the GEMMs, the ragged-batch kernels, the status word
-SERVE_STEMS = ("status", "gemm_tcgen05", "gemm_tcgen05_2cta", "gemm_simt", "serve_layers", "serve_attention",
-               "serve_attention_tc", "serve_softmax", "serve_softmax_tc", "serve_streams", "retention", "retention_mma", "ssm",
-               "ssm_mma")
-SERVE_LIB = OUT_DIR / "libapb200_serve.so"
+# what serving any stateful architecture needs: the status word, the GEMMs, the kernels of a ragged batch; each names the
+# sources of its own layers in models/registry.py
+SERVE_STEMS = ("status", "gemm_tcgen05", "gemm_tcgen05_2cta", "gemm_simt", "serve_layers")
+
+
+def serve_lib(architecture: str) -> Path:
+    return OUT_DIR / f"libapb200_{architecture.lower()}.so"
+
+
 RT_SERVE_LIB = OUT_DIR / "libapb200_rt_serve.so"       # the page allocator (runtime.cpp)
 
 

@@ -62,12 +62,14 @@ def make_engine(model_dir: str, dtype: str, max_tokens: int):
     from ..engine.stateful_sampler import StatefulSampler
     from ..models import registry
     from ..models.factory import LoaderContext, ModelSpec, build_model
+    from ..ops import _lib
     spec = ModelSpec(model_dir, dtype=dtype)
     cfg = LoaderContext(spec).hf_config
     if not registry.is_stateful(cfg):
         raise SystemExit(f"{model_dir}: traces replay on the stateful engine ({', '.join(registry.architectures())})")
     if not torch.cuda.is_available():
         raise SystemExit("trace_run needs a CUDA device")
+    _lib.serve_only(cfg.architecture)
     model = build_model(spec, device="cuda").model
     return StatefulSampler(cfg, "cuda", model=model, kv_cache_tokens=max_tokens, max_batch=MAX_LIVE,
                            max_seq_len=max(max_tokens, 64))
@@ -76,7 +78,6 @@ def make_engine(model_dir: str, dtype: str, max_tokens: int):
 def main(argv=None) -> int:
     args = parse_args(argv)
     from ..ops import _lib
-    _lib.serve_only()
     engine = make_engine(args.model, args.dtype, args.max_tokens)
     replay = Replay(engine, args.out)
     for line in sys.stdin:

@@ -1,8 +1,9 @@
 """Architectures that are not described by :class:`~arctic_platform_b200.models.config.DecoderConfig`.
 
 A checkpoint directory whose ``config.json`` has an ``architecture`` key names one of these.  An entry gives the
-configuration class (``from_dict``, ``PRESETS``) and the model class; both are imported on first use.  The model class
-implements the serving protocol of :mod:`arctic_platform_b200.engine.stateful_sampler`.
+configuration class (``from_dict``, ``PRESETS``) and the model class -- both are imported on first use -- and the kernel
+sources (``csrc/*.cu``) of its layers.  The model class implements the serving protocol of
+:mod:`arctic_platform_b200.engine.stateful_sampler`.
 """
 from __future__ import annotations
 
@@ -10,14 +11,23 @@ import importlib
 from typing import Any, Dict, Tuple
 
 _ARCHITECTURES: Dict[str, Tuple[str, str, str]] = {}        # architecture -> (module, config class, model class)
+_KERNELS: Dict[str, Tuple[str, ...]] = {}
 
 
-def register_architecture(name: str, module: str, config_class: str, model_class: str) -> None:
+def register_architecture(name: str, module: str, config_class: str, model_class: str, kernels: Tuple[str, ...] = ()) -> None:
     _ARCHITECTURES[name] = (module, config_class, model_class)
+    _KERNELS[name] = tuple(kernels)
 
 
-register_architecture("Reninex", "arctic_platform_b200.models.reninex", "ReninexConfig", "ReninexLM")
-register_architecture("Rigulorn", "arctic_platform_b200.models.rigulorn", "RigulornConfig", "RigulornLM")
+register_architecture("Reninex", "arctic_platform_b200.models.reninex", "ReninexConfig", "ReninexLM",
+                      ("serve_attention", "serve_attention_tc", "retention", "retention_mma"))
+register_architecture("Rigulorn", "arctic_platform_b200.models.rigulorn", "RigulornConfig", "RigulornLM",
+                      ("serve_streams", "serve_softmax", "serve_softmax_tc", "ssm", "ssm_mma"))
+
+
+def kernel_sources(architecture: str) -> Tuple[str, ...]:
+    """Sources of the kernels of the architecture's own layers (without extension)."""
+    return _KERNELS[architecture]
 
 
 def architectures() -> Tuple[str, ...]:

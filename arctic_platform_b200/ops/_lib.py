@@ -11,7 +11,7 @@ from __future__ import annotations
 import ctypes
 import threading
 from pathlib import Path
-from typing import Tuple
+from typing import Optional, Tuple
 
 import torch
 
@@ -55,19 +55,22 @@ def _load(path: Path, builder):
         raise NativeLibraryError(f"cannot load {path}: {exc}") from exc
 
 
-_serve_only = False
+_serve: Optional[Tuple[Path, Tuple[str, ...]]] = None        # kernel library of one architecture and its sources
 
 
-def serve_only() -> None:
-    """For processes that only serve a stateful architecture: unless the full kernel library is built and current,
+def serve_only(architecture: str) -> None:
+    """For processes that only serve this stateful architecture: unless the full kernel library is built and current,
     compile and load just the kernels such a model needs.  Call it before the first kernel."""
-    global _serve_only
-    _serve_only = not _build.cuda_up_to_date()
-    if _serve_only:
-        try:
-            _build.build_cuda_subset(_build.SERVE_STEMS, _build.SERVE_LIB)
-        except Exception as exc:
-            raise NativeLibraryError(f"{_build.SERVE_LIB.name} could not be built: {exc}") from exc
+    global _serve
+    if _build.cuda_up_to_date():
+        _serve = None
+        return
+    from ..models import registry
+    _serve = _build.serve_lib(architecture), _build.SERVE_STEMS + registry.kernel_sources(architecture)
+    try:
+        _build.build_cuda_subset(_serve[1], _serve[0])
+    except Exception as exc:
+        raise NativeLibraryError(f"{_serve[0].name} could not be built: {exc}") from exc
 
 
 def cuda_lib() -> ctypes.CDLL:
@@ -75,8 +78,9 @@ def cuda_lib() -> ctypes.CDLL:
     if _cuda is None:
         with _lock:
             if _cuda is None:
-                if _serve_only:
-                    lib = _load(_build.SERVE_LIB, lambda: _build.build_cuda_subset(_build.SERVE_STEMS, _build.SERVE_LIB))
+                if _serve is not None:
+                    path, stems = _serve
+                    lib = _load(path, lambda: _build.build_cuda_subset(stems, path))
                 else:
                     lib = _load(_build.CUDA_LIB, _build.build_cuda)
                 _declare_cuda(lib)
@@ -89,7 +93,7 @@ def rt_lib() -> ctypes.CDLL:
     if _rt is None:
         with _lock:
             if _rt is None:
-                if _serve_only and not _build.RT_LIB.exists():
+                if _serve is not None and not _build.RT_LIB.exists():
                     lib = _load(_build.RT_SERVE_LIB,
                                 lambda: _build.build_runtime(stems=("runtime",), lib=_build.RT_SERVE_LIB))
                 else:

@@ -181,3 +181,13 @@ def test_row_tiles_skip_single_tokens():
     from arctic_platform_b200.ops.serving import row_tiles
     host = np.array([[0, 33, 0, 0], [33, 1, 1, 9], [34, 16, 2, 0]])
     assert row_tiles(host, 16).tolist() == [[0, 0], [0, 16], [0, 32], [2, 0]]
+
+
+def test_a_serving_process_compiles_only_its_own_kernels():
+    from arctic_platform_b200 import _build
+    from arctic_platform_b200.models import registry
+    own = {a: set(registry.kernel_sources(a)) for a in registry.architectures()}
+    names = {p.stem for p in _build.cuda_sources()}
+    assert all(k and k <= names and not k & set(_build.SERVE_STEMS) for k in own.values())
+    assert not own["Rigulorn"] & own["Reninex"] and set(_build.SERVE_STEMS) <= names
+    assert _build.serve_lib("Rigulorn") != _build.serve_lib("Reninex")
