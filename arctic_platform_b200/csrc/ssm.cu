@@ -16,6 +16,7 @@ namespace apb {
 
 // ---------------------------------------------------------------------------- one token
 constexpr int kSsmDecThreads = 256;
+constexpr int kSsmDecAhead = 8;    // state rows per thread that are on their way while the convolution is computed
 
 template <typename T, int VEC>
 __global__ void __launch_bounds__(kSsmDecThreads)
@@ -40,6 +41,18 @@ ssm_decode_kernel(const SsmParams p) {
     old_h = p.hist + (static_cast<long long>(slot) * 2 + par) * hist * channels;
     new_h = p.hist + (static_cast<long long>(slot) * 2 + (par ^ 1)) * hist * channels;
   }
+  float* S = p.state + (static_cast<long long>(slot) * p.H + h) * N * E;
+  const int nx = min(E / VEC, kSsmDecThreads), ny = kSsmDecThreads / nx;
+  const int tx = threadIdx.x % nx, ty = threadIdx.x / nx;
+  float4 ahead[kSsmDecAhead];
+  if (VEC == 4) {
+#pragma unroll
+    for (int k = 0; k < kSsmDecAhead; ++k) {
+      const int d = ty + k * ny;
+      ahead[k] = make_float4(0.f, 0.f, 0.f, 0.f);            // position 0: the slot may hold anything
+      if (pos > 0 && ty < ny && d < N) ahead[k] = __ldcs(reinterpret_cast<const float4*>(S + static_cast<long long>(d) * E + tx * 4));
+    }
+  }
   const bool group_owner = h % rep == 0;                     // writes the history of its group's B and C
   for (int i = threadIdx.x; i < E + 2 * N; i += kSsmDecThreads) {
     const int c = i < E ? h * E + i : (i < E + N ? p.H * E + g * N + i - E : p.H * E + (p.G + g) * N + i - E - N);
@@ -57,9 +70,6 @@ ssm_decode_kernel(const SsmParams p) {
   const float2 st = ssm_step_of<T>(p, row, h);
   const float dt = st.x, dec = pos == 0 ? 0.f : exp2f(st.y);
   __syncthreads();
-  float* S = p.state + (static_cast<long long>(slot) * p.H + h) * N * E;
-  const int nx = min(E / VEC, kSsmDecThreads), ny = kSsmDecThreads / nx;
-  const int tx = threadIdx.x % nx, ty = threadIdx.x / nx;
   if (ty < ny) {
     for (int cx = tx; cx < E / VEC; cx += nx) {
       float acc[VEC], v[VEC];
@@ -68,13 +78,29 @@ ssm_decode_kernel(const SsmParams p) {
         acc[i] = 0.f;
         v[i] = xs[cx * VEC + i] * dt;
       }
-#pragma unroll 8
-      for (int d = ty; d < N; d += ny) {
+      int d = ty;
+      if (VEC == 4 && cx == tx) {
+#pragma unroll
+        for (int k = 0; k < kSsmDecAhead; ++k, d += ny)
+          if (d < N) {
+            const float bd = bs[d], cd = cs[d];
+            const float4 o = ahead[k];
+            const float4 n = make_float4(o.x * dec + bd * v[0], o.y * dec + bd * v[1 % VEC], o.z * dec + bd * v[2 % VEC],
+                                         o.w * dec + bd * v[3 % VEC]);
+            acc[0] += n.x * cd;
+            acc[1 % VEC] += n.y * cd;
+            acc[2 % VEC] += n.z * cd;
+            acc[3 % VEC] += n.w * cd;
+            __stcs(reinterpret_cast<float4*>(S + static_cast<long long>(d) * E + cx * 4), n);
+          }
+      }
+#pragma unroll 4
+      for (; d < N; d += ny) {
         float* sp = S + static_cast<long long>(d) * E + cx * VEC;
         float s[VEC];
 #pragma unroll
         for (int i = 0; i < VEC; ++i) s[i] = 0.f;
-        if (pos > 0) {             // at position 0 the slot may hold anything
+        if (pos > 0) {
           if (VEC == 4) {
             const float4 t = __ldcs(reinterpret_cast<const float4*>(sp));
             s[0] = t.x;
