@@ -19,6 +19,7 @@ enum GemmEpilogue : int {
   kEpiBf16ScatterPeer = 8, // GEMM -> all-to-all: bf16 row stored to (peer, row) = row_map[m] (MoE combine)
   kEpiGeGLU = 9,       // as kEpiSwiGLU with the tanh form of GELU as the activation of the gate
   kEpiClampGLU = 10,   // as kEpiSwiGLU: g = min(gate, limit), u = clamp(up, -limit, limit), g sigmoid(1.702 g) (u + 1)
+  kEpiSigmoidGate = 11,    // C(bf16) = acc * sigmoid(gate), gate (bf16) laid out like C
 };
 
 __host__ __device__ inline bool is_glu_epilogue(int epi) {
@@ -65,6 +66,10 @@ struct GemmParams {
   const int2* row_map;     // kEpiBf16ScatterPeer: (rank, destination row) per output row, rank < 0 = drop
   int a_peer_rows;         // > 0: A is row-sharded over ranks, this many rows each, read through per-rank maps
   int world;
+  // products per head: C[:, h c_step + n] = A[:, h a_step + k] B[h N + n, k] (0 heads: an ordinary product)
+  int heads, a_step, c_step;
+  const __nv_bfloat16* gate;   // kEpiSigmoidGate
+  long long ldg;
   int chained;             // 1: launched in chained mode -- B (weights nobody in the chain writes) is prefetched
                            // before the wait for the previous kernel, everything else after it
 };
@@ -84,19 +89,34 @@ __device__ __forceinline__ float clamped_glu_f(float g, float u, float limit) {
 // One output row, 32 consecutive accumulator columns starting at `col0` (raw fp32 bits in `r`).  Covers every
 // epilogue except the two lm-head ones, which keep running state across the chunks of a tile.
 // `ncols` (32, or 16 for the last chunk of a tile width that is not a multiple of 32) clips the chunk at the tile
-// edge; columns at or beyond p.N are never written either.
+// edge; columns at or beyond p.N are never written either.  `c_shift`: first column of the head in C (products per head).
 __device__ __forceinline__ void gemm_store_chunk(const GemmParams& p, int row, int col0, const uint32_t (&r)[32],
-                                                 int ncols = 32) {
+                                                 int ncols = 32, int c_shift = 0) {
   float v[32];
 #pragma unroll
   for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(r[j]) * p.alpha;
-  if (p.epi == kEpiBf16 || (is_glu_epilogue(p.epi) && p.C != nullptr)) {
+  if (p.epi == kEpiSigmoidGate) {
+    const __nv_bfloat16* g = p.gate + static_cast<long long>(row) * p.ldg + c_shift + col0;
+#pragma unroll
+    for (int j = 0; j < 32; j += 8)
+      if (j < ncols && col0 + j < p.N) {
+        const uint4 raw = *reinterpret_cast<const uint4*>(g + j);
+        const uint32_t w[4] = {raw.x, raw.y, raw.z, raw.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[i]));
+          v[j + 2 * i] /= 1.f + __expf(-f.x);
+          v[j + 2 * i + 1] /= 1.f + __expf(-f.y);
+        }
+      }
+  }
+  if (p.epi == kEpiBf16 || p.epi == kEpiSigmoidGate || (is_glu_epilogue(p.epi) && p.C != nullptr)) {
     if (p.bias) {
 #pragma unroll
       for (int j = 0; j < 32; ++j)
         if (col0 + j < p.N) v[j] += __bfloat162float(p.bias[col0 + j]);
     }
-    __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(p.C) + static_cast<long long>(row) * p.ldc + col0;
+    __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(p.C) + static_cast<long long>(row) * p.ldc + c_shift + col0;
 #pragma unroll
     for (int q = 0; q < 4; ++q) {
       if (q * 8 < ncols && col0 + q * 8 < p.N) {

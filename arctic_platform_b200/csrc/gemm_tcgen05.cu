@@ -58,8 +58,9 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tma_a, const CUtens
 
   const int tiles_m = (p.M + kBM - 1) / kBM;
   const int tiles_n = (p.N + BN - 1) / BN;
+  if (p.tile_map) pdl_wait();     // the tables may come from the previous kernel of a chained launch
   const int mn_tiles = p.tile_map ? (p.num_tiles_dev ? min(*p.num_tiles_dev, p.num_map_tiles) : p.num_map_tiles)
-                                  : tiles_m * tiles_n;
+                                  : tiles_m * tiles_n * max(1, p.heads);
   const int total_tiles = mn_tiles * p.splits;
   const int k_blocks = (p.K + kBK - 1) / kBK;
 
@@ -92,6 +93,7 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tma_a, const CUtens
   // one n-band before moving on, so CTAs running at the same time share B in L2.
   // c_off / bk_off: see GemmParams::tile_ext (0 without it)
   int c_off = 0, bk_off = 0;
+  int a_col = 0, c_col = 0;     // first column of the tile's head in A and C
   auto decode = [&](int t, int& m0, int& m_end, int& b_row, int& n0, int& kb0, int& kb1) {
     const int split = t / mn_tiles;
     const int tt = t - split * mn_tiles;
@@ -113,6 +115,14 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tma_a, const CUtens
           if (kb1 < kb0) kb1 = kb0;
         }
       }
+    } else if (p.heads) {
+      const int per_head = tiles_m * tiles_n, h = tt / per_head, r = tt - h * per_head;
+      a_col = h * p.a_step;
+      c_col = h * p.c_step;
+      m0 = (r % tiles_m) * kBM;
+      m_end = p.M;
+      n0 = (r / tiles_m) * BN;
+      b_row = h * p.N + n0;
     } else {
       constexpr int G = 8;
       const int per_group = G * tiles_n;
@@ -191,7 +201,7 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tma_a, const CUtens
                           row - peer * p.a_peer_rows);
             }
           } else if (!p.a_mn) {
-            tma_load_2d(sa, &tma_a, &full_bar[stage], kb * kBK, m0);
+            tma_load_2d(sa, &tma_a, &full_bar[stage], kb * kBK + a_col, m0);
           } else {
 #pragma unroll
             for (int c = 0; c < kBM / 64; ++c)
@@ -392,7 +402,7 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap& tma_a, const CUtens
           tmem_ld_wait();
         }
         if (!row_ok) continue;
-        gemm_store_chunk(p, row + c_off, col0, r, ncols);
+        gemm_store_chunk(p, row + c_off, col0, r, ncols, c_col);
       }
       tc_fence_before();
       __syncwarp();
@@ -454,7 +464,7 @@ static int launch_gemm(const CUtensorMap& ta, const CUtensorMap& tb, const GemmP
   }
   const int tiles_m = (p.M + kBM - 1) / kBM;
   const int tiles_n = (p.N + BN - 1) / BN;
-  const int mn_tiles = p.tile_map ? p.num_map_tiles : tiles_m * tiles_n;
+  const int mn_tiles = p.tile_map ? p.num_map_tiles : tiles_m * tiles_n * (p.heads > 0 ? p.heads : 1);
   const long long total = static_cast<long long>(mn_tiles) * p.splits;
   int grid = static_cast<int>(total < sm_count() ? total : sm_count());
   if (max_ctas > 0 && grid > max_ctas) grid = max_ctas;
@@ -477,7 +487,7 @@ static int launch_gemm_x2(const CUtensorMap& ta, const CUtensorMap& tb, const Ge
   }
   const int tiles_m = (p.M + kBM - 1) / kBM;
   const int tiles_n = (p.N + BN - 1) / BN;
-  const int mn_tiles = p.tile_map ? p.num_map_tiles : tiles_m * tiles_n;
+  const int mn_tiles = p.tile_map ? p.num_map_tiles : tiles_m * tiles_n * (p.heads > 0 ? p.heads : 1);
   const long long total = static_cast<long long>(mn_tiles) * p.splits;
   const int cap = 2 * sm_count();
   const int grid = static_cast<int>(total < cap ? total : cap);
@@ -615,7 +625,7 @@ static int gemm_bf16_impl(const void* A, const void* B, void* C, int M, int N, i
   p.labels = nullptr;
   p.partial = nullptr;
   p.row_lse = p.row_ent = p.row_glp = p.row_gent = nullptr;
-  p.chained = chained_launch_on() ? 1 : 0;
+  p.chained = chained_launch_on() && !tile_map ? 1 : 0;
   if (x2) return bn == 64 ? launch_gemm_x2<64>(ta, tb, p, stream) : launch_gemm_x2<128>(ta, tb, p, stream);
   if (bn == 64) return launch_gemm<64>(ta, tb, p, max_ctas, stream);
   if (bn == 144) return launch_gemm<144>(ta, tb, p, max_ctas, stream);
@@ -638,6 +648,44 @@ int apb_gemm_bf16_glu(const void* A, const void* B, int M, int N, int K, long lo
   if (!apb::is_glu_epilogue(epi)) return apb::kBadArgument;
   return gemm_bf16_impl(A, B, nullptr, M, N, K, lda, ldb, 0, 0, 0, epi, 1, 1.f, nullptr, C2, ldc2, nullptr, 0, nullptr, 0, 0,
                         0, stream, nullptr, 0, limit);
+}
+
+// Products per head: C[:, h c_step + n] = A[:, h a_step + k] B[h N + n, k] for h < heads, bf16; epi 0 or 11 (gate [M, heads c_step]
+// laid out like C).  The columns of A behind a head's K (up to the next multiple of 64) are read too and meet zeros; they have
+// to be finite.  N, a_step, c_step and the leading dimensions are multiples of 8.
+int apb_gemm_bf16_heads(const void* A, const void* B, void* C, int M, int N, int K, int heads, long long lda, long long ldb,
+                        long long ldc, int a_step, int c_step, int epi, const void* gate, long long ldg, cudaStream_t stream) {
+  using namespace apb;
+  if (M <= 0 || N <= 0 || K <= 0) return 0;
+  if (heads <= 0 || (N % 8) || (lda % 8) || (ldb % 8) || (ldc % 8) || (a_step % 8) || (c_step % 8) ||
+      ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(B) | reinterpret_cast<uintptr_t>(C)) & 15) ||
+      (epi != kEpiBf16 && epi != kEpiSigmoidGate) ||
+      (epi == kEpiSigmoidGate && (!gate || (ldg % 8) || (reinterpret_cast<uintptr_t>(gate) & 15))))
+    return kBadArgument;
+  const long long tm = (M + kBM - 1) / kBM;
+  const int bn = tm * ((N + 127) / 128) * heads * 10 < sm_count() * 7 ? 64 : 128;
+  CUtensorMap ta, tb;
+  int rc = make_tmap_2d(&ta, A, 2, static_cast<uint64_t>(M), static_cast<uint64_t>(heads - 1) * a_step + K, lda, 64, kBM);
+  if (rc) return 1000 + rc;
+  rc = make_tmap_2d(&tb, B, 2, static_cast<uint64_t>(heads) * N, static_cast<uint64_t>(K), ldb, 64, bn);
+  if (rc) return 2000 + rc;
+  GemmParams p{};
+  p.M = M;
+  p.N = N;
+  p.K = K;
+  p.epi = epi;
+  p.splits = 1;
+  p.C = C;
+  p.ldc = ldc;
+  p.alpha = 1.f;
+  p.heads = heads;
+  p.a_step = a_step;
+  p.c_step = c_step;
+  p.gate = static_cast<const __nv_bfloat16*>(gate);
+  p.ldg = ldg;
+  p.status = status_device_ptr();
+  p.chained = chained_launch_on() ? 1 : 0;
+  return bn == 64 ? launch_gemm<64>(ta, tb, p, 0, stream) : launch_gemm<128>(ta, tb, p, 0, stream);
 }
 
 // Grouped GEMM whose tile table was written by a kernel: `tile_map` has room for `max_tiles` entries, the number in

@@ -282,12 +282,12 @@ norm_conv_vec_kernel(const float* __restrict__ x, const T* __restrict__ gain, co
   }
 }
 
-// Final norm of selected rows: out[i] = x[rows[i]] / rms * g (rows == null: row i), with one gain (gain_step 0) or one per
-// channel (gain_step 1).  One block per row.
+// Final norm of selected rows: out[i] = x[rows[i]] / rms * (offset + g) (rows == null: row i), with one gain (gain_step 0) or
+// one per channel (gain_step 1).  One block per row.
 template <typename T>
 __global__ void __launch_bounds__(256)
 gain_norm_rows_kernel(const float* __restrict__ x, const int* __restrict__ rows, const T* __restrict__ gain,
-                      int gain_step, T* __restrict__ out, int W, float eps) {
+                      int gain_step, float offset, T* __restrict__ out, int W, float eps) {
   pdl_entry();
   __shared__ float red[8];
   const float* xr = x + static_cast<long long>(rows ? rows[blockIdx.x] : static_cast<int>(blockIdx.x)) * W;
@@ -301,7 +301,7 @@ gain_norm_rows_kernel(const float* __restrict__ x, const int* __restrict__ rows,
   for (int i = 0; i < 8; ++i) ss += red[i];
   const float f = 1.f / sqrtf(ss / W + eps);
   for (int c = threadIdx.x; c < W; c += 256)
-    out[static_cast<long long>(blockIdx.x) * W + c] = from_f32<T>(xr[c] * f * to_f32(gain[c * gain_step]));
+    out[static_cast<long long>(blockIdx.x) * W + c] = from_f32<T>(xr[c] * f * (offset + to_f32(gain[c * gain_step])));
 }
 
 // ---------------------------------------------------------------------------- q/k norm + paged cache write
@@ -428,6 +428,112 @@ rope_cache_kernel(T* __restrict__ p, long long ld, int q_col, int k_col, int v_c
   }
 }
 
+// ---------------------------------------------------------------------------- norm of whole projections + rotation + page write
+// p [rows, ld]: H query heads of D columns at q_col, G key heads at k_col, G value heads of E at v_col.  All query columns are
+// divided by their common root mean square and multiplied by wq [H D], the key columns likewise (wk [G D]); then the first
+// `rot` columns of every head are rotated, dimension i with i + rot / 2, by the angles of the row's position.  q goes back in
+// place, k and v to their cache slot.  One block per row; a thread owns V neighbouring columns and their partners.
+constexpr int kRowNormThreads = 256;
+
+template <typename T, int V>
+__device__ __forceinline__ void load_cols(const T* p, float (&v)[V]) {
+  if constexpr (V == 8) {
+    const uint4 r = *reinterpret_cast<const uint4*>(p);
+    const uint32_t w[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[i]));
+      v[2 * i] = f.x;
+      v[2 * i + 1] = f.y;
+    }
+  } else {
+    v[0] = to_f32(*p);
+  }
+}
+template <typename T, int V>
+__device__ __forceinline__ void store_cols(T* p, const float (&v)[V]) {
+  if constexpr (V == 8)
+    *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
+  else
+    *p = from_f32<T>(v[0]);
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(kRowNormThreads)
+row_norm_rope_cache_kernel(T* __restrict__ p, long long ld, int q_col, int k_col, int v_col, const T* __restrict__ wq,
+                           const T* __restrict__ wk, const int* __restrict__ row_entry, const ServeEntries e,
+                           const int* __restrict__ kv_slot, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
+                           int rot, T* __restrict__ kcache, T* __restrict__ vcache, int H, int G, int D, int E, float eps) {
+  pdl_entry();
+  __shared__ float red[2][kRowNormThreads / 32];
+  const int row = blockIdx.x;
+  const int en = row_entry ? row_entry[row] : row;
+  const int at = row - e.start[en];
+  if (at < 0 || at >= e.len[en]) return;
+  T* pr = p + static_cast<long long>(row) * ld;
+  float s[2] = {0.f, 0.f};
+  for (int i = threadIdx.x * V; i < (H + G) * D; i += kRowNormThreads * V) {
+    float v[V];
+    const bool k = i >= H * D;
+    load_cols<T, V>(k ? pr + k_col + (i - H * D) : pr + q_col + i, v);
+#pragma unroll
+    for (int j = 0; j < V; ++j) s[k ? 1 : 0] += v[j] * v[j];
+  }
+#pragma unroll
+  for (int k = 0; k < 2; ++k) {
+    s[k] = warp_sum(s[k]);
+    if ((threadIdx.x & 31) == 0) red[k][threadIdx.x >> 5] = s[k];
+  }
+  __syncthreads();
+#pragma unroll
+  for (int k = 0; k < 2; ++k) {
+    s[k] = 0.f;
+#pragma unroll
+    for (int i = 0; i < kRowNormThreads / 32; ++i) s[k] += red[k][i];
+    s[k] = 1.f / sqrtf(s[k] / ((k ? G : H) * D) + eps);
+  }
+  const int slot = kv_slot[row];
+  const long long page = slot / kServePage, off = slot % kServePage;
+  const int half = rot >> 1, per = (D - half) / V;              // units of a head: pairs of runs, then runs that are not rotated
+  const long long tr = static_cast<long long>(e.pos0[en] + at) * half;
+  for (int u = threadIdx.x; u < (H + G) * per; u += kRowNormThreads) {
+    const int hh = u / per, c = (u % per) * V;
+    const bool k = hh >= H;
+    const int head = k ? hh - H : hh;
+    if (k && slot < 0) continue;
+    const T* src = pr + (k ? k_col : q_col) + head * D;
+    const T* w = (k ? wk : wq) + head * D;
+    T* dst = k ? kcache + ((page * G + head) * kServePage + off) * D : pr + q_col + head * D;
+    const float r = s[k ? 1 : 0];
+    const int c0 = c < half ? c : c + half;
+    float a[V], g[V];
+    load_cols<T, V>(src + c0, a);
+    load_cols<T, V>(w + c0, g);
+#pragma unroll
+    for (int j = 0; j < V; ++j) a[j] *= r * g[j];
+    if (c < half) {
+      float b[V];
+      load_cols<T, V>(src + c0 + half, b);
+      load_cols<T, V>(w + c0 + half, g);
+#pragma unroll
+      for (int j = 0; j < V; ++j) {
+        b[j] *= r * g[j];
+        const float cs = cos_t[tr + c0 + j], sn = sin_t[tr + c0 + j], x = a[j];
+        a[j] = x * cs - b[j] * sn;
+        b[j] = b[j] * cs + x * sn;
+      }
+      store_cols<T, V>(dst + c0 + half, b);
+    }
+    store_cols<T, V>(dst + c0, a);
+  }
+  if (slot < 0) return;
+  for (int i = threadIdx.x * V; i < G * E; i += kRowNormThreads * V) {
+    float v[V];
+    load_cols<T, V>(pr + v_col + i, v);
+    store_cols<T, V>(vcache + ((page * G + i / E) * kServePage + off) * E + i % E, v);
+  }
+}
+
 // ---------------------------------------------------------------------------- end of a step
 // Every entry that fed tokens: remember its last token and flip the parity of its double-buffered state.
 __global__ void __launch_bounds__(128)
@@ -497,11 +603,11 @@ int apb_norm_conv(const float* x, const void* gain, const void* w1, const void* 
                              static_cast<T*>(out1), static_cast<T*>(out2), state, parity, e, tiles, W, taps, eps)));
 }
 
-int apb_gain_norm_rows(const float* x, const int* rows, const void* gain, int gain_step, void* out, int n, int W, float eps,
-                       int dtype, cudaStream_t s) {
+int apb_gain_norm_rows(const float* x, const int* rows, const void* gain, int gain_step, float offset, void* out, int n, int W,
+                       float eps, int dtype, cudaStream_t s) {
   if (n <= 0) return 0;
   APB_SERVE_DTYPE(dtype, return static_cast<int>(launch_kernel(gain_norm_rows_kernel<T>, dim3(n), dim3(256), 0, s, x, rows,
-                                                               static_cast<const T*>(gain), gain_step,
+                                                               static_cast<const T*>(gain), gain_step, offset,
                                                                static_cast<T*>(out), W, eps)));
 }
 
@@ -539,6 +645,28 @@ int apb_rope_cache(void* p, long long ld, int q_col, int k_col, int v_col, const
   if (vec) APB_ROPE(__nv_bfloat16, 8);
   APB_SERVE_DTYPE(dtype, APB_ROPE(T, 2));
 #undef APB_ROPE
+}
+
+// row_entry [rows] or null (row i belongs to entry i); wq [H D], wk [G D].
+int apb_row_norm_rope_cache(void* p, long long ld, int q_col, int k_col, int v_col, const void* wq, const void* wk,
+                            const int* row_entry, const int* e_start, const int* e_len, const int* e_slot, const int* e_pos0,
+                            const int* kv_slot, const float* cos_t, const float* sin_t, int rot, void* kcache, void* vcache,
+                            int rows, int H, int G, int D, int E, float eps, int dtype, cudaStream_t s) {
+  if (rows <= 0) return 0;
+  if (H <= 0 || G <= 0 || D <= 0 || E <= 0 || rot < 0 || (rot & 1) || rot > D || (rot && (!cos_t || !sin_t)) || !kv_slot)
+    return kBadArgument;
+  const ServeEntries e{e_start, e_len, e_slot, e_pos0};
+  const bool vec = dtype == 0 && !((D | E | q_col | k_col | v_col) & 7) && !(rot & 15) && !(ld & 7) &&
+                   !((reinterpret_cast<uintptr_t>(p) | reinterpret_cast<uintptr_t>(kcache) | reinterpret_cast<uintptr_t>(vcache) |
+                      reinterpret_cast<uintptr_t>(wq) | reinterpret_cast<uintptr_t>(wk)) & 15);
+#define APB_ROW_NORM(TT, VV)                                                                                               \
+  return static_cast<int>(launch_kernel(row_norm_rope_cache_kernel<TT, VV>, dim3(rows), dim3(kRowNormThreads), 0, s,       \
+                                        static_cast<TT*>(p), ld, q_col, k_col, v_col, static_cast<const TT*>(wq),          \
+                                        static_cast<const TT*>(wk), row_entry, e, kv_slot, cos_t, sin_t, rot,              \
+                                        static_cast<TT*>(kcache), static_cast<TT*>(vcache), H, G, D, E, eps))
+  if (vec) APB_ROW_NORM(__nv_bfloat16, 8);
+  APB_SERVE_DTYPE(dtype, APB_ROW_NORM(T, 1));
+#undef APB_ROW_NORM
 }
 
 int apb_serve_commit(const int* tokens, const int* e_start, const int* e_len, const int* e_slot, const int* e_pos0,

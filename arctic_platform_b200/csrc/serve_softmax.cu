@@ -1,10 +1,12 @@
 // Paged causal softmax attention for ragged serving batches: optional score cap, optional chunks (a query sees its own
-// chunk of positions only), one or two maps per head (differential attention).  See SoftmaxSpec.
+// chunk of positions only) and sliding windows, sinks, output gates, one or two maps per head (differential attention).  See
+// SoftmaxSpec.
 //
-// Keys and values live in pages of 16 tokens (kcache [pages, G, 16, maps * D], vcache [pages, G, 16, E]); the step's own keys
-// are already there when these kernels run, so prompts, portions of prompts and decoded tokens read the same memory.
+// Keys and values live in pages of 16 tokens (kcache [pages, G, 16, maps * D], vcache [pages, G, 16, E]; without a vcache the
+// values are the first E columns of the key rows); the step's own keys are already there when these kernels run, so prompts,
+// portions of prompts and decoded tokens read the same memory.
 //
-//  * softmax_attn_kernel      any D and E up to 512, bf16 or fp32, fp32 arithmetic throughout (the fp32 engine, odd sizes);
+//  * softmax_attn_kernel      any D up to 1024, E up to 512, bf16 or fp32, fp32 arithmetic throughout (the fp32 engine, odd sizes);
 //  * softmax_attn_mma_kernel  bf16, D and E multiples of 8, maps * D and E up to 256: m16n8k16 tensor-core tiles whose 16
 //                             rows are (query, head of one KV head, map) triples -- decoded tokens and short portions.  A
 //                             row's query is zero in the columns of the other map, so one product with the whole cache row
@@ -24,7 +26,7 @@ template <typename T, int NV, int MAPS>
 __global__ void __launch_bounds__(kSoftThreads)
 softmax_attn_kernel(const T* __restrict__ q, long long ldq, const int* __restrict__ row_entry, const ServeEntries e,
                     const int* __restrict__ page_table, int max_pages, const T* __restrict__ kcache,
-                    const T* __restrict__ vcache, T* __restrict__ out, long long ldo, int H, int G, int D, int E,
+                    const T* __restrict__ vcache, int v_row, T* __restrict__ out, long long ldo, int H, int G, int D, int E,
                     const SoftmaxSpec sp) {
   pdl_entry();
   extern __shared__ float sx_smem[];
@@ -49,7 +51,7 @@ softmax_attn_kernel(const T* __restrict__ q, long long ldq, const int* __restric
 #pragma unroll
     for (int i = 0; i < NV; ++i) acc[a][i] = 0.f;
   }
-  for (int k0 = chunk_begin(pos, sp.chunk) + warp * 32; k0 <= pos; k0 += 128) {
+  for (int k0 = visible_begin(pos, sp) + warp * 32; k0 <= pos; k0 += 128) {
     const int key = k0 + lane;
     float p[MAPS];
     long long tok = 0;                      // (page, kv head, offset) row of the key
@@ -74,7 +76,7 @@ softmax_attn_kernel(const T* __restrict__ q, long long ldq, const int* __restric
     }
     const int n = min(32, pos + 1 - k0);
     for (int j = 0; j < n; ++j) {
-      const T* vp = vcache + __shfl_sync(0xffffffffu, tok, j) * E;
+      const T* vp = vcache + __shfl_sync(0xffffffffu, tok, j) * v_row;
       float pj[MAPS];
 #pragma unroll
       for (int a = 0; a < MAPS; ++a) pj[a] = __shfl_sync(0xffffffffu, p[a], j);
@@ -109,8 +111,9 @@ softmax_attn_kernel(const T* __restrict__ q, long long ldq, const int* __restric
       f[w][a] = ml[w][a][1] > 0.f ? expf(ml[w][a][0] - mx) : 0.f;
       sum += f[w][a] * ml[w][a][1];
     }
+    const float inv = inverse_sum(sp, h, mx * 1.4426950408889634f, sum);
 #pragma unroll
-    for (int w = 0; w < 4; ++w) f[w][a] /= sum;
+    for (int w = 0; w < 4; ++w) f[w][a] *= inv;
   }
   const float lam = MAPS == 2 ? *sp.lambda : 0.f;
   float ss = 0.f;
@@ -135,7 +138,7 @@ softmax_attn_kernel(const T* __restrict__ q, long long ldq, const int* __restric
     __syncthreads();
     post = sp.post_scale / sqrtf((part[0] + part[1] + part[2] + part[3]) / E + sp.eps);
   }
-  for (int i = threadIdx.x; i < E; i += kSoftThreads) dst[i] = from_f32<T>(red[i] * post);
+  for (int i = threadIdx.x; i < E; i += kSoftThreads) dst[i] = from_f32<T>(red[i] * post * output_gate<T>(sp, row, h, i));
 }
 
 // ---------------------------------------------------------------------------- tensor-core tiles for few queries
@@ -153,7 +156,7 @@ struct SoftmaxMmaParams {
   const int* page_table;
   int max_pages;
   const __nv_bfloat16* kcache;
-  const __nv_bfloat16* vcache;
+  const __nv_bfloat16* vcache;    // null: the values are the first E columns of the key rows
   __nv_bfloat16* out;
   long long ldo;
   float* part;            // [entries, max_len, H, maps, splits, E + 2] fp32 (sums, maximum, weight sum) when splits > 1
@@ -183,9 +186,13 @@ __device__ __forceinline__ void sx_mma(float (&c)[4], const uint32_t (&a)[4], ui
 // The output stage of one (query, head): `read(a, c)` gives the normalised output of map a at column c, for the columns of
 // this lane.  One warp.
 template <typename F>
-__device__ __forceinline__ void softmax_finish(const SoftmaxSpec& sp, int E, __nv_bfloat16* dst, int lane, F read) {
+__device__ __forceinline__ void softmax_finish(const SoftmaxSpec& sp, int E, long long row, int head, __nv_bfloat16* dst,
+                                               int lane, F read) {
   if (sp.maps == 1) {
-    for (int c = lane; c < E; c += 32) dst[c] = __float2bfloat16(read(0, c));
+    const bool per_head = sp.gate_cols == 1;
+    const float g = per_head ? output_gate<__nv_bfloat16>(sp, row, head, 0) : 1.f;
+    for (int c = lane; c < E; c += 32)
+      dst[c] = __float2bfloat16(read(0, c) * (per_head ? g : output_gate<__nv_bfloat16>(sp, row, head, c)));
     return;
   }
   const float lam = *sp.lambda;
@@ -215,8 +222,10 @@ softmax_attn_mma_kernel(const SoftmaxMmaParams p) {
   const int M = p.sp.maps;
   const int DK = FULL ? NK * 16 : p.D * M, E = FULL ? NE * 16 : p.E, R = p.H / p.G, D = p.D;
   const int d16 = (DK + 15) >> 4, e16 = (E + 15) >> 4;
-  const int k_row = d16 * 32 + 16, v_row = e16 * 32 + 16;            // ring row bytes
-  const int stage_bytes = kServePage * (k_row + v_row);
+  const bool own_v = p.vcache != nullptr;
+  const int k_row = d16 * 32 + 16, v_row = own_v ? e16 * 32 + 16 : k_row;      // ring row bytes
+  const int v_off = own_v ? kServePage * k_row : 0;
+  const int stage_bytes = kServePage * k_row + (own_v ? kServePage * v_row : 0);
   const int split = blockIdx.y, splits = gridDim.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int start = p.e.start[en], pos0 = p.e.pos0[en];
@@ -234,7 +243,7 @@ softmax_attn_mma_kernel(const SoftmaxMmaParams p) {
 
   for (int f0 = blockIdx.z * 16; f0 < n_rows; f0 += gridDim.z * 16) {
     const int q_first = f0 / (R * M), q_last = (min(f0 + 16, n_rows) - 1) / (R * M);
-    const int page_lo = chunk_begin(pos0 + q_first, p.sp.chunk) / kServePage;
+    const int page_lo = visible_begin(pos0 + q_first, p.sp) / kServePage;
     const int n_pages = (pos0 + q_last + kServePage) / kServePage;   // pages up to the last query of the pass
     const int per = (n_pages - page_lo + splits - 1) / splits;
     const int p0 = page_lo + split * per, p1 = min(n_pages, p0 + per);
@@ -251,7 +260,7 @@ softmax_attn_mma_kernel(const SoftmaxMmaParams p) {
       const bool ok = f < n_rows;
       const int map = ok ? f % M : 0, qi = ok ? f / (R * M) : 0, head = g * R + (ok ? f / M % R : 0);
       hi[h] = ok ? pos0 + qi : -1;
-      lo[h] = chunk_begin(pos0 + qi, p.sp.chunk);
+      lo[h] = visible_begin(pos0 + qi, p.sp);
       const __nv_bfloat16* qp = p.q + static_cast<long long>(start + qi) * p.ldq + static_cast<long long>(head) * DK;
       const int d_lo = map * D, d_hi = d_lo + D;
 #pragma unroll
@@ -272,12 +281,13 @@ softmax_attn_mma_kernel(const SoftmaxMmaParams p) {
         const long long base = (static_cast<long long>(pages[p0 + warp + 4 * j]) * p.G + g) * kServePage;
         const uint32_t dst = ring + (j % kSxStages) * stage_bytes;
         const __nv_bfloat16* kp = p.kcache + base * DK;
-        const __nv_bfloat16* vp = p.vcache + base * E;
 #pragma unroll
         for (int i = lane; i < kServePage * kc; i += 32) sx_cp_async16(dst + (i / kc) * k_row + (i % kc) * 16, kp + i * 8);
+        if (own_v) {
+          const __nv_bfloat16* vp = p.vcache + base * E;
 #pragma unroll
-        for (int i = lane; i < kServePage * vc; i += 32)
-          sx_cp_async16(dst + kServePage * k_row + (i / vc) * v_row + (i % vc) * 16, vp + i * 8);
+          for (int i = lane; i < kServePage * vc; i += 32) sx_cp_async16(dst + v_off + (i / vc) * v_row + (i % vc) * 16, vp + i * 8);
+        }
       }
       asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -289,7 +299,7 @@ softmax_attn_mma_kernel(const SoftmaxMmaParams p) {
       asm volatile("cp.async.wait_group %0;" ::"n"(kSxStages - 1) : "memory");
       __syncwarp();
       const uint32_t ks_addr = ring + (j % kSxStages) * stage_bytes;
-      const uint32_t vs_addr = ks_addr + kServePage * k_row;
+      const uint32_t vs_addr = ks_addr + v_off;
       float sc[2][4];
 #pragma unroll
       for (int nt = 0; nt < 2; ++nt) sc[nt][0] = sc[nt][1] = sc[nt][2] = sc[nt][3] = 0.f;
@@ -409,8 +419,8 @@ softmax_attn_mma_kernel(const SoftmaxMmaParams p) {
           }
         }
       } else {
-        const float i0 = 1.f / sum[0], i1 = M == 2 ? 1.f / sum[1] : 0.f;
-        softmax_finish(p.sp, E, p.out + static_cast<long long>(start + qi) * p.ldo + static_cast<long long>(head) * E, lane,
+        const float i0 = inverse_sum(p.sp, head, mx[0], sum[0]), i1 = M == 2 ? 1.f / sum[1] : 0.f;
+        softmax_finish(p.sp, E, start + qi, head, p.out + static_cast<long long>(start + qi) * p.ldo + static_cast<long long>(head) * E, lane,
                        [&](int a, int c) { return total(a, c) * (a ? i1 : i0); });
       }
     }
@@ -440,9 +450,9 @@ softmax_merge_kernel(const SoftmaxMmaParams p, int n_entries, int splits) {
     float sum = 0.f;
     for (int i = 0; i < splits; ++i)
       if (s[i * (E + 2) + E + 1] > 0.f) sum += exp2f(s[i * (E + 2) + E] - mx[a]) * s[i * (E + 2) + E + 1];
-    inv[a] = 1.f / sum;
+    inv[a] = inverse_sum(p.sp, head, mx[a], sum);
   }
-  softmax_finish(p.sp, E, p.out + static_cast<long long>(p.e.start[en] + qi) * p.ldo + static_cast<long long>(head) * E, lane,
+  softmax_finish(p.sp, E, p.e.start[en] + qi, head, p.out + static_cast<long long>(p.e.start[en] + qi) * p.ldo + static_cast<long long>(head) * E, lane,
                  [&](int a, int c) {
                    const float* s = src + a * splits * (E + 2);
                    const float top = a ? mx[1] : mx[0];
@@ -463,19 +473,22 @@ using namespace apb;
 int apb_softmax_attn(const void* q, long long ldq, const int* row_entry, const int* e_start, const int* e_len,
                      const int* e_slot, const int* e_pos0, const int* page_table, int max_pages, const void* kcache,
                      const void* vcache, void* out, long long ldo, int rows, int H, int G, int D, int E, float scale,
-                     float cap, int chunk, int maps, const float* lambda, float post_scale, float eps, int dtype,
-                     cudaStream_t s) {
+                     float cap, int chunk, int maps, const float* lambda, float post_scale, float eps, int window,
+                     const float* sink, const void* gate, long long ldg, int gate_cols, int dtype, cudaStream_t s) {
   if (rows <= 0) return 0;
-  if (H <= 0 || G <= 0 || H % G || D <= 0 || E <= 0 || D > 512 || E > 512 || maps < 1 || maps > 2 || (maps == 2 && !lambda) ||
-      chunk < 0)
+  if (H <= 0 || G <= 0 || H % G || D <= 0 || E <= 0 || D > 1024 || E > 512 || maps < 1 || maps > 2 || (maps == 2 && !lambda) ||
+      chunk < 0 || window < 0 || (maps == 2 && (sink || gate)) || (!vcache && E > maps * D) ||
+      (gate && gate_cols != 1 && gate_cols != E))
     return kBadArgument;
+  const int v_row = vcache ? E : maps * D;
+  if (!vcache) vcache = kcache;
   const ServeEntries e{e_start, e_len, e_slot, e_pos0};
-  const SoftmaxSpec sp{scale, cap, chunk, maps, lambda, post_scale, eps};
-  const size_t smem = maps * (D + 4 * E) * sizeof(float);              // at most 20 KB
+  const SoftmaxSpec sp{scale, cap, chunk, maps, lambda, post_scale, eps, window, sink, gate, ldg, gate_cols};
+  const size_t smem = maps * (D + 4 * E) * sizeof(float);              // at most 24 KB
 #define APB_SX(NVV, MM)                                                                                              \
   return static_cast<int>(launch_kernel(softmax_attn_kernel<T, NVV, MM>, dim3(rows, H), dim3(kSoftThreads), smem, s, \
                                         static_cast<const T*>(q), ldq, row_entry, e, page_table, max_pages,          \
-                                        static_cast<const T*>(kcache), static_cast<const T*>(vcache),                \
+                                        static_cast<const T*>(kcache), static_cast<const T*>(vcache), v_row,         \
                                         static_cast<T*>(out), ldo, H, G, D, E, sp))
   APB_SERVE_DTYPE(dtype, if (maps == 2 && E <= 128) APB_SX(4, 2); if (maps == 2) APB_SX(16, 2);
                   if (E <= 128) APB_SX(4, 1); APB_SX(16, 1));
@@ -488,18 +501,20 @@ int apb_softmax_attn_mma(const void* q, long long ldq, const int* e_start, const
                          const int* e_pos0, int n_entries, const int* page_table, int max_pages, const void* kcache,
                          const void* vcache, void* out, long long ldo, float* part, int H, int G, int D, int E, int min_len,
                          int max_len, int splits, float scale, float cap, int chunk, int maps, const float* lambda,
-                         float post_scale, float eps, cudaStream_t s) {
+                         float post_scale, float eps, int window, const float* sink, const void* gate, long long ldg,
+                         int gate_cols, cudaStream_t s) {
   if (n_entries <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G || D <= 0 || E <= 0 || (D % 8) || (E % 8) || maps < 1 || maps > 2 || maps * D > 256 || E > 256 ||
       (ldq % 8) || (reinterpret_cast<uintptr_t>(q) & 15) || min_len < 1 || max_len < min_len || splits < 1 ||
-      (splits > 1 && !part) || (maps == 2 && !lambda) || chunk < 0)
+      (splits > 1 && !part) || (maps == 2 && !lambda) || chunk < 0 || window < 0 || (maps == 2 && (sink || gate)) ||
+      (!vcache && E > maps * D) || (gate && gate_cols != 1 && gate_cols != E))
     return kBadArgument;
   SoftmaxMmaParams p{static_cast<const __nv_bfloat16*>(q), ldq, ServeEntries{e_start, e_len, e_slot, e_pos0}, page_table,
                      max_pages, static_cast<const __nv_bfloat16*>(kcache), static_cast<const __nv_bfloat16*>(vcache),
                      static_cast<__nv_bfloat16*>(out), ldo, part, H, G, D, E, min_len, max_len,
-                     SoftmaxSpec{scale, cap, chunk, maps, lambda, post_scale, eps}};
+                     SoftmaxSpec{scale, cap, chunk, maps, lambda, post_scale, eps, window, sink, gate, ldg, gate_cols}};
   const int DK = maps * D, d16 = (DK + 15) / 16, e16 = (E + 15) / 16;
-  const int ring = 4 * kSxStages * kServePage * (d16 * 32 + e16 * 32 + 32), sums = 4 * 16 * e16 * 16 * 4;
+  const int ring = 4 * kSxStages * kServePage * (d16 * 32 + 16 + (vcache ? e16 * 32 + 16 : 0)), sums = 4 * 16 * e16 * 16 * 4;
   const int smem = ring > sums ? ring : sums;
   const int passes = static_cast<int>((static_cast<long long>(max_len) * (H / G) * maps + 15) / 16);
   const dim3 grid(n_entries * G, splits, passes < 256 ? passes : 256);

@@ -370,7 +370,7 @@ int apb_softmax_attn_tc(const void* q, long long ldq, int rows, const int* work,
   rc = make_tmap_2d(&tv, vcache, 2, cache_rows, E, E, 64, kServePage);
   if (rc) return 3000 + rc;
   SoftmaxTcParams p{work, page_table, max_pages, static_cast<__nv_bfloat16*>(out), ldo, G, D, E,
-                    SoftmaxSpec{scale, cap, 0, 2, lambda, post_scale, eps}, status_device_ptr()};
+                    SoftmaxSpec{scale, cap, 0, 2, lambda, post_scale, eps, 0, nullptr, nullptr, 0, 0}, status_device_ptr()};
   const cudaError_t e = cudaFuncSetAttribute(softmax_attn_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kXtcSmem);
   if (e != cudaSuccess) return static_cast<int>(e);
   softmax_attn_tc_kernel<<<n_work, kXtcThreads, kXtcSmem, stream>>>(tq, tk, tv, p);

@@ -4,8 +4,8 @@
 allocator, slots, sampling kernels, CUDA-graph decode loop, ``generate`` -- with the layers and their memory supplied by
 the model through a small protocol (``models/registry.py`` lists the architectures):
 
-* ``model.cache_layout()``       what each layer run keeps per sequence: paged K/V with its own head sizes (or the run
-                                 whose pages it reads), an fp32 recurrent state, the history of a short convolution (any
+* ``model.cache_layout()``       what each layer run keeps per sequence: paged K/V with its own head sizes (value size 0: key
+                                 rows only; or the run whose pages it reads), an fp32 recurrent state, the history of a short convolution (any
                                  of them may be absent);
 * ``model.prepare_serving(n)``   tables for ``n`` positions;
 * ``model.serve_rows(batch, cache)``   one pass over a ragged :class:`~arctic_platform_b200.ops.serving.StepBatch`,
@@ -54,7 +54,7 @@ class StateCache:
                 continue
             # zero-filled: the unwritten tail of a last page is multiplied by weight 0 and must be finite
             self.k.append(torch.zeros((pages, kv[0], PAGE, kv[1]), device=device, dtype=dtype) if kv else None)
-            self.v.append(torch.zeros((pages, kv[0], PAGE, kv[2]), device=device, dtype=dtype) if kv else None)
+            self.v.append(torch.zeros((pages, kv[0], PAGE, kv[2]), device=device, dtype=dtype) if kv and kv[2] else None)
             self.state.append(torch.zeros((slots,) + tuple(st), **f32) if st else None)
             self.conv.append(torch.zeros((slots, 2) + tuple(cv), **f32) if cv and cv[0] else None)
         self.prev = torch.zeros(slots, device=device, dtype=torch.int32)      # last token fed

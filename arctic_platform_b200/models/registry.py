@@ -23,6 +23,8 @@ register_architecture("Reninex", "arctic_platform_b200.models.reninex", "Reninex
                       ("serve_attention", "serve_attention_tc", "retention", "retention_mma"))
 register_architecture("Rigulorn", "arctic_platform_b200.models.rigulorn", "RigulornConfig", "RigulornLM",
                       ("serve_streams", "serve_softmax", "serve_softmax_tc", "ssm", "ssm_mma"))
+register_architecture("Titatar", "arctic_platform_b200.models.titatar", "TitatarConfig", "TitatarLM",
+                      ("serve_residual", "serve_latent", "serve_moe", "serve_softmax"))
 
 
 def kernel_sources(architecture: str) -> Tuple[str, ...]:

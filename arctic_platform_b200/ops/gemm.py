@@ -21,6 +21,7 @@ EPI_F32_ACCUM = 3
 EPI_SWIGLU = 4
 EPI_GEGLU = 9
 EPI_CLAMP_GLU = 10
+EPI_SIGMOID_GATE = 11
 
 
 def _check2d(t: torch.Tensor, name: str) -> None:

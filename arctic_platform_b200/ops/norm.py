@@ -8,6 +8,8 @@ the place of the Liger kernels patched in by the reference
 """
 from __future__ import annotations
 
+import math
+from dataclasses import dataclass
 from typing import Optional, Tuple
 
 import torch
@@ -25,10 +27,29 @@ def rmsnorm_ref(x, w, eps: float, res=None, w_offset: float = 0.0):
     return y.to(x.dtype), xs.to(x.dtype)
 
 
-def rope_tables(max_pos: int, dim: int, theta: float, device) -> Tuple[torch.Tensor, torch.Tensor]:
-    inv = 1.0 / (theta ** (torch.arange(0, dim, 2, dtype=torch.float64) / dim))
+@dataclass(frozen=True)
+class Yarn:
+    """Rotary frequencies stretched for contexts beyond ``original`` positions: pairs that turn more than ``fast`` times over them
+    keep their frequency, pairs that turn less than ``slow`` times are slowed down by ``factor``, with a linear blend over the
+    pairs between; cos and sin grow by ``0.1 ln(factor) + 1``."""
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+    def apply(self, inv: torch.Tensor, dim: int, theta: float) -> Tuple[torch.Tensor, float]:
+        at = lambda turns: dim * math.log(self.original / (2.0 * math.pi * turns)) / (2.0 * math.log(theta))
+        lo, hi = max(math.floor(at(self.fast)), 0), min(math.ceil(at(self.slow)), dim - 1)
+        slowed = ((torch.arange(dim // 2, dtype=torch.float64) - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+        return inv / self.factor * slowed + inv * (1.0 - slowed), 0.1 * math.log(self.factor) + 1.0
+
+
+def rope_tables(max_pos: int, dim: int, theta: float, device, yarn: Optional[Yarn] = None) -> Tuple[torch.Tensor, torch.Tensor]:
+    inv, gain = 1.0 / (theta ** (torch.arange(0, dim, 2, dtype=torch.float64) / dim)), 1.0
+    if yarn is not None:
+        inv, gain = yarn.apply(inv, dim, theta)
     ang = torch.arange(max_pos, dtype=torch.float64)[:, None] * inv[None, :]
-    return ang.cos().float().to(device).contiguous(), ang.sin().float().to(device).contiguous()
+    return (ang.cos() * gain).float().to(device).contiguous(), (ang.sin() * gain).float().to(device).contiguous()
 
 
 def qknorm_rope_ref(q, k, wq, wk, cos_t, sin_t, pos, eps: float):

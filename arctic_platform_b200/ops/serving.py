@@ -2,7 +2,7 @@
 
 A step advances several sequences at once, each by its own run of new tokens: a portion of a prompt of any length, or
 one decoded token.  :class:`StepBatch` is the device-side description of such a step; the functions below launch the
-kernels of ``serve_*.cu``, ``retention*.cu``, ``ssm*.cu`` and ``gemm_simt.cu`` on it.  They take bf16 or fp32 activations;
+kernels of ``serve_*.cu``, ``retention*.cu``, ``ssm*.cu`` and ``gemm_*.cu`` on it.  They take bf16 or fp32 activations;
 the residual streams and all carried state are fp32.
 """
 from __future__ import annotations
@@ -31,12 +31,24 @@ def _fn(name: str):
             "apb_embed_hash": [vp] * 9 + [ll, ll, ll, i, i, f, i, vp, vp, ll, vp, i, vp, i, i, vp],
             "apb_loop_begin": [vp, vp, i, i, vp, ll, i, vp],
             "apb_norm_conv": [vp] * 13 + [i, i, i, f, i, vp],
-            "apb_gain_norm_rows": [vp, vp, vp, i, vp, i, i, f, i, vp],
+            "apb_gain_norm_rows": [vp, vp, vp, i, f, vp, i, i, f, i, vp],
             "apb_qk_norm_cache": [vp, ll, i, i, i, vp, vp, vp, i, i, i, i, i, f, i, vp],
             "apb_rope_cache": [vp, ll, i, i, i] + [vp] * 8 + [i, vp, vp] + [i] * 7 + [vp],
             "apb_stream_step": [vp] * 7 + [i] * 5 + [f, i, vp],
-            "apb_softmax_attn": [vp, ll] + [vp] * 6 + [i, vp, vp, vp, ll] + [i] * 5 + [f, f, i, i, vp, f, f, i, vp],
-            "apb_softmax_attn_mma": [vp, ll] + [vp] * 4 + [i, vp, i, vp, vp, vp, ll, vp] + [i] * 7 + [f, f, i, i, vp, f, f, vp],
+            "apb_softmax_attn": [vp, ll] + [vp] * 6 + [i, vp, vp, vp, ll] + [i] * 5 + [f, f, i, i, vp, f, f, i, vp, vp, ll, i, i, vp],
+            "apb_softmax_attn_mma": [vp, ll] + [vp] * 4 + [i, vp, i, vp, vp, vp, ll, vp] + [i] * 7
+                                    + [f, f, i, i, vp, f, f, i, vp, vp, ll, i, vp],
+            "apb_row_norm_rope_cache": [vp, ll, i, i, i] + [vp] * 10 + [i, vp, vp] + [i] * 5 + [f, i, vp],
+            "apb_residual_step": [vp] * 7 + [i, f] + [vp] * 5 + [i, i, i, f, f, i, i, i, vp],
+            "apb_latent_norm_cache": [vp, ll, i, i] + [vp] * 11 + [i, i, i, i, f, i, vp],
+            "apb_latent_rotate": [vp, ll] + [vp] * 8 + [i] * 6 + [vp],
+            "apb_latent_gather": [vp, vp, i, vp, i, vp, vp, i, i, vp],
+            "apb_moe_serve_route": [vp, ll, vp, vp, i, i, i, i] + [vp] * 9 + [i, i, i, i, vp],
+            "apb_moe_serve_gather": [vp, i, ll, vp, vp, vp, i, vp, vp, vp],
+            "apb_gemm_simt_grouped": [vp, vp, vp, i, i, i, ll, ll, ll, i, vp, ll, vp, i, vp, i, vp],
+            "apb_gemm_simt_heads": [vp, vp, vp, i, i, i, i, ll, ll, ll, ll, ll, i, vp, ll, i, vp],
+            "apb_gemm_bf16_grouped_dev": [vp, vp, vp, i, i, i, ll, ll, ll, i, f, vp, ll, vp, i, vp, ll, vp],
+            "apb_gemm_bf16_heads": [vp, vp, vp, i, i, i, i, ll, ll, ll, i, i, i, vp, ll, vp],
             "apb_softmax_attn_tc": [vp, ll, i, vp, i, vp, i, vp, vp, i, vp, ll, i, i, i, i, f, f, vp, f, f, vp],
             "apb_ssm": [vp, ll, i, i, vp, vp, i] + [vp] * 6 + [ll] + [vp] * 7 + [i, vp] + [i] * 8 + [vp],
             "apb_ssm_mma": [vp, ll] + [vp] * 9 + [i, vp, vp, vp] + [i] * 5 + [vp],
@@ -96,6 +108,7 @@ class StepBatch:
     tables: Dict[tuple, torch.Tensor] = field(default_factory=dict)       # derived tables, on the device / host
     host_tables: Dict[tuple, dict] = field(default_factory=dict)
     host: Optional[np.ndarray] = None      # [entries, 4] start, len, slot, pos0 (None for a captured decode step)
+    parts: Dict[tuple, "StepBatch"] = field(default_factory=dict)
 
     @staticmethod
     def plan(entries: Sequence[StepEntry]) -> Dict[str, np.ndarray]:
@@ -142,6 +155,21 @@ class StepBatch:
             self.tables[key] = to_device(torch.from_numpy(make()).pin_memory(), self.tokens.device)
         return self.tables[key]
 
+    def part(self, e0: int, e1: int) -> "StepBatch":
+        """The entries ``[e0, e1)`` as a batch of their own over rows that start at 0 (views of this one)."""
+        if self.host is None or (e0, e1) == (0, self.n_entries):
+            return self
+        if (e0, e1) not in self.parts:
+            host = self.host[e0:e1].copy()
+            r0, r1 = int(host[0, 0]), int(host[-1, 0] + host[-1, 1])
+            host[:, 0] -= r0
+            lens = host[:, 1]
+            self.parts[e0, e1] = StepBatch(
+                r1 - r0, e1 - e0, self.tokens[r0:r1], self.row_entry[r0:r1] - e0, self.start[e0:e1] - r0, self.len[e0:e1],
+                self.slot[e0:e1], self.pos0[e0:e1], self.page_table[e0:e1], self.kv_slot[r0:r1], None,
+                bool((lens == 1).any()), bool((lens > 1).any()), host=host)
+        return self.parts[e0, e1]
+
     def entry_ptrs(self):
         return _lib.ptr(self.start), _lib.ptr(self.len), _lib.ptr(self.slot), _lib.ptr(self.pos0)
 
@@ -181,10 +209,13 @@ def norm_conv(b: StepBatch, x: torch.Tensor, gain: torch.Tensor, w1: Optional[to
     return o1, o2
 
 
-def gain_norm_rows(x: torch.Tensor, rows: Optional[torch.Tensor], gain: torch.Tensor, eps: float) -> torch.Tensor:
+def gain_norm_rows(x: torch.Tensor, rows: Optional[torch.Tensor], gain: torch.Tensor, eps: float,
+                   offset: float = 0.0) -> torch.Tensor:
+    """``x / rms(x) * (offset + gain)`` of some rows, in the activation type."""
     n = x.shape[0] if rows is None else rows.shape[0]
     out = torch.empty((n, x.shape[1]), device=x.device, dtype=gain.dtype)
-    _call("apb_gain_norm_rows", _lib.ptr(x), _lib.ptr(rows), _lib.ptr(gain), int(gain.numel() > 1), _lib.ptr(out), n, x.shape[1], float(eps),
+    _call("apb_gain_norm_rows", _lib.ptr(x), _lib.ptr(rows), _lib.ptr(gain), int(gain.numel() > 1), float(offset),
+          _lib.ptr(out), n, x.shape[1], float(eps),
           dtype_code(gain.dtype))
     return out
 
@@ -207,6 +238,47 @@ def rope_cache(b: StepBatch, p: torch.Tensor, cols: Tuple[int, ...], rope: Tuple
     _call("apb_rope_cache", _lib.ptr(p), p.stride(0), q_col, k_col, v_col, _lib.ptr(b.row_entry), *b.entry_ptrs(),
           _lib.ptr(b.kv_slot), _lib.ptr(rope[0]), _lib.ptr(rope[1]), rot_dims, _lib.ptr(kcache), _lib.ptr(vcache), b.rows,
           q_heads, G * (kcache.shape[3] // dim) if write else 0, G, dim, E, dtype_code(p.dtype))
+
+
+def row_norm_rope_cache(b: StepBatch, p: torch.Tensor, cols: Tuple[int, int, int], wq: torch.Tensor, wk: torch.Tensor,
+                        rope: Tuple[torch.Tensor, torch.Tensor], rot_dims: int, heads: int, kcache: torch.Tensor,
+                        vcache: torch.Tensor, eps: float) -> None:
+    """q and k columns of ``p`` normed over the whole projection (weights ``wq``, ``wk``), then the first ``rot_dims`` of every
+    head rotated (dimension i with i + rot_dims / 2); q in place, k and v into the page cache."""
+    G, D, E = kcache.shape[1], kcache.shape[3], vcache.shape[3]
+    _call("apb_row_norm_rope_cache", _lib.ptr(p), p.stride(0), *cols, _lib.ptr(wq), _lib.ptr(wk), _lib.ptr(b.row_entry),
+          *b.entry_ptrs(), _lib.ptr(b.kv_slot), _lib.ptr(rope[0]), _lib.ptr(rope[1]), rot_dims, _lib.ptr(kcache), _lib.ptr(vcache),
+          b.rows, heads, G, D, E, float(eps), dtype_code(p.dtype))
+
+
+# --------------------------------------------------------------------------------------------- normed residual
+@dataclass
+class ExpertMix:
+    """Output of a mixture of experts that has not been summed yet: rows ``out [slots, W]`` of the routed experts with the
+    rows ``slots [rows, top]`` (-1: none) and ``weights [rows, top]`` of every token, and ``ident [rows]`` times its input."""
+    out: torch.Tensor
+    slots: torch.Tensor
+    weights: torch.Tensor
+    ident: torch.Tensor
+    h: torch.Tensor
+
+
+def residual_step(x: torch.Tensor, y: Optional[torch.Tensor], post: Optional[torch.Tensor], pre: Optional[torch.Tensor], eps: float,
+                  *, mix: Optional[ExpertMix] = None, offset: float = 1.0, again: Optional[tuple] = None, write: bool = True,
+                  clear: bool = False, dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+    """One pass over the residual ``x [rows, W]`` (fp32): ``x <- x + s / rms(s) * (offset + post)`` with ``s`` = ``y`` (fp32) plus
+    the sum of ``mix`` (both may be absent; without ``post`` s itself), plus the embedding output if ``again`` = (tokens, table,
+    scale) is given; then ``x / rms(x) * (offset + pre)`` in the activation type, without ``pre`` the fp32 x.  ``write`` False
+    leaves ``x`` as it was; ``clear`` zeroes ``y`` after reading it."""
+    T, W = x.shape
+    dt = next((t.dtype for t in (pre, post) if t is not None), dtype)
+    out = torch.empty((T, W), device=x.device, dtype=dt if pre is not None else torch.float32)
+    tok, table, scale = again or (None, None, 0.0)
+    m = (mix.out, mix.slots, mix.weights, mix.ident, mix.h) if mix is not None else (None,) * 5
+    _call("apb_residual_step", _lib.ptr(x), _lib.ptr(y), _lib.ptr(post), _lib.ptr(pre), _lib.ptr(out), _lib.ptr(tok), _lib.ptr(table),
+          0 if table is None else table.shape[0], float(scale), *(_lib.ptr(t) for t in m), 0 if mix is None else mix.slots.shape[1],
+          T, W, float(offset), float(eps), int(write), int(clear), dtype_code(dt or torch.float32))
+    return out
 
 
 # --------------------------------------------------------------------------------------------- parallel residual streams
@@ -278,6 +350,11 @@ def gate_up_gelu(x: torch.Tensor, w_gu: torch.Tensor, out: torch.Tensor) -> None
     gate_up(x, w_gu, out, gemm.EPI_GEGLU)
 
 
+def gate_up_silu(x: torch.Tensor, w_gu: torch.Tensor, out: torch.Tensor) -> None:
+    """silu(gate) * up."""
+    gate_up(x, w_gu, out, gemm.EPI_SWIGLU)
+
+
 def gate_up_clamped(x: torch.Tensor, w_gu: torch.Tensor, out: torch.Tensor, limit: float) -> None:
     """g sigmoid(1.702 g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit)."""
     gate_up(x, w_gu, out, gemm.EPI_CLAMP_GLU, limit)
@@ -303,6 +380,68 @@ def _gemm_simt(a, w, out, epi, out2=None, limit=0.0) -> None:
     _call("apb_gemm_simt", _lib.ptr(a), _lib.ptr(w), _lib.ptr(out), a.shape[0], w.shape[0], a.shape[1], a.stride(0),
           w.stride(0), 0 if out is None else out.stride(0), epi, None, _lib.ptr(out2),
           0 if out2 is None else out2.stride(0), float(limit), dtype_code(a.dtype))
+
+
+def heads_linear(a: torch.Tensor, a_step: int, w: torch.Tensor, heads: int, k: int, out: torch.Tensor, out_step: int,
+                 gate: Optional[torch.Tensor] = None) -> None:
+    """Product per head: ``out[:, h out_step + n] = a[:, h a_step + k] w[h N + n, k]``, optionally times the sigmoid of ``gate``
+    (laid out like ``out``).  Behind a head's ``k`` columns ``a`` holds finite values."""
+    N = w.shape[0] // heads
+    gp, gs = (_lib.ptr(gate), gate.stride(0)) if gate is not None else (None, 0)
+    epi = gemm.EPI_SIGMOID_GATE if gate is not None else gemm.EPI_BF16
+    odd = _simt(a, w, out) or N % 8 or a_step % 8 or out_step % 8
+    if gate is not None:
+        odd = odd or gate.stride(0) % 8 or gate.data_ptr() & 15
+    args = (_lib.ptr(a), _lib.ptr(w), _lib.ptr(out), a.shape[0], N, k, heads, a.stride(0), w.stride(0), out.stride(0), a_step,
+            out_step, epi, gp, gs)
+    if odd:
+        _call("apb_gemm_simt_heads", *args, dtype_code(a.dtype))
+    else:
+        _call("apb_gemm_bf16_heads", *args)
+
+
+# --------------------------------------------------------------------------------------------- mixture of experts
+def experts(b: StepBatch, h: torch.Tensor, logits: torch.Tensor, correction: Optional[torch.Tensor], counters: torch.Tensor,
+            w_gu: torch.Tensor, w_down: torch.Tensor, n: int, n_experts: int, top: int, ff: int) -> ExpertMix:
+    """Routes every row of ``h`` by its fp32 ``logits`` (``n`` scores, the first ``n_experts`` of them experts with weights, the
+    others identity experts) and runs the gated SiLU experts as two grouped products.  ``w_gu [experts * 2 ff, W]`` (gate and up
+    interleaved), ``w_down [experts * W, >= ff]``; ``counters [experts + 1]`` int32 are zero between calls."""
+    T, W = h.shape
+    dev, E, P = h.device, n_experts, T * top
+    I, ldf = 2 * ff, w_down.shape[1]
+    simt = h.dtype == torch.float32 or bool(W % 8 or I % 16 or w_gu.stride(0) % 8 or ldf % 8)
+    tile = 64 if simt else 128
+    blocks = (P + tile - 1) // tile + min(E, P)
+    max1, max2 = blocks * ((I + tile - 1) // tile), blocks * ((W + tile - 1) // tile)
+    i32 = dict(device=dev, dtype=torch.int32)
+    f32 = dict(device=dev, dtype=torch.float32)
+    o1 = (3 * P + E + 2 + 3) // 4 * 4                                             # tile tables on 16-byte boundaries
+    ints = torch.empty(o1 + 4 * (max1 + max2), **i32)                             # one allocation for all tables
+    expert, rank, slots = (ints[i * P:(i + 1) * P].view(T, top) for i in range(3))
+    first, n_tiles = ints[3 * P:3 * P + E], ints[3 * P + E:3 * P + E + 2]
+    tiles1, tiles2 = ints[o1:o1 + 4 * max1], ints[o1 + 4 * max1:o1 + 4 * (max1 + max2)]
+    weights, ident = torch.empty((T, top), **f32), torch.empty(T, **f32)
+    _call("apb_moe_serve_route", _lib.ptr(logits), logits.stride(0), _lib.ptr(correction), _lib.ptr(b.kv_slot), T, n, E, top,
+          _lib.ptr(expert), _lib.ptr(rank), _lib.ptr(weights), _lib.ptr(ident), _lib.ptr(counters), _lib.ptr(first), _lib.ptr(tiles1),
+          _lib.ptr(tiles2), _lib.ptr(n_tiles), I, W, tile, dtype_code(h.dtype))
+    xs = torch.empty((P, W), device=dev, dtype=h.dtype)
+    _call("apb_moe_serve_gather", _lib.ptr(h), T, W * h.element_size(), _lib.ptr(expert), _lib.ptr(rank), _lib.ptr(first), top,
+          _lib.ptr(slots), _lib.ptr(xs))
+    act = (torch.zeros if ldf != ff else torch.empty)((P, ldf), device=dev, dtype=h.dtype)
+    out = torch.empty((P, W), device=dev, dtype=h.dtype)
+    n1, n2 = _lib.ptr(n_tiles), _lib.ptr(n_tiles[1:])
+    if simt:
+        dt = dtype_code(h.dtype)
+        _call("apb_gemm_simt_grouped", _lib.ptr(xs), _lib.ptr(w_gu), None, P, I, W, W, w_gu.stride(0), 0, gemm.EPI_SWIGLU, _lib.ptr(act),
+              ldf, _lib.ptr(tiles1), max1, n1, dt)
+        _call("apb_gemm_simt_grouped", _lib.ptr(act), _lib.ptr(w_down), _lib.ptr(out), P, W, ff, ldf, w_down.stride(0), W, gemm.EPI_BF16,
+              None, 0, _lib.ptr(tiles2), max2, n2, dt)
+    else:
+        _call("apb_gemm_bf16_grouped_dev", _lib.ptr(xs), _lib.ptr(w_gu), None, P, I, W, W, w_gu.stride(0), 0, gemm.EPI_SWIGLU, 1.0,
+              _lib.ptr(act), ldf, _lib.ptr(tiles1), max1, n1, w_gu.shape[0])
+        _call("apb_gemm_bf16_grouped_dev", _lib.ptr(act), _lib.ptr(w_down), _lib.ptr(out), P, W, ff, ldf, w_down.stride(0), W,
+              gemm.EPI_BF16, 1.0, None, 0, _lib.ptr(tiles2), max2, n2, w_down.shape[0])
+    return ExpertMix(out, slots, weights, ident, h)
 
 
 # --------------------------------------------------------------------------------------------- sequence mixers
@@ -379,14 +518,15 @@ def sigmoid_attention(b: StepBatch, q: torch.Tensor, heads: int, kcache: torch.T
 @dataclass(frozen=True)
 class SoftmaxSpec:
     """Softmax attention over the page cache: ``score = scale q.k``, capped to ``cap tanh(score / cap)`` (0: no cap), chunks of
-    ``chunk`` positions (0: none).  ``maps`` 2: differential attention, ``out = o / rms(o) * post_scale`` with
-    ``o = a1 - lambda a2``."""
+    ``chunk`` positions and windows of the last ``window`` positions (0: none).  ``maps`` 2: differential attention,
+    ``out = o / rms(o) * post_scale`` with ``o = a1 - lambda a2``."""
     scale: float
     cap: float = 0.0
     chunk: int = 0
     maps: int = 1
     post_scale: float = 1.0
     eps: float = 1e-5
+    window: int = 0
 
 
 MAX_FIXED_CAP = 64.0    # the tcgen05 kernel's bound on the score cap
@@ -422,13 +562,19 @@ def chunk_tiles(host: np.ndarray, heads: int, kv_heads: int, min_len: int, chunk
     return np.ascontiguousarray(work[np.argsort(work[:, 6] - work[:, 5] - work[:, 4], kind="stable")], dtype=np.int32)
 
 
-def softmax_attention(b: StepBatch, q: torch.Tensor, heads: int, kcache: torch.Tensor, vcache: torch.Tensor,
-                      spec: SoftmaxSpec, lam: Optional[torch.Tensor], out: torch.Tensor) -> None:
+def softmax_attention(b: StepBatch, q: torch.Tensor, heads: int, kcache: torch.Tensor, vcache: Optional[torch.Tensor],
+                      spec: SoftmaxSpec, lam: Optional[torch.Tensor], out: torch.Tensor, *, vdim: int = 0,
+                      sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, gate_cols: int = 1) -> None:
     """``q [rows, heads * maps * D]`` (column slice, rotated) over the entries' pages -> ``out [rows, heads * E]`` (column
-    slice).  bf16 with head sizes that are multiples of 8 runs on tensor cores; fp32 and odd sizes on CUDA cores."""
-    G, DK, E = kcache.shape[1], kcache.shape[3], vcache.shape[3]
+    slice).  Without a ``vcache`` the values are the first ``vdim`` columns of the key rows.  ``sink [heads]`` fp32: a score per
+    head that counts in the denominator only; ``gate``: columns of the activations whose sigmoid multiplies the output, one per
+    head (``gate_cols`` 1) or one per output column (``gate_cols`` E).
+    bf16 with head sizes that are multiples of 8 runs on tensor cores; fp32 and odd sizes on CUDA cores."""
+    G, DK = kcache.shape[1], kcache.shape[3]
+    E = vdim if vcache is None else vcache.shape[3]
     D = DK // spec.maps
-    tail = (float(spec.scale), float(spec.cap), spec.chunk, spec.maps, _lib.ptr(lam), float(spec.post_scale), float(spec.eps))
+    shape = (float(spec.scale), float(spec.cap), spec.chunk, spec.maps, _lib.ptr(lam), float(spec.post_scale), float(spec.eps))
+    tail = shape + (spec.window, _lib.ptr(sink), _lib.ptr(gate), 0 if gate is None else gate.stride(0), gate_cols)
     aligned = not (D % 8 or E % 8 or q.stride(0) % 8 or out.stride(0) % 8 or (q.data_ptr() | out.data_ptr()) & 15)
     if q.dtype != torch.bfloat16 or not aligned or max(DK, E) > 256:
         _call("apb_softmax_attn", _lib.ptr(q), q.stride(0), _lib.ptr(b.row_entry), *b.entry_ptrs(), _lib.ptr(b.page_table),
@@ -452,7 +598,76 @@ def softmax_attention(b: StepBatch, q: torch.Tensor, heads: int, kcache: torch.T
         work = b.table(("softmax", heads, G, spec.chunk), lambda: chunk_tiles(b.host, heads, G, limit + 1, spec.chunk))
         _call("apb_softmax_attn_tc", _lib.ptr(q), q.stride(0), b.rows, _lib.ptr(work), work.shape[0], _lib.ptr(b.page_table),
               b.page_table.stride(0), _lib.ptr(kcache), _lib.ptr(vcache), kcache.shape[0], _lib.ptr(out), out.stride(0), heads,
-              G, D, E, *tail[:2], *tail[4:])
+              G, D, E, *shape[:2], *shape[4:])
+
+
+# --------------------------------------------------------------------------------------------- latent attention
+@dataclass(frozen=True)
+class LatentSpec:
+    """Latent attention: heads of ``dim`` plain and ``rot`` rotated query / key columns and ``vdim`` value columns; the cache
+    keeps ``rank`` latent and ``rot`` rotated key columns per token, shared by all heads."""
+    heads: int
+    dim: int
+    rot: int
+    vdim: int
+    rank: int
+    scale: float
+
+
+def latent_norm_cache(b: StepBatch, p: torch.Tensor, q_col: int, c_col: int, q_gain: torch.Tensor, c_gain: torch.Tensor,
+                      rope: Tuple[torch.Tensor, torch.Tensor], cache: torch.Tensor, eps: float) -> None:
+    """Norm of the query latent (columns ``q_col`` of ``p``, in place) and of the key / value latent (``c_col``), rotation of the
+    shared key part behind it; both go to the page cache ``[pages, 1, PAGE, rank + rot]``."""
+    Q, C = q_gain.numel(), c_gain.numel()
+    _call("apb_latent_norm_cache", _lib.ptr(p), p.stride(0), q_col, c_col, _lib.ptr(q_gain), _lib.ptr(c_gain), _lib.ptr(b.row_entry),
+          *b.entry_ptrs(), _lib.ptr(b.kv_slot), _lib.ptr(rope[0]), _lib.ptr(rope[1]), _lib.ptr(cache), b.rows, Q, C,
+          cache.shape[3] - C, float(eps), dtype_code(p.dtype))
+
+
+def latent_rotate(b: StepBatch, q: torch.Tensor, s: LatentSpec, rope: Tuple[torch.Tensor, torch.Tensor],
+                  dst: Optional[torch.Tensor] = None) -> None:
+    """Rotates the rotated part of every head of ``q [rows, heads * (dim + rot)]``, in place or into the last ``rot`` columns of
+    the heads of ``dst [rows, heads * (rank + rot)]``."""
+    _call("apb_latent_rotate", _lib.ptr(q), q.stride(0), _lib.ptr(b.row_entry), *b.entry_ptrs(), _lib.ptr(rope[0]), _lib.ptr(rope[1]),
+          _lib.ptr(dst), b.rows, s.heads, s.dim, s.rot, s.rank, dtype_code(q.dtype))
+
+
+def entry_runs(host: Optional[np.ndarray], n_entries: int, limit: int) -> list:
+    """Maximal runs ``(e0, e1)`` of neighbouring entries of at most ``limit`` rows (no host table: all entries are single rows)."""
+    if host is None:
+        return [(0, n_entries)]
+    out, e0 = [], None
+    for e, n in enumerate(host[:, 1].tolist() + [limit + 1]):
+        if n <= limit and e0 is None:
+            e0 = e
+        elif n > limit and e0 is not None:
+            out.append((e0, e))
+            e0 = None
+    return out
+
+
+def latent_attention(b: StepBatch, q: torch.Tensor, s: LatentSpec, cache: torch.Tensor, w_absorb: torch.Tensor,
+                     w_expand: torch.Tensor, sink: Optional[torch.Tensor], gate: Optional[torch.Tensor],
+                     rope: Tuple[torch.Tensor, torch.Tensor], out: torch.Tensor) -> None:
+    """``q [rows, heads * (dim + rot)]`` (not rotated yet) over the entries' latents -> ``out [rows, heads * vdim]`` (column
+    slice), times the sigmoid of the ``gate`` columns.  ``w_expand`` holds the key rows (heads * dim) and then the value rows
+    (heads * vdim) over the latent, ``w_absorb [heads * rank, dim]`` the key rows transposed per head.
+
+    The key projection is applied to the query and the value projection to the weighted sum of the latents."""
+    H, D, R, C, E = s.heads, s.dim, s.rot, s.rank, s.vdim
+    spec = SoftmaxSpec(s.scale)
+    w_value = w_expand[w_expand.shape[0] - H * E:]
+    limit = b.rows
+    for e0, e1 in entry_runs(b.host, b.n_entries, limit):
+        p = b.part(e0, e1)
+        r0 = 0 if b.host is None else int(b.host[e0, 0])
+        rows = slice(r0, r0 + p.rows)
+        ql = torch.empty((p.rows, H * (C + R)), device=q.device, dtype=q.dtype)
+        heads_linear(q[rows], D + R, w_absorb, H, D, ql, C + R)
+        latent_rotate(p, q[rows], s, rope, ql)
+        o = torch.empty((p.rows, H * C), device=q.device, dtype=q.dtype)
+        softmax_attention(p, ql, H, cache, None, spec, None, o, vdim=C, sink=sink)
+        heads_linear(o, C, w_value, H, C, out[rows], E, None if gate is None else gate[rows])
 
 
 MIN_SEGMENT = 256       # tokens; a multiple of the kernel's chunk
