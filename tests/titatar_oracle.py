@@ -7,8 +7,7 @@ by name and returns ``(logits [T, V], residual stream after every layer run [run
 
 ``faults`` (a set of names) plants a deliberate mistake, so that a test can show that its inputs would reveal one:
 ``window_early`` / ``window_late`` (the window one token shorter / longer), ``no_window``, ``no_sink``, ``no_head_sink``,
-``sink_scaled`` (a learned sink multiplied like a score), ``no_gate``, ``gate_after`` (the gate behind the output projection is
-left out), ``head_norm`` (q and k normalised per head), ``norm_after_rotation``, ``neighbour_pairs`` (pairs (2i, 2i + 1) in the
+``sink_scaled`` (a learned sink multiplied like a score), ``no_gate``, ``head_norm`` (q and k normalised per head), ``norm_after_rotation``, ``neighbour_pairs`` (pairs (2i, 2i + 1) in the
 grouped attention), ``half_pairs`` (pairs (i, i + dims/2) in the latent attention), ``no_yarn``, ``no_yarn_gain``,
 ``yarn_scale`` (the score scale multiplied by the squared gain too), ``first_rotated`` (the rotated part in front of a query
 head), ``rot_normed`` (the norm of the latent spans the rotated key part), ``no_latent_norm``, ``plain_gain`` (layer norms
