@@ -1,0 +1,373 @@
+// Causal softmax attention on tcgen05 tensor cores for long portions of prompts: one map, optional sliding window, sinks and
+// output gates (see SoftmaxSpec), no bound on the scores.
+//
+// A CTA = two tiles of 128 query rows that share their keys: two query heads of one KV head on the same rows, or two
+// consecutive row tiles of one head.  320 threads: warp 0 TMA producer, warp 1 MMA issuer, warps 2-5 and 6-9 the weight groups,
+// one per tile, which ping-pong on the tensor core.
+//
+// Keys and values come from the page cache (16-row boxes, one page of one KV head each) or from a contiguous copy of the
+// entry's context (128-row boxes; a head's columns side by side).  A key may have a second part that all heads share (the
+// rotated part of latent attention), read through a tensor map of its own; queries hold both parts side by side.
+//
+// K and V travel in chunks of 64 columns x 128 keys through one ring.  The weights are taken relative to a reference that
+// follows the running maximum only when it falls behind by more than 2^8: the products of all key blocks accumulate in tensor
+// memory and are rescaled there on those rare occasions.
+#include "common.cuh"
+#include "host_utils.cuh"
+#include "serve_softmax.cuh"
+
+namespace apb {
+
+constexpr int kFlThreads = 320;
+constexpr int kFlKeys = 128;                           // keys per block
+constexpr int kFlChunk = 128 * 64 * 2;                 // 64 columns of 128 rows
+constexpr int kFlChunks = 14;                          // query chunks and ring slots together
+constexpr int kFlMaxRing = 12;
+constexpr int kFlSmem = kFlChunks * kFlChunk + 1024 + 512;
+constexpr float kFlLag = 8.f;                          // in log2: how far the reference may lag behind the maximum
+
+struct FlashParams {
+  const int* work;        // [n][12]: entry, KV head, first key of the walk (a multiple of the page size), row of the entry's key 0 in
+                          // the contiguous copy; then per tile: first row, valid rows (0: no second tile), head, position
+  const int* page_table;  // null: contiguous keys
+  int max_pages;
+  __nv_bfloat16* out;
+  long long ldo;
+  int G, D, R, E;         // R: columns of the shared second part
+  SoftmaxSpec sp;
+  int* status;
+};
+
+__global__ void __launch_bounds__(kFlThreads, 1)
+flash_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_k,
+                const __grid_constant__ CUtensorMap tma_k2, const __grid_constant__ CUtensorMap tma_v, const FlashParams p) {
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  uint64_t* full = reinterpret_cast<uint64_t*>(smem + kFlChunks * kFlChunk);
+  uint64_t* empty = full + kFlMaxRing;
+  uint64_t* q_full = empty + kFlMaxRing;
+  uint64_t* s_full = q_full + 1;    // [2] scores of a tile are in tensor memory
+  uint64_t* p_full = s_full + 2;    // [2] its weights are
+  uint64_t* o_full = p_full + 2;    // [2] every product of the tile has completed
+  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(o_full + 2);
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int* w = p.work + static_cast<long long>(blockIdx.x) * 12;
+  const int entry = w[0], kvh = w[1], k0 = w[2], base_row = w[3];
+  const int n_tiles = w[9] > 0 ? 2 : 1;
+  const int k1 = (p.D + 63) >> 6, kch = k1 + ((p.R + 63) >> 6), vch = (p.E + 63) >> 6;
+  const int ring = min(kFlMaxRing, kFlChunks - 2 * kch), per = kch + vch;
+  uint8_t* smem_q = smem;                              // [2 tiles][kch]
+  uint8_t* smem_kv = smem + 2 * kch * kFlChunk;
+  auto blocks_of = [&](int g) { return (w[4 + 4 * g + 3] + w[4 + 4 * g + 1] - k0 + kFlKeys - 1) / kFlKeys; };
+  const int nb0 = blocks_of(0), nb1 = n_tiles == 2 ? blocks_of(1) : 0, n_blocks = max(nb0, nb1);
+
+  if (threadIdx.x == 0) {
+    for (int s = 0; s < ring; ++s) {
+      mbar_init(&full[s], 1);
+      mbar_init(&empty[s], 1);
+    }
+    mbar_init(q_full, 1);
+    for (int g = 0; g < 2; ++g) {
+      mbar_init(&s_full[g], 1);
+      mbar_init(&p_full[g], 128);
+      mbar_init(&o_full[g], 1);
+    }
+    mbar_fence_init();
+  }
+  if (warp == 1) {
+    tmem_alloc(tmem_holder, 512);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_base = *tmem_holder;
+  // TMEM: S / P of tile g at columns [g * 128, +128), O of tile g at [256 + g * 128, +E)
+
+  if (warp == 0) {
+    // ---------------------------------------------------------------- producer (lanes 0-7: one page each)
+    if (lane == 0) {
+      mbar_expect_tx(q_full, n_tiles * kch * kFlChunk);
+      for (int g = 0; g < n_tiles; ++g)
+        for (int c = 0; c < kch; ++c)
+          tma_load_2d(smem_q + (g * kch + c) * kFlChunk, &tma_q, q_full,
+                      w[4 + 4 * g + 2] * (p.D + p.R) + (c < k1 ? c * 64 : p.D + (c - k1) * 64), w[4 + 4 * g]);
+    }
+    // paged: the blocks' tails beyond the last key repeat the last page (their weights are 0)
+    const bool paged = p.page_table != nullptr;
+    const int last = max(w[7] + w[5], n_tiles == 2 ? w[11] + w[9] : 0);                 // keys of the walk's end
+    const int page0 = k0 / kServePage, n_pages = (last + kServePage - 1) / kServePage;
+    const int* pages = p.page_table + static_cast<long long>(entry) * p.max_pages;
+    bool ok = true;
+    int n = 0;
+    for (int j = 0; j < n_blocks && ok; ++j) {
+      int row = 0;
+      if (paged && lane < kFlKeys / kServePage)
+        row = (pages[min(page0 + j * (kFlKeys / kServePage) + lane, n_pages - 1)] * p.G + kvh) * kServePage;
+      for (int c = 0; c < per; ++c, ++n) {
+        const int slot = n % ring;
+        ok = mbar_wait(&empty[slot], ((n / ring) & 1) ^ 1, p.status, kTimeoutEmpty);
+        ok = __all_sync(0xffffffffu, ok);
+        if (!ok) break;
+        if (lane == 0) mbar_expect_tx(&full[slot], kFlChunk);
+        __syncwarp();
+        uint8_t* dst = smem_kv + slot * kFlChunk;
+        const bool second = c >= k1 && c < kch;
+        const CUtensorMap* map = c < k1 ? &tma_k : second ? &tma_k2 : &tma_v;
+        const int col = c < k1 ? c * 64 : second ? (c - k1) * 64 : (c - kch) * 64;
+        if (paged) {
+          if (lane < kFlKeys / kServePage) tma_load_2d(dst + lane * (kServePage * 128), map, &full[slot], col, row);
+        } else if (lane == 0) {
+          tma_load_2d(dst, map, &full[slot], second ? col : kvh * (c < k1 ? p.D : p.E) + col, base_row + k0 + j * kFlKeys);
+        }
+      }
+    }
+    if (!ok) {                         // give copies in flight time to land before the block ends
+      const uint64_t t0 = global_timer_ns();
+      while (global_timer_ns() - t0 < 100000ull) {
+      }
+    }
+  } else if (warp == 1) {
+    // ---------------------------------------------------------------- MMA issuer
+    if (lane == 0) {
+      const int e16 = (p.E + 15) & ~15;
+      const uint32_t idesc_s = umma_idesc_bf16(128, kFlKeys, 0, 0);
+      const uint32_t idesc_o = umma_idesc_bf16(128, e16, 0, 1);
+      const uint32_t idesc_lo = umma_idesc_bf16(128, 64, 0, 1), idesc_hi = umma_idesc_bf16(128, e16 - 64 > 0 ? e16 - 64 : 16, 0, 1);
+      const uint32_t kv = smem_u32(smem_kv);
+      bool ok = mbar_wait(q_full, 0, p.status, kTimeoutFull);
+      auto wait_item = [&](int n) { return mbar_wait(&full[n % ring], (n / ring) & 1, p.status, kTimeoutFull); };
+      auto wait_items = [&](int n, int count) {
+        for (int c = 0; c < count; ++c)
+          if (!wait_item(n + c)) return false;
+        return true;
+      };
+      auto release = [&](int n, int count) {
+        for (int c = 0; c < count; ++c) tc_commit(&empty[(n + c) % ring]);
+      };
+      auto issue_s = [&](int g, int n) {               // n: ring item of the block's first key chunk
+        uint32_t more = 0;
+        for (int c = 0; c < kch; ++c) {
+          const uint32_t qa = smem_u32(smem_q + (g * kch + c) * kFlChunk), ka = kv + ((n + c) % ring) * kFlChunk;
+          const int cols = c < k1 ? min(64, p.D - c * 64) : min(64, p.R - (c - k1) * 64);
+          for (int k = 0; k < cols >> 4; ++k) {
+            umma_bf16_ss(tmem_base + g * 128, umma_smem_desc(qa + k * 32, 0, 1024), umma_smem_desc(ka + k * 32, 0, 1024), idesc_s, more);
+            more = 1;
+          }
+        }
+        tc_commit(&s_full[g]);
+      };
+      auto issue_o = [&](int g, int n, bool first_block) {
+        const uint32_t t_o = tmem_base + 256 + g * 128, t_p = tmem_base + g * 128;
+        const int s0 = n % ring;
+        if (vch == 1 || s0 + 1 < ring) {
+          const uint32_t va = kv + s0 * kFlChunk;
+#pragma unroll
+          for (int k = 0; k < kFlKeys / 16; ++k)
+            umma_bf16_ts(t_o, t_p + k * 8, umma_smem_desc(va + k * 2048, kFlChunk, 1024), idesc_o, first_block && k == 0 ? 0u : 1u);
+        } else {                                       // the value chunks lie at both ends of the ring
+          const uint32_t va = kv + s0 * kFlChunk;
+          for (int k = 0; k < kFlKeys / 16; ++k)
+            umma_bf16_ts(t_o, t_p + k * 8, umma_smem_desc(va + k * 2048, kFlChunk, 1024), idesc_lo, first_block && k == 0 ? 0u : 1u);
+          for (int k = 0; k < kFlKeys / 16; ++k)
+            umma_bf16_ts(t_o + 64, t_p + k * 8, umma_smem_desc(kv + k * 2048, kFlChunk, 1024), idesc_hi, first_block && k == 0 ? 0u : 1u);
+        }
+      };
+      if (ok) ok = wait_items(0, kch);
+      if (ok) {
+        tc_fence_after();
+        for (int g = 0; g < n_tiles; ++g) issue_s(g, 0);
+        release(0, kch);
+      }
+      for (int j = 0; j < n_blocks && ok; ++j) {
+        const int nv = j * per + kch, nk = (j + 1) * per;
+        const bool more = j + 1 < n_blocks;
+        if (!wait_items(nv, vch) || (more && !wait_items(nk, kch))) {
+          ok = false;
+          break;
+        }
+        tc_fence_after();
+        for (int g = 0; g < n_tiles; ++g) {
+          const int nb = g ? nb1 : nb0;
+          if (j >= nb) continue;
+          if (!mbar_wait(&p_full[g], j & 1, p.status, kTimeoutTmemEmpty)) {
+            ok = false;
+            break;
+          }
+          tc_fence_after();
+          issue_o(g, nv, j == 0);
+          if (j + 1 < nb)
+            issue_s(g, nk);                            // runs after the product above has read the weights
+          else
+            tc_commit(&o_full[g]);
+        }
+        if (!ok) break;
+        release(nv, vch);
+        if (more) release(nk, kch);
+      }
+    }
+  } else if (((warp - 2) >> 2) < n_tiles) {
+    // ---------------------------------------------------------------- weight groups, one per tile
+    const int g = (warp - 2) >> 2;
+    const int quarter = warp & 3, row = quarter * 32 + lane;
+    const int row0 = w[4 + 4 * g], valid = w[4 + 4 * g + 1], head = w[4 + 4 * g + 2], pos0 = w[4 + 4 * g + 3];
+    const int nb = g ? nb1 : nb0, window = p.sp.window;
+    const uint32_t lane_off = static_cast<uint32_t>(quarter * 32) << 16;
+    const uint32_t t_s = tmem_base + lane_off + g * 128, t_o = tmem_base + lane_off + 256 + g * 128;
+    const float scale = p.sp.scale * 1.4426950408889634f;
+    const uint64_t scale2 = xtc_pair(scale, scale);
+    const int pos = pos0 + min(row, valid - 1);
+    float ref = -INFINITY;                             // reference of the weights (log2)
+    uint64_t sum2 = xtc_pair(0.f, 0.f);
+    bool ok = true;
+    for (int j = 0; j < nb; ++j) {
+      if (!mbar_wait(&s_full[g], j & 1, p.status, kTimeoutTmemFull)) {
+        ok = false;
+        break;
+      }
+      tc_fence_after();
+      const int base = k0 + j * kFlKeys;                                 // position of the block's first key
+      const int limit = pos + 1 - base;                                  // visible keys: [skip, limit) of the block
+      const int skip = window > 0 ? pos + 1 - window - base : 0;
+      const bool whole = pos0 + 1 - base >= kFlKeys && (window <= 0 || pos0 + valid - window - base <= 0);   // all 128 for every row
+      uint32_t pk[4][16];
+      for (int pass = 0; pass < 2; ++pass) {           // a second time if the reference had to move
+        const float off = ref == -INFINITY ? 0.f : -ref;
+        const uint64_t off2 = xtc_pair(off, off);
+        float top = -INFINITY;                         // largest score relative to the reference
+        uint64_t block2 = xtc_pair(0.f, 0.f);
+        uint32_t stage[2][32];
+        tmem_ld_32x32(t_s, stage[0]);
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {                  // the next 32 scores are on their way while these are worked on
+          uint32_t(&r)[32] = stage[c & 1];
+          xtc_wait_load(r);
+          if (c < 3) tmem_ld_32x32(t_s + (c + 1) * 32, stage[(c + 1) & 1]);
+#pragma unroll
+          for (int i = 0; i < 16; ++i) {
+            float2 v = xtc_unpair(xtc_fma2(xtc_pair(__uint_as_float(r[2 * i]), __uint_as_float(r[2 * i + 1])), scale2, off2));
+            if (!whole) {
+              const int a = c * 32 + 2 * i;
+              if (a >= limit || a < skip) v.x = -INFINITY;
+              if (a + 1 >= limit || a + 1 < skip) v.y = -INFINITY;
+            }
+            top = fmaxf(fmaxf(top, v.x), v.y);
+            const float w0 = xtc_ex2(v.x), w1 = xtc_ex2(v.y);
+            block2 = xtc_add2(block2, xtc_pair(w0, w1));
+            pk[c][i] = pack_bf16x2(w0, w1);
+          }
+        }
+        const bool behind = top > kFlLag || (ref == -INFINITY && top > -INFINITY);
+        if (pass == 1 || !__any_sync(0xffffffffu, behind)) {
+          sum2 = xtc_add2(sum2, block2);
+          break;
+        }
+        const float next = fmaxf(ref, top - off);
+        const float f = ref == next ? 1.f : xtc_ex2(ref - next);         // 0 while nothing has been seen
+        ref = next;
+        sum2 = xtc_mul2(sum2, xtc_pair(f, f));
+        if (j > 0) {                                   // the products of the blocks before have completed: S_j came behind them
+          for (int c = 0; c < p.E; c += 32) {
+            uint32_t o[32];
+            tmem_ld_32x32(t_o + c, o);
+            xtc_wait_load(o);
+#pragma unroll
+            for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * f);
+            tmem_st_32x32(t_o + c, o);
+          }
+        }
+      }
+#pragma unroll
+      for (int c = 0; c < 4; ++c) tmem_st_32x16(t_s + c * 16, pk[c]);
+      tmem_st_wait();
+      tc_fence_before();
+      mbar_arrive(&p_full[g]);
+    }
+    if (ok) ok = mbar_wait(&o_full[g], 0, p.status, kTimeoutTmemFull);
+    if (ok) {
+      tc_fence_after();
+      const float2 halves = xtc_unpair(sum2);
+      const long long t = static_cast<long long>(row0) + row;
+      const bool live = row < valid, per_column = p.sp.gate && p.sp.gate_cols != 1;
+      const float inv = live ? inverse_sum(p.sp, head, ref, halves.x + halves.y) * (per_column ? 1.f : output_gate<__nv_bfloat16>(p.sp, t, head, 0))
+                             : 0.f;
+      __nv_bfloat16* dst = p.out + t * p.ldo + static_cast<long long>(head) * p.E;
+      const __nv_bfloat16* gate = static_cast<const __nv_bfloat16*>(p.sp.gate) + t * p.sp.ldg + static_cast<long long>(head) * p.E;
+#pragma unroll 1
+      for (int c = 0; c < p.E; c += 32) {
+        uint32_t o[32];
+        tmem_ld_32x32(t_o + c, o);
+        xtc_wait_load(o);
+        if (!live) continue;
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+          if (c + q * 8 >= p.E) continue;
+          float v[8];
+#pragma unroll
+          for (int i = 0; i < 8; ++i) v[i] = __uint_as_float(o[q * 8 + i]) * inv;
+          if (per_column) {
+            const uint4 raw = *reinterpret_cast<const uint4*>(gate + c + q * 8);
+            const uint32_t gw[4] = {raw.x, raw.y, raw.z, raw.w};
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+              const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gw[i]));
+              v[2 * i] /= 1.f + __expf(-f.x);
+              v[2 * i + 1] /= 1.f + __expf(-f.y);
+            }
+          }
+          *reinterpret_cast<uint4*>(dst + c + q * 8) =
+              make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
+        }
+      }
+      tc_fence_before();
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem_base, 512);
+  }
+}
+
+}  // namespace apb
+
+extern "C" {
+
+// q: [rows, H * (D + R)] columns of a row-major buffer (row stride ldq); out [rows, H * E] (row stride ldo), 16-byte aligned rows.
+// With a page table: k [pages, G, 16, D], v [pages, G, 16, E], key_rows = pages * G * 16, R = 0.  Without: k [key_rows, G * D]
+// (row stride ldk), k2 [key_rows, R] (contiguous, R > 0), v [key_rows, G * E] (ldv).  D and R multiples of 16, at most 4 chunks of
+// 64 columns together, E a multiple of 8 up to 128; gate (if any): rows of 16-byte aligned columns.
+int apb_flash_tc(const void* q, long long ldq, int rows, const int* work, int n_work, const int* page_table, int max_pages,
+                 const void* k, long long ldk, const void* k2, const void* v, long long ldv, long long key_rows, void* out,
+                 long long ldo, int H, int G, int D, int R, int E, float scale, int window, const float* sink, const void* gate,
+                 long long ldg, int gate_cols, cudaStream_t stream) {
+  using namespace apb;
+  if (n_work <= 0) return 0;
+  const int kch = (D + 63) / 64 + (R + 63) / 64;
+  if (H <= 0 || G <= 0 || H % G || D <= 0 || R < 0 || E <= 0 || (D % 16) || (R % 16) || (E % 8) || kch > 4 || E > 128 ||
+      (ldq % 8) || (ldo % 8) || (ldk % 8) || (ldv % 8) || key_rows <= 0 || !work || (page_table && R) || (R && !k2) || window < 0 ||
+      ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(k) |
+        reinterpret_cast<uintptr_t>(k2) | reinterpret_cast<uintptr_t>(v)) & 15) ||
+      (gate && gate_cols != 1 && (gate_cols != E || (ldg % 8) || (reinterpret_cast<uintptr_t>(gate) & 15))))
+    return kBadArgument;
+  CUtensorMap tq, tk, tk2, tv;
+  const int box = page_table ? kServePage : kFlKeys, heads = page_table ? 1 : G;
+  int rc = make_tmap_2d(&tq, q, 2, rows, static_cast<uint64_t>(H) * (D + R), ldq, 64, 128);
+  if (rc) return 1000 + rc;
+  rc = make_tmap_2d(&tk, k, 2, key_rows, static_cast<uint64_t>(heads) * D, ldk, 64, box);
+  if (rc) return 2000 + rc;
+  rc = R ? make_tmap_2d(&tk2, k2, 2, key_rows, R, R, 64, box) : 0;
+  if (rc) return 3000 + rc;
+  if (!R) tk2 = tk;
+  rc = make_tmap_2d(&tv, v, 2, key_rows, static_cast<uint64_t>(heads) * E, ldv, 64, box);
+  if (rc) return 4000 + rc;
+  const FlashParams p{work, page_table, max_pages, static_cast<__nv_bfloat16*>(out), ldo, G, D, R, E,
+                      SoftmaxSpec{scale, 0.f, 0, 1, nullptr, 1.f, 0.f, window, sink, gate, ldg, gate_cols}, status_device_ptr()};
+  const cudaError_t e = cudaFuncSetAttribute(flash_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kFlSmem);
+  if (e != cudaSuccess) return static_cast<int>(e);
+  flash_tc_kernel<<<n_work, kFlThreads, kFlSmem, stream>>>(tq, tk, tk2, tv, p);
+  return static_cast<int>(cudaGetLastError());
+}
+}

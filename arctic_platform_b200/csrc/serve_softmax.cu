@@ -15,7 +15,7 @@
 // Long portions run on tcgen05 (serve_softmax_tc.cu).
 #include "common.cuh"
 #include "host_utils.cuh"
-#include "serve_softmax.cuh"
+#include "serve_softmax_mma.cuh"
 
 namespace apb {
 
@@ -148,66 +148,6 @@ softmax_attn_kernel(const T* __restrict__ q, long long ldq, const int* __restric
 // m16n8k16 MMAs; the warps' sums are combined at the end.  Ring rows are an odd multiple of 16 bytes apart, so the 8 rows of
 // an ldmatrix tile fall into different banks.
 constexpr int kSxStages = 3;
-
-struct SoftmaxMmaParams {
-  const __nv_bfloat16* q;
-  long long ldq;
-  ServeEntries e;
-  const int* page_table;
-  int max_pages;
-  const __nv_bfloat16* kcache;
-  const __nv_bfloat16* vcache;    // null: the values are the first E columns of the key rows
-  __nv_bfloat16* out;
-  long long ldo;
-  float* part;            // [entries, max_len, H, maps, splits, E + 2] fp32 (sums, maximum, weight sum) when splits > 1
-  int H, G, D, E, min_len, max_len;
-  SoftmaxSpec sp;
-};
-
-__device__ __forceinline__ void sx_cp_async16(uint32_t dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
-}
-__device__ __forceinline__ void sx_ldsm_x4(uint32_t addr, uint32_t (&r)[4]) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void sx_ldsm_x4_t(uint32_t addr, uint32_t (&r)[4]) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void sx_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
-      "{%0, %1, %2, %3};"
-      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-
-// The output stage of one (query, head): `read(a, c)` gives the normalised output of map a at column c, for the columns of
-// this lane.  One warp.
-template <typename F>
-__device__ __forceinline__ void softmax_finish(const SoftmaxSpec& sp, int E, long long row, int head, __nv_bfloat16* dst,
-                                               int lane, F read) {
-  if (sp.maps == 1) {
-    const bool per_head = sp.gate_cols == 1;
-    const float g = per_head ? output_gate<__nv_bfloat16>(sp, row, head, 0) : 1.f;
-    for (int c = lane; c < E; c += 32)
-      dst[c] = __float2bfloat16(read(0, c) * (per_head ? g : output_gate<__nv_bfloat16>(sp, row, head, c)));
-    return;
-  }
-  const float lam = *sp.lambda;
-  float o[8], ss = 0.f;                      // E <= 256
-#pragma unroll
-  for (int i = 0; i < 8; ++i) {
-    const int c = lane + i * 32;
-    o[i] = c < E ? read(0, c) - lam * read(1, c) : 0.f;
-    ss += o[i] * o[i];
-  }
-  const float post = sp.post_scale / sqrtf(warp_sum(ss) / E + sp.eps);
-#pragma unroll
-  for (int i = 0; i < 8; ++i)
-    if (lane + i * 32 < E) dst[lane + i * 32] = __float2bfloat16(o[i] * post);
-}
 
 // NK, NE: upper bounds of maps * D / 16 and E / 16; FULL: both are equal to them (constant index arithmetic).
 // RUNNING: keep a running maximum (no score cap, or a large one); otherwise the scores' reference is fixed.
@@ -463,6 +403,12 @@ softmax_merge_kernel(const SoftmaxMmaParams p, int n_entries, int splits) {
                  });
 }
 
+int launch_softmax_merge(const SoftmaxMmaParams& p, int n_entries, int splits, cudaStream_t s) {
+  const long long warps = static_cast<long long>(n_entries) * p.max_len * p.H;
+  return static_cast<int>(launch_kernel(softmax_merge_kernel, dim3(static_cast<unsigned>((warps + 7) / 8)), dim3(256), 0, s, p,
+                                        n_entries, splits));
+}
+
 }  // namespace apb
 
 extern "C" {
@@ -539,7 +485,6 @@ int apb_softmax_attn_mma(const void* q, long long ldq, const int* e_start, const
     rc = n16 <= 4 ? run(softmax_attn_mma_kernel<4, 4, false, true>)
          : n16 <= 8 ? run(softmax_attn_mma_kernel<8, 8, false, true>) : run(softmax_attn_mma_kernel<16, 16, false, true>);
   if (rc || splits == 1) return rc;
-  const int mg = static_cast<int>((static_cast<long long>(n_entries) * max_len * H * 32 + 255) / 256);
-  return static_cast<int>(launch_kernel(softmax_merge_kernel, dim3(mg), dim3(256), 0, s, p, n_entries, splits));
+  return launch_softmax_merge(p, n_entries, splits, s);
 }
 }

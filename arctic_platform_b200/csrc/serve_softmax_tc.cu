@@ -39,47 +39,6 @@ struct SoftmaxTcParams {
   int* status;
 };
 
-__device__ __forceinline__ float xtc_ex2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-// Pairs of fp32 values in one 64-bit register: half the issue slots of the scalar forms.
-__device__ __forceinline__ uint64_t xtc_pair(float lo, float hi) {
-  uint64_t v;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(v) : "f"(lo), "f"(hi));
-  return v;
-}
-__device__ __forceinline__ float2 xtc_unpair(uint64_t v) {
-  float2 f;
-  asm("mov.b64 {%0, %1}, %2;" : "=f"(f.x), "=f"(f.y) : "l"(v));
-  return f;
-}
-__device__ __forceinline__ uint64_t xtc_mul2(uint64_t a, uint64_t b) {
-  uint64_t v;
-  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(v) : "l"(a), "l"(b));
-  return v;
-}
-__device__ __forceinline__ uint64_t xtc_fma2(uint64_t a, uint64_t b, uint64_t c) {
-  uint64_t v;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(v) : "l"(a), "l"(b), "l"(c));
-  return v;
-}
-__device__ __forceinline__ uint64_t xtc_add2(uint64_t a, uint64_t b) {
-  uint64_t v;
-  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(v) : "l"(a), "l"(b));
-  return v;
-}
-// Waits for a tensor-memory load into r; nothing that reads r can move in front of it.
-__device__ __forceinline__ void xtc_wait_load(uint32_t (&r)[32]) {
-  asm volatile("tcgen05.wait::ld.sync.aligned;"
-               : "+r"(r[0]), "+r"(r[1]), "+r"(r[2]), "+r"(r[3]), "+r"(r[4]), "+r"(r[5]), "+r"(r[6]), "+r"(r[7]),
-               "+r"(r[8]), "+r"(r[9]), "+r"(r[10]), "+r"(r[11]), "+r"(r[12]), "+r"(r[13]), "+r"(r[14]),
-               "+r"(r[15]), "+r"(r[16]), "+r"(r[17]), "+r"(r[18]), "+r"(r[19]), "+r"(r[20]), "+r"(r[21]),
-               "+r"(r[22]), "+r"(r[23]), "+r"(r[24]), "+r"(r[25]), "+r"(r[26]), "+r"(r[27]), "+r"(r[28]),
-               "+r"(r[29]), "+r"(r[30]), "+r"(r[31])
-               :: "memory");
-}
 __device__ __forceinline__ void xtc_group_barrier() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
 
 __global__ void __launch_bounds__(kXtcThreads, 1)

@@ -24,7 +24,7 @@ register_architecture("Reninex", "arctic_platform_b200.models.reninex", "Reninex
 register_architecture("Rigulorn", "arctic_platform_b200.models.rigulorn", "RigulornConfig", "RigulornLM",
                       ("serve_streams", "serve_softmax", "serve_softmax_tc", "ssm", "ssm_mma"))
 register_architecture("Titatar", "arctic_platform_b200.models.titatar", "TitatarConfig", "TitatarLM",
-                      ("serve_residual", "serve_latent", "serve_moe", "serve_softmax"))
+                      ("serve_residual", "serve_latent", "serve_moe", "serve_softmax", "serve_softmax_wide", "serve_flash_tc"))
 
 
 def kernel_sources(architecture: str) -> Tuple[str, ...]:

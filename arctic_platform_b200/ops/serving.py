@@ -49,6 +49,8 @@ def _fn(name: str):
             "apb_gemm_simt_heads": [vp, vp, vp, i, i, i, i, ll, ll, ll, ll, ll, i, vp, ll, i, vp],
             "apb_gemm_bf16_grouped_dev": [vp, vp, vp, i, i, i, ll, ll, ll, i, f, vp, ll, vp, i, vp, ll, vp],
             "apb_gemm_bf16_heads": [vp, vp, vp, i, i, i, i, ll, ll, ll, i, i, i, vp, ll, vp],
+            "apb_softmax_attn_wide": [vp, ll] + [vp] * 4 + [i, vp, i, vp, vp, ll, vp] + [i] * 7 + [f, i, vp, vp, ll, i, vp],
+            "apb_flash_tc": [vp, ll, i, vp, i, vp, i, vp, ll, vp, vp, ll, ll, vp, ll] + [i] * 5 + [f, i, vp, vp, ll, i, vp],
             "apb_softmax_attn_tc": [vp, ll, i, vp, i, vp, i, vp, vp, i, vp, ll, i, i, i, i, f, f, vp, f, f, vp],
             "apb_ssm": [vp, ll, i, i, vp, vp, i] + [vp] * 6 + [ll] + [vp] * 7 + [i, vp] + [i] * 8 + [vp],
             "apb_ssm_mma": [vp, ll] + [vp] * 9 + [i, vp, vp, vp] + [i] * 5 + [vp],
@@ -562,6 +564,56 @@ def chunk_tiles(host: np.ndarray, heads: int, kv_heads: int, min_len: int, chunk
     return np.ascontiguousarray(work[np.argsort(work[:, 6] - work[:, 5] - work[:, 4], kind="stable")], dtype=np.int32)
 
 
+def flash_fits(dim: int, rot: int, vdim: int) -> bool:
+    """Whether the tcgen05 kernel with a running reference takes heads of these sizes."""
+    return dim % 16 == 0 and rot % 16 == 0 and vdim % 8 == 0 and vdim <= 128 and -(-dim // 64) + -(-rot // 64) <= 4
+
+
+def flash_tiles(host: np.ndarray, heads: int, kv_heads: int, min_len: int, window: int, base: Optional[np.ndarray] = None,
+                tile: int = 128) -> np.ndarray:
+    """Work items of the tcgen05 kernel with a running reference for the entries of at least ``min_len`` rows, longest key range
+    first: ``[n, 12]`` int32 = entry, KV head, first key of the walk (a multiple of ``PAGE``), ``base`` of the entry, then for
+    each of two tiles (first row, valid rows, head, position of the first row).  The tiles are two query heads of a KV head on the
+    same rows; a head left over pairs consecutive row tiles (``valid = 0``: no second tile)."""
+    R = heads // kv_heads
+    parts = []
+    for en, (start, n, _slot, pos0) in enumerate(host.tolist()):
+        if n < min_len:
+            continue
+        t = np.arange(0, n, tile)
+        rows, valid, pos = start + t, np.minimum(tile, n - t), pos0 + t
+
+        def items(sel0, h0, sel1, h1):
+            a = [x[sel0] for x in (rows, valid, pos)]
+            c = [x[sel1] for x in (rows, valid, pos)]
+            m, m1 = len(a[0]), len(c[0])
+            it = np.zeros((kv_heads, m, 12), dtype=np.int64)
+            g = np.arange(kv_heads)[:, None]
+            it[..., 0], it[..., 1], it[..., 3] = en, g, 0 if base is None else base[en]
+            it[..., 2] = (np.maximum(0, a[2] - window + 1) if window else np.zeros_like(a[2])) // PAGE * PAGE
+            it[..., 4], it[..., 5], it[..., 6], it[..., 7] = a[0], a[1], g * R + h0, a[2]
+            it[:, :m1, 8], it[:, :m1, 9], it[:, :m1, 10], it[:, :m1, 11] = c[0], c[1], g * R + h1, c[2]
+            parts.append(it.reshape(-1, 12))
+
+        for h in range(0, R - 1, 2):
+            items(slice(None), h, slice(None), h + 1)
+        if R % 2:
+            items(slice(0, None, 2), R - 1, slice(1, None, 2), R - 1)
+    if not parts:
+        return np.zeros((0, 12), dtype=np.int32)
+    work = np.concatenate(parts)
+    keys = np.maximum(work[:, 7] + work[:, 5], work[:, 11] + work[:, 9]) - work[:, 2]
+    return np.ascontiguousarray(work[np.argsort(-keys, kind="stable")], dtype=np.int32)
+
+
+MAX_WIDE_SPLITS = 16
+
+
+def wide_splits(blocks: int, sms: int) -> int:
+    """Key splits of the wide-row kernel (one CTA per SM): full waves, against the cost of writing and merging the parts."""
+    return min(range(1, MAX_WIDE_SPLITS + 1), key=lambda s: -(-blocks * s // sms) / s + 0.04 * (s - 1) * blocks / sms)
+
+
 def softmax_attention(b: StepBatch, q: torch.Tensor, heads: int, kcache: torch.Tensor, vcache: Optional[torch.Tensor],
                       spec: SoftmaxSpec, lam: Optional[torch.Tensor], out: torch.Tensor, *, vdim: int = 0,
                       sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, gate_cols: int = 1) -> None:
@@ -576,25 +628,42 @@ def softmax_attention(b: StepBatch, q: torch.Tensor, heads: int, kcache: torch.T
     shape = (float(spec.scale), float(spec.cap), spec.chunk, spec.maps, _lib.ptr(lam), float(spec.post_scale), float(spec.eps))
     tail = shape + (spec.window, _lib.ptr(sink), _lib.ptr(gate), 0 if gate is None else gate.stride(0), gate_cols)
     aligned = not (D % 8 or E % 8 or q.stride(0) % 8 or out.stride(0) % 8 or (q.data_ptr() | out.data_ptr()) & 15)
-    if q.dtype != torch.bfloat16 or not aligned or max(DK, E) > 256:
+    if q.dtype != torch.bfloat16 or not aligned or (max(DK, E) > 256 and not (vcache is None and DK <= 640 and E <= 512 and spec.maps == 1)):
         _call("apb_softmax_attn", _lib.ptr(q), q.stride(0), _lib.ptr(b.row_entry), *b.entry_ptrs(), _lib.ptr(b.page_table),
               b.page_table.stride(0), _lib.ptr(kcache), _lib.ptr(vcache), _lib.ptr(out), out.stride(0), b.rows, heads, G, D, E,
               *tail, dtype_code(q.dtype))
         return
+    plain = spec.maps == 1 and not spec.cap and not spec.chunk
     tc = spec.maps == 2 and D % 16 == 0 and D <= 64 and E <= 128 and 0 < spec.cap <= MAX_FIXED_CAP
+    flash = plain and vcache is not None and flash_fits(D, 0, E) and not out.data_ptr() & 15
+    wide = plain and vcache is None and (DK > 256 or heads // G > 16)
     lens = np.ones(1, dtype=np.int64) if b.host is None else b.host[:, 1]
-    limit = SHORT_ROWS if tc else int(lens.max())
+    limit = SHORT_ROWS if tc or flash else int(lens.max())
     short = lens[lens <= limit]
     if len(short):
         longest = int(short.max())
-        passes = min(256, (longest * (heads // G) * spec.maps + 15) // 16)
-        splits = max(1, min(MAX_SPLITS, 2 * _sm_count(q.device) // (b.n_entries * G * passes)))
-        part = torch.empty((b.n_entries, longest, heads, spec.maps, splits, E + 2), device=q.device, dtype=torch.float32) \
-            if splits > 1 else None
-        _call("apb_softmax_attn_mma", _lib.ptr(q), q.stride(0), *b.entry_ptrs(), b.n_entries, _lib.ptr(b.page_table),
-              b.page_table.stride(0), _lib.ptr(kcache), _lib.ptr(vcache), _lib.ptr(out), out.stride(0), _lib.ptr(part), heads, G,
-              D, E, 1, longest, splits, *tail)
-    if len(short) < len(lens):
+        f32 = dict(device=q.device, dtype=torch.float32)
+        if wide:
+            splits = wide_splits(b.n_entries * G * -(-longest * (heads // G) // 32), _sm_count(q.device))
+            part = torch.empty((b.n_entries, longest, heads, splits, E + 2), **f32) if splits > 1 else None
+            _call("apb_softmax_attn_wide", _lib.ptr(q), q.stride(0), *b.entry_ptrs(), b.n_entries, _lib.ptr(b.page_table),
+                  b.page_table.stride(0), _lib.ptr(kcache), _lib.ptr(out), out.stride(0), _lib.ptr(part), heads, G, D, E, 1, longest,
+                  splits, float(spec.scale), *tail[7:])
+        else:
+            passes = min(256, (longest * (heads // G) * spec.maps + 15) // 16)
+            splits = max(1, min(MAX_SPLITS, 2 * _sm_count(q.device) // (b.n_entries * G * passes)))
+            part = torch.empty((b.n_entries, longest, heads, spec.maps, splits, E + 2), **f32) if splits > 1 else None
+            _call("apb_softmax_attn_mma", _lib.ptr(q), q.stride(0), *b.entry_ptrs(), b.n_entries, _lib.ptr(b.page_table),
+                  b.page_table.stride(0), _lib.ptr(kcache), _lib.ptr(vcache), _lib.ptr(out), out.stride(0), _lib.ptr(part), heads, G,
+                  D, E, 1, longest, splits, *tail)
+    if len(short) == len(lens):
+        return
+    if flash:
+        work = b.table(("flash", heads, G, spec.window), lambda: flash_tiles(b.host, heads, G, limit + 1, spec.window))
+        _call("apb_flash_tc", _lib.ptr(q), q.stride(0), b.rows, _lib.ptr(work), work.shape[0], _lib.ptr(b.page_table),
+              b.page_table.stride(0), _lib.ptr(kcache), D, None, _lib.ptr(vcache), E, kcache.shape[0] * G * PAGE, _lib.ptr(out),
+              out.stride(0), heads, G, D, 0, E, float(spec.scale), *tail[7:])
+    else:
         work = b.table(("softmax", heads, G, spec.chunk), lambda: chunk_tiles(b.host, heads, G, limit + 1, spec.chunk))
         _call("apb_softmax_attn_tc", _lib.ptr(q), q.stride(0), b.rows, _lib.ptr(work), work.shape[0], _lib.ptr(b.page_table),
               b.page_table.stride(0), _lib.ptr(kcache), _lib.ptr(vcache), kcache.shape[0], _lib.ptr(out), out.stride(0), heads,
@@ -646,18 +715,53 @@ def entry_runs(host: Optional[np.ndarray], n_entries: int, limit: int) -> list:
     return out
 
 
+LATENT_ROWS = 32        # entries up to this length work on the latents themselves
+EXPAND_TOKENS = 65536   # tokens of context whose keys and values are expanded at a time (a longer entry alone)
+
+
+def expansion_plan(host: np.ndarray, heads: int, min_len: int, budget: int = EXPAND_TOKENS) -> list:
+    """Groups of the entries of at least ``min_len`` rows whose contexts are expanded together: ``pages [n, 4]`` int32 (entry,
+    page of the entry, first row of the copy, tokens) for the gather kernel and ``work`` (:func:`flash_tiles`)."""
+    groups, at = [], 0
+    for en, (_start, n, _slot, pos0) in enumerate(host.tolist()):
+        if n < min_len:
+            continue
+        size = -(-(pos0 + n) // PAGE) * PAGE
+        if not groups or at + size > budget:
+            groups.append([])
+            at = 0
+        groups[-1].append((en, at, size))
+        at += size
+    plans = []
+    for group in groups:
+        base = np.zeros(len(host), dtype=np.int64)
+        mine = host.copy()
+        mine[:, 1] = 0
+        for en, row, _ in group:
+            base[en], mine[en, 1] = row, host[en, 1]
+        pages = [np.stack([np.full(size // PAGE, en), np.arange(size // PAGE), row + np.arange(0, size, PAGE),
+                           np.full(size // PAGE, PAGE)], 1) for en, row, size in group]
+        plans.append({"pages": np.concatenate(pages).astype(np.int32), "work": flash_tiles(mine, heads, heads, min_len, 0, base)})
+    return plans
+
+
 def latent_attention(b: StepBatch, q: torch.Tensor, s: LatentSpec, cache: torch.Tensor, w_absorb: torch.Tensor,
                      w_expand: torch.Tensor, sink: Optional[torch.Tensor], gate: Optional[torch.Tensor],
                      rope: Tuple[torch.Tensor, torch.Tensor], out: torch.Tensor) -> None:
     """``q [rows, heads * (dim + rot)]`` (not rotated yet) over the entries' latents -> ``out [rows, heads * vdim]`` (column
-    slice), times the sigmoid of the ``gate`` columns.  ``w_expand`` holds the key rows (heads * dim) and then the value rows
-    (heads * vdim) over the latent, ``w_absorb [heads * rank, dim]`` the key rows transposed per head.
+    slice), times the sigmoid of the ``gate`` columns.  ``w_expand`` holds the key rows (heads * dim) and, from the next multiple of
+    8 on, the value rows (heads * vdim) over the latent, ``w_absorb [heads * rank, dim]`` the key rows transposed per head.
 
-    The key projection is applied to the query and the value projection to the weighted sum of the latents."""
+    Short entries work on the latents: the key projection is applied to the query and the value projection to the weighted sum.
+    Long ones expand the keys and values of all heads from the latents of their whole context first."""
     H, D, R, C, E = s.heads, s.dim, s.rot, s.rank, s.vdim
     spec = SoftmaxSpec(s.scale)
-    w_value = w_expand[w_expand.shape[0] - H * E:]
-    limit = b.rows
+    v_col = (H * D + 7) // 8 * 8
+    w_value = w_expand[v_col:][:H * E]
+    gated = [] if gate is None else [gate]
+    aligned = not (C % 8 or any(t.stride(0) % 8 or t.data_ptr() & 15 for t in [q, out] + gated))
+    expand = b.host is not None and q.dtype == torch.bfloat16 and aligned and flash_fits(D, R, E) and R > 0
+    limit = LATENT_ROWS if expand else b.rows
     for e0, e1 in entry_runs(b.host, b.n_entries, limit):
         p = b.part(e0, e1)
         r0 = 0 if b.host is None else int(b.host[e0, 0])
@@ -668,6 +772,23 @@ def latent_attention(b: StepBatch, q: torch.Tensor, s: LatentSpec, cache: torch.
         o = torch.empty((p.rows, H * C), device=q.device, dtype=q.dtype)
         softmax_attention(p, ql, H, cache, None, spec, None, o, vdim=C, sink=sink)
         heads_linear(o, C, w_value, H, C, out[rows], E, None if gate is None else gate[rows])
+    if not expand or not (b.host[:, 1] > limit).any():
+        return
+    latent_rotate(b, q, s, rope)
+    key = ("expanded", H)
+    if key not in b.host_tables:
+        b.host_tables[key] = expansion_plan(b.host, H, limit + 1)
+    for n, plan in enumerate(b.host_tables[key]):
+        pages, work = (b.table(key + (n, t), lambda t=t: plan[t]) for t in ("pages", "work"))
+        keys = plan["pages"].shape[0] * PAGE
+        latents, rotated = (torch.empty((keys, w), device=q.device, dtype=q.dtype) for w in (C, R))
+        _call("apb_latent_gather", _lib.ptr(cache), _lib.ptr(pages), pages.shape[0], _lib.ptr(b.page_table), b.page_table.stride(0),
+              _lib.ptr(latents), _lib.ptr(rotated), C, R)
+        kv = linear(latents, w_expand[:, :C])
+        v = kv[:, v_col:]
+        _call("apb_flash_tc", _lib.ptr(q), q.stride(0), b.rows, _lib.ptr(work), work.shape[0], None, 0, _lib.ptr(kv), kv.stride(0),
+              _lib.ptr(rotated), _lib.ptr(v), kv.stride(0), keys, _lib.ptr(out), out.stride(0), H, H, D, R, E, float(s.scale), 0,
+              _lib.ptr(sink), _lib.ptr(gate), 0 if gate is None else gate.stride(0), E)
 
 
 MIN_SEGMENT = 256       # tokens; a multiple of the kernel's chunk

@@ -176,3 +176,48 @@ def test_runs_of_short_entries():
     from arctic_platform_b200.ops.serving import entry_runs
     host = np.array([[0, 1, 0, 5], [1, 40, 1, 0], [41, 2, 2, 9], [43, 1, 3, 7], [44, 90, 4, 0]])
     assert entry_runs(host, 5, 16) == [(0, 1), (2, 4)] and entry_runs(host, 5, 100) == [(0, 5)] and entry_runs(None, 7, 1) == [(0, 7)]
+
+
+@pytest.mark.parametrize("window", [0, 1, 50, 128, 200, 4096])
+@pytest.mark.parametrize("heads,kv", [(4, 2), (3, 1), (5, 5)])
+def test_attention_work_items_cover_every_row_once_and_walk_all_visible_keys(heads, kv, window):
+    from arctic_platform_b200.ops.serving import PAGE, flash_tiles
+    host = np.array([[0, 300, 1, 40], [300, 5, 0, 1000], [305, 129, 2, 0], [434, 128, 3, 7], [562, 17, 4, 2047]])
+    work = flash_tiles(host, heads, kv, 17, window, np.arange(5) * 10000)
+    seen, keys = {}, []
+    for en, g, k0, base, *tiles in work.tolist():
+        start, n, _, pos0 = host[en]
+        assert k0 % PAGE == 0 and base == en * 10000 and tiles[1] > 0
+        ends = []
+        for row, valid, head, pos in (tiles[:4], tiles[4:]):
+            if not valid:
+                continue
+            assert head // (heads // kv) == g and 0 < valid <= 128 and row + valid <= start + n and pos - pos0 == row - start
+            assert k0 <= max(0, pos - window + 1 if window else 0)
+            ends.append(pos + valid)
+            for r in range(row, row + valid):
+                seen[r, head] = seen.get((r, head), 0) + 1
+        keys.append(max(ends) - k0)
+    rows = [r for s, n, _, _ in host.tolist() if n > 16 for r in range(s, s + n)]
+    assert seen == {(r, h): 1 for r in rows for h in range(heads)}
+    assert (np.diff(keys) <= 0).all()
+    assert flash_tiles(host, heads, kv, 1000, window).shape == (0, 12)
+
+
+def test_contexts_are_expanded_in_groups_of_bounded_size():
+    from arctic_platform_b200.ops.serving import PAGE, expansion_plan
+    host = np.array([[0, 40, 1, 100], [40, 3, 0, 900], [43, 60, 2, 0], [103, 64, 3, 1000]])
+    plans = expansion_plan(host, 2, 33, 256)
+    assert [sorted({int(e) for e in p["pages"][:, 0]}) for p in plans] == [[0, 2], [3]]
+    for p in plans:
+        rows = p["pages"][:, 2]
+        assert rows.tolist() == list(range(0, len(rows) * PAGE, PAGE)) and (p["pages"][:, 3] == PAGE).all()
+        for en, _, _, base, *_ in p["work"].tolist():
+            mine = p["pages"][p["pages"][:, 0] == en]
+            assert mine[0, 2] == base and mine[:, 1].tolist() == list(range(-(-(host[en, 3] + host[en, 1]) // PAGE)))
+
+
+def test_splits_of_wide_rows():
+    from arctic_platform_b200.ops.serving import MAX_WIDE_SPLITS, wide_splits
+    assert wide_splits(1, 148) == MAX_WIDE_SPLITS and wide_splits(128, 148) == 1 and wide_splits(64, 148) == 2
+    assert all(1 <= wide_splits(n, 148) <= MAX_WIDE_SPLITS for n in range(1, 2000, 37))
