@@ -8,11 +8,14 @@ For every model (random weights, synthetic prompts) two parts are measured on on
 * kernels: each step of ONE layer of every kind on a prefill batch (4 prompts x 2048 tokens) and on a decode batch (128
   sequences after 2048 tokens), next to the like kernel of the closest model: for Reninex a Qwen3-style layer of the same
   width, heads and feed-forward (for retention the gated delta rule of the hybrid family at the same heads and sizes); for
-  Rigulorn a Reninex layer whose K/V rows, state and feed-forward have the same size.  ``floor_ms`` is the slower of
+  Rigulorn a Reninex layer whose K/V rows, state and feed-forward have the same size; for Titatar the dense decoder's layer
+  with the heads of its windowed attention, and the decoder family's mixture of experts with as many experts and (on average)
+  as many routed rows.  ``floor_ms`` is the slower of
   algorithmic bytes over the measured copy bandwidth and FLOPs over the measured bf16 GEMM peak, ``frac`` = floor / time.
   CUDA events around every launch, L2 overwritten before it, median over the iterations.
 * engine: prefill and decode tokens/s through ``generate`` of the model, of the dense decoder with as many layers as the
-  model has layer runs and, for Rigulorn, of the Reninex preset of the same width.
+  model has layer runs (for Titatar: with a mixture of experts of the same size in every layer) and, for Rigulorn, of the
+  Reninex preset of the same width.
 
 Prints one JSON line per measurement.
 """
@@ -87,7 +90,7 @@ def phase_batch(phase):
 
 def stateful_ops(cfg, phase):
     """``(name, fn, bytes, flops)`` of the steps of the model's layers on the phase's batch."""
-    return {"Reninex": reninex_ops, "Rigulorn": rigulorn_ops}[cfg.architecture](cfg, phase)
+    return {"Reninex": reninex_ops, "Rigulorn": rigulorn_ops, "Titatar": titatar_ops}[cfg.architecture](cfg, phase)
 
 
 def reninex_ops(cfg, phase):
@@ -196,6 +199,139 @@ def rigulorn_ops(cfg, phase):
     ]
 
 
+def titatar_ops(cfg, phase):
+    import dataclasses
+    import math
+    from arctic_platform_b200.engine.stateful_sampler import StateCache
+    from arctic_platform_b200.models.titatar import MoeSpec, TitatarLM
+    from arctic_platform_b200.ops import serving
+    lat = next(s for s in cfg.layers if s.latent and isinstance(s.mlp, MoeSpec))
+    win = next(s for s in cfg.layers if not s.latent)
+    ff = next(s.mlp for s in cfg.layers if isinstance(s.mlp, int))
+    one = dataclasses.replace(cfg, layers=(lat, dataclasses.replace(win, mlp=ff)), loop=None, vocab_size=1024)
+    model = TitatarLM(one, "cuda", torch.bfloat16).init_weights(0)
+    model.prepare_serving(SEQ + 8)
+    b, n, n_pages, keys = phase_batch(phase)
+    cache = StateCache(model.cache_layout(), n_pages, n, "cuda", torch.bfloat16)
+    for t in cache._paged():
+        t.normal_()
+    T, W, L, A, M = b.rows, cfg.hidden_size, lat.mixer, win.mixer, lat.mlp
+    lb, wb = model.blocks
+    lm, wm, moe, glu = lb.mixer, wb.mixer, lb.mlp, wb.mlp
+    x = torch.randn(T, W, device="cuda")
+    serving.embed(b, model.embed, None, None, cache.prev, torch.empty_like(x))
+    clear = serving.accumulates(T, W, x.device)
+    y, h = torch.zeros(T, W, device="cuda"), _bf(T, W)
+    pl, pw = serving.linear(h, lm.w_in), serving.linear(h, wm.w_in)
+    lc, wc = lm.in_cols, wm.in_cols
+    rl, rw = model._rope[L.rot], model._rope[A.rot]
+    q = _bf(T, lm.w_q.shape[0])
+    ql = pl[:, lc["dq"][0]:lc["dq"][0] + L.q_rank]
+    lo, wo, fo = _bf(T, lm.n_out), _bf(T, wm.n_out), _bf(T, ff)
+    z = serving.linear(h, moe.router, out_dtype=torch.float32)
+
+    def experts():
+        return serving.experts(b, h, z, moe.correction, moe.counters, moe.w_gu, moe.w_down, M.scores, M.experts, M.top, M.ff)
+
+    mix = experts()
+    pairs = T * M.top * M.experts / M.scores
+    touched = M.experts * (1 - math.exp(-pairs / M.experts))
+    C, R, D, E, H = L.kv_rank, L.rot_dim, L.dim, L.vdim, L.heads
+    row = (C + R) * 2
+    ctx = T if phase == "prefill" else keys
+    seen = keys                                          # keys inside the window, summed over the rows
+    if A.window:
+        seen = n * sum(min(i + 1, A.window) for i in range(SEQ)) if phase == "prefill" else n * min(A.window, SEQ + 1)
+    wctx = T if phase == "prefill" else seen
+    kv_row = A.kv_heads * (A.dim + A.vdim) * 2
+    expand = lm.w_expand.numel() * 2
+    if phase == "prefill":
+        lat_flops = 2 * keys * H * (D + R + E) + 2 * T * C * H * (D + E)
+    else:
+        lat_flops = 2 * keys * H * (2 * C + R) + 2 * T * C * H * (D + E)
+    gemm = lambda N, K: (2 * (T * K + N * K + T * N), 2 * T * N * K)
+    out = lambda K: (2 * (T * K + K * W) + (8 if clear else 4) * T * W, 2 * T * W * K)
+    return [
+        ("residual update + norms", lambda: serving.residual_step(x, y, lb.norm1b, lb.norm2, 1e-6, clear=clear),
+         T * W * (8 + 4 + 2 + (4 if clear else 0)), 0),
+        ("residual update + expert sum + norms", lambda: serving.residual_step(x, y, lb.norm1b, lb.norm2, 1e-6, clear=clear, mix=mix),
+         T * W * (8 + 4 + 2 + (4 if clear else 0) + 2) + 2 * pairs * W, 0),
+        ("latent input projections (GEMM)", lambda: serving.linear(h, lm.w_in, pl), *gemm(pl.shape[1], W)),
+        ("latent norms + cache write", lambda: serving.latent_norm_cache(b, pl, lc["dq"][0], lc["dkv"][0], lm.q_norm, lm.kv_norm, rl,
+                                                                        cache.k[0], 1e-6), 2 * T * (2 * L.q_rank + 2 * (C + R)), 0),
+        ("query projection (GEMM)", lambda: serving.linear(ql, lm.w_q[:, :L.q_rank], q), *gemm(q.shape[1], L.q_rank)),
+        ("latent attention", lambda: serving.latent_attention(b, q, lm.spec, cache.k[0], lm.w_absorb, lm.w_expand, lm.sink32,
+                                                              pl[:, lc["g"][0]:], rl, lo),
+         ctx * row + expand + 2 * T * H * (D + R + 2 * E), lat_flops),
+        ("latent output projection (GEMM)", lambda: serving.project(lo, lm.w_out, y), *out(lm.n_out)),
+        ("windowed input projections (GEMM)", lambda: serving.linear(h, wm.w_in, pw), *gemm(pw.shape[1], W)),
+        ("q/k norm + rotation + cache write", lambda: serving.row_norm_rope_cache(b, pw, (wc["q"][0], wc["k"][0], wc["v"][0]), wm.q_norm,
+                                                                                wm.k_norm, rw, A.rot.dims, A.heads, cache.k[1], cache.v[1], 1e-6),
+         2 * T * (2 * A.heads * A.dim) + 2 * T * kv_row, 0),
+        ("windowed attention", lambda: serving.softmax_attention(b, pw, A.heads, cache.k[1], cache.v[1], wm.spec, None, wo, sink=wm.sink,
+                                                                 gate=pw[:, wc["g"][0]:]),
+         wctx * kv_row + 2 * T * A.heads * (A.dim + A.vdim), 2 * seen * A.heads * (A.dim + A.vdim)),
+        ("windowed output projection (GEMM)", lambda: serving.project(wo, wm.w_out, y), *out(wm.n_out)),
+        ("router (GEMM)", lambda: serving.linear(h, moe.router, z), 2 * T * W + 2 * z.shape[1] * W + 4 * T * z.shape[1], 2 * T * W * z.shape[1]),
+        ("routed experts", experts, touched * 6 * W * M.ff + 2 * T * W + 2 * pairs * W, 6 * pairs * W * M.ff),
+        ("gate/up + SiLU (GEMM)", lambda: serving.gate_up_silu(h, glu.w_gu, fo), 2 * (T * W + 2 * ff * W + T * ff), 4 * T * W * ff),
+        ("down projection (GEMM)", lambda: serving.project(fo, glu.w_down, y), *out(ff)),
+    ]
+
+
+# step of a Titatar layer -> the like step of the dense decoder's layer (experts: of its mixture)
+TITATAR_LIKE = {
+    "residual update + norms": "norm + 2 input convolutions", "residual update + expert sum + norms": "norm + 2 input convolutions",
+    "latent input projections (GEMM)": "input projections (GEMM)", "latent norms + cache write": "q/k norm + cache write",
+    "query projection (GEMM)": "attention output projection (GEMM)", "latent attention": "attention",
+    "latent output projection (GEMM)": "attention output projection (GEMM)",
+    "windowed input projections (GEMM)": "input projections (GEMM)", "q/k norm + rotation + cache write": "q/k norm + cache write",
+    "windowed attention": "attention", "windowed output projection (GEMM)": "attention output projection (GEMM)",
+    "router (GEMM)": "router (GEMM)", "routed experts": "routed experts", "gate/up + SiLU (GEMM)": "gate/up + GELU (GEMM)",
+    "down projection (GEMM)": "output projections (GEMM, += fp32)",
+}
+
+
+def titatar_like(cfg):
+    """The layer sizes of the windowed attention and the dense feed-forward, in the form ``dense_ops`` takes."""
+    from arctic_platform_b200.models.reninex import ReninexConfig, _uniform
+    A = next(s for s in cfg.layers if not s.latent).mixer
+    ff = next(s.mlp for s in cfg.layers if isinstance(s.mlp, int))
+    layers = _uniform(1, (A.heads, A.kv_heads, A.dim, A.vdim), (2, 64, 64, 64), ff)
+    return ReninexConfig(cfg.vocab_size, cfg.hidden_size, layers, cfg.norm_eps, 4, None, None, f"titatar-like-{cfg.hidden_size}")
+
+
+def moe_config(cfg):
+    """The decoder family's mixture-of-experts model beside a Titatar model: its windowed attention's heads, its experts without
+    the identity ones, as many of them per token as Titatar chooses on average, one layer per run."""
+    import dataclasses
+    m = next(s.mlp for s in cfg.layers if not isinstance(s.mlp, int) and s.mlp is not None)
+    return dataclasses.replace(dense_config(titatar_like(cfg)), num_layers=len(cfg.layer_runs()), num_experts=m.experts,
+                               num_experts_per_tok=round(m.top * m.experts / m.scores), moe_intermediate_size=m.ff,
+                               name=f"moe-{cfg.hidden_size}")
+
+
+def moe_ops(cfg, phase):
+    import math
+    from arctic_platform_b200.models.moe import MoEFeedForward
+    from arctic_platform_b200.ops import gemm
+    d = moe_config(cfg)
+    n = PREFILL_SEQS * SEQ if phase == "prefill" else DECODE_SEQS
+    W, F, E = d.hidden_size, d.moe_intermediate_size, d.num_experts
+    ff = MoEFeedForward(d, "cuda", torch.bfloat16)
+    for t in ff.parameters():
+        t.data.normal_(std=0.02)
+    x = _bf(n, W)
+    pairs = n * d.num_experts_per_tok
+    touched = E * (1 - math.exp(-pairs / E))
+
+    def run():
+        with torch.no_grad():
+            ff._routed(x)
+    return {"routed experts": (run, touched * 6 * W * F + 4 * n * W, 6 * pairs * W * F),
+            "router (GEMM)": (lambda: gemm.matmul_nt(x, ff.router.data), 2 * (n * W + E * W + n * E), 2 * n * W * E)}
+
+
 # step of a Rigulorn layer -> (model, the like step of its layer); products next to the dense decoder's of the same shape
 RIGULORN_LIKE = {
     "stream update + norm": ("reninex", "norm + 2 input convolutions"),
@@ -221,6 +357,9 @@ def reninex_like(cfg):
 
 def like_ops(cfg, phase):
     """Steps of the closest older model, keyed by the names of ``stateful_ops``: ``name -> (fn, bytes, flops)``."""
+    if cfg.architecture == "Titatar":
+        ops = {**dense_ops(titatar_like(cfg), phase), **moe_ops(cfg, phase)}
+        return {mine: ops[theirs] for mine, theirs in TITATAR_LIKE.items()}
     if cfg.architecture != "Rigulorn":
         return dense_ops(cfg, phase)
     like = reninex_like(cfg)
@@ -371,8 +510,7 @@ def bench_engine(name, cfg, seqs, new_tokens):
     from arctic_platform_b200.models.config import resolve_config
     prompts = [np.random.default_rng(i).integers(1, cfg.vocab_size, SEQ).tolist() for i in range(seqs)]
     limits = dict(kv_cache_tokens=seqs * (SEQ + new_tokens + 32), max_batch=seqs, max_seq_len=SEQ + new_tokens + 16)
-    d = dense_config(cfg)
-    models = [cfg, d]
+    models = [cfg, moe_config(cfg) if cfg.architecture == "Titatar" else dense_config(cfg)]
     if cfg.architecture == "Rigulorn" and f"reninex-{cfg.hidden_size}" in registry.presets():
         models.append(resolve_config(f"reninex-{cfg.hidden_size}"))
     for m in models:
@@ -422,7 +560,7 @@ def main(models, kernels_only=False, only=None, iters=20, seqs=64, new_tokens=12
 
 if __name__ == "__main__":
     ap = argparse.ArgumentParser()
-    ap.add_argument("--models", default="reninex-2048,reninex-4096,rigulorn-2048,rigulorn-4096")
+    ap.add_argument("--models", default="reninex-2048,reninex-4096,rigulorn-2048,rigulorn-4096,titatar-2048,titatar-4096")
     ap.add_argument("--kernels-only", action="store_true")
     ap.add_argument("--only", choices=["prefill", "decode", "none"], help="which kernels are timed")
     ap.add_argument("--step", help="only the steps whose name contains this")
