@@ -1,7 +1,7 @@
 // Latent attention: the small steps around its products.
 //
 // A token keeps one latent of C columns and one rotated key part of R columns that all heads share; both lie side by side in a
-// page row [pages, 1, 16, C + R].  A head's keys and values are projections of the latent, so attention can run either on the
+// page row [pages, 1, 16, ldk] of at least C + R columns.  A head's keys and values are projections of the latent, so attention can run either on the
 // expanded keys and values, or -- with the key projection moved to the query and the value projection behind the sum -- on
 // the latents themselves.  Rotary positions pair neighbouring dimensions.
 #include "common.cuh"
@@ -29,7 +29,7 @@ __global__ void __launch_bounds__(kLatThreads)
 latent_norm_cache_kernel(T* __restrict__ p, long long ld, int q_col, int c_col, const T* __restrict__ q_gain,
                          const T* __restrict__ c_gain, const int* __restrict__ row_entry, const ServeEntries e,
                          const int* __restrict__ kv_slot, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
-                         T* __restrict__ cache, int Q, int C, int R, float eps) {
+                         T* __restrict__ cache, int ldk, int Q, int C, int R, float eps) {
   pdl_entry();
   __shared__ float red[2][kLatThreads / 32];
   const int row = blockIdx.x;
@@ -48,7 +48,7 @@ latent_norm_cache_kernel(T* __restrict__ p, long long ld, int q_col, int c_col, 
   for (int i = threadIdx.x; i < Q; i += kLatThreads) q[i] = from_f32<T>(to_f32(q[i]) * rq * to_f32(q_gain[i]));
   const int slot = kv_slot[row];
   if (slot < 0) return;
-  T* dst = cache + static_cast<long long>(slot) * (C + R);
+  T* dst = cache + static_cast<long long>(slot) * ldk;
   for (int i = threadIdx.x; i < C; i += kLatThreads) dst[i] = from_f32<T>(to_f32(c[i]) * rc * to_f32(c_gain[i]));
   const int en = row_entry ? row_entry[row] : row;
   const long long tr = static_cast<long long>(e.pos0[en] + row - e.start[en]) * (R >> 1);
@@ -88,13 +88,13 @@ latent_rotate_kernel(T* __restrict__ q, long long ld, const int* __restrict__ ro
 template <typename V>
 __global__ void __launch_bounds__(128)
 latent_gather_kernel(const V* __restrict__ cache, const int* __restrict__ work, const int* __restrict__ page_table, int max_pages,
-                     V* __restrict__ latents, V* __restrict__ rotated, int C, int R) {
+                     V* __restrict__ latents, V* __restrict__ rotated, int ldk, int C, int R) {
   pdl_entry();
   const int4 w = reinterpret_cast<const int4*>(work)[blockIdx.x];
-  const V* src = cache + static_cast<long long>(page_table[static_cast<long long>(w.x) * max_pages + w.y]) * kServePage * (C + R);
+  const V* src = cache + static_cast<long long>(page_table[static_cast<long long>(w.x) * max_pages + w.y]) * kServePage * ldk;
   for (int i = threadIdx.x; i < w.w * (C + R); i += 128) {
     const int t = i / (C + R), c = i % (C + R);
-    const V v = src[i];
+    const V v = src[t * ldk + c];
     if (c < C)
       latents[static_cast<long long>(w.z + t) * C + c] = v;
     else
@@ -109,15 +109,15 @@ using namespace apb;
 
 int apb_latent_norm_cache(void* p, long long ld, int q_col, int c_col, const void* q_gain, const void* c_gain,
                           const int* row_entry, const int* e_start, const int* e_len, const int* e_slot, const int* e_pos0,
-                          const int* kv_slot, const float* cos_t, const float* sin_t, void* cache, int rows, int Q, int C, int R,
-                          float eps, int dtype, cudaStream_t s) {
+                          const int* kv_slot, const float* cos_t, const float* sin_t, void* cache, int ldk, int rows, int Q, int C,
+                          int R, float eps, int dtype, cudaStream_t s) {
   if (rows <= 0) return 0;
-  if (Q <= 0 || C <= 0 || R < 0 || (R & 1) || !kv_slot || !cache || (R && (!cos_t || !sin_t))) return kBadArgument;
+  if (Q <= 0 || C <= 0 || R < 0 || (R & 1) || ldk < C + R || !kv_slot || !cache || (R && (!cos_t || !sin_t))) return kBadArgument;
   const ServeEntries e{e_start, e_len, e_slot, e_pos0};
   APB_SERVE_DTYPE(dtype, return static_cast<int>(launch_kernel(
                              latent_norm_cache_kernel<T>, dim3(rows), dim3(kLatThreads), 0, s, static_cast<T*>(p), ld, q_col,
                              c_col, static_cast<const T*>(q_gain), static_cast<const T*>(c_gain), row_entry, e, kv_slot, cos_t,
-                             sin_t, static_cast<T*>(cache), Q, C, R, eps)));
+                             sin_t, static_cast<T*>(cache), ldk, Q, C, R, eps)));
 }
 
 int apb_latent_rotate(void* q, long long ld, const int* row_entry, const int* e_start, const int* e_len, const int* e_slot,
@@ -133,13 +133,13 @@ int apb_latent_rotate(void* q, long long ld, const int* row_entry, const int* e_
                                                                static_cast<T*>(dst), rows, H, D, R, C)));
 }
 
-// bf16; C and R multiples of 8.
+// bf16; C, R and ldk multiples of 8.
 int apb_latent_gather(const void* cache, const int* work, int n_work, const int* page_table, int max_pages, void* latents,
-                      void* rotated, int C, int R, cudaStream_t s) {
+                      void* rotated, int ldk, int C, int R, cudaStream_t s) {
   if (n_work <= 0) return 0;
-  if (C <= 0 || R < 0 || (C & 7) || (R & 7) || !work || !page_table) return kBadArgument;
+  if (C <= 0 || R < 0 || (C & 7) || (R & 7) || (ldk & 7) || ldk < C + R || !work || !page_table) return kBadArgument;
   return static_cast<int>(launch_kernel(latent_gather_kernel<uint4>, dim3(n_work), dim3(128), 0, s,
                                         static_cast<const uint4*>(cache), work, page_table, max_pages,
-                                        static_cast<uint4*>(latents), static_cast<uint4*>(rotated), C / 8, R / 8));
+                                        static_cast<uint4*>(latents), static_cast<uint4*>(rotated), ldk / 8, C / 8, R / 8));
 }
 }

@@ -3,7 +3,7 @@
 // SoftmaxSpec.
 //
 // Keys and values live in pages of 16 tokens (kcache [pages, G, 16, maps * D], vcache [pages, G, 16, E]; without a vcache the
-// values are the first E columns of the key rows); the step's own keys are already there when these kernels run, so prompts,
+// values are the first E columns of the key rows -- softmax_attn_kernel only); the step's own keys are already there when these kernels run, so prompts,
 // portions of prompts and decoded tokens read the same memory.
 //
 //  * softmax_attn_kernel      any D up to 1024, E up to 512, bf16 or fp32, fp32 arithmetic throughout (the fp32 engine, odd sizes);
@@ -162,10 +162,8 @@ softmax_attn_mma_kernel(const SoftmaxMmaParams p) {
   const int M = p.sp.maps;
   const int DK = FULL ? NK * 16 : p.D * M, E = FULL ? NE * 16 : p.E, R = p.H / p.G, D = p.D;
   const int d16 = (DK + 15) >> 4, e16 = (E + 15) >> 4;
-  const bool own_v = p.vcache != nullptr;
-  const int k_row = d16 * 32 + 16, v_row = own_v ? e16 * 32 + 16 : k_row;      // ring row bytes
-  const int v_off = own_v ? kServePage * k_row : 0;
-  const int stage_bytes = kServePage * k_row + (own_v ? kServePage * v_row : 0);
+  const int k_row = d16 * 32 + 16, v_row = e16 * 32 + 16;            // ring row bytes
+  const int stage_bytes = kServePage * (k_row + v_row);
   const int split = blockIdx.y, splits = gridDim.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int start = p.e.start[en], pos0 = p.e.pos0[en];
@@ -223,11 +221,10 @@ softmax_attn_mma_kernel(const SoftmaxMmaParams p) {
         const __nv_bfloat16* kp = p.kcache + base * DK;
 #pragma unroll
         for (int i = lane; i < kServePage * kc; i += 32) sx_cp_async16(dst + (i / kc) * k_row + (i % kc) * 16, kp + i * 8);
-        if (own_v) {
-          const __nv_bfloat16* vp = p.vcache + base * E;
+        const __nv_bfloat16* vp = p.vcache + base * E;
 #pragma unroll
-          for (int i = lane; i < kServePage * vc; i += 32) sx_cp_async16(dst + v_off + (i / vc) * v_row + (i % vc) * 16, vp + i * 8);
-        }
+        for (int i = lane; i < kServePage * vc; i += 32)
+          sx_cp_async16(dst + kServePage * k_row + (i / vc) * v_row + (i % vc) * 16, vp + i * 8);
       }
       asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -239,7 +236,7 @@ softmax_attn_mma_kernel(const SoftmaxMmaParams p) {
       asm volatile("cp.async.wait_group %0;" ::"n"(kSxStages - 1) : "memory");
       __syncwarp();
       const uint32_t ks_addr = ring + (j % kSxStages) * stage_bytes;
-      const uint32_t vs_addr = ks_addr + v_off;
+      const uint32_t vs_addr = ks_addr + kServePage * k_row;
       float sc[2][4];
 #pragma unroll
       for (int nt = 0; nt < 2; ++nt) sc[nt][0] = sc[nt][1] = sc[nt][2] = sc[nt][3] = 0.f;
@@ -453,14 +450,14 @@ int apb_softmax_attn_mma(const void* q, long long ldq, const int* e_start, const
   if (H <= 0 || G <= 0 || H % G || D <= 0 || E <= 0 || (D % 8) || (E % 8) || maps < 1 || maps > 2 || maps * D > 256 || E > 256 ||
       (ldq % 8) || (reinterpret_cast<uintptr_t>(q) & 15) || min_len < 1 || max_len < min_len || splits < 1 ||
       (splits > 1 && !part) || (maps == 2 && !lambda) || chunk < 0 || window < 0 || (maps == 2 && (sink || gate)) ||
-      (!vcache && E > maps * D) || (gate && gate_cols != 1 && gate_cols != E))
+      !vcache || (gate && gate_cols != 1 && gate_cols != E))
     return kBadArgument;
   SoftmaxMmaParams p{static_cast<const __nv_bfloat16*>(q), ldq, ServeEntries{e_start, e_len, e_slot, e_pos0}, page_table,
                      max_pages, static_cast<const __nv_bfloat16*>(kcache), static_cast<const __nv_bfloat16*>(vcache),
                      static_cast<__nv_bfloat16*>(out), ldo, part, H, G, D, E, min_len, max_len,
                      SoftmaxSpec{scale, cap, chunk, maps, lambda, post_scale, eps, window, sink, gate, ldg, gate_cols}};
   const int DK = maps * D, d16 = (DK + 15) / 16, e16 = (E + 15) / 16;
-  const int ring = 4 * kSxStages * kServePage * (d16 * 32 + 16 + (vcache ? e16 * 32 + 16 : 0)), sums = 4 * 16 * e16 * 16 * 4;
+  const int ring = 4 * kSxStages * kServePage * (d16 * 32 + e16 * 32 + 32), sums = 4 * 16 * e16 * 16 * 4;
   const int smem = ring > sums ? ring : sums;
   const int passes = static_cast<int>((static_cast<long long>(max_len) * (H / G) * maps + 15) / 16);
   const dim3 grid(n_entries * G, splits, passes < 256 ? passes : 256);

@@ -11,7 +11,7 @@ struct SoftmaxMmaParams {
   const int* page_table;
   int max_pages;
   const __nv_bfloat16* kcache;
-  const __nv_bfloat16* vcache;    // null: the values are the first E columns of the key rows
+  const __nv_bfloat16* vcache;    // unused where the values are the first E columns of the key rows
   __nv_bfloat16* out;
   long long ldo;
   float* part;            // [entries, max_len, H, maps, splits, E + 2] fp32 (sums, maximum, weight sum) when splits > 1

@@ -1,207 +1,261 @@
 // Paged causal softmax attention over wide key rows whose first columns are the values (absorbed latent attention): decoded
 // tokens and short portions, one map.  See SoftmaxSpec.
 //
+// A key row lies in the page cache as in shared memory: its columns, zeros up to a multiple of 16 and 8 columns more, an odd number
+// of 16-byte pieces, so that the rows of a page arrive by one copy and fall into different banks.
+//
 // Many query heads share one key row of up to 640 columns, so a row is read once and meets MT * 16 (query, head) rows on m16n8k16
-// tensor-core tiles.  A CTA = one entry, KV head, group of rows and share of the keys; 8 warps.  Blocks of 64 keys (four pages)
-// are double-buffered in shared memory and serve both products: for the scores the warps split rows and keys, for the weighted
-// sums they split the value columns.  The running maximum and the weights pass through shared memory in between.
+// tensor-core tiles.  A CTA = one entry, KV head, group of rows and share of the keys.  13 warps: a producer that copies pages
+// into a ring of 32-key blocks, four score warps and eight value warps.  A block serves both products: the score warps split its
+// keys (and the rows), agree on the rows' maximum and leave weights and rescaling factors in shared memory; the value warps, which
+// split the value columns, work on one block while the score warps are at the next and the others are on their way.
 #include "common.cuh"
 #include "host_utils.cuh"
 #include "serve_softmax_mma.cuh"
 
 namespace apb {
 
-constexpr int kWideThreads = 256;
-constexpr int kWideKeys = 64;
+constexpr int kWideThreads = 13 * 32;
+constexpr int kWideKeys = 32;                          // keys per block
+constexpr int kWideMaxStages = 8;
+constexpr int kWideMaxSmem = 227 * 1024 - 3 * 1024;    // besides the static arrays
 constexpr int kWideMaxDK = 640, kWideMaxE = 512;
 constexpr int kWidePRow = kWideKeys * 2 + 16;          // bytes of a row of weights
 
+// Contiguous bytes (a multiple of 16, both ends 16-byte aligned) to shared memory; counts on `bar`.
+__device__ __forceinline__ void bulk_load(uint32_t dst, const void* src, uint32_t bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src),
+               "r"(bytes), "r"(smem_u32(bar))
+               : "memory");
+}
+__device__ __forceinline__ void wide_score_barrier() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
+
+// A wait that runs out is recorded, and the loops go on without waiting: the block ends and frees what it holds.
+struct WideWait {
+  int* status;
+  bool ok = true;
+  __device__ __forceinline__ void operator()(uint64_t* bar, uint32_t parity, int code) {
+    if (ok) ok = mbar_wait(bar, parity, status, code);
+    __syncwarp();
+  }
+};
+
 template <int MT>
 __global__ void __launch_bounds__(kWideThreads, 1)
-softmax_attn_wide_kernel(const SoftmaxMmaParams p) {
+softmax_attn_wide_kernel(const SoftmaxMmaParams p, const int stages, int* status) {
   pdl_entry();
   extern __shared__ __align__(128) uint8_t smem[];
   constexpr int kRows = MT * 16;
-  constexpr int kParts = MT == 2 ? 4 : 8;              // warps that share a row, by keys
-  constexpr int kNt = MT == 2 ? 2 : 1;                 // key tiles of 8 per warp
-  __shared__ float s_max[kRows][8], s_sum[kRows][8];
+  constexpr int kParts = 4 / MT;                       // score warps that share a row, by keys
+  constexpr int kNt = MT;                              // key tiles of 8 per score warp
+  __shared__ __align__(16) float s_max[2][kRows][4];
+  __shared__ float s_fac[2][kRows], s_sum[kRows][4], s_ref[kRows];
+  __shared__ uint64_t full[kWideMaxStages], empty[kWideMaxStages], p_full[2], p_empty[2];
   const int en = blockIdx.x / p.G, g = blockIdx.x % p.G;
   const int len = p.e.len[en];
   if (len < p.min_len || len > p.max_len) return;
   const int DK = p.D, E = p.E, R = p.H / p.G;
+  const int n_rows = len * R, f0 = blockIdx.z * kRows;
+  if (f0 >= n_rows) return;
   const int d16 = (DK + 15) >> 4, e16 = (E + 15) >> 4;
   const int row_b = d16 * 32 + 16;                     // bytes of a row of queries or keys
-  const uint32_t sq = smem_u32(smem), sp = sq + kRows * row_b, sk = sp + kRows * kWidePRow;
+  const uint32_t sq = smem_u32(smem), sp = sq + kRows * row_b, sk = sp + 2 * kRows * kWidePRow;
   const int split = blockIdx.y, splits = gridDim.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int start = p.e.start[en], pos0 = p.e.pos0[en];
-  const int* pages = p.page_table + static_cast<long long>(en) * p.max_pages;
-  const int n_rows = len * R;
-  const int mt = MT == 2 ? warp & 1 : 0, part = MT == 2 ? warp >> 1 : warp;
-  const float scale = p.sp.scale * 1.4426950408889634f;
+  const int q_first = f0 / R, q_last = (min(f0 + kRows, n_rows) - 1) / R;
+  const int key_lo = visible_begin(pos0 + q_first, p.sp) / kServePage * kServePage, key_hi = pos0 + q_last + 1;
+  const int blocks = (key_hi - key_lo + kWideKeys - 1) / kWideKeys, per = (blocks + splits - 1) / splits;
+  const int b0 = split * per, n = max(0, min(blocks, b0 + per) - b0);          // blocks [b0, b0 + n)
+  const int cols = d16 * 2;                            // 16-byte pieces of a row
 
-  for (int f0 = blockIdx.z * kRows; f0 < n_rows; f0 += gridDim.z * kRows) {
-    const int q_first = f0 / R, q_last = (min(f0 + kRows, n_rows) - 1) / R;
-    const int key_lo = visible_begin(pos0 + q_first, p.sp) / kServePage * kServePage, key_hi = pos0 + q_last + 1;
-    const int blocks = (key_hi - key_lo + kWideKeys - 1) / kWideKeys, per = (blocks + splits - 1) / splits;
-    const int b0 = split * per, b1 = min(blocks, b0 + per);
-    const int last_page = (key_hi - 1) / kServePage;
-    const int cols = d16 * 2;                          // 16-byte pieces of a row
-    __syncthreads();                                   // the pass before has left the shared memory
-    auto load_block = [&](int b) {
-      const uint32_t dst = sk + (b & 1) * kWideKeys * row_b;
-      const int k0 = key_lo + b * kWideKeys;
-      for (int i = threadIdx.x; i < kWideKeys * cols; i += kWideThreads) {
-        const int t = i / cols, c = i - t * cols;
-        const int pg = min((k0 + t) / kServePage, last_page);            // beyond the last key: weight 0
-        const __nv_bfloat16* src = p.kcache + ((static_cast<long long>(pages[pg]) * p.G + g) * kServePage + (t & (kServePage - 1))) * DK + c * 8;
-        if (c * 8 < DK) sx_cp_async16(dst + t * row_b + c * 16, src);
-      }
-      asm volatile("cp.async.commit_group;" ::: "memory");
-    };
-    if (b0 < b1) load_block(b0);
-    // queries; what lies behind the last column of queries and keys is zero
-    for (int i = threadIdx.x; i < kRows * cols; i += kWideThreads) {
-      const int r = i / cols, c = i - r * cols, f = f0 + r;
-      uint4 v = make_uint4(0, 0, 0, 0);
-      if (f < n_rows && c * 8 < DK)
-        v = *reinterpret_cast<const uint4*>(p.q + static_cast<long long>(start + f / R) * p.ldq + static_cast<long long>(g * R + f % R) * DK + c * 8);
-      *reinterpret_cast<uint4*>(smem + r * row_b + c * 16) = v;
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < stages; ++i) {
+      mbar_init(&full[i], 1);
+      mbar_init(&empty[i], 8);
     }
-    if (cols * 8 > DK)
-      for (int t = threadIdx.x; t < 2 * kWideKeys; t += kWideThreads)
-        *reinterpret_cast<uint4*>(smem + (sk - sq) + t * row_b + (cols - 1) * 16) = make_uint4(0, 0, 0, 0);
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&p_full[i], 128);
+      mbar_init(&p_empty[i], 8);
+    }
+    mbar_fence_init();
+  }
+  // queries; zeros behind the last column
+  for (int i = threadIdx.x; i < kRows * cols; i += kWideThreads) {
+    const int r = i / cols, c = i - r * cols, f = f0 + r;
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (f < n_rows && c * 8 < DK)
+      v = *reinterpret_cast<const uint4*>(p.q + static_cast<long long>(start + f / R) * p.ldq + static_cast<long long>(g * R + f % R) * DK + c * 8);
+    *reinterpret_cast<uint4*>(smem + r * row_b + c * 16) = v;
+  }
+  __syncthreads();
 
-    // rows of this thread, for its score tile and for all tiles of the sums
+  WideWait wait{status};
+  if (warp == 12) {
+    // ---------------------------------------------------------------- producer (a page per lane)
+    const int* pages = p.page_table + static_cast<long long>(en) * p.max_pages;
+    const int last_page = (key_hi - 1) / kServePage, page0 = key_lo / kServePage + b0 * (kWideKeys / kServePage);
+    for (int i = 0, stage = 0, phase = 1; i < n; ++i) {
+      wait(&empty[stage], phase, kTimeoutEmpty);
+      if (!__all_sync(0xffffffffu, wait.ok)) break;
+      if (lane == 0) mbar_expect_tx(&full[stage], kWideKeys * row_b);
+      __syncwarp();
+      if (lane < kWideKeys / kServePage) {
+        const int pg = pages[min(page0 + i * (kWideKeys / kServePage) + lane, last_page)];      // beyond the last key: weight 0
+        bulk_load(sk + (stage * kWideKeys + lane * kServePage) * row_b,
+                  p.kcache + (static_cast<long long>(pg) * p.G + g) * kServePage * (row_b / 2), kServePage * row_b, &full[stage]);
+      }
+      if (++stage == stages) stage = 0, phase ^= 1;
+    }
+    if (!wait.ok) {                    // give copies in flight time to land before the block ends
+      const uint64_t t0 = global_timer_ns();
+      while (global_timer_ns() - t0 < 100000ull) {
+      }
+    }
+  } else if (warp < 4) {
+    // ---------------------------------------------------------------- scores of one row tile and 8 kNt keys of every block
+    const int mt = MT == 2 ? warp & 1 : 0, part = MT == 2 ? warp >> 1 : warp;
+    const float scale = p.sp.scale * 1.4426950408889634f;
     int hi[2], lo[2];
+    float mx[2] = {-INFINITY, -INFINITY}, sum[2] = {0.f, 0.f};
+    const int row0 = mt * 16 + (lane >> 2);            // this thread's rows: row0 and row0 + 8
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
-      const int f = f0 + mt * 16 + (lane >> 2) + 8 * h;
+      const int f = f0 + row0 + 8 * h;
       hi[h] = f < n_rows ? pos0 + f / R : -1;
       lo[h] = f < n_rows ? visible_begin(pos0 + f / R, p.sp) : 0;
     }
-    float mx[MT][2], sum[2] = {0.f, 0.f};
-    float acc[MT][4][2][4];                            // value tiles warp, warp + 8, ... of 16 columns
-#pragma unroll
-    for (int m = 0; m < MT; ++m) {
-      mx[m][0] = mx[m][1] = -INFINITY;
-#pragma unroll
-      for (int i = 0; i < 4; ++i)
-#pragma unroll
-        for (int n = 0; n < 2; ++n) acc[m][i][n][0] = acc[m][i][n][1] = acc[m][i][n][2] = acc[m][i][n][3] = 0.f;
-    }
-
-    for (int b = b0; b < b1; ++b) {
-      asm volatile("cp.async.wait_group 0;" ::: "memory");
-      __syncthreads();                                 // block b is there, block b - 1 has been used
-      if (b + 1 < b1) load_block(b + 1);
-      const uint32_t kb = sk + (b & 1) * kWideKeys * row_b;
-      const int k0 = key_lo + b * kWideKeys;
-      // ---- scores: rows of tile mt, keys [part * 8 kNt, +8 kNt)
+    const uint32_t qa = sq + (mt * 16 + (lane & 15)) * row_b + (lane >> 4) * 16;
+    // a load covers 16 keys x 16 columns, or 8 keys x 32 columns
+    const uint32_t k_off = MT == 2 ? (part * 16 + (lane & 7) + ((lane >> 4) << 3)) * row_b + ((lane >> 3) & 1) * 16
+                                   : (part * 8 + (lane & 7)) * row_b + (lane >> 3) * 16;
+    for (int j = 0, stage = 0, phase = 0; j < n; ++j) {
+      wait(&full[stage], phase, kTimeoutFull);
+      const uint32_t ka = sk + stage * kWideKeys * row_b + k_off;
       float sc[2][kNt][4];                             // two chains per tile
 #pragma unroll
-      for (int a = 0; a < 2; ++a)
+      for (int c = 0; c < 2; ++c)
 #pragma unroll
-        for (int n = 0; n < kNt; ++n) sc[a][n][0] = sc[a][n][1] = sc[a][n][2] = sc[a][n][3] = 0.f;
-      const uint32_t qa = sq + (mt * 16 + (lane & 15)) * row_b + (lane >> 4) * 16;
-      if (kNt == 2) {
-        const uint32_t ka = kb + (part * 16 + (lane & 7) + ((lane >> 4) << 3)) * row_b + ((lane >> 3) & 1) * 16;
+        for (int t = 0; t < kNt; ++t) sc[c][t][0] = sc[c][t][1] = sc[c][t][2] = sc[c][t][3] = 0.f;
+      int k = 0;
 #pragma unroll 4
-        for (int k = 0; k < d16; ++k) {
-          uint32_t a[4], v[4];
-          sx_ldsm_x4(qa + k * 32, a);
-          sx_ldsm_x4(ka + k * 32, v);
-          if (k & 1) {
-            sx_mma(sc[1][0], a, v[0], v[1]);
-            sx_mma(sc[1][kNt - 1], a, v[2], v[3]);
-          } else {
-            sx_mma(sc[0][0], a, v[0], v[1]);
-            sx_mma(sc[0][kNt - 1], a, v[2], v[3]);
-          }
-        }
-      } else {                                         // 8 keys: one load covers 32 columns
-        const uint32_t ka = kb + (part * 8 + (lane & 7)) * row_b + (lane >> 3) * 16;
-#pragma unroll 4
-        for (int k = 0; k < d16; k += 2) {
-          uint32_t a[4], v[4];
-          sx_ldsm_x4(qa + k * 32, a);
-          // an odd last step reads 32 bytes behind the row: the next row's, or the margin behind the last one
-          sx_ldsm_x4(ka + k * 32, v);
-          sx_mma(sc[0][0], a, v[0], v[1]);
-          if (k + 1 < d16) {
-            sx_ldsm_x4(qa + k * 32 + 32, a);
-            sx_mma(sc[1][0], a, v[2], v[3]);
-          }
+      for (; k + 1 < d16; k += 2) {
+        uint32_t a[2][4], v[2][4];
+        sx_ldsm_x4(qa + k * 32, a[0]);
+        sx_ldsm_x4(qa + k * 32 + 32, a[1]);
+        sx_ldsm_x4(ka + k * 32, v[0]);
+        if (MT == 2) sx_ldsm_x4(ka + k * 32 + 32, v[1]);
+        sx_mma(sc[0][0], a[0], v[0][0], v[0][1]);
+        if (MT == 2) {
+          sx_mma(sc[0][kNt - 1], a[0], v[0][2], v[0][3]);
+          sx_mma(sc[1][0], a[1], v[1][0], v[1][1]);
+          sx_mma(sc[1][kNt - 1], a[1], v[1][2], v[1][3]);
+        } else {
+          sx_mma(sc[1][0], a[1], v[0][2], v[0][3]);
         }
       }
-      float top[2] = {-INFINITY, -INFINITY}, s[kNt][4];
+      if (k < d16) {                                   // with 8 keys the load's upper half lies behind the row and is not used
+        uint32_t a[4], v[4];
+        sx_ldsm_x4(qa + k * 32, a);
+        sx_ldsm_x4(ka + k * 32, v);
+        sx_mma(sc[0][0], a, v[0], v[1]);
+        if (MT == 2) sx_mma(sc[0][kNt - 1], a, v[2], v[3]);
+      }
+      const int key0 = key_lo + (b0 + j) * kWideKeys + part * 8 * kNt + (lane & 3) * 2;
+      float s[kNt][4], top[2] = {-INFINITY, -INFINITY};
 #pragma unroll
-      for (int n = 0; n < kNt; ++n)
+      for (int t = 0; t < kNt; ++t)
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const int key = k0 + part * 8 * kNt + n * 8 + (lane & 3) * 2 + (i & 1), h = i >> 1;
-          s[n][i] = key <= hi[h] && key >= lo[h] ? (sc[0][n][i] + sc[1][n][i]) * scale : -INFINITY;
-          top[h] = fmaxf(top[h], s[n][i]);
+        for (int q = 0; q < 4; ++q) {
+          const int key = key0 + t * 8 + (q & 1), h = q >> 1;
+          s[t][q] = key <= hi[h] && key >= lo[h] ? (sc[0][t][q] + sc[1][t][q]) * scale : -INFINITY;
+          top[h] = fmaxf(top[h], s[t][q]);
         }
 #pragma unroll
       for (int h = 0; h < 2; ++h) {
         top[h] = fmaxf(top[h], __shfl_xor_sync(0xffffffffu, top[h], 1));
         top[h] = fmaxf(top[h], __shfl_xor_sync(0xffffffffu, top[h], 2));
-        if ((lane & 3) == 0) s_max[mt * 16 + (lane >> 2) + 8 * h][part] = top[h];
+        if ((lane & 3) == 0) s_max[j & 1][row0 + 8 * h][part] = top[h];
       }
-      __syncthreads();
-      float fac[MT][2];
-#pragma unroll
-      for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int h = 0; h < 2; ++h) {
-          float t = mx[m][h];
-#pragma unroll
-          for (int w = 0; w < kParts; ++w) t = fmaxf(t, s_max[m * 16 + (lane >> 2) + 8 * h][w]);
-          fac[m][h] = t == -INFINITY ? 1.f : exp2f(mx[m][h] - t);
-          mx[m][h] = t;
-        }
-      float ref[2], fmine[2];
+      wait(&p_empty[j & 1], ((j >> 1) & 1) ^ 1, kTimeoutEmpty);                // the weights of block j - 2 have been used
+      wide_score_barrier();
+      float ref[2];
 #pragma unroll
       for (int h = 0; h < 2; ++h) {
-        ref[h] = MT == 2 && mt ? mx[MT - 1][h] : mx[0][h];
-        fmine[h] = MT == 2 && mt ? fac[MT - 1][h] : fac[0][h];
-        if (ref[h] == -INFINITY) ref[h] = 0.f;
-        sum[h] *= fmine[h];
+        const int row = row0 + 8 * h;
+        float t = mx[h];
+#pragma unroll
+        for (int w = 0; w < kParts; ++w) t = fmaxf(t, s_max[j & 1][row][w]);
+        const float f = t == -INFINITY ? 1.f : exp2f(mx[h] - t);
+        mx[h] = t;
+        sum[h] *= f;
+        ref[h] = t == -INFINITY ? 0.f : t;
+        if (part == 0 && (lane & 3) == 0) s_fac[j & 1][row] = f;
       }
 #pragma unroll
-      for (int n = 0; n < kNt; ++n) {
+      for (int t = 0; t < kNt; ++t) {
         float w[4];
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          w[i] = exp2f(s[n][i] - ref[i >> 1]);
-          sum[i >> 1] += w[i];
+        for (int q = 0; q < 4; ++q) {
+          w[q] = exp2f(s[t][q] - ref[q >> 1]);
+          sum[q >> 1] += w[q];
         }
-        uint8_t* dst = smem + (sp - sq) + (mt * 16 + (lane >> 2)) * kWidePRow + (part * 8 * kNt + n * 8 + (lane & 3) * 2) * 2;
+        uint8_t* dst = smem + (sp - sq) + ((j & 1) * kRows + row0) * kWidePRow + (part * 8 * kNt + t * 8 + (lane & 3) * 2) * 2;
         *reinterpret_cast<uint32_t*>(dst) = pack_bf16x2(w[0], w[1]);
         *reinterpret_cast<uint32_t*>(dst + 8 * kWidePRow) = pack_bf16x2(w[2], w[3]);
       }
-      __syncthreads();
-      // ---- weighted sums: all rows, this warp's value tiles
+      mbar_arrive(&p_full[j & 1]);
+      if (++stage == stages) stage = 0, phase ^= 1;
+    }
 #pragma unroll
-      for (int m = 0; m < MT; ++m)
+    for (int h = 0; h < 2; ++h) {
+      float t = sum[h];
+      t += __shfl_xor_sync(0xffffffffu, t, 1);
+      t += __shfl_xor_sync(0xffffffffu, t, 2);
+      if ((lane & 3) == 0) s_sum[row0 + 8 * h][part] = t;
+      if (part == 0 && (lane & 3) == 0) s_ref[row0 + 8 * h] = mx[h];
+    }
+  }
+  // ------------------------------------------------------------------ weighted sums: value tiles vw, vw + 8, ... of 16 columns
+  const int vw = warp - 4;
+  float acc[MT][4][2][4];
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int t = 0; t < 2; ++t) acc[m][i][t][0] = acc[m][i][t][1] = acc[m][i][t][2] = acc[m][i][t][3] = 0.f;
+  if (vw >= 0 && vw < 8) {
+    for (int j = 0, stage = 0, phase = 0; j < n; ++j) {
+      wait(&p_full[j & 1], (j >> 1) & 1, kTimeoutFull);
+      // the keys are there too, but only the score warps have seen it: every reader of copied bytes observes the barrier
+      wait(&full[stage], phase, kTimeoutFull);
+#pragma unroll
+      for (int m = 0; m < MT; ++m) {
+        const float g0 = s_fac[j & 1][m * 16 + (lane >> 2)], g1 = s_fac[j & 1][m * 16 + (lane >> 2) + 8];
 #pragma unroll
         for (int i = 0; i < 4; ++i)
 #pragma unroll
-          for (int n = 0; n < 2; ++n)
-#pragma unroll
-            for (int q = 0; q < 4; ++q) acc[m][i][n][q] *= fac[m][q >> 1];
+          for (int t = 0; t < 2; ++t) {
+            acc[m][i][t][0] *= g0;
+            acc[m][i][t][1] *= g0;
+            acc[m][i][t][2] *= g1;
+            acc[m][i][t][3] *= g1;
+          }
+      }
 #pragma unroll
       for (int k = 0; k < kWideKeys / 16; ++k) {
+        const uint32_t kb = sk + (stage * kWideKeys + k * 16 + (lane & 15)) * row_b + (lane >> 4) * 16;
         uint32_t a[MT][4];
 #pragma unroll
-        for (int m = 0; m < MT; ++m) sx_ldsm_x4(sp + (m * 16 + (lane & 15)) * kWidePRow + k * 32 + (lane >> 4) * 16, a[m]);
+        for (int m = 0; m < MT; ++m)
+          sx_ldsm_x4(sp + ((j & 1) * kRows + m * 16 + (lane & 15)) * kWidePRow + k * 32 + (lane >> 4) * 16, a[m]);
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
-          const int tile = warp + 8 * i;
+          const int tile = vw + 8 * i;
           if (tile >= e16) break;
           uint32_t v[4];
-          sx_ldsm_x4_t(kb + (k * 16 + (lane & 15)) * row_b + tile * 32 + (lane >> 4) * 16, v);
+          sx_ldsm_x4_t(kb + tile * 32, v);
 #pragma unroll
           for (int m = 0; m < MT; ++m) {
             sx_mma(acc[m][i][0], a[m], v[0], v[1]);
@@ -209,67 +263,69 @@ softmax_attn_wide_kernel(const SoftmaxMmaParams p) {
           }
         }
       }
+      __syncwarp();
+      if (lane == 0) {
+        mbar_arrive(&empty[stage]);
+        mbar_arrive(&p_empty[j & 1]);
+      }
+      if (++stage == stages) stage = 0, phase ^= 1;
     }
-    // ---- output
+  }
+  __syncthreads();
+  if (vw < 0 || vw >= 8) return;
+  // ------------------------------------------------------------------ output
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
-      sum[h] += __shfl_xor_sync(0xffffffffu, sum[h], 1);
-      sum[h] += __shfl_xor_sync(0xffffffffu, sum[h], 2);
-      if ((lane & 3) == 0) s_sum[mt * 16 + (lane >> 2) + 8 * h][part] = sum[h];
-    }
-    __syncthreads();
+      const int rr = m * 16 + (lane >> 2) + 8 * h, f = f0 + rr;
+      if (f >= n_rows) continue;
+      const float ref = s_ref[rr];
+      float total = 0.f;
 #pragma unroll
-    for (int m = 0; m < MT; ++m)
+      for (int w = 0; w < kParts; ++w) total += s_sum[rr][w];
+      const int qi = f / R, head = g * R + f % R;
+      if (splits > 1) {
+        float* dst = p.part + (((static_cast<long long>(en) * p.max_len + qi) * p.H + head) * splits + split) * (E + 2);
 #pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        const int rr = m * 16 + (lane >> 2) + 8 * h, f = f0 + rr;
-        if (f >= n_rows) continue;
-        float total = 0.f;
+        for (int i = 0; i < 4; ++i)
 #pragma unroll
-        for (int w = 0; w < kParts; ++w) total += s_sum[rr][w];
-        const int qi = f / R, head = g * R + f % R;
-        if (splits > 1) {
-          float* dst = p.part + (((static_cast<long long>(en) * p.max_len + qi) * p.H + head) * splits + split) * (E + 2);
-#pragma unroll
-          for (int i = 0; i < 4; ++i)
-#pragma unroll
-            for (int n = 0; n < 2; ++n) {
-              const int c = (warp + 8 * i) * 16 + n * 8 + (lane & 3) * 2;
-              if (c < E) *reinterpret_cast<float2*>(dst + c) = make_float2(acc[m][i][n][2 * h], acc[m][i][n][2 * h + 1]);
-            }
-          if (warp == 0 && (lane & 3) == 0) {
-            dst[E] = mx[m][h];
-            dst[E + 1] = total;
+          for (int t = 0; t < 2; ++t) {
+            const int c = (vw + 8 * i) * 16 + t * 8 + (lane & 3) * 2;
+            if (c < E) *reinterpret_cast<float2*>(dst + c) = make_float2(acc[m][i][t][2 * h], acc[m][i][t][2 * h + 1]);
           }
-        } else {
-          const long long row = start + qi;
-          const bool per_column = p.sp.gate && p.sp.gate_cols != 1;
-          const float inv = inverse_sum(p.sp, head, mx[m][h], total) * (per_column ? 1.f : output_gate<__nv_bfloat16>(p.sp, row, head, 0));
-          __nv_bfloat16* dst = p.out + row * p.ldo + static_cast<long long>(head) * E;
-#pragma unroll
-          for (int i = 0; i < 4; ++i)
-#pragma unroll
-            for (int n = 0; n < 2; ++n) {
-              const int c = (warp + 8 * i) * 16 + n * 8 + (lane & 3) * 2;
-              if (c >= E) continue;
-              float u = acc[m][i][n][2 * h] * inv, v = acc[m][i][n][2 * h + 1] * inv;
-              if (per_column) {
-                u *= output_gate<__nv_bfloat16>(p.sp, row, head, c);
-                v *= output_gate<__nv_bfloat16>(p.sp, row, head, c + 1);
-              }
-              *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16x2(u, v);
-            }
+        if (vw == 0 && (lane & 3) == 0) {
+          dst[E] = ref;
+          dst[E + 1] = total;
         }
+      } else {
+        const long long row = start + qi;
+        const bool per_column = p.sp.gate && p.sp.gate_cols != 1;
+        const float inv = inverse_sum(p.sp, head, ref, total) * (per_column ? 1.f : output_gate<__nv_bfloat16>(p.sp, row, head, 0));
+        __nv_bfloat16* dst = p.out + row * p.ldo + static_cast<long long>(head) * E;
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+          for (int t = 0; t < 2; ++t) {
+            const int c = (vw + 8 * i) * 16 + t * 8 + (lane & 3) * 2;
+            if (c >= E) continue;
+            float u = acc[m][i][t][2 * h] * inv, v = acc[m][i][t][2 * h + 1] * inv;
+            if (per_column) {
+              u *= output_gate<__nv_bfloat16>(p.sp, row, head, c);
+              v *= output_gate<__nv_bfloat16>(p.sp, row, head, c + 1);
+            }
+            *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16x2(u, v);
+          }
       }
-  }
+    }
 }
 
 }  // namespace apb
 
 extern "C" {
 
-// bf16; kcache [pages, G, 16, D] whose first E columns are the values; D and E multiples of 8, D up to 640, E up to 512; entries of
-// min_len .. max_len rows.  part: fp32 scratch [entries, max_len, H, splits, E + 2] when splits > 1.
+// bf16; kcache [pages, G, 16, D rounded up to a multiple of 16, plus 8] whose first E columns are the values and whose columns behind
+// D are zeros; D and E multiples of 8, D up to 640, E up to 512; entries of min_len .. max_len rows.  part: fp32 scratch [entries, max_len, H, splits, E + 2] when splits > 1.
 int apb_softmax_attn_wide(const void* q, long long ldq, const int* e_start, const int* e_len, const int* e_slot, const int* e_pos0,
                           int n_entries, const int* page_table, int max_pages, const void* kcache, void* out, long long ldo,
                           float* part, int H, int G, int D, int E, int min_len, int max_len, int splits, float scale, int window,
@@ -285,13 +341,15 @@ int apb_softmax_attn_wide(const void* q, long long ldq, const int* e_start, cons
                            min_len, max_len, SoftmaxSpec{scale, 0.f, 0, 1, nullptr, 1.f, 0.f, window, sink, gate, ldg, gate_cols}};
   const long long rows = static_cast<long long>(max_len) * (H / G);
   const int mt = rows > 16 ? 2 : 1, row_b = (D + 15) / 16 * 32 + 16;
-  const int smem = mt * 16 * (row_b + kWidePRow) + 2 * kWideKeys * row_b + 64;
+  const int fixed = mt * 16 * (row_b + 2 * kWidePRow) + 32, fit = (kWideMaxSmem - fixed) / (kWideKeys * row_b);
+  const int stages = fit < kWideMaxStages ? fit : kWideMaxStages, smem = fixed + stages * kWideKeys * row_b;
   const long long passes = (rows + mt * 16 - 1) / (mt * 16);
-  const dim3 grid(n_entries * G, splits, static_cast<unsigned>(passes < 1024 ? passes : 1024));
+  if (passes > 65535 || stages < 2) return kBadArgument;
+  const dim3 grid(n_entries * G, splits, static_cast<unsigned>(passes));
   auto run = [&](auto fn) -> int {
     const cudaError_t e = cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return static_cast<int>(e);
-    return static_cast<int>(launch_kernel(fn, grid, dim3(kWideThreads), smem, s, p));
+    return static_cast<int>(launch_kernel(fn, grid, dim3(kWideThreads), smem, s, p, stages, status_device_ptr()));
   };
   const int rc = mt == 2 ? run(softmax_attn_wide_kernel<2>) : run(softmax_attn_wide_kernel<1>);
   return rc || splits == 1 ? rc : launch_softmax_merge(p, n_entries, splits, s);

@@ -326,13 +326,13 @@ class _LatentMixer(nn.Module):
             self.sink32.copy_(self.sink.data)
 
     def cache_layout(self) -> Dict[str, Any]:
-        return {"kv": (1, self.m.kv_rank + self.m.rot_dim, 0)}
+        return {"kv": (1, serving.shared_row(self.m.kv_rank + self.m.rot_dim, self.m.kv_rank, self.sink.dtype), 0)}
 
     def serve(self, b: serving.StepBatch, h: torch.Tensor, y: torch.Tensor, cache, run: int, rope) -> None:
         m, c = self.m, self.in_cols
         p = serving.linear(h, self.w_in)
         latents = cache.k[run]
-        serving.latent_norm_cache(b, p, c["dq"][0], c["dkv"][0], self.q_norm, self.kv_norm, rope[m.rot], latents, self.eps)
+        serving.latent_norm_cache(b, p, c["dq"][0], c["dkv"][0], self.q_norm, self.kv_norm, rope[m.rot], latents, self.eps, m.rot_dim)
         q = serving.linear(p[:, c["dq"][0]:c["dq"][0] + m.q_rank], self.w_q[:, :m.q_rank])
         a = _activations(b.rows, self.n_out, h)
         serving.latent_attention(b, q, self.spec, latents, self.w_absorb, self.w_expand, self.sink32, p[:, c["g"][0]:], rope[m.rot], a)

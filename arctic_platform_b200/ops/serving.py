@@ -40,9 +40,9 @@ def _fn(name: str):
                                     + [f, f, i, i, vp, f, f, i, vp, vp, ll, i, vp],
             "apb_row_norm_rope_cache": [vp, ll, i, i, i] + [vp] * 10 + [i, vp, vp] + [i] * 5 + [f, i, vp],
             "apb_residual_step": [vp] * 7 + [i, f] + [vp] * 5 + [i, i, i, f, f, i, i, i, vp],
-            "apb_latent_norm_cache": [vp, ll, i, i] + [vp] * 11 + [i, i, i, i, f, i, vp],
+            "apb_latent_norm_cache": [vp, ll, i, i] + [vp] * 11 + [i, i, i, i, i, f, i, vp],
             "apb_latent_rotate": [vp, ll] + [vp] * 8 + [i] * 6 + [vp],
-            "apb_latent_gather": [vp, vp, i, vp, i, vp, vp, i, i, vp],
+            "apb_latent_gather": [vp, vp, i, vp, i, vp, vp, i, i, i, vp],
             "apb_moe_serve_route": [vp, ll, vp, vp, i, i, i, i] + [vp] * 9 + [i, i, i, i, vp],
             "apb_moe_serve_gather": [vp, i, ll, vp, vp, vp, i, vp, vp, vp],
             "apb_gemm_simt_grouped": [vp, vp, vp, i, i, i, ll, ll, ll, i, vp, ll, vp, i, vp, i, vp],
@@ -606,6 +606,13 @@ def flash_tiles(host: np.ndarray, heads: int, kv_heads: int, min_len: int, windo
     return np.ascontiguousarray(work[np.argsort(-keys, kind="stable")], dtype=np.int32)
 
 
+def shared_row(dim: int, vdim: int, dtype: torch.dtype) -> int:
+    """Columns of a cache row of ``dim`` key columns whose first ``vdim`` are the values.  Where the tensor-core kernel takes the
+    sizes: padded to a multiple of 16 (zeros) and by 8 more, which spreads the rows over the shared-memory banks."""
+    fits = dtype == torch.bfloat16 and dim % 8 == 0 and vdim % 8 == 0 and dim <= 640 and vdim <= 512
+    return (dim + 15) // 16 * 16 + 8 if fits else dim
+
+
 MAX_WIDE_SPLITS = 16
 
 
@@ -615,20 +622,21 @@ def wide_splits(blocks: int, sms: int) -> int:
 
 
 def softmax_attention(b: StepBatch, q: torch.Tensor, heads: int, kcache: torch.Tensor, vcache: Optional[torch.Tensor],
-                      spec: SoftmaxSpec, lam: Optional[torch.Tensor], out: torch.Tensor, *, vdim: int = 0,
+                      spec: SoftmaxSpec, lam: Optional[torch.Tensor], out: torch.Tensor, *, dim: int = 0, vdim: int = 0,
                       sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, gate_cols: int = 1) -> None:
     """``q [rows, heads * maps * D]`` (column slice, rotated) over the entries' pages -> ``out [rows, heads * E]`` (column
-    slice).  Without a ``vcache`` the values are the first ``vdim`` columns of the key rows.  ``sink [heads]`` fp32: a score per
+    slice).  Without a ``vcache`` the values are the first ``vdim`` of the ``dim`` columns of the key rows (:func:`shared_row`).  ``sink [heads]`` fp32: a score per
     head that counts in the denominator only; ``gate``: columns of the activations whose sigmoid multiplies the output, one per
     head (``gate_cols`` 1) or one per output column (``gate_cols`` E).
     bf16 with head sizes that are multiples of 8 runs on tensor cores; fp32 and odd sizes on CUDA cores."""
     G, DK = kcache.shape[1], kcache.shape[3]
     E = vdim if vcache is None else vcache.shape[3]
-    D = DK // spec.maps
+    D = DK // spec.maps if vcache is not None else dim
     shape = (float(spec.scale), float(spec.cap), spec.chunk, spec.maps, _lib.ptr(lam), float(spec.post_scale), float(spec.eps))
     tail = shape + (spec.window, _lib.ptr(sink), _lib.ptr(gate), 0 if gate is None else gate.stride(0), gate_cols)
     aligned = not (D % 8 or E % 8 or q.stride(0) % 8 or out.stride(0) % 8 or (q.data_ptr() | out.data_ptr()) & 15)
-    if q.dtype != torch.bfloat16 or not aligned or (max(DK, E) > 256 and not (vcache is None and DK <= 640 and E <= 512 and spec.maps == 1)):
+    wide = vcache is None and DK > D
+    if not wide and (vcache is None or q.dtype != torch.bfloat16 or not aligned or max(DK, E) > 256):
         _call("apb_softmax_attn", _lib.ptr(q), q.stride(0), _lib.ptr(b.row_entry), *b.entry_ptrs(), _lib.ptr(b.page_table),
               b.page_table.stride(0), _lib.ptr(kcache), _lib.ptr(vcache), _lib.ptr(out), out.stride(0), b.rows, heads, G, D, E,
               *tail, dtype_code(q.dtype))
@@ -636,7 +644,6 @@ def softmax_attention(b: StepBatch, q: torch.Tensor, heads: int, kcache: torch.T
     plain = spec.maps == 1 and not spec.cap and not spec.chunk
     tc = spec.maps == 2 and D % 16 == 0 and D <= 64 and E <= 128 and 0 < spec.cap <= MAX_FIXED_CAP
     flash = plain and vcache is not None and flash_fits(D, 0, E) and not out.data_ptr() & 15
-    wide = plain and vcache is None and (DK > 256 or heads // G > 16)
     lens = np.ones(1, dtype=np.int64) if b.host is None else b.host[:, 1]
     limit = SHORT_ROWS if tc or flash else int(lens.max())
     short = lens[lens <= limit]
@@ -684,13 +691,13 @@ class LatentSpec:
 
 
 def latent_norm_cache(b: StepBatch, p: torch.Tensor, q_col: int, c_col: int, q_gain: torch.Tensor, c_gain: torch.Tensor,
-                      rope: Tuple[torch.Tensor, torch.Tensor], cache: torch.Tensor, eps: float) -> None:
+                      rope: Tuple[torch.Tensor, torch.Tensor], cache: torch.Tensor, eps: float, rot: int) -> None:
     """Norm of the query latent (columns ``q_col`` of ``p``, in place) and of the key / value latent (``c_col``), rotation of the
-    shared key part behind it; both go to the page cache ``[pages, 1, PAGE, rank + rot]``."""
+    shared key part of ``rot`` columns behind it; both go to the page cache ``[pages, 1, PAGE, >= rank + rot]``."""
     Q, C = q_gain.numel(), c_gain.numel()
     _call("apb_latent_norm_cache", _lib.ptr(p), p.stride(0), q_col, c_col, _lib.ptr(q_gain), _lib.ptr(c_gain), _lib.ptr(b.row_entry),
-          *b.entry_ptrs(), _lib.ptr(b.kv_slot), _lib.ptr(rope[0]), _lib.ptr(rope[1]), _lib.ptr(cache), b.rows, Q, C,
-          cache.shape[3] - C, float(eps), dtype_code(p.dtype))
+          *b.entry_ptrs(), _lib.ptr(b.kv_slot), _lib.ptr(rope[0]), _lib.ptr(rope[1]), _lib.ptr(cache), cache.shape[3],
+          b.rows, Q, C, rot, float(eps), dtype_code(p.dtype))
 
 
 def latent_rotate(b: StepBatch, q: torch.Tensor, s: LatentSpec, rope: Tuple[torch.Tensor, torch.Tensor],
@@ -770,7 +777,7 @@ def latent_attention(b: StepBatch, q: torch.Tensor, s: LatentSpec, cache: torch.
         heads_linear(q[rows], D + R, w_absorb, H, D, ql, C + R)
         latent_rotate(p, q[rows], s, rope, ql)
         o = torch.empty((p.rows, H * C), device=q.device, dtype=q.dtype)
-        softmax_attention(p, ql, H, cache, None, spec, None, o, vdim=C, sink=sink)
+        softmax_attention(p, ql, H, cache, None, spec, None, o, dim=C + R, vdim=C, sink=sink)
         heads_linear(o, C, w_value, H, C, out[rows], E, None if gate is None else gate[rows])
     if not expand or not (b.host[:, 1] > limit).any():
         return
@@ -783,7 +790,7 @@ def latent_attention(b: StepBatch, q: torch.Tensor, s: LatentSpec, cache: torch.
         keys = plan["pages"].shape[0] * PAGE
         latents, rotated = (torch.empty((keys, w), device=q.device, dtype=q.dtype) for w in (C, R))
         _call("apb_latent_gather", _lib.ptr(cache), _lib.ptr(pages), pages.shape[0], _lib.ptr(b.page_table), b.page_table.stride(0),
-              _lib.ptr(latents), _lib.ptr(rotated), C, R)
+              _lib.ptr(latents), _lib.ptr(rotated), cache.shape[3], C, R)
         kv = linear(latents, w_expand[:, :C])
         v = kv[:, v_col:]
         _call("apb_flash_tc", _lib.ptr(q), q.stride(0), b.rows, _lib.ptr(work), work.shape[0], None, 0, _lib.ptr(kv), kv.stride(0),

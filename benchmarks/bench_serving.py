@@ -258,7 +258,7 @@ def titatar_ops(cfg, phase):
          T * W * (8 + 4 + 2 + (4 if clear else 0) + 2) + 2 * pairs * W, 0),
         ("latent input projections (GEMM)", lambda: serving.linear(h, lm.w_in, pl), *gemm(pl.shape[1], W)),
         ("latent norms + cache write", lambda: serving.latent_norm_cache(b, pl, lc["dq"][0], lc["dkv"][0], lm.q_norm, lm.kv_norm, rl,
-                                                                        cache.k[0], 1e-6), 2 * T * (2 * L.q_rank + 2 * (C + R)), 0),
+                                                                        cache.k[0], 1e-6, R), 2 * T * (2 * L.q_rank + 2 * (C + R)), 0),
         ("query projection (GEMM)", lambda: serving.linear(ql, lm.w_q[:, :L.q_rank], q), *gemm(q.shape[1], L.q_rank)),
         ("latent attention", lambda: serving.latent_attention(b, q, lm.spec, cache.k[0], lm.w_absorb, lm.w_expand, lm.sink32,
                                                               pl[:, lc["g"][0]:], rl, lo),

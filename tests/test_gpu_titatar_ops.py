@@ -156,7 +156,7 @@ def _run_softmax(dtype, heads, lens, cuts, seed=0, faults=()):
             out.append(o)
         want.append(torch.cat(out, -1))
     pages, pool = _pages(lens, seed)
-    kc = torch.zeros(pool, G, PAGE, D, device="cuda", dtype=dtype)
+    kc = torch.zeros(pool, G, PAGE, D if own else serving.shared_row(D, E, dtype), device="cuda", dtype=dtype)
     vc = torch.zeros(pool, G, PAGE, E, device="cuda", dtype=dtype)
     got = [[] for _ in lens]
     for step in _schedule(lens, cuts):
@@ -164,11 +164,11 @@ def _run_softmax(dtype, heads, lens, cuts, seed=0, faults=()):
         p = torch.cat([P[i][a:a + n] for i, a, n in step]).cuda()
         rows = torch.tensor([int(pages[i][t // PAGE]) for i, a, n in step for t in range(a, a + n)], device="cuda")
         off = torch.tensor([t % PAGE for i, a, n in step for t in range(a, a + n)], device="cuda")
-        kc[rows, :, off] = p[:, ck:ck + G * D].view(-1, G, D)
+        kc[rows, :, off, :D] = p[:, ck:ck + G * D].view(-1, G, D)
         if own:
             vc[rows, :, off] = p[:, cv:cv + G * E].view(-1, G, E)
         out = torch.full((b.rows, _pad8(H * E) + 16), 3.0, device="cuda", dtype=dtype)
-        serving.softmax_attention(b, p, H, kc, vc if own else None, spec, None, out[:, 8:], vdim=E,
+        serving.softmax_attention(b, p, H, kc, vc if own else None, spec, None, out[:, 8:], dim=D, vdim=E,
                                   sink=None if sink is None else sink.cuda(), gate=p[:, cg:] if gate else None, gate_cols=1 if gate == 1 else E)
         assert (out[:, :8] == 3).all() and (out[:, 8 + H * E:] == 3).all()
         r = 0
@@ -258,7 +258,7 @@ def _run_latent(dtype, shape, lens, cuts, seed=0, faults=()):
         want.append(oracle.latent_attention_mixer(m, W64, "", h.double(), eps, faults))
     pages, pool = _pages(lens, seed)
     rope = norm.rope_tables(max(lens), R, 2000.0, "cuda", yarn)
-    cache = torch.zeros(pool, 1, PAGE, C + R, device="cuda", dtype=dtype)
+    cache = torch.zeros(pool, 1, PAGE, serving.shared_row(C + R, C, dtype), device="cuda", dtype=dtype)
     got = [[] for _ in lens]
     c = mixer.in_cols
     for step in _schedule(lens, cuts):
@@ -271,7 +271,7 @@ def _run_latent(dtype, shape, lens, cuts, seed=0, faults=()):
             o, k = c[n]
             p[:, o:o + k] = h[:, at:at + k]
             at += k
-        serving.latent_norm_cache(b, p, c["dq"][0], c["dkv"][0], mixer.q_norm, mixer.kv_norm, rope, cache, eps)
+        serving.latent_norm_cache(b, p, c["dq"][0], c["dkv"][0], mixer.q_norm, mixer.kv_norm, rope, cache, eps, R)
         q = serving.linear(p[:, c["dq"][0]:c["dq"][0] + Q], mixer.w_q[:, :Q])
         out = torch.full((b.rows, _pad8(H * E) + 16), 3.0, device="cuda", dtype=dtype)
         serving.latent_attention(b, q, mixer.spec, cache, mixer.w_absorb, mixer.w_expand, mixer.sink32, p[:, c["g"][0]:], rope, out[:, 8:])
