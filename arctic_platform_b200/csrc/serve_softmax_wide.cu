@@ -5,10 +5,10 @@
 // of 16-byte pieces, so that the rows of a page arrive by one copy and fall into different banks.
 //
 // Many query heads share one key row of up to 640 columns, so a row is read once and meets MT * 16 (query, head) rows on m16n8k16
-// tensor-core tiles.  A CTA = one entry, KV head, group of rows and share of the keys.  13 warps: a producer that copies pages
-// into a ring of 32-key blocks, four score warps and eight value warps.  A block serves both products: the score warps split its
-// keys (and the rows), agree on the rows' maximum and leave weights and rescaling factors in shared memory; the value warps, which
-// split the value columns, work on one block while the score warps are at the next and the others are on their way.
+// tensor-core tiles.  A CTA = one entry, KV head, group of rows and share of the keys.  13 warps: a producer that copies pages into
+// a ring, four score warps and eight value warps.  A page serves both products.  The score warps take the pages in turn: each
+// computes a page's scores for all rows, then -- in the order of the pages -- moves the rows' running maximum, and leaves weights
+// and rescaling factors in shared memory; the value warps split the value columns and follow page by page.
 #include "common.cuh"
 #include "host_utils.cuh"
 #include "serve_softmax_mma.cuh"
@@ -16,11 +16,11 @@
 namespace apb {
 
 constexpr int kWideThreads = 13 * 32;
-constexpr int kWideKeys = 32;                          // keys per block
-constexpr int kWideMaxStages = 8;
+constexpr int kWideScore = 4;                          // score warps
+constexpr int kWideMaxStages = 12;
 constexpr int kWideMaxSmem = 227 * 1024 - 3 * 1024;    // besides the static arrays
 constexpr int kWideMaxDK = 640, kWideMaxE = 512;
-constexpr int kWidePRow = kWideKeys * 2 + 16;          // bytes of a row of weights
+constexpr int kWidePRow = kServePage * 2 + 16;         // bytes of a row of weights
 
 // Contiguous bytes (a multiple of 16, both ends 16-byte aligned) to shared memory; counts on `bar`.
 __device__ __forceinline__ void bulk_load(uint32_t dst, const void* src, uint32_t bytes, uint64_t* bar) {
@@ -28,7 +28,6 @@ __device__ __forceinline__ void bulk_load(uint32_t dst, const void* src, uint32_
                "r"(bytes), "r"(smem_u32(bar))
                : "memory");
 }
-__device__ __forceinline__ void wide_score_barrier() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
 
 // A wait that runs out is recorded, and the loops go on without waiting: the block ends and frees what it holds.
 struct WideWait {
@@ -46,11 +45,8 @@ softmax_attn_wide_kernel(const SoftmaxMmaParams p, const int stages, int* status
   pdl_entry();
   extern __shared__ __align__(128) uint8_t smem[];
   constexpr int kRows = MT * 16;
-  constexpr int kParts = 4 / MT;                       // score warps that share a row, by keys
-  constexpr int kNt = MT;                              // key tiles of 8 per score warp
-  __shared__ __align__(16) float s_max[2][kRows][4];
-  __shared__ float s_fac[2][kRows], s_sum[kRows][4], s_ref[kRows];
-  __shared__ uint64_t full[kWideMaxStages], empty[kWideMaxStages], p_full[2], p_empty[2];
+  __shared__ float s_run[kRows], s_fac[kWideScore][kRows], s_sum[kWideScore][kRows], s_last[kWideScore][kRows];
+  __shared__ uint64_t full[kWideMaxStages], empty[kWideMaxStages], p_full[kWideScore], p_empty[kWideScore], turn[kWideScore];
   const int en = blockIdx.x / p.G, g = blockIdx.x % p.G;
   const int len = p.e.len[en];
   if (len < p.min_len || len > p.max_len) return;
@@ -59,14 +55,14 @@ softmax_attn_wide_kernel(const SoftmaxMmaParams p, const int stages, int* status
   if (f0 >= n_rows) return;
   const int d16 = (DK + 15) >> 4, e16 = (E + 15) >> 4;
   const int row_b = d16 * 32 + 16;                     // bytes of a row of queries or keys
-  const uint32_t sq = smem_u32(smem), sp = sq + kRows * row_b, sk = sp + 2 * kRows * kWidePRow;
+  const uint32_t sq = smem_u32(smem), sp = sq + kRows * row_b, sk = sp + kWideScore * kRows * kWidePRow;
   const int split = blockIdx.y, splits = gridDim.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int start = p.e.start[en], pos0 = p.e.pos0[en];
   const int q_first = f0 / R, q_last = (min(f0 + kRows, n_rows) - 1) / R;
-  const int key_lo = visible_begin(pos0 + q_first, p.sp) / kServePage * kServePage, key_hi = pos0 + q_last + 1;
-  const int blocks = (key_hi - key_lo + kWideKeys - 1) / kWideKeys, per = (blocks + splits - 1) / splits;
-  const int b0 = split * per, n = max(0, min(blocks, b0 + per) - b0);          // blocks [b0, b0 + n)
+  const int page_lo = visible_begin(pos0 + q_first, p.sp) / kServePage, page_hi = (pos0 + q_last) / kServePage + 1;
+  const int per = (page_hi - page_lo + splits - 1) / splits;
+  const int b0 = page_lo + split * per, n = max(0, min(page_hi, b0 + per) - b0);        // pages [b0, b0 + n)
   const int cols = d16 * 2;                            // 16-byte pieces of a row
 
   if (threadIdx.x == 0) {
@@ -74,12 +70,15 @@ softmax_attn_wide_kernel(const SoftmaxMmaParams p, const int stages, int* status
       mbar_init(&full[i], 1);
       mbar_init(&empty[i], 8);
     }
-    for (int i = 0; i < 2; ++i) {
-      mbar_init(&p_full[i], 128);
+    for (int i = 0; i < kWideScore; ++i) {
+      mbar_init(&p_full[i], 1);
       mbar_init(&p_empty[i], 8);
+      mbar_init(&turn[i], 1);
     }
     mbar_fence_init();
+    mbar_arrive(&turn[0]);
   }
+  if (threadIdx.x < kRows) s_run[threadIdx.x] = -INFINITY;
   // queries; zeros behind the last column
   for (int i = threadIdx.x; i < kRows * cols; i += kWideThreads) {
     const int r = i / cols, c = i - r * cols, f = f0 + r;
@@ -92,129 +91,151 @@ softmax_attn_wide_kernel(const SoftmaxMmaParams p, const int stages, int* status
 
   WideWait wait{status};
   if (warp == 12) {
-    // ---------------------------------------------------------------- producer (a page per lane)
-    const int* pages = p.page_table + static_cast<long long>(en) * p.max_pages;
-    const int last_page = (key_hi - 1) / kServePage, page0 = key_lo / kServePage + b0 * (kWideKeys / kServePage);
-    for (int i = 0, stage = 0, phase = 1; i < n; ++i) {
-      wait(&empty[stage], phase, kTimeoutEmpty);
-      if (!__all_sync(0xffffffffu, wait.ok)) break;
-      if (lane == 0) mbar_expect_tx(&full[stage], kWideKeys * row_b);
-      __syncwarp();
-      if (lane < kWideKeys / kServePage) {
-        const int pg = pages[min(page0 + i * (kWideKeys / kServePage) + lane, last_page)];      // beyond the last key: weight 0
-        bulk_load(sk + (stage * kWideKeys + lane * kServePage) * row_b,
-                  p.kcache + (static_cast<long long>(pg) * p.G + g) * kServePage * (row_b / 2), kServePage * row_b, &full[stage]);
+    // ---------------------------------------------------------------- producer
+    if (lane == 0) {
+      const int* pages = p.page_table + static_cast<long long>(en) * p.max_pages;
+      for (int i = 0, stage = 0, phase = 1; i < n; ++i) {
+        const int pg = pages[b0 + i];
+        if (!mbar_wait(&empty[stage], phase, status, kTimeoutEmpty)) {
+          wait.ok = false;
+          break;
+        }
+        mbar_expect_tx(&full[stage], kServePage * row_b);
+        bulk_load(sk + stage * kServePage * row_b, p.kcache + (static_cast<long long>(pg) * p.G + g) * kServePage * (row_b / 2),
+                  kServePage * row_b, &full[stage]);
+        if (++stage == stages) stage = 0, phase ^= 1;
       }
-      if (++stage == stages) stage = 0, phase ^= 1;
     }
     if (!wait.ok) {                    // give copies in flight time to land before the block ends
       const uint64_t t0 = global_timer_ns();
       while (global_timer_ns() - t0 < 100000ull) {
       }
     }
-  } else if (warp < 4) {
-    // ---------------------------------------------------------------- scores of one row tile and 8 kNt keys of every block
-    const int mt = MT == 2 ? warp & 1 : 0, part = MT == 2 ? warp >> 1 : warp;
+  } else if (warp < kWideScore) {
+    // ---------------------------------------------------------------- scores of the pages warp, warp + 4, ...; all rows
     const float scale = p.sp.scale * 1.4426950408889634f;
-    int hi[2], lo[2];
-    float mx[2] = {-INFINITY, -INFINITY}, sum[2] = {0.f, 0.f};
-    const int row0 = mt * 16 + (lane >> 2);            // this thread's rows: row0 and row0 + 8
+    int hi[MT][2], lo[MT][2];
+    float last[MT][2], sum[MT][2];                     // this warp's share of the weight sums, relative to 2^last
 #pragma unroll
-    for (int h = 0; h < 2; ++h) {
-      const int f = f0 + row0 + 8 * h;
-      hi[h] = f < n_rows ? pos0 + f / R : -1;
-      lo[h] = f < n_rows ? visible_begin(pos0 + f / R, p.sp) : 0;
-    }
-    const uint32_t qa = sq + (mt * 16 + (lane & 15)) * row_b + (lane >> 4) * 16;
-    // a load covers 16 keys x 16 columns, or 8 keys x 32 columns
-    const uint32_t k_off = MT == 2 ? (part * 16 + (lane & 7) + ((lane >> 4) << 3)) * row_b + ((lane >> 3) & 1) * 16
-                                   : (part * 8 + (lane & 7)) * row_b + (lane >> 3) * 16;
-    for (int j = 0, stage = 0, phase = 0; j < n; ++j) {
-      wait(&full[stage], phase, kTimeoutFull);
-      const uint32_t ka = sk + stage * kWideKeys * row_b + k_off;
-      float sc[2][kNt][4];                             // two chains per tile
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int f = f0 + m * 16 + (lane >> 2) + 8 * h;
+        hi[m][h] = f < n_rows ? pos0 + f / R : -1;
+        lo[m][h] = f < n_rows ? visible_begin(pos0 + f / R, p.sp) : 0;
+        last[m][h] = -INFINITY;
+        sum[m][h] = 0.f;
+      }
+    const uint32_t qa = sq + (lane & 15) * row_b + (lane >> 4) * 16;
+    const uint32_t k_off = ((lane & 7) + ((lane >> 4) << 3)) * row_b + ((lane >> 3) & 1) * 16;
+    for (int j = warp; j < n; j += kWideScore) {
+      const int stage = j % stages, turns = j / kWideScore;
+      wait(&full[stage], (j / stages) & 1, kTimeoutFull);
+      const uint32_t ka = sk + stage * kServePage * row_b + k_off;
+      float sc[2][MT][2][4];                           // two chains per tile
 #pragma unroll
       for (int c = 0; c < 2; ++c)
 #pragma unroll
-        for (int t = 0; t < kNt; ++t) sc[c][t][0] = sc[c][t][1] = sc[c][t][2] = sc[c][t][3] = 0.f;
-      int k = 0;
-#pragma unroll 4
-      for (; k + 1 < d16; k += 2) {
-        uint32_t a[2][4], v[2][4];
-        sx_ldsm_x4(qa + k * 32, a[0]);
-        sx_ldsm_x4(qa + k * 32 + 32, a[1]);
-        sx_ldsm_x4(ka + k * 32, v[0]);
-        if (MT == 2) sx_ldsm_x4(ka + k * 32 + 32, v[1]);
-        sx_mma(sc[0][0], a[0], v[0][0], v[0][1]);
-        if (MT == 2) {
-          sx_mma(sc[0][kNt - 1], a[0], v[0][2], v[0][3]);
-          sx_mma(sc[1][0], a[1], v[1][0], v[1][1]);
-          sx_mma(sc[1][kNt - 1], a[1], v[1][2], v[1][3]);
-        } else {
-          sx_mma(sc[1][0], a[1], v[0][2], v[0][3]);
-        }
-      }
-      if (k < d16) {                                   // with 8 keys the load's upper half lies behind the row and is not used
-        uint32_t a[4], v[4];
-        sx_ldsm_x4(qa + k * 32, a);
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+          for (int t = 0; t < 2; ++t) sc[c][m][t][0] = sc[c][m][t][1] = sc[c][m][t][2] = sc[c][m][t][3] = 0.f;
+      auto steps = [&](int k, int c) {
+        uint32_t v[4], a[MT][4];
         sx_ldsm_x4(ka + k * 32, v);
-        sx_mma(sc[0][0], a, v[0], v[1]);
-        if (MT == 2) sx_mma(sc[0][kNt - 1], a, v[2], v[3]);
+#pragma unroll
+        for (int m = 0; m < MT; ++m) sx_ldsm_x4(qa + m * 16 * row_b + k * 32, a[m]);
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          sx_mma(sc[c][m][0], a[m], v[0], v[1]);
+          sx_mma(sc[c][m][1], a[m], v[2], v[3]);
+        }
+      };
+      int k = 0;
+#pragma unroll 3
+      for (; k + 1 < d16; k += 2) {
+        steps(k, 0);
+        steps(k + 1, 1);
       }
-      const int key0 = key_lo + (b0 + j) * kWideKeys + part * 8 * kNt + (lane & 3) * 2;
-      float s[kNt][4], top[2] = {-INFINITY, -INFINITY};
+      if (k < d16) steps(k, 0);
+      const int key0 = (b0 + j) * kServePage + (lane & 3) * 2;
+      float s[MT][2][4], top[MT][2];
 #pragma unroll
-      for (int t = 0; t < kNt; ++t)
+      for (int m = 0; m < MT; ++m) {
+        top[m][0] = top[m][1] = -INFINITY;
 #pragma unroll
-        for (int q = 0; q < 4; ++q) {
-          const int key = key0 + t * 8 + (q & 1), h = q >> 1;
-          s[t][q] = key <= hi[h] && key >= lo[h] ? (sc[0][t][q] + sc[1][t][q]) * scale : -INFINITY;
-          top[h] = fmaxf(top[h], s[t][q]);
+        for (int t = 0; t < 2; ++t)
+#pragma unroll
+          for (int q = 0; q < 4; ++q) {
+            const int key = key0 + t * 8 + (q & 1), h = q >> 1;
+            s[m][t][q] = key <= hi[m][h] && key >= lo[m][h] ? (sc[0][m][t][q] + sc[1][m][t][q]) * scale : -INFINITY;
+            top[m][h] = fmaxf(top[m][h], s[m][t][q]);
+          }
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          top[m][h] = fmaxf(top[m][h], __shfl_xor_sync(0xffffffffu, top[m][h], 1));
+          top[m][h] = fmaxf(top[m][h], __shfl_xor_sync(0xffffffffu, top[m][h], 2));
+        }
+      }
+      // ---- in the order of the pages: the running maximum
+      wait(&turn[warp], turns & 1, kTimeoutFull);
+      float before[MT][2];
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          before[m][h] = s_run[m * 16 + (lane >> 2) + 8 * h];
+          top[m][h] = fmaxf(top[m][h], before[m][h]);
+        }
+      __syncwarp();
+      if ((lane & 3) == 0)
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+          for (int h = 0; h < 2; ++h) s_run[m * 16 + (lane >> 2) + 8 * h] = top[m][h];
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&turn[(warp + 1) % kWideScore]);
+      // ---- weights
+      wait(&p_empty[warp], (turns & 1) ^ 1, kTimeoutEmpty);                    // this warp's last weights have been used
+#pragma unroll
+      for (int m = 0; m < MT; ++m) {
+        float ref[2];
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          const float t = top[m][h];
+          ref[h] = t == -INFINITY ? 0.f : t;
+          if (t != -INFINITY) sum[m][h] *= exp2f(last[m][h] - t);
+          last[m][h] = t;
+          if ((lane & 3) == 0) s_fac[warp][m * 16 + (lane >> 2) + 8 * h] = t == -INFINITY ? 1.f : exp2f(before[m][h] - t);
         }
 #pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        top[h] = fmaxf(top[h], __shfl_xor_sync(0xffffffffu, top[h], 1));
-        top[h] = fmaxf(top[h], __shfl_xor_sync(0xffffffffu, top[h], 2));
-        if ((lane & 3) == 0) s_max[j & 1][row0 + 8 * h][part] = top[h];
-      }
-      wait(&p_empty[j & 1], ((j >> 1) & 1) ^ 1, kTimeoutEmpty);                // the weights of block j - 2 have been used
-      wide_score_barrier();
-      float ref[2];
+        for (int t = 0; t < 2; ++t) {
+          float w[4];
 #pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        const int row = row0 + 8 * h;
-        float t = mx[h];
-#pragma unroll
-        for (int w = 0; w < kParts; ++w) t = fmaxf(t, s_max[j & 1][row][w]);
-        const float f = t == -INFINITY ? 1.f : exp2f(mx[h] - t);
-        mx[h] = t;
-        sum[h] *= f;
-        ref[h] = t == -INFINITY ? 0.f : t;
-        if (part == 0 && (lane & 3) == 0) s_fac[j & 1][row] = f;
-      }
-#pragma unroll
-      for (int t = 0; t < kNt; ++t) {
-        float w[4];
-#pragma unroll
-        for (int q = 0; q < 4; ++q) {
-          w[q] = exp2f(s[t][q] - ref[q >> 1]);
-          sum[q >> 1] += w[q];
+          for (int q = 0; q < 4; ++q) {
+            w[q] = exp2f(s[m][t][q] - ref[q >> 1]);
+            sum[m][q >> 1] += w[q];
+          }
+          uint8_t* dst = smem + (sp - sq) + (warp * kRows + m * 16 + (lane >> 2)) * kWidePRow + (t * 8 + (lane & 3) * 2) * 2;
+          *reinterpret_cast<uint32_t*>(dst) = pack_bf16x2(w[0], w[1]);
+          *reinterpret_cast<uint32_t*>(dst + 8 * kWidePRow) = pack_bf16x2(w[2], w[3]);
         }
-        uint8_t* dst = smem + (sp - sq) + ((j & 1) * kRows + row0) * kWidePRow + (part * 8 * kNt + t * 8 + (lane & 3) * 2) * 2;
-        *reinterpret_cast<uint32_t*>(dst) = pack_bf16x2(w[0], w[1]);
-        *reinterpret_cast<uint32_t*>(dst + 8 * kWidePRow) = pack_bf16x2(w[2], w[3]);
       }
-      mbar_arrive(&p_full[j & 1]);
-      if (++stage == stages) stage = 0, phase ^= 1;
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&p_full[warp]);
     }
 #pragma unroll
-    for (int h = 0; h < 2; ++h) {
-      float t = sum[h];
-      t += __shfl_xor_sync(0xffffffffu, t, 1);
-      t += __shfl_xor_sync(0xffffffffu, t, 2);
-      if ((lane & 3) == 0) s_sum[row0 + 8 * h][part] = t;
-      if (part == 0 && (lane & 3) == 0) s_ref[row0 + 8 * h] = mx[h];
-    }
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int row = m * 16 + (lane >> 2) + 8 * h;
+        float t = sum[m][h];
+        t += __shfl_xor_sync(0xffffffffu, t, 1);
+        t += __shfl_xor_sync(0xffffffffu, t, 2);
+        if ((lane & 3) == 0) {
+          s_sum[warp][row] = t;
+          s_last[warp][row] = last[m][h];
+        }
+      }
   }
   // ------------------------------------------------------------------ weighted sums: value tiles vw, vw + 8, ... of 16 columns
   const int vw = warp - 4;
@@ -227,46 +248,48 @@ softmax_attn_wide_kernel(const SoftmaxMmaParams p, const int stages, int* status
       for (int t = 0; t < 2; ++t) acc[m][i][t][0] = acc[m][i][t][1] = acc[m][i][t][2] = acc[m][i][t][3] = 0.f;
   if (vw >= 0 && vw < 8) {
     for (int j = 0, stage = 0, phase = 0; j < n; ++j) {
-      wait(&p_full[j & 1], (j >> 1) & 1, kTimeoutFull);
-      // the keys are there too, but only the score warps have seen it: every reader of copied bytes observes the barrier
+      const int buf = j % kWideScore;
+      wait(&p_full[buf], (j / kWideScore) & 1, kTimeoutFull);
+      // the keys are there too, but only a score warp has seen it: every reader of copied bytes observes the barrier
       wait(&full[stage], phase, kTimeoutFull);
+      float fac[MT][2];
+      bool same = true;
 #pragma unroll
-      for (int m = 0; m < MT; ++m) {
-        const float g0 = s_fac[j & 1][m * 16 + (lane >> 2)], g1 = s_fac[j & 1][m * 16 + (lane >> 2) + 8];
+      for (int m = 0; m < MT; ++m)
 #pragma unroll
-        for (int i = 0; i < 4; ++i)
+        for (int h = 0; h < 2; ++h) {
+          fac[m][h] = s_fac[buf][m * 16 + (lane >> 2) + 8 * h];
+          same = same && fac[m][h] == 1.f;
+        }
+      uint32_t a[MT][4], v[4][4];
 #pragma unroll
-          for (int t = 0; t < 2; ++t) {
-            acc[m][i][t][0] *= g0;
-            acc[m][i][t][1] *= g0;
-            acc[m][i][t][2] *= g1;
-            acc[m][i][t][3] *= g1;
-          }
-      }
+      for (int m = 0; m < MT; ++m) sx_ldsm_x4(sp + (buf * kRows + m * 16 + (lane & 15)) * kWidePRow + (lane >> 4) * 16, a[m]);
+      const uint32_t kb = sk + (stage * kServePage + (lane & 15)) * row_b + (lane >> 4) * 16;
 #pragma unroll
-      for (int k = 0; k < kWideKeys / 16; ++k) {
-        const uint32_t kb = sk + (stage * kWideKeys + k * 16 + (lane & 15)) * row_b + (lane >> 4) * 16;
-        uint32_t a[MT][4];
+      for (int i = 0; i < 4; ++i)
+        if (vw + 8 * i < e16) sx_ldsm_x4_t(kb + (vw + 8 * i) * 32, v[i]);
+      if (!__all_sync(0xffffffffu, same)) {
 #pragma unroll
         for (int m = 0; m < MT; ++m)
-          sx_ldsm_x4(sp + ((j & 1) * kRows + m * 16 + (lane & 15)) * kWidePRow + k * 32 + (lane >> 4) * 16, a[m]);
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const int tile = vw + 8 * i;
-          if (tile >= e16) break;
-          uint32_t v[4];
-          sx_ldsm_x4_t(kb + tile * 32, v);
+          for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int t = 0; t < 2; ++t)
+#pragma unroll
+              for (int q = 0; q < 4; ++q) acc[m][i][t][q] *= fac[m][q >> 1];
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (vw + 8 * i < e16)
 #pragma unroll
           for (int m = 0; m < MT; ++m) {
-            sx_mma(acc[m][i][0], a[m], v[0], v[1]);
-            sx_mma(acc[m][i][1], a[m], v[2], v[3]);
+            sx_mma(acc[m][i][0], a[m], v[i][0], v[i][1]);
+            sx_mma(acc[m][i][1], a[m], v[i][2], v[i][3]);
           }
-        }
-      }
       __syncwarp();
       if (lane == 0) {
         mbar_arrive(&empty[stage]);
-        mbar_arrive(&p_empty[j & 1]);
+        mbar_arrive(&p_empty[buf]);
       }
       if (++stage == stages) stage = 0, phase ^= 1;
     }
@@ -280,10 +303,11 @@ softmax_attn_wide_kernel(const SoftmaxMmaParams p, const int stages, int* status
     for (int h = 0; h < 2; ++h) {
       const int rr = m * 16 + (lane >> 2) + 8 * h, f = f0 + rr;
       if (f >= n_rows) continue;
-      const float ref = s_ref[rr];
+      const float ref = s_run[rr];
       float total = 0.f;
 #pragma unroll
-      for (int w = 0; w < kParts; ++w) total += s_sum[rr][w];
+      for (int w = 0; w < kWideScore; ++w)
+        if (s_last[w][rr] != -INFINITY) total += s_sum[w][rr] * exp2f(s_last[w][rr] - ref);
       const int qi = f / R, head = g * R + f % R;
       if (splits > 1) {
         float* dst = p.part + (((static_cast<long long>(en) * p.max_len + qi) * p.H + head) * splits + split) * (E + 2);
@@ -341,8 +365,8 @@ int apb_softmax_attn_wide(const void* q, long long ldq, const int* e_start, cons
                            min_len, max_len, SoftmaxSpec{scale, 0.f, 0, 1, nullptr, 1.f, 0.f, window, sink, gate, ldg, gate_cols}};
   const long long rows = static_cast<long long>(max_len) * (H / G);
   const int mt = rows > 16 ? 2 : 1, row_b = (D + 15) / 16 * 32 + 16;
-  const int fixed = mt * 16 * (row_b + 2 * kWidePRow) + 32, fit = (kWideMaxSmem - fixed) / (kWideKeys * row_b);
-  const int stages = fit < kWideMaxStages ? fit : kWideMaxStages, smem = fixed + stages * kWideKeys * row_b;
+  const int fixed = mt * 16 * (row_b + kWideScore * kWidePRow), fit = (kWideMaxSmem - fixed) / (kServePage * row_b);
+  const int stages = fit < kWideMaxStages ? fit : kWideMaxStages, smem = fixed + stages * kServePage * row_b;
   const long long passes = (rows + mt * 16 - 1) / (mt * 16);
   if (passes > 65535 || stages < 2) return kBadArgument;
   const dim3 grid(n_entries * G, splits, static_cast<unsigned>(passes));
