@@ -2,8 +2,8 @@
 // output gates (see SoftmaxSpec), no bound on the scores.
 //
 // A CTA = two tiles of 128 query rows that share their keys: two query heads of one KV head on the same rows, or two
-// consecutive row tiles of one head.  320 threads: warp 0 TMA producer, warp 1 MMA issuer, warps 2-5 and 6-9 the weight groups,
-// one per tile, which ping-pong on the tensor core.
+// consecutive row tiles of one head.  352 threads: warp 0 TMA producer, warps 2-5 and 6-9 the weight groups and warps 1 and 10 the MMA
+// issuers, one per tile; the tiles ping-pong on the tensor core.
 //
 // Keys and values come from the page cache (16-row boxes, one page of one KV head each) or from a contiguous copy of the
 // entry's context (128-row boxes; a head's columns side by side).  A key may have a second part that all heads share (the
@@ -18,7 +18,7 @@
 
 namespace apb {
 
-constexpr int kFlThreads = 320;
+constexpr int kFlThreads = 352;
 constexpr int kFlKeys = 128;                           // keys per block
 constexpr int kFlChunk = 128 * 64 * 2;                 // 64 columns of 128 rows
 constexpr int kFlChunks = 14;                          // query chunks and ring slots together
@@ -37,6 +37,40 @@ struct FlashParams {
   SoftmaxSpec sp;
   int* status;
 };
+
+// Weights 2^(score scale + off) of a row's 128 scores at t_s, packed, and their sum in two halves; top: the largest exponent.
+// WHOLE: every key counts, otherwise those in [skip, limit).
+template <bool WHOLE>
+__device__ __forceinline__ uint64_t flash_weights(uint32_t t_s, uint64_t scale2, float off, int limit, int skip, float& top,
+                                                  uint32_t (&pk)[4][16]) {
+  const uint64_t off2 = xtc_pair(off, off);
+  uint64_t sum[2] = {xtc_pair(0.f, 0.f), xtc_pair(0.f, 0.f)};
+  float t0 = -INFINITY, t1 = -INFINITY;
+  uint32_t stage[2][32];
+  tmem_ld_32x32(t_s, stage[0]);
+#pragma unroll
+  for (int c = 0; c < 4; ++c) {                        // the next 32 scores are on their way while these are worked on
+    uint32_t(&r)[32] = stage[c & 1];
+    xtc_wait_load(r);
+    if (c < 3) tmem_ld_32x32(t_s + (c + 1) * 32, stage[(c + 1) & 1]);
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+      float2 v = xtc_unpair(xtc_fma2(xtc_pair(__uint_as_float(r[2 * i]), __uint_as_float(r[2 * i + 1])), scale2, off2));
+      if (!WHOLE) {
+        const int a = c * 32 + 2 * i;
+        if (a >= limit || a < skip) v.x = -INFINITY;
+        if (a + 1 >= limit || a + 1 < skip) v.y = -INFINITY;
+      }
+      t0 = fmaxf(t0, v.x);
+      t1 = fmaxf(t1, v.y);
+      const float w0 = xtc_ex2(v.x), w1 = xtc_ex2(v.y);
+      sum[i & 1] = xtc_add2(sum[i & 1], xtc_pair(w0, w1));
+      pk[c][i] = pack_bf16x2(w0, w1);
+    }
+  }
+  top = fmaxf(t0, t1);
+  return xtc_add2(sum[0], sum[1]);
+}
 
 __global__ void __launch_bounds__(kFlThreads, 1)
 flash_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_k,
@@ -65,7 +99,7 @@ flash_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
   if (threadIdx.x == 0) {
     for (int s = 0; s < ring; ++s) {
       mbar_init(&full[s], 1);
-      mbar_init(&empty[s], 1);
+      mbar_init(&empty[s], n_tiles);
     }
     mbar_init(q_full, 1);
     for (int g = 0; g < 2; ++g) {
@@ -100,14 +134,14 @@ flash_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
     const int page0 = k0 / kServePage, n_pages = (last + kServePage - 1) / kServePage;
     const int* pages = p.page_table + static_cast<long long>(entry) * p.max_pages;
     bool ok = true;
-    int n = 0;
+    int slot = 0;
+    uint32_t phase = 1;
     for (int j = 0; j < n_blocks && ok; ++j) {
       int row = 0;
       if (paged && lane < kFlKeys / kServePage)
         row = (pages[min(page0 + j * (kFlKeys / kServePage) + lane, n_pages - 1)] * p.G + kvh) * kServePage;
-      for (int c = 0; c < per; ++c, ++n) {
-        const int slot = n % ring;
-        ok = mbar_wait(&empty[slot], ((n / ring) & 1) ^ 1, p.status, kTimeoutEmpty);
+      for (int c = 0; c < per; ++c) {
+        ok = mbar_wait(&empty[slot], phase, p.status, kTimeoutEmpty);
         ok = __all_sync(0xffffffffu, ok);
         if (!ok) break;
         if (lane == 0) mbar_expect_tx(&full[slot], kFlChunk);
@@ -121,6 +155,7 @@ flash_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
         } else if (lane == 0) {
           tma_load_2d(dst, map, &full[slot], second ? col : kvh * (c < k1 ? p.D : p.E) + col, base_row + k0 + j * kFlKeys);
         }
+        if (++slot == ring) slot = 0, phase ^= 1;
       }
     }
     if (!ok) {                         // give copies in flight time to land before the block ends
@@ -128,86 +163,93 @@ flash_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
       while (global_timer_ns() - t0 < 100000ull) {
       }
     }
-  } else if (warp == 1) {
-    // ---------------------------------------------------------------- MMA issuer
-    if (lane == 0) {
-      const int e16 = (p.E + 15) & ~15;
+  } else if (warp == 1 || warp == 10) {
+    // ---------------------------------------------------------------- MMA issuers, one per tile
+    const int g = warp == 10;
+    if (lane == 0 && g < n_tiles) {
+      const int nb = g ? nb1 : nb0, e16 = (p.E + 15) & ~15;
       const uint32_t idesc_s = umma_idesc_bf16(128, kFlKeys, 0, 0);
       const uint32_t idesc_o = umma_idesc_bf16(128, e16, 0, 1);
       const uint32_t idesc_lo = umma_idesc_bf16(128, 64, 0, 1), idesc_hi = umma_idesc_bf16(128, e16 - 64 > 0 ? e16 - 64 : 16, 0, 1);
-      const uint32_t kv = smem_u32(smem_kv);
-      bool ok = mbar_wait(q_full, 0, p.status, kTimeoutFull);
-      auto wait_item = [&](int n) { return mbar_wait(&full[n % ring], (n / ring) & 1, p.status, kTimeoutFull); };
-      auto wait_items = [&](int n, int count) {
-        for (int c = 0; c < count; ++c)
-          if (!wait_item(n + c)) return false;
+      // descriptors differ in their address field (16-byte units) only
+      const uint64_t k_desc = umma_smem_desc(0, 0, 1024), v_desc = umma_smem_desc(0, kFlChunk, 1024);
+      constexpr uint32_t kChunk16 = kFlChunk >> 4;
+      const uint32_t q16 = smem_u32(smem_q + g * kch * kFlChunk) >> 4, kv16 = smem_u32(smem_kv) >> 4;
+      const uint32_t t_s = tmem_base + g * 128, t_o = tmem_base + 256 + g * 128;
+      const int steps1 = (p.D - (k1 - 1) * 64) >> 4, steps2 = p.R ? (p.R - (kch - k1 - 1) * 64) >> 4 : 0;   // of the parts' last chunks
+      int slot = 0;                                    // of the next item, and the parity of its phase
+      uint32_t phase = 0;
+      auto wait_items = [&](int count) {
+        for (int c = 0; c < count; ++c) {
+          if (!mbar_wait(&full[slot], phase, p.status, kTimeoutFull)) return false;
+          if (++slot == ring) slot = 0, phase ^= 1;
+        }
         return true;
       };
-      auto release = [&](int n, int count) {
-        for (int c = 0; c < count; ++c) tc_commit(&empty[(n + c) % ring]);
+      auto release = [&](int first, int count) {
+        for (int c = 0; c < count; ++c, first = first + 1 == ring ? 0 : first + 1) tc_commit(&empty[first]);
       };
-      auto issue_s = [&](int g, int n) {               // n: ring item of the block's first key chunk
+      auto issue_s = [&](int first) {                  // slot of the block's first key chunk
+        uint64_t qd = k_desc + q16;
         uint32_t more = 0;
         for (int c = 0; c < kch; ++c) {
-          const uint32_t qa = smem_u32(smem_q + (g * kch + c) * kFlChunk), ka = kv + ((n + c) % ring) * kFlChunk;
-          const int cols = c < k1 ? min(64, p.D - c * 64) : min(64, p.R - (c - k1) * 64);
-          for (int k = 0; k < cols >> 4; ++k) {
-            umma_bf16_ss(tmem_base + g * 128, umma_smem_desc(qa + k * 32, 0, 1024), umma_smem_desc(ka + k * 32, 0, 1024), idesc_s, more);
-            more = 1;
-          }
+          const uint64_t kd = k_desc + (kv16 + first * kChunk16);
+          const int steps = c == k1 - 1 ? steps1 : c == kch - 1 ? steps2 : 4;
+#pragma unroll
+          for (int k = 0; k < 4; ++k)
+            if (k < steps) {
+              umma_bf16_ss(t_s, qd + k * 2, kd + k * 2, idesc_s, more);
+              more = 1;
+            }
+          qd += kChunk16;
+          first = first + 1 == ring ? 0 : first + 1;
         }
         tc_commit(&s_full[g]);
       };
-      auto issue_o = [&](int g, int n, bool first_block) {
-        const uint32_t t_o = tmem_base + 256 + g * 128, t_p = tmem_base + g * 128;
-        const int s0 = n % ring;
-        if (vch == 1 || s0 + 1 < ring) {
-          const uint32_t va = kv + s0 * kFlChunk;
+      auto issue_o = [&](int first, bool first_block) {
+        const uint64_t vd = v_desc + (kv16 + first * kChunk16);
+        const bool split = vch == 2 && first + 1 == ring;                // the value chunks lie at both ends of the ring
+        const uint32_t idesc = split ? idesc_lo : idesc_o;
 #pragma unroll
-          for (int k = 0; k < kFlKeys / 16; ++k)
-            umma_bf16_ts(t_o, t_p + k * 8, umma_smem_desc(va + k * 2048, kFlChunk, 1024), idesc_o, first_block && k == 0 ? 0u : 1u);
-        } else {                                       // the value chunks lie at both ends of the ring
-          const uint32_t va = kv + s0 * kFlChunk;
-          for (int k = 0; k < kFlKeys / 16; ++k)
-            umma_bf16_ts(t_o, t_p + k * 8, umma_smem_desc(va + k * 2048, kFlChunk, 1024), idesc_lo, first_block && k == 0 ? 0u : 1u);
-          for (int k = 0; k < kFlKeys / 16; ++k)
-            umma_bf16_ts(t_o + 64, t_p + k * 8, umma_smem_desc(kv + k * 2048, kFlChunk, 1024), idesc_hi, first_block && k == 0 ? 0u : 1u);
+        for (int k = 0; k < kFlKeys / 16; ++k) umma_bf16_ts(t_o, t_s + k * 8, vd + k * 128, idesc, first_block && k == 0 ? 0u : 1u);
+        if (split) {
+          const uint64_t v2 = v_desc + kv16;
+#pragma unroll
+          for (int k = 0; k < kFlKeys / 16; ++k) umma_bf16_ts(t_o + 64, t_s + k * 8, v2 + k * 128, idesc_hi, first_block && k == 0 ? 0u : 1u);
         }
       };
-      if (ok) ok = wait_items(0, kch);
+      bool ok = mbar_wait(q_full, 0, p.status, kTimeoutFull) && wait_items(kch);
       if (ok) {
         tc_fence_after();
-        for (int g = 0; g < n_tiles; ++g) issue_s(g, 0);
+        issue_s(0);
         release(0, kch);
       }
       for (int j = 0; j < n_blocks && ok; ++j) {
-        const int nv = j * per + kch, nk = (j + 1) * per;
-        const bool more = j + 1 < n_blocks;
-        if (!wait_items(nv, vch) || (more && !wait_items(nk, kch))) {
-          ok = false;
-          break;
-        }
-        tc_fence_after();
-        for (int g = 0; g < n_tiles; ++g) {
-          const int nb = g ? nb1 : nb0;
-          if (j >= nb) continue;
-          if (!mbar_wait(&p_full[g], j & 1, p.status, kTimeoutTmemEmpty)) {
-            ok = false;
-            break;
-          }
+        const bool more = j + 1 < n_blocks;            // of the other tile, perhaps
+        const int sv = slot;
+        if (!wait_items(vch)) break;
+        if (j < nb) {
+          if (!mbar_wait(&p_full[g], j & 1, p.status, kTimeoutTmemEmpty)) break;
           tc_fence_after();
-          issue_o(g, nv, j == 0);
-          if (j + 1 < nb)
-            issue_s(g, nk);                            // runs after the product above has read the weights
-          else
-            tc_commit(&o_full[g]);
+          issue_o(sv, j == 0);
+          if (more) release(sv, vch);
+          if (j + 1 == nb) tc_commit(&o_full[g]);
+        } else if (more) {
+          for (int c = 0, at = sv; c < vch; ++c, at = at + 1 == ring ? 0 : at + 1) mbar_arrive(&empty[at]);
         }
-        if (!ok) break;
-        release(nv, vch);
-        if (more) release(nk, kch);
+        if (!more) break;
+        const int sk = slot;
+        if (!wait_items(kch)) break;
+        if (j + 1 < nb) {                              // these scores run after the product above has read the weights
+          tc_fence_after();
+          issue_s(sk);
+          release(sk, kch);
+        } else {
+          for (int c = 0, at = sk; c < kch; ++c, at = at + 1 == ring ? 0 : at + 1) mbar_arrive(&empty[at]);
+        }
       }
     }
-  } else if (((warp - 2) >> 2) < n_tiles) {
+  } else if (warp < 10 && ((warp - 2) >> 2) < n_tiles) {
     // ---------------------------------------------------------------- weight groups, one per tile
     const int g = (warp - 2) >> 2;
     const int quarter = warp & 3, row = quarter * 32 + lane;
@@ -234,30 +276,9 @@ flash_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
       uint32_t pk[4][16];
       for (int pass = 0; pass < 2; ++pass) {           // a second time if the reference had to move
         const float off = ref == -INFINITY ? 0.f : -ref;
-        const uint64_t off2 = xtc_pair(off, off);
-        float top = -INFINITY;                         // largest score relative to the reference
-        uint64_t block2 = xtc_pair(0.f, 0.f);
-        uint32_t stage[2][32];
-        tmem_ld_32x32(t_s, stage[0]);
-#pragma unroll
-        for (int c = 0; c < 4; ++c) {                  // the next 32 scores are on their way while these are worked on
-          uint32_t(&r)[32] = stage[c & 1];
-          xtc_wait_load(r);
-          if (c < 3) tmem_ld_32x32(t_s + (c + 1) * 32, stage[(c + 1) & 1]);
-#pragma unroll
-          for (int i = 0; i < 16; ++i) {
-            float2 v = xtc_unpair(xtc_fma2(xtc_pair(__uint_as_float(r[2 * i]), __uint_as_float(r[2 * i + 1])), scale2, off2));
-            if (!whole) {
-              const int a = c * 32 + 2 * i;
-              if (a >= limit || a < skip) v.x = -INFINITY;
-              if (a + 1 >= limit || a + 1 < skip) v.y = -INFINITY;
-            }
-            top = fmaxf(fmaxf(top, v.x), v.y);
-            const float w0 = xtc_ex2(v.x), w1 = xtc_ex2(v.y);
-            block2 = xtc_add2(block2, xtc_pair(w0, w1));
-            pk[c][i] = pack_bf16x2(w0, w1);
-          }
-        }
+        float top;                                     // largest score relative to the reference
+        const uint64_t block2 = whole ? flash_weights<true>(t_s, scale2, off, limit, skip, top, pk)
+                                      : flash_weights<false>(t_s, scale2, off, limit, skip, top, pk);
         const bool behind = top > kFlLag || (ref == -INFINITY && top > -INFINITY);
         if (pass == 1 || !__any_sync(0xffffffffu, behind)) {
           sum2 = xtc_add2(sum2, block2);
