@@ -305,6 +305,12 @@ flash_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
       tc_fence_before();
       mbar_arrive(&p_full[g]);
     }
+    if (p.sp.gate && row < valid) {                    // the row's gates come closer while the last products run
+      const __nv_bfloat16* gate = static_cast<const __nv_bfloat16*>(p.sp.gate) + (static_cast<long long>(row0) + row) * p.sp.ldg +
+                                  static_cast<long long>(head) * p.sp.gate_cols;
+      for (int c = 0; c < p.sp.gate_cols; c += 64) asm volatile("prefetch.global.L1 [%0];" ::"l"(gate + c));
+    }
+    __syncwarp();
     if (ok) ok = mbar_wait(&o_full[g], 0, p.status, kTimeoutTmemFull);
     if (ok) {
       tc_fence_after();
@@ -333,8 +339,8 @@ flash_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
               const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gw[i]));
-              v[2 * i] /= 1.f + __expf(-f.x);
-              v[2 * i + 1] /= 1.f + __expf(-f.y);
+              v[2 * i] = __fdividef(v[2 * i], 1.f + __expf(-f.x));
+              v[2 * i + 1] = __fdividef(v[2 * i + 1], 1.f + __expf(-f.y));
             }
           }
           *reinterpret_cast<uint4*>(dst + c + q * 8) =

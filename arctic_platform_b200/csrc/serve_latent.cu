@@ -60,27 +60,41 @@ latent_norm_cache_kernel(T* __restrict__ p, long long ld, int q_col, int c_col, 
 }
 
 // The rotated part (R columns behind D) of every head of q [rows, H * (D + R)]: in place, or (dst) into column C of the head's
-// row of dst [rows, H * (C + R)].  One thread per pair.
-template <typename T>
+// row of dst [rows, H * (C + R)].  One thread per V pairs (V 4: 16-byte accesses, bf16).
+template <typename T, int V>
 __global__ void __launch_bounds__(256)
 latent_rotate_kernel(T* __restrict__ q, long long ld, const int* __restrict__ row_entry, const ServeEntries e,
                      const float* __restrict__ cos_t, const float* __restrict__ sin_t, T* __restrict__ dst, int rows, int H,
                      int D, int R, int C) {
   pdl_entry();
-  const int half = R >> 1;
+  const int half = R >> 1, per = half / V;
   const long long idx = blockIdx.x * 256LL + threadIdx.x;
-  if (idx >= static_cast<long long>(rows) * H * half) return;
-  const int i = static_cast<int>(idx % half), h = static_cast<int>(idx / half % H);
-  const int row = static_cast<int>(idx / half / H);
+  if (idx >= static_cast<long long>(rows) * H * per) return;
+  const int i = static_cast<int>(idx % per) * V, h = static_cast<int>(idx / per % H);
+  const int row = static_cast<int>(idx / per / H);
   const int en = row_entry ? row_entry[row] : row;
   const int at = row - e.start[en];
   if (at < 0 || at >= e.len[en]) return;
   const long long tr = static_cast<long long>(e.pos0[en] + at) * half + i;
   T* src = q + static_cast<long long>(row) * ld + static_cast<long long>(h) * (D + R) + D + 2 * i;
   T* out = dst ? dst + (static_cast<long long>(row) * H + h) * (C + R) + C + 2 * i : src;
-  const float u = to_f32(src[0]), v = to_f32(src[1]), cs = cos_t[tr], sn = sin_t[tr];
-  out[0] = from_f32<T>(u * cs - v * sn);
-  out[1] = from_f32<T>(v * cs + u * sn);
+  if constexpr (V == 4) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(src);
+    const float4 cs = *reinterpret_cast<const float4*>(cos_t + tr), sn = *reinterpret_cast<const float4*>(sin_t + tr);
+    const uint32_t w[4] = {raw.x, raw.y, raw.z, raw.w};
+    const float c[4] = {cs.x, cs.y, cs.z, cs.w}, s[4] = {sn.x, sn.y, sn.z, sn.w};
+    uint32_t o[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[j]));
+      o[j] = pack_bf16x2(f.x * c[j] - f.y * s[j], f.y * c[j] + f.x * s[j]);
+    }
+    *reinterpret_cast<uint4*>(out) = make_uint4(o[0], o[1], o[2], o[3]);
+  } else {
+    const float u = to_f32(src[0]), v = to_f32(src[1]), cs = cos_t[tr], sn = sin_t[tr];
+    out[0] = from_f32<T>(u * cs - v * sn);
+    out[1] = from_f32<T>(v * cs + u * sn);
+  }
 }
 
 // Page rows of some entries side by side: work [n][4] = entry, page of the entry, first row of the copy, tokens.
@@ -126,11 +140,17 @@ int apb_latent_rotate(void* q, long long ld, const int* row_entry, const int* e_
   if (rows <= 0 || R == 0) return 0;
   if (H <= 0 || D < 0 || R < 0 || (R & 1) || !cos_t || !sin_t) return kBadArgument;
   const ServeEntries e{e_start, e_len, e_slot, e_pos0};
-  const long long n = static_cast<long long>(rows) * H * (R >> 1);
+  const bool vec = dtype == 0 && !((D | R | ld | (dst ? C : 0)) & 7) &&
+                   !((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(dst) | reinterpret_cast<uintptr_t>(cos_t) |
+                      reinterpret_cast<uintptr_t>(sin_t)) & 15);
+  const long long n = static_cast<long long>(rows) * H * (R >> 1) / (vec ? 4 : 1);
   const dim3 grid(static_cast<unsigned>((n + 255) / 256));
-  APB_SERVE_DTYPE(dtype, return static_cast<int>(launch_kernel(latent_rotate_kernel<T>, grid, dim3(256), 0, s,
-                                                               static_cast<T*>(q), ld, row_entry, e, cos_t, sin_t,
-                                                               static_cast<T*>(dst), rows, H, D, R, C)));
+#define APB_ROTATE(TT, VV)                                                                                                  \
+  return static_cast<int>(launch_kernel(latent_rotate_kernel<TT, VV>, grid, dim3(256), 0, s, static_cast<TT*>(q), ld, row_entry, \
+                                        e, cos_t, sin_t, static_cast<TT*>(dst), rows, H, D, R, C))
+  if (vec) APB_ROTATE(__nv_bfloat16, 4);
+  APB_SERVE_DTYPE(dtype, APB_ROTATE(T, 1));
+#undef APB_ROTATE
 }
 
 // bf16; C, R and ldk multiples of 8.
