@@ -1,9 +1,9 @@
 // Latent attention: the small steps around its products.
 //
 // A token keeps one latent of C columns and one rotated key part of R columns that all heads share; both lie side by side in a
-// page row [pages, 1, 16, ldk] of at least C + R columns.  A head's keys and values are projections of the latent, so attention can run either on the
-// expanded keys and values, or -- with the key projection moved to the query and the value projection behind the sum -- on
-// the latents themselves.  Rotary positions pair neighbouring dimensions.
+// page row [pages, 1, 16, ldk] of at least C + R columns.  A head's keys and values are projections of the latent, so attention
+// can run either on the expanded keys and values, or -- with the key projection moved to the query and the value projection
+// behind the sum -- on the latents themselves.  Rotary positions pair neighbouring dimensions.
 #include "common.cuh"
 #include "host_utils.cuh"
 #include "serve_common.cuh"

@@ -2,9 +2,9 @@
 // chunk of positions only) and sliding windows, sinks, output gates, one or two maps per head (differential attention).  See
 // SoftmaxSpec.
 //
-// Keys and values live in pages of 16 tokens (kcache [pages, G, 16, maps * D], vcache [pages, G, 16, E]; without a vcache the
-// values are the first E columns of the key rows -- softmax_attn_kernel only); the step's own keys are already there when these kernels run, so prompts,
-// portions of prompts and decoded tokens read the same memory.
+// Keys and values live in pages of 16 tokens (kcache [pages, G, 16, maps * D], vcache [pages, G, 16, E]; the first kernel also
+// takes no vcache: the values are then the first E columns of the key rows); the step's own keys are already there when these
+// kernels run, so prompts, portions of prompts and decoded tokens read the same memory.
 //
 //  * softmax_attn_kernel      any D up to 1024, E up to 512, bf16 or fp32, fp32 arithmetic throughout (the fp32 engine, odd sizes);
 //  * softmax_attn_mma_kernel  bf16, D and E multiples of 8, maps * D and E up to 256: m16n8k16 tensor-core tiles whose 16

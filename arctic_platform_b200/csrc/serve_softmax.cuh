@@ -1,4 +1,4 @@
-// Declarations shared by the paged softmax attention kernels (serve_softmax.cu, serve_softmax_tc.cu).
+// Declarations shared by the paged softmax attention kernels (serve_softmax*.cu, serve_flash_tc.cu).
 #pragma once
 #include "serve_common.cuh"
 
@@ -64,7 +64,6 @@ __device__ __forceinline__ float tanh_series(float z) {
 }
 __device__ __forceinline__ float tanh_exp(float z) { return 1.f - __fdividef(2.f, 1.f + __expf(2.f * z)); }
 __device__ __forceinline__ float tanh_any(float z) { return fabsf(z) <= kSmallTanh ? tanh_series(z) : tanh_exp(z); }
-
 
 // ---------------------------------------------------------------------------- pieces of the tcgen05 kernels
 __device__ __forceinline__ float xtc_ex2(float x) {

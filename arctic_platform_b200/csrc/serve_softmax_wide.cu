@@ -84,7 +84,8 @@ softmax_attn_wide_kernel(const SoftmaxMmaParams p, const int stages, int* status
     const int r = i / cols, c = i - r * cols, f = f0 + r;
     uint4 v = make_uint4(0, 0, 0, 0);
     if (f < n_rows && c * 8 < DK)
-      v = *reinterpret_cast<const uint4*>(p.q + static_cast<long long>(start + f / R) * p.ldq + static_cast<long long>(g * R + f % R) * DK + c * 8);
+      v = *reinterpret_cast<const uint4*>(p.q + static_cast<long long>(start + f / R) * p.ldq +
+                                          static_cast<long long>(g * R + f % R) * DK + c * 8);
     *reinterpret_cast<uint4*>(smem + r * row_b + c * 16) = v;
   }
   __syncthreads();
@@ -349,7 +350,8 @@ softmax_attn_wide_kernel(const SoftmaxMmaParams p, const int stages, int* status
 extern "C" {
 
 // bf16; kcache [pages, G, 16, D rounded up to a multiple of 16, plus 8] whose first E columns are the values and whose columns behind
-// D are zeros; D and E multiples of 8, D up to 640, E up to 512; entries of min_len .. max_len rows.  part: fp32 scratch [entries, max_len, H, splits, E + 2] when splits > 1.
+// D are zeros; D and E multiples of 8, D up to 640, E up to 512; entries of min_len .. max_len rows.  part: fp32 scratch
+// [entries, max_len, H, splits, E + 2] when splits > 1.
 int apb_softmax_attn_wide(const void* q, long long ldq, const int* e_start, const int* e_len, const int* e_slot, const int* e_pos0,
                           int n_entries, const int* page_table, int max_pages, const void* kcache, void* out, long long ldo,
                           float* part, int H, int G, int D, int E, int min_len, int max_len, int splits, float scale, int window,
