@@ -132,10 +132,10 @@ int apb_gemm_simt(const void* A, const void* B, void* C, int M, int N, int K, lo
 
 // A tile table written by a kernel, 64 x 64 tiles: rows of A and C by group, B stacked.
 int apb_gemm_simt_grouped(const void* A, const void* B, void* C, int M, int N, int K, long long lda, long long ldb, long long ldc,
-                          int epi, void* C2, long long ldc2, const void* tile_map, int max_tiles, const int* num_tiles, int dtype,
-                          cudaStream_t s) {
+                          int epi, void* C2, long long ldc2, float glu_limit, const void* tile_map, int max_tiles,
+                          const int* num_tiles, int dtype, cudaStream_t s) {
   if (!tile_map || !num_tiles || max_tiles <= 0) return kBadArgument;
-  return gemm_simt_impl(SimtParams{A, B, C, lda, ldb, ldc, M, N, K, epi, nullptr, C2, ldc2, 0.f, static_cast<const int4*>(tile_map),
+  return gemm_simt_impl(SimtParams{A, B, C, lda, ldb, ldc, M, N, K, epi, nullptr, C2, ldc2, glu_limit, static_cast<const int4*>(tile_map),
                                    num_tiles}, 1, max_tiles, dtype, s);
 }
 

@@ -698,6 +698,15 @@ int apb_gemm_bf16_grouped_dev(const void* A, const void* B, void* C, int M, int 
                         num_tiles_dev, b_rows, 128, 0, stream);
 }
 
+// The same with a GLU epilogue (kEpiClampGLU with its limit): C2[m, n / 2] from interleaved (gate, up) columns.
+int apb_gemm_bf16_grouped_glu(const void* A, const void* B, int M, int N, int K, long long lda, long long ldb, int epi, float limit,
+                              void* C2, long long ldc2, const void* tile_map, int max_tiles, const int* num_tiles_dev,
+                              long long b_rows, cudaStream_t stream) {
+  if (!tile_map || !num_tiles_dev || max_tiles <= 0 || !apb::is_glu_epilogue(epi)) return apb::kBadArgument;
+  return gemm_bf16_impl(A, B, nullptr, M, N, K, lda, ldb, 0, 0, 0, epi, 1, 1.f, nullptr, C2, ldc2, tile_map, max_tiles,
+                        num_tiles_dev, b_rows, 128, 0, stream, nullptr, 0, limit);
+}
+
 // The grouped backward passes of an expert layer, tables written by a kernel (apb_moe_plan):
 //   data gradient    dX[rows of e] = dY[rows of e] @ W[e],  W stacked [E * K, N] (b_mn = 1, bk_off = e * K per tile);
 //   weight gradient  dW[e] (+)= dY[rows of e]^T @ X[rows of e]: a_mn = b_mn = 1, K = the row axis, every tile walks

@@ -287,21 +287,18 @@ norm_conv_vec_kernel(const float* __restrict__ x, const T* __restrict__ gain, co
 template <typename T>
 __global__ void __launch_bounds__(256)
 gain_norm_rows_kernel(const float* __restrict__ x, const int* __restrict__ rows, const T* __restrict__ gain,
-                      int gain_step, float offset, T* __restrict__ out, int W, float eps) {
+                      int gain_step, float offset, T* __restrict__ out, int W, int groups, float eps) {
   pdl_entry();
-  __shared__ float red[8];
+  extern __shared__ float gn_sums[];           // [max(8, groups)]
   const float* xr = x + static_cast<long long>(rows ? rows[blockIdx.x] : static_cast<int>(blockIdx.x)) * W;
-  float ss = 0.f;
-  for (int c = threadIdx.x; c < W; c += 256) ss += xr[c] * xr[c];
-  ss = warp_sum(ss);
-  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+  const int size = W / groups, parts = group_parts(groups);
+  group_sums(groups, size, gn_sums, [&](int c) { return xr[c]; });
   __syncthreads();
-  ss = 0.f;
-#pragma unroll
-  for (int i = 0; i < 8; ++i) ss += red[i];
-  const float f = 1.f / sqrtf(ss / W + eps);
-  for (int c = threadIdx.x; c < W; c += 256)
+  float f = groups == 1 ? group_rms_inverse(gn_sums, 0, parts, size, eps) : 0.f;
+  for (int c = threadIdx.x; c < W; c += 256) {
+    if (groups > 1) f = group_rms_inverse(gn_sums, c / size, parts, size, eps);
     out[static_cast<long long>(blockIdx.x) * W + c] = from_f32<T>(xr[c] * f * (offset + to_f32(gain[c * gain_step])));
+  }
 }
 
 // ---------------------------------------------------------------------------- q/k norm + paged cache write
@@ -446,6 +443,10 @@ __device__ __forceinline__ void load_cols(const T* p, float (&v)[V]) {
       v[2 * i] = f.x;
       v[2 * i + 1] = f.y;
     }
+  } else if constexpr (V == 2) {
+    const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
+    v[0] = f.x;
+    v[1] = f.y;
   } else {
     v[0] = to_f32(*p);
   }
@@ -454,6 +455,8 @@ template <typename T, int V>
 __device__ __forceinline__ void store_cols(T* p, const float (&v)[V]) {
   if constexpr (V == 8)
     *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
+  else if constexpr (V == 2)
+    *reinterpret_cast<uint32_t*>(p) = pack_bf16x2(v[0], v[1]);
   else
     *p = from_f32<T>(v[0]);
 }
@@ -534,6 +537,78 @@ row_norm_rope_cache_kernel(T* __restrict__ p, long long ld, int q_col, int k_col
   }
 }
 
+// ---------------------------------------------------------------------------- half-split rotation + value norm + page write
+// p [rows, ld]: H query heads of D columns at q_col, G key heads at k_col, G value heads of E at v_col.  The first `rot` columns of
+// every query and key head are rotated, dimension i with i + rot / 2, by the angles of the row's position; with v_eps >= 0 every
+// value head is divided by its root mean square.  q goes back in place, k and v to their cache slot.  One warp per (row, head).
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+half_rope_cache_kernel(T* __restrict__ p, long long ld, int q_col, int k_col, int v_col, const int* __restrict__ row_entry,
+                       const ServeEntries e, const int* __restrict__ kv_slot, const float* __restrict__ cos_t,
+                       const float* __restrict__ sin_t, int rot, T* __restrict__ kcache, T* __restrict__ vcache, int rows, int H,
+                       int G, int D, int E, float v_eps) {
+  pdl_entry();
+  const int lane = threadIdx.x & 31, heads = H + 2 * G;
+  const long long gw = (blockIdx.x * 256LL + threadIdx.x) >> 5;
+  if (gw >= static_cast<long long>(rows) * heads) return;
+  const int row = static_cast<int>(gw / heads), hh = static_cast<int>(gw % heads);
+  const int en = row_entry ? row_entry[row] : row;
+  const int at = row - e.start[en];
+  if (at < 0 || at >= e.len[en]) return;
+  const bool is_q = hh < H, is_v = hh >= H + G;
+  const int head = is_q ? hh : is_v ? hh - H - G : hh - H;
+  const int slot = is_q ? 0 : kv_slot[row];
+  if (slot < 0) return;
+  T* pr = p + static_cast<long long>(row) * ld;
+  const long long tok = (static_cast<long long>(slot / kServePage) * G + head) * kServePage + slot % kServePage;
+  if (is_v) {
+    const T* src = pr + v_col + head * E;
+    T* dst = vcache + tok * E;
+    float r = 1.f;
+    if (v_eps >= 0.f) {
+      float ss = 0.f;
+      for (int c = lane * V; c < E; c += 32 * V) {
+        float a[V];
+        load_cols<T, V>(src + c, a);
+#pragma unroll
+        for (int i = 0; i < V; ++i) ss += a[i] * a[i];
+      }
+      r = 1.f / sqrtf(warp_sum(ss) / E + v_eps);
+    }
+    for (int c = lane * V; c < E; c += 32 * V) {
+      float a[V];
+      load_cols<T, V>(src + c, a);
+#pragma unroll
+      for (int i = 0; i < V; ++i) a[i] *= r;
+      store_cols<T, V>(dst + c, a);
+    }
+    return;
+  }
+  T* src = pr + (is_q ? q_col : k_col) + head * D;
+  T* dst = is_q ? src : kcache + tok * D;
+  const int half = rot >> 1;
+  const long long tr = static_cast<long long>(e.pos0[en] + at) * half;
+  for (int c = lane * V; c < half; c += 32 * V) {
+    float a[V], b[V];
+    load_cols<T, V>(src + c, a);
+    load_cols<T, V>(src + c + half, b);
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      const float cs = cos_t[tr + c + i], sn = sin_t[tr + c + i], u = a[i];
+      a[i] = u * cs - b[i] * sn;
+      b[i] = b[i] * cs + u * sn;
+    }
+    store_cols<T, V>(dst + c, a);
+    store_cols<T, V>(dst + c + half, b);
+  }
+  if (!is_q)
+    for (int c = rot + lane * V; c < D; c += 32 * V) {
+      float a[V];
+      load_cols<T, V>(src + c, a);
+      store_cols<T, V>(dst + c, a);
+    }
+}
+
 // ---------------------------------------------------------------------------- end of a step
 // Every entry that fed tokens: remember its last token and flip the parity of its double-buffered state.
 __global__ void __launch_bounds__(128)
@@ -604,11 +679,13 @@ int apb_norm_conv(const float* x, const void* gain, const void* w1, const void* 
 }
 
 int apb_gain_norm_rows(const float* x, const int* rows, const void* gain, int gain_step, float offset, void* out, int n, int W,
-                       float eps, int dtype, cudaStream_t s) {
+                       int groups, float eps, int dtype, cudaStream_t s) {
   if (n <= 0) return 0;
-  APB_SERVE_DTYPE(dtype, return static_cast<int>(launch_kernel(gain_norm_rows_kernel<T>, dim3(n), dim3(256), 0, s, x, rows,
+  if (W <= 0 || groups < 1 || W % groups || groups > 8192) return kBadArgument;
+  const size_t smem = (groups > 8 ? groups : 8) * sizeof(float);
+  APB_SERVE_DTYPE(dtype, return static_cast<int>(launch_kernel(gain_norm_rows_kernel<T>, dim3(n), dim3(256), smem, s, x, rows,
                                                                static_cast<const T*>(gain), gain_step, offset,
-                                                               static_cast<T*>(out), W, eps)));
+                                                               static_cast<T*>(out), W, groups, eps)));
 }
 
 int apb_qk_norm_cache(void* p, long long ld, int q_col, int k_col, int v_col, const int* kv_slot, void* kcache,
@@ -667,6 +744,29 @@ int apb_row_norm_rope_cache(void* p, long long ld, int q_col, int k_col, int v_c
   if (vec) APB_ROW_NORM(__nv_bfloat16, 8);
   APB_SERVE_DTYPE(dtype, APB_ROW_NORM(T, 1));
 #undef APB_ROW_NORM
+}
+
+// row_entry [rows] or null (row i belongs to entry i); v_eps < 0: values are stored as they are.
+int apb_half_rope_cache(void* p, long long ld, int q_col, int k_col, int v_col, const int* row_entry, const int* e_start,
+                        const int* e_len, const int* e_slot, const int* e_pos0, const int* kv_slot, const float* cos_t,
+                        const float* sin_t, int rot, void* kcache, void* vcache, int rows, int H, int G, int D, int E, float v_eps,
+                        int dtype, cudaStream_t s) {
+  if (rows <= 0) return 0;
+  if (H <= 0 || G <= 0 || D <= 0 || E <= 0 || rot < 0 || (rot & 1) || rot > D || (rot && (!cos_t || !sin_t)) || !kv_slot || !kcache ||
+      !vcache)
+    return kBadArgument;
+  const ServeEntries e{e_start, e_len, e_slot, e_pos0};
+  const bool vec = dtype == 0 && !((D | E | q_col | k_col | v_col) & 1) && !(rot & 3) && !(ld & 1) &&
+                   !((reinterpret_cast<uintptr_t>(p) | reinterpret_cast<uintptr_t>(kcache) | reinterpret_cast<uintptr_t>(vcache)) & 3);
+  const long long warps = static_cast<long long>(rows) * (H + 2 * G);
+  const dim3 grid(static_cast<unsigned>((warps + 7) / 8));
+#define APB_HALF_ROPE(TT, VV)                                                                                             \
+  return static_cast<int>(launch_kernel(half_rope_cache_kernel<TT, VV>, grid, dim3(256), 0, s, static_cast<TT*>(p), ld,   \
+                                        q_col, k_col, v_col, row_entry, e, kv_slot, cos_t, sin_t, rot,                    \
+                                        static_cast<TT*>(kcache), static_cast<TT*>(vcache), rows, H, G, D, E, v_eps))
+  if (vec) APB_HALF_ROPE(__nv_bfloat16, 2);
+  APB_SERVE_DTYPE(dtype, APB_HALF_ROPE(T, 1));
+#undef APB_HALF_ROPE
 }
 
 int apb_serve_commit(const int* tokens, const int* e_start, const int* e_len, const int* e_slot, const int* e_pos0,

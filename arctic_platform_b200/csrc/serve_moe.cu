@@ -1,11 +1,12 @@
 // Routing of a mixture of experts in a serving step, without a host round trip.
 //
-//   scores = softmax(logits) over N experts, the last of which may be identity experts (their output is the input);
+//   scores = softmax(logits), or sigmoid(logits), over N experts, the last of which may be identity experts (their output is the
+//   input);
 //   the `top` experts with the largest scores + correction are chosen, their weights are the scores without it.
 //
 // moe_serve_route_kernel: one warp per row chooses, blocks count the rows of every expert, and the last block to finish turns
 // the counts into first rows and into the tile tables of the two grouped products.  moe_serve_gather_kernel copies every row
-// to the rows of its experts.  Where a row lands inside its expert does not matter: rows of a product do not mix.
+// to the rows of its experts, the scaled form multiplied by its weight (experts that weigh their input).  Where a row lands inside its expert does not matter: rows of a product do not mix.
 #include "common.cuh"
 #include "host_utils.cuh"
 #include "serve_common.cuh"
@@ -22,6 +23,7 @@ struct MoeRouteParams {
   long long ld;
   const void* correction;  // [N] activation type or null
   const int* live;         // [rows] or null: rows with a negative entry take no expert
+  int sigmoid;             // scores are sigmoids of the logits (0: their softmax)
   int rows, N, E, top;     // E routed experts in front of N - E identity experts
   int* expert;             // [rows, top] routed expert, -1: none
   int* rank;               // [rows, top] row inside the expert
@@ -57,18 +59,24 @@ moe_serve_route_kernel(const MoeRouteParams p) {
       sc[j] = e < p.N ? z[e] : -INFINITY;
       mx = fmaxf(mx, sc[j]);
     }
-    mx = warp_max(mx);
-    float sum = 0.f;
+    if (p.sigmoid) {
 #pragma unroll
-    for (int j = 0; j < kMoePerLane; ++j) {
-      sc[j] = lane + 32 * j < p.N ? expf(sc[j] - mx) : 0.f;
-      sum += sc[j];
+      for (int j = 0; j < kMoePerLane; ++j) sc[j] = 1.f / (1.f + expf(-sc[j]));
+    } else {
+      mx = warp_max(mx);
+      float sum = 0.f;
+#pragma unroll
+      for (int j = 0; j < kMoePerLane; ++j) {
+        sc[j] = lane + 32 * j < p.N ? expf(sc[j] - mx) : 0.f;
+        sum += sc[j];
+      }
+      sum = warp_sum(sum);
+#pragma unroll
+      for (int j = 0; j < kMoePerLane; ++j) sc[j] /= sum;
     }
-    sum = warp_sum(sum);
 #pragma unroll
     for (int j = 0; j < kMoePerLane; ++j) {
       const int e = lane + 32 * j;
-      sc[j] /= sum;
       pick[j] = e < p.N ? sc[j] + (p.correction ? to_f32(static_cast<const T*>(p.correction)[e]) : 0.f) : -INFINITY;
     }
     for (int r = 0; r < p.top; ++r) {
@@ -190,6 +198,51 @@ moe_serve_gather_kernel(const V* __restrict__ h, int n, const int* __restrict__ 
   }
 }
 
+// The same, every row multiplied by its weight.
+template <typename T, int V>
+__global__ void __launch_bounds__(128)
+moe_serve_gather_scaled_kernel(const T* __restrict__ h, int n, const int* __restrict__ expert, const int* __restrict__ rank,
+                               const int* __restrict__ first, const float* __restrict__ weight, int top, int* __restrict__ slots,
+                               T* __restrict__ xs) {
+  pdl_entry();
+  __shared__ int s[32];
+  __shared__ float w[32];
+  const long long row = blockIdx.x;
+  if (threadIdx.x < top) {
+    const int e = expert[row * top + threadIdx.x];
+    const int v = e >= 0 ? first[e] + rank[row * top + threadIdx.x] : -1;
+    s[threadIdx.x] = v;
+    w[threadIdx.x] = weight[row * top + threadIdx.x];
+    slots[row * top + threadIdx.x] = v;
+  }
+  __syncthreads();
+  for (int c = threadIdx.x * V; c < n; c += 128 * V) {
+    float v[V];
+    if constexpr (V == 8) {
+      const uint4 raw = *reinterpret_cast<const uint4*>(h + row * n + c);
+      const uint32_t u[4] = {raw.x, raw.y, raw.z, raw.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u[i]));
+        v[2 * i] = f.x;
+        v[2 * i + 1] = f.y;
+      }
+    } else {
+      v[0] = to_f32(h[row * n + c]);
+    }
+    for (int k = 0; k < top; ++k) {
+      if (s[k] < 0) continue;
+      T* dst = xs + static_cast<long long>(s[k]) * n + c;
+      const float f = w[k];
+      if constexpr (V == 8)
+        *reinterpret_cast<uint4*>(dst) = make_uint4(pack_bf16x2(v[0] * f, v[1] * f), pack_bf16x2(v[2] * f, v[3] * f),
+                                                    pack_bf16x2(v[4] * f, v[5] * f), pack_bf16x2(v[6] * f, v[7] * f));
+      else
+        *dst = from_f32<T>(v[0] * f);
+    }
+  }
+}
+
 }  // namespace apb
 
 extern "C" {
@@ -197,10 +250,10 @@ using namespace apb;
 
 int apb_moe_serve_route(const float* logits, long long ld, const void* correction, const int* live, int rows, int N, int E,
                         int top, int* expert, int* rank, float* weight, float* ident, int* counters, int* first, void* tiles1,
-                        void* tiles2, int* n_tiles, int n_out1, int n_out2, int tile, int dtype, cudaStream_t s) {
+                        void* tiles2, int* n_tiles, int n_out1, int n_out2, int tile, int sigmoid, int dtype, cudaStream_t s) {
   if (rows <= 0) return 0;
   if (E <= 0 || N < E || N > kMoeMax || top < 1 || top > 32 || top > N || ld < N || tile < 1 || !counters) return kBadArgument;
-  const MoeRouteParams p{logits, ld, correction, live, rows, N, E, top, expert, rank, weight, ident, counters, first,
+  const MoeRouteParams p{logits, ld, correction, live, sigmoid, rows, N, E, top, expert, rank, weight, ident, counters, first,
                          static_cast<int4*>(tiles1), static_cast<int4*>(tiles2), n_tiles, n_out1, n_out2, tile};
   const dim3 grid((rows + kMoeWarps - 1) / kMoeWarps);
   APB_SERVE_DTYPE(dtype, return static_cast<int>(launch_kernel(moe_serve_route_kernel<T>, grid, dim3(kMoeThreads), 0, s, p)));
@@ -219,6 +272,20 @@ int apb_moe_serve_gather(const void* h, int rows, long long row_bytes, const int
   if ((a & 15) == 0) APB_GATHER(uint4);
   if ((a & 3) == 0) APB_GATHER(uint32_t);
   APB_GATHER(uint16_t);
+#undef APB_GATHER
+}
+
+// The same with every row times its weight; h and xs [rows, n] of the activation type.
+int apb_moe_serve_gather_scaled(const void* h, int rows, int n, const int* expert, const int* rank, const int* first,
+                                const float* weight, int top, int* slots, void* xs, int dtype, cudaStream_t s) {
+  if (rows <= 0) return 0;
+  if (top < 1 || top > 32 || n <= 0 || !weight) return kBadArgument;
+  const bool vec = dtype == 0 && !(n & 7) && !((reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(xs)) & 15);
+#define APB_GATHER(TT, VV)                                                                                                   \
+  return static_cast<int>(launch_kernel(moe_serve_gather_scaled_kernel<TT, VV>, dim3(rows), dim3(128), 0, s,                 \
+                                        static_cast<const TT*>(h), n, expert, rank, first, weight, top, slots, static_cast<TT*>(xs)))
+  if (vec) APB_GATHER(__nv_bfloat16, 8);
+  APB_SERVE_DTYPE(dtype, APB_GATHER(T, 1));
 #undef APB_GATHER
 }
 }

@@ -1,12 +1,14 @@
-// Residual update between two sublayers of a decoder that norms a sublayer's output as well as its input.
+// Residual update between two sublayers of a decoder that may norm a sublayer's output as well as its input.
 //
 // With y [rows, W] the (fp32) output of the last sublayer,
-//     x <- x + y / rms(y) * (offset + post)  (+ embed[token] * scale: the embedding output, ahead of a pass over looped layers)
-//     h  = x / rms(x) * (offset + pre)
+//     x <- x + mult * sigmoid(gate + bias) * (y / rms(y) * (offset + post) + y2 / rms(y2) * (offset + post2))
+//            (+ embed[token] * scale: the embedding output, ahead of a pass over looped layers)
+//     h  = x / rms(x) * (offset + pre)       rms over `groups` equal parts of the row
 // in one pass: read x and y once, write x and h once.  y may come in parts: routed experts leave rows `eo` that are weighted and
 // summed here, identity experts return the sublayer's own input h_in times their weight (ExpertParts).  Without `post` y is
-// added as it is, without y nothing is; without `pre` the fp32 x is written instead of h; write_x = 0 leaves x alone (a look at
-// the stream in between).  clear_y resets y to zero after reading it, for producers that add into it.
+// added as it is, without y nothing is; y2, the output of a second mixer beside the first, and the gate may be absent; without
+// `pre` the fp32 x is written instead of h; write_x = 0 leaves x alone (a look at the stream in between).  clear_y resets y and y2
+// to zero after reading them, for producers that add into them.
 #include "common.cuh"
 #include "host_utils.cuh"
 #include "serve_common.cuh"
@@ -18,8 +20,8 @@ constexpr int kResThreads = 256;
 struct ExpertParts {
   const void* eo;          // [slots, W] outputs of the routed experts (activation type), or null
   const int* slots;        // [rows, top] row of eo, -1: none
-  const float* weights;    // [rows, top]
-  const float* ident;      // [rows] weight of h_in
+  const float* weights;    // [rows, top], or null: all 1
+  const float* ident;      // [rows] weight of h_in, or null: none
   const void* h_in;        // [rows, W] activation type
   int top;
 };
@@ -36,6 +38,14 @@ struct ResidualParams {
   float embed_scale, offset, eps;
   int W, write_x, clear_y;
   ExpertParts ex;
+  float* y2;               // second output, or null
+  const void* post2;
+  const void* gate;        // [rows, ld_gate] columns (activation type, or fp32 with gate_f32), or null
+  long long ld_gate;
+  int gate_f32;
+  const void* gate_bias;   // [W] activation type
+  float mult;
+  int groups;              // of the norm ahead of the next sublayer
 };
 
 template <int V>
@@ -80,14 +90,32 @@ __device__ __forceinline__ float sumsq(const Run<V>& a) {
   return s;
 }
 
-__device__ __forceinline__ float block_sum_residual(float v, float* red) {
-  v = warp_sum(v);
-  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+// Sum over the block of two values per thread.
+__device__ __forceinline__ float2 block_sum_residual(float a, float b, float (*red)[kResThreads / 32]) {
+  a = warp_sum(a);
+  b = warp_sum(b);
+  if ((threadIdx.x & 31) == 0) {
+    red[0][threadIdx.x >> 5] = a;
+    red[1][threadIdx.x >> 5] = b;
+  }
   __syncthreads();
-  v = 0.f;
+  a = b = 0.f;
 #pragma unroll
-  for (int i = 0; i < kResThreads / 32; ++i) v += red[i];
-  return v;
+  for (int i = 0; i < kResThreads / 32; ++i) {
+    a += red[0][i];
+    b += red[1][i];
+  }
+  return make_float2(a, b);
+}
+
+template <typename T, int V>
+__device__ __forceinline__ Run<V> gate_run(const ResidualParams& p, int row, int c) {
+  const long long o = static_cast<long long>(row) * p.ld_gate + c;
+  Run<V> z = p.gate_f32 ? load_run<V>(static_cast<const float*>(p.gate) + o) : load_run<V>(static_cast<const T*>(p.gate) + o);
+  const Run<V> b = load_run<V>(static_cast<const T*>(p.gate_bias) + c);
+#pragma unroll
+  for (int i = 0; i < V; ++i) z.v[i] = 1.f / (1.f + expf(-(z.v[i] + b.v[i])));
+  return z;
 }
 
 // One block per row; every thread keeps its own columns in shared memory between the passes.
@@ -95,18 +123,20 @@ template <typename T, int V>
 __global__ void __launch_bounds__(kResThreads)
 residual_step_kernel(const ResidualParams p) {
   pdl_entry();
-  extern __shared__ __align__(16) float buf[];     // [W]
-  __shared__ float red[2][kResThreads / 32];
+  extern __shared__ __align__(16) float buf[];     // [W], with y2 [2 W], then [max(8, groups)] partial sums of the groups
+  __shared__ float red[2][kResThreads / 32], red2[2][kResThreads / 32];
   const int row = blockIdx.x, W = p.W;
   float* x = p.x + static_cast<long long>(row) * W;
   float* y = p.y ? p.y + static_cast<long long>(row) * W : nullptr;
+  float* y2 = p.y2 ? p.y2 + static_cast<long long>(row) * W : nullptr;
+  float* buf2 = buf + W;
   const bool has_y = y || p.ex.eo;
-  float ry = 1.f;
+  float2 ry = make_float2(1.f, 1.f);
   if (has_y) {
-    float ss = 0.f;
+    float ss = 0.f, ss2 = 0.f;
     const int* slots = p.ex.slots + static_cast<long long>(row) * p.ex.top;
-    const float* wts = p.ex.weights + static_cast<long long>(row) * p.ex.top;
-    const float ident = p.ex.eo ? p.ex.ident[row] : 0.f;
+    const float* wts = p.ex.weights ? p.ex.weights + static_cast<long long>(row) * p.ex.top : nullptr;
+    const float ident = p.ex.eo && p.ex.ident ? p.ex.ident[row] : 0.f;
 #pragma unroll 2
     for (int c = threadIdx.x * V; c < W; c += kResThreads * V) {
       Run<V> v = {};
@@ -114,17 +144,26 @@ residual_step_kernel(const ResidualParams p) {
         v = load_run<V>(y + c);
         if (p.clear_y) store_run<V>(y + c, Run<V>{});
       }
+      if (y2) {
+        const Run<V> v2 = load_run<V>(y2 + c);
+        if (p.clear_y) store_run<V>(y2 + c, Run<V>{});
+        store_run<V>(buf2 + c, v2);
+        ss2 += sumsq<V>(v2);
+      }
       if (p.ex.eo) {
         for (int k = 0; k < p.ex.top; ++k) {
           const int s = slots[k];
-          if (s >= 0) axpy<V>(v, wts[k], load_run<V>(static_cast<const T*>(p.ex.eo) + static_cast<long long>(s) * W + c));
+          if (s >= 0) axpy<V>(v, wts ? wts[k] : 1.f, load_run<V>(static_cast<const T*>(p.ex.eo) + static_cast<long long>(s) * W + c));
         }
         if (ident != 0.f) axpy<V>(v, ident, load_run<V>(static_cast<const T*>(p.ex.h_in) + static_cast<long long>(row) * W + c));
       }
       store_run<V>(buf + c, v);
       ss += sumsq<V>(v);
     }
-    if (p.post) ry = 1.f / sqrtf(block_sum_residual(ss, red[0]) / W + p.eps);
+    if (p.post) {
+      const float2 s = block_sum_residual(ss, ss2, red);
+      ry = make_float2(1.f / sqrtf(s.x / W + p.eps), 1.f / sqrtf(s.y / W + p.eps));
+    }
   }
   const T* e = nullptr;
   if (p.embed) {
@@ -140,9 +179,19 @@ residual_step_kernel(const ResidualParams p) {
       if (p.post) {
         const Run<V> g = load_run<V>(static_cast<const T*>(p.post) + c);
 #pragma unroll
-        for (int i = 0; i < V; ++i) u.v[i] *= ry * (p.offset + g.v[i]);
+        for (int i = 0; i < V; ++i) u.v[i] *= ry.x * (p.offset + g.v[i]);
       }
-      axpy<V>(v, 1.f, u);
+      if (y2) {
+        const Run<V> u2 = load_run<V>(buf2 + c), g = load_run<V>(static_cast<const T*>(p.post2) + c);
+#pragma unroll
+        for (int i = 0; i < V; ++i) u.v[i] += u2.v[i] * ry.y * (p.offset + g.v[i]);
+      }
+      if (p.gate) {
+        const Run<V> g = gate_run<T, V>(p, row, c);
+#pragma unroll
+        for (int i = 0; i < V; ++i) u.v[i] *= g.v[i];
+      }
+      axpy<V>(v, p.mult, u);
     }
     if (e) axpy<V>(v, p.embed_scale, load_run<V>(e + c));
     if (p.write_x && (has_y || e)) store_run<V>(x + c, v);
@@ -154,14 +203,33 @@ residual_step_kernel(const ResidualParams p) {
     }
   }
   if (!p.pre) return;
-  const float r = 1.f / sqrtf(block_sum_residual(ss, red[1]) / W + p.eps);
   T* h = static_cast<T*>(p.h) + static_cast<long long>(row) * W;
+  if (p.groups == 1) {
+    const float r = 1.f / sqrtf(block_sum_residual(ss, 0.f, red2).x / W + p.eps);
 #pragma unroll 2
+    for (int c = threadIdx.x * V; c < W; c += kResThreads * V) {
+      Run<V> v = load_run<V>(buf + c);
+      const Run<V> g = load_run<V>(static_cast<const T*>(p.pre) + c);
+#pragma unroll
+      for (int i = 0; i < V; ++i) v.v[i] *= r * (p.offset + g.v[i]);
+      store_run<V>(h + c, v);
+    }
+    return;
+  }
+  float* sums = buf + (p.y2 ? 2 * W : W);
+  const int size = W / p.groups, parts = group_parts(p.groups);
+  __syncthreads();
+  group_sums(p.groups, size, sums, [&](int c) { return buf[c]; });
+  __syncthreads();
   for (int c = threadIdx.x * V; c < W; c += kResThreads * V) {
     Run<V> v = load_run<V>(buf + c);
     const Run<V> g = load_run<V>(static_cast<const T*>(p.pre) + c);
+    float r = 0.f;
 #pragma unroll
-    for (int i = 0; i < V; ++i) v.v[i] *= r * (p.offset + g.v[i]);
+    for (int i = 0; i < V; ++i) {
+      if (i == 0 || (c + i) % size == 0) r = group_rms_inverse(sums, (c + i) / size, parts, size, p.eps);
+      v.v[i] *= r * (p.offset + g.v[i]);
+    }
     store_run<V>(h + c, v);
   }
 }
@@ -171,17 +239,19 @@ residual_step_kernel(const ResidualParams p) {
 extern "C" {
 using namespace apb;
 
+// gate [rows, ld_gate] (fp32 with gate_f32) and gate_bias [W], or null; y2 and post2 only beside y and post.
 int apb_residual_step(float* x, float* y, const void* post, const void* pre, void* h, const int* tokens, const void* embed,
                       int vocab, float embed_scale, const void* eo, const int* slots, const float* weights,
                       const float* ident, const void* h_in, int top, int rows, int W, float offset, float eps, int write_x,
-                      int clear_y, int dtype, cudaStream_t s) {
+                      int clear_y, float* y2, const void* post2, const void* gate, long long ld_gate, int gate_f32,
+                      const void* gate_bias, float mult, int groups, int dtype, cudaStream_t s) {
   if (rows <= 0) return 0;
-  if (!x || !h || W <= 0 || W > 49152 || (embed && (!tokens || vocab <= 0)) ||
-      (eo && (!slots || !weights || !ident || !h_in || top < 1)))
+  if (!x || !h || W <= 0 || W > 49152 || (embed && (!tokens || vocab <= 0)) || (eo && (!slots || top < 1 || (ident && !h_in))) ||
+      (y2 && (!y || !post || !post2 || W > 24576)) || (gate && (!gate_bias || ld_gate < W)) || groups < 1 || W % groups)
     return kBadArgument;
   const ResidualParams p{x, y, post, pre, h, tokens, embed, vocab, embed_scale, offset, eps, W, write_x, clear_y,
-                         ExpertParts{eo, slots, weights, ident, h_in, top}};
-  const int smem = W * static_cast<int>(sizeof(float));
+                         ExpertParts{eo, slots, weights, ident, h_in, top}, y2, post2, gate, ld_gate, gate_f32, gate_bias, mult, groups};
+  const int smem = ((y2 ? 2 * W : W) + (groups > 8 ? groups : 8)) * static_cast<int>(sizeof(float));
   auto run = [&](auto fn) -> int {
     if (smem > 46 * 1024) {                  // the default limit counts the static arrays too
       const cudaError_t e = cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
@@ -189,6 +259,7 @@ int apb_residual_step(float* x, float* y, const void* post, const void* pre, voi
     }
     return static_cast<int>(launch_kernel(fn, dim3(rows), dim3(kResThreads), smem, s, p));
   };
-  APB_SERVE_DTYPE(dtype, if ((W & 3) == 0) return run(residual_step_kernel<T, 4>); return run(residual_step_kernel<T, 1>));
+  const bool vec = (W & 3) == 0 && (!gate || (!(ld_gate & 3) && !(reinterpret_cast<uintptr_t>(gate) & 15)));
+  APB_SERVE_DTYPE(dtype, if (vec) return run(residual_step_kernel<T, 4>); return run(residual_step_kernel<T, 1>));
 }
 }

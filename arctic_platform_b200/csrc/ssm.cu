@@ -151,7 +151,7 @@ ssm_conv_kernel(const SsmParams p, const int* __restrict__ tiles) {
   const int nr = min(kSsmRows, len - r0);
   const long long start = p.e.start[en];
   const int pos0 = p.e.pos0[en], slot = p.e.slot[en];
-  if (blockIdx.y == 0)
+  if (blockIdx.y == 0 && p.steps)
     for (int i = threadIdx.x; i < nr * p.H; i += kSsmConvThreads) {
       const long long row = start + r0 + i / p.H;
       p.steps[row * p.H + i % p.H] = ssm_step_of<T>(p, row, i % p.H);
@@ -192,7 +192,7 @@ ssm_conv_kernel(const SsmParams p, const int* __restrict__ tiles) {
       if (pair) out[i * p.ldx + 1] = v.y;
     }
   };
-  const float2 bias = make_float2(to_f32(cb[c]), pair ? to_f32(cb[c + 1]) : 0.f);
+  const float2 bias = cb ? make_float2(to_f32(cb[c]), pair ? to_f32(cb[c + 1]) : 0.f) : make_float2(0.f, 0.f);
   if constexpr (TAPS > 0) {
     constexpr int kHist = TAPS - 1;
     float2 w[TAPS], x[kHist + kSsmRows];
@@ -403,6 +403,18 @@ static int ssm_smem_limit(F fn, size_t bytes) {
   return bytes <= 46 * 1024 ? 0 : static_cast<int>(cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes)));
 }
 
+static int ssm_conv_run(const SsmParams& a, int channels, const int* tiles, int n_tiles, int dtype, cudaStream_t s) {
+  const dim3 grid(n_tiles, (channels + 2 * kSsmConvThreads - 1) / (2 * kSsmConvThreads));
+  auto run = [&](auto fn) -> int { return static_cast<int>(launch_kernel(fn, grid, dim3(kSsmConvThreads), 0, s, a, tiles)); };
+#define APB_SSM_CONV(T)                                                                                     \
+  return a.taps == 2 ? run(ssm_conv_kernel<T, 2>) : a.taps == 3 ? run(ssm_conv_kernel<T, 3>) : a.taps == 4  \
+           ? run(ssm_conv_kernel<T, 4>) : run(ssm_conv_kernel<T, 0>)
+  if (dtype == 0) APB_SSM_CONV(__nv_bfloat16);
+  if (dtype == 1) APB_SSM_CONV(float);
+#undef APB_SSM_CONV
+  return kBadArgument;
+}
+
 }  // namespace apb
 
 extern "C" {
@@ -436,15 +448,7 @@ int apb_ssm(const void* p, long long ld, int xbc_col, int dt_col, const void* co
     if (rc) return rc;
   }
   if (n_tiles > 0) {
-    const dim3 grid(n_tiles, (channels + 2 * kSsmConvThreads - 1) / (2 * kSsmConvThreads));
-    auto run = [&](auto fn) -> int { return static_cast<int>(launch_kernel(fn, grid, dim3(kSsmConvThreads), 0, s, a, tiles)); };
-    int rc = kBadArgument;
-#define APB_SSM_CONV(T)                                                                                     \
-  rc = taps == 2 ? run(ssm_conv_kernel<T, 2>) : taps == 3 ? run(ssm_conv_kernel<T, 3>) : taps == 4          \
-           ? run(ssm_conv_kernel<T, 4>) : run(ssm_conv_kernel<T, 0>)
-    if (dtype == 0) APB_SSM_CONV(__nv_bfloat16);
-    if (dtype == 1) APB_SSM_CONV(float);
-#undef APB_SSM_CONV
+    const int rc = ssm_conv_run(a, channels, tiles, n_tiles, dtype, s);
     if (rc) return rc;
   }
   if (scan) {
@@ -458,6 +462,30 @@ int apb_ssm(const void* p, long long ld, int xbc_col, int dt_col, const void* co
     return kBadArgument;
   }
   return 0;
+}
+
+// The convolution alone, over `channels` columns from `col` on, for the entries longer than one token: out [rows, ldx] (ldx even) =
+// silu(conv); bias may be null.
+int apb_short_conv(const void* p, long long ld, int col, const void* conv_w, const void* bias, int taps, float* hist, const int* parity,
+                   void* out, long long ldx, int channels, const int* e_start, const int* e_len, const int* e_slot, const int* e_pos0,
+                   const int* tiles, int n_tiles, int dtype, cudaStream_t s) {
+  if (n_tiles <= 0) return 0;
+  if (!p || !conv_w || !out || !tiles || channels <= 0 || taps < 1 || (taps > 1 && (!hist || !parity)) || (ldx & 1)) return kBadArgument;
+  SsmParams a{};
+  a.e = ServeEntries{e_start, e_len, e_slot, e_pos0};
+  a.p = p;
+  a.ld = ld;
+  a.xbc_col = col;
+  a.conv_w = conv_w;
+  a.conv_b = bias;
+  a.taps = taps;
+  a.hist = hist;
+  a.parity = parity;
+  a.xbc = out;
+  a.ldx = ldx;
+  a.H = 1;
+  a.E = channels;
+  return ssm_conv_run(a, channels, tiles, n_tiles, dtype, s);
 }
 
 // y [rows, inner] fp32, z [rows, inner] columns (row stride ldz), w [inner]; inner a multiple of parts.

@@ -5,8 +5,8 @@ allocator, slots, sampling kernels, CUDA-graph decode loop, ``generate`` -- with
 the model through a small protocol (``models/registry.py`` lists the architectures):
 
 * ``model.cache_layout()``       what each layer run keeps per sequence: paged K/V with its own head sizes (value size 0: key
-                                 rows only; or the run whose pages it reads), an fp32 recurrent state, the history of a short convolution (any
-                                 of them may be absent);
+                                 rows only; or the run whose pages it reads), an fp32 recurrent state and what else its recurrence carries
+                                 (``aux``), the history of a short convolution (any of them may be absent);
 * ``model.prepare_serving(n)``   tables for ``n`` positions;
 * ``model.serve_rows(batch, cache)``   one pass over a ragged :class:`~arctic_platform_b200.ops.serving.StepBatch`,
                                  reading and advancing caches and states; the same code for prompts, portions, decoded
@@ -42,20 +42,22 @@ class StateCache:
         self.k: List[Optional[torch.Tensor]] = []
         self.v: List[Optional[torch.Tensor]] = []
         self.state: List[Optional[torch.Tensor]] = []
+        self.aux: List[Optional[torch.Tensor]] = []
         self.conv: List[Optional[torch.Tensor]] = []
         f32 = dict(device=device, dtype=torch.float32)
         for run in layout:
-            kv, st, cv = run.get("kv"), run.get("state"), run.get("conv")
+            kv, st, ax, cv = (run.get(n) for n in ("kv", "state", "aux", "conv"))
             if "kv_from" in run:                              # reads the pages an earlier run writes
                 self.k.append(self.k[run["kv_from"]])
                 self.v.append(self.v[run["kv_from"]])
-                self.state.append(None)
-                self.conv.append(None)
+                for kept in (self.state, self.aux, self.conv):
+                    kept.append(None)
                 continue
             # zero-filled: the unwritten tail of a last page is multiplied by weight 0 and must be finite
             self.k.append(torch.zeros((pages, kv[0], PAGE, kv[1]), device=device, dtype=dtype) if kv else None)
             self.v.append(torch.zeros((pages, kv[0], PAGE, kv[2]), device=device, dtype=dtype) if kv and kv[2] else None)
             self.state.append(torch.zeros((slots,) + tuple(st), **f32) if st else None)
+            self.aux.append(torch.zeros((slots,) + tuple(ax), **f32) if ax else None)
             self.conv.append(torch.zeros((slots, 2) + tuple(cv), **f32) if cv and cv[0] else None)
         self.prev = torch.zeros(slots, device=device, dtype=torch.int32)      # last token fed
         self.parity = torch.zeros(slots, device=device, dtype=torch.int32)    # valid half of double-buffered state
@@ -64,7 +66,7 @@ class StateCache:
         return list({id(t): t for t in self.k + self.v if t is not None}.values())
 
     def _slotted(self):
-        return [t for t in self.state + self.conv if t is not None] + [self.prev, self.parity]
+        return [t for t in self.state + self.aux + self.conv if t is not None] + [self.prev, self.parity]
 
     def num_bytes(self) -> int:
         return sum(t.numel() * t.element_size() for t in self._paged() + self._slotted())

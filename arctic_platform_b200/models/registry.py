@@ -25,6 +25,8 @@ register_architecture("Rigulorn", "arctic_platform_b200.models.rigulorn", "Rigul
                       ("serve_streams", "serve_softmax", "serve_softmax_tc", "ssm", "ssm_mma"))
 register_architecture("Titatar", "arctic_platform_b200.models.titatar", "TitatarConfig", "TitatarLM",
                       ("serve_residual", "serve_latent", "serve_moe", "serve_softmax", "serve_softmax_wide", "serve_flash_tc"))
+register_architecture("Meronex", "arctic_platform_b200.models.meronex", "MeronexConfig", "MeronexLM",
+                      ("serve_residual", "serve_moe", "serve_softmax", "serve_flash_tc", "ssm", "recurrent"))
 
 
 def kernel_sources(architecture: str) -> Tuple[str, ...]:

@@ -2,7 +2,7 @@
 
 A step advances several sequences at once, each by its own run of new tokens: a portion of a prompt of any length, or
 one decoded token.  :class:`StepBatch` is the device-side description of such a step; the functions below launch the
-kernels of ``serve_*.cu``, ``retention*.cu``, ``ssm*.cu`` and ``gemm_*.cu`` on it.  They take bf16 or fp32 activations;
+kernels of ``serve_*.cu``, ``retention*.cu``, ``ssm*.cu``, ``recurrent.cu``, ``*_mma.cu`` and ``gemm_*.cu`` on it.  They take bf16 or fp32 activations;
 the residual streams and all carried state are fp32.
 """
 from __future__ import annotations
@@ -31,7 +31,7 @@ def _fn(name: str):
             "apb_embed_hash": [vp] * 9 + [ll, ll, ll, i, i, f, i, vp, vp, ll, vp, i, vp, i, i, vp],
             "apb_loop_begin": [vp, vp, i, i, vp, ll, i, vp],
             "apb_norm_conv": [vp] * 13 + [i, i, i, f, i, vp],
-            "apb_gain_norm_rows": [vp, vp, vp, i, f, vp, i, i, f, i, vp],
+            "apb_gain_norm_rows": [vp, vp, vp, i, f, vp, i, i, i, f, i, vp],
             "apb_qk_norm_cache": [vp, ll, i, i, i, vp, vp, vp, i, i, i, i, i, f, i, vp],
             "apb_rope_cache": [vp, ll, i, i, i] + [vp] * 8 + [i, vp, vp] + [i] * 7 + [vp],
             "apb_stream_step": [vp] * 7 + [i] * 5 + [f, i, vp],
@@ -39,13 +39,20 @@ def _fn(name: str):
             "apb_softmax_attn_mma": [vp, ll] + [vp] * 4 + [i, vp, i, vp, vp, vp, ll, vp] + [i] * 7
                                     + [f, f, i, i, vp, f, f, i, vp, vp, ll, i, vp],
             "apb_row_norm_rope_cache": [vp, ll, i, i, i] + [vp] * 10 + [i, vp, vp] + [i] * 5 + [f, i, vp],
-            "apb_residual_step": [vp] * 7 + [i, f] + [vp] * 5 + [i, i, i, f, f, i, i, i, vp],
+            "apb_residual_step": [vp] * 7 + [i, f] + [vp] * 5 + [i, i, i, f, f, i, i, vp, vp, vp, ll, i, vp, f, i, i, vp],
+            "apb_half_rope_cache": [vp, ll, i, i, i] + [vp] * 8 + [i, vp, vp] + [i] * 5 + [f, i, vp],
+            "apb_recurrent": [i, vp, vp] + [i] * 6 + [vp],
+            "apb_short_conv": [vp, ll, i, vp, vp, i, vp, vp, vp, ll, i] + [vp] * 5 + [i, i, vp],
+            "apb_token_shift": [vp] * 10 + [i, i, i, vp, vp, i, i, vp, i, vp],
+            "apb_tanh_rows": [vp, ll, i, i, i, vp],
             "apb_latent_norm_cache": [vp, ll, i, i] + [vp] * 11 + [i, i, i, i, i, f, i, vp],
             "apb_latent_rotate": [vp, ll] + [vp] * 8 + [i] * 6 + [vp],
             "apb_latent_gather": [vp, vp, i, vp, i, vp, vp, i, i, i, vp],
-            "apb_moe_serve_route": [vp, ll, vp, vp, i, i, i, i] + [vp] * 9 + [i, i, i, i, vp],
+            "apb_moe_serve_route": [vp, ll, vp, vp, i, i, i, i] + [vp] * 9 + [i, i, i, i, i, vp],
             "apb_moe_serve_gather": [vp, i, ll, vp, vp, vp, i, vp, vp, vp],
-            "apb_gemm_simt_grouped": [vp, vp, vp, i, i, i, ll, ll, ll, i, vp, ll, vp, i, vp, i, vp],
+            "apb_moe_serve_gather_scaled": [vp, i, i, vp, vp, vp, vp, i, vp, vp, i, vp],
+            "apb_gemm_simt_grouped": [vp, vp, vp, i, i, i, ll, ll, ll, i, vp, ll, f, vp, i, vp, i, vp],
+            "apb_gemm_bf16_grouped_glu": [vp, vp, i, i, i, ll, ll, i, f, vp, ll, vp, i, vp, ll, vp],
             "apb_gemm_simt_heads": [vp, vp, vp, i, i, i, i, ll, ll, ll, ll, ll, i, vp, ll, i, vp],
             "apb_gemm_bf16_grouped_dev": [vp, vp, vp, i, i, i, ll, ll, ll, i, f, vp, ll, vp, i, vp, ll, vp],
             "apb_gemm_bf16_heads": [vp, vp, vp, i, i, i, i, ll, ll, ll, i, i, i, vp, ll, vp],
@@ -212,12 +219,12 @@ def norm_conv(b: StepBatch, x: torch.Tensor, gain: torch.Tensor, w1: Optional[to
 
 
 def gain_norm_rows(x: torch.Tensor, rows: Optional[torch.Tensor], gain: torch.Tensor, eps: float,
-                   offset: float = 0.0) -> torch.Tensor:
-    """``x / rms(x) * (offset + gain)`` of some rows, in the activation type."""
+                   offset: float = 0.0, groups: int = 1) -> torch.Tensor:
+    """``x / rms(x) * (offset + gain)`` of some rows, in the activation type; rms over ``groups`` equal parts of a row."""
     n = x.shape[0] if rows is None else rows.shape[0]
     out = torch.empty((n, x.shape[1]), device=x.device, dtype=gain.dtype)
     _call("apb_gain_norm_rows", _lib.ptr(x), _lib.ptr(rows), _lib.ptr(gain), int(gain.numel() > 1), float(offset),
-          _lib.ptr(out), n, x.shape[1], float(eps),
+          _lib.ptr(out), n, x.shape[1], groups, float(eps),
           dtype_code(gain.dtype))
     return out
 
@@ -253,33 +260,50 @@ def row_norm_rope_cache(b: StepBatch, p: torch.Tensor, cols: Tuple[int, int, int
           b.rows, heads, G, D, E, float(eps), dtype_code(p.dtype))
 
 
+def half_rope_cache(b: StepBatch, p: torch.Tensor, cols: Tuple[int, int, int], rope: Tuple[torch.Tensor, torch.Tensor], rot_dims: int,
+                    heads: int, kcache: torch.Tensor, vcache: torch.Tensor, value_eps: Optional[float] = None) -> None:
+    """Rotates the first ``rot_dims`` of every query and key head of ``p`` (dimension i with i + rot_dims / 2); q in place, k and v into
+    the page cache.  ``value_eps``: every value head is divided by its root mean square first."""
+    G, D, E = kcache.shape[1], kcache.shape[3], vcache.shape[3]
+    _call("apb_half_rope_cache", _lib.ptr(p), p.stride(0), *cols, _lib.ptr(b.row_entry), *b.entry_ptrs(), _lib.ptr(b.kv_slot),
+          _lib.ptr(rope[0]), _lib.ptr(rope[1]), rot_dims, _lib.ptr(kcache), _lib.ptr(vcache), b.rows, heads, G, D, E,
+          -1.0 if value_eps is None else float(value_eps), dtype_code(p.dtype))
+
+
 # --------------------------------------------------------------------------------------------- normed residual
 @dataclass
 class ExpertMix:
     """Output of a mixture of experts that has not been summed yet: rows ``out [slots, W]`` of the routed experts with the
-    rows ``slots [rows, top]`` (-1: none) and ``weights [rows, top]`` of every token, and ``ident [rows]`` times its input."""
+    rows ``slots [rows, top]`` (-1: none) and ``weights [rows, top]`` (None: all 1) of every token, and ``ident [rows]`` (None: 0)
+    times its input."""
     out: torch.Tensor
     slots: torch.Tensor
-    weights: torch.Tensor
-    ident: torch.Tensor
+    weights: Optional[torch.Tensor]
+    ident: Optional[torch.Tensor]
     h: torch.Tensor
 
 
 def residual_step(x: torch.Tensor, y: Optional[torch.Tensor], post: Optional[torch.Tensor], pre: Optional[torch.Tensor], eps: float,
                   *, mix: Optional[ExpertMix] = None, offset: float = 1.0, again: Optional[tuple] = None, write: bool = True,
-                  clear: bool = False, dtype: Optional[torch.dtype] = None) -> torch.Tensor:
-    """One pass over the residual ``x [rows, W]`` (fp32): ``x <- x + s / rms(s) * (offset + post)`` with ``s`` = ``y`` (fp32) plus
-    the sum of ``mix`` (both may be absent; without ``post`` s itself), plus the embedding output if ``again`` = (tokens, table,
-    scale) is given; then ``x / rms(x) * (offset + pre)`` in the activation type, without ``pre`` the fp32 x.  ``write`` False
-    leaves ``x`` as it was; ``clear`` zeroes ``y`` after reading it."""
+                  clear: bool = False, dtype: Optional[torch.dtype] = None, y2: Optional[torch.Tensor] = None,
+                  post2: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, gate_bias: Optional[torch.Tensor] = None,
+                  mult: float = 1.0, groups: int = 1) -> torch.Tensor:
+    """One pass over the residual ``x [rows, W]`` (fp32): ``x <- x + mult * sigmoid(gate + gate_bias) * s / rms(s) * (offset + post)``
+    with ``s`` = ``y`` (fp32) plus the sum of ``mix`` (both may be absent; without ``post`` s itself), plus the same of a second output
+    ``y2`` with ``post2`` under the same gate, plus the embedding output if ``again`` = (tokens, table, scale) is given; then
+    ``x / rms(x) * (offset + pre)`` in the activation type (rms over ``groups`` equal parts), without ``pre`` the fp32 x.  ``gate``
+    ``[rows, W]`` columns in fp32 or the activation type (None: 1).  ``write`` False leaves ``x`` as it was; ``clear`` zeroes ``y`` and
+    ``y2`` after reading them."""
     T, W = x.shape
-    dt = next((t.dtype for t in (pre, post) if t is not None), dtype)
+    dt = next((t.dtype for t in (pre, post, gate_bias) if t is not None), dtype)
     out = torch.empty((T, W), device=x.device, dtype=dt if pre is not None else torch.float32)
     tok, table, scale = again or (None, None, 0.0)
     m = (mix.out, mix.slots, mix.weights, mix.ident, mix.h) if mix is not None else (None,) * 5
     _call("apb_residual_step", _lib.ptr(x), _lib.ptr(y), _lib.ptr(post), _lib.ptr(pre), _lib.ptr(out), _lib.ptr(tok), _lib.ptr(table),
           0 if table is None else table.shape[0], float(scale), *(_lib.ptr(t) for t in m), 0 if mix is None else mix.slots.shape[1],
-          T, W, float(offset), float(eps), int(write), int(clear), dtype_code(dt or torch.float32))
+          T, W, float(offset), float(eps), int(write), int(clear), _lib.ptr(y2), _lib.ptr(post2), _lib.ptr(gate),
+          0 if gate is None else gate.stride(0), int(gate is not None and gate.dtype == torch.float32), _lib.ptr(gate_bias), float(mult),
+          groups, dtype_code(dt or torch.float32))
     return out
 
 
@@ -404,10 +428,13 @@ def heads_linear(a: torch.Tensor, a_step: int, w: torch.Tensor, heads: int, k: i
 
 # --------------------------------------------------------------------------------------------- mixture of experts
 def experts(b: StepBatch, h: torch.Tensor, logits: torch.Tensor, correction: Optional[torch.Tensor], counters: torch.Tensor,
-            w_gu: torch.Tensor, w_down: torch.Tensor, n: int, n_experts: int, top: int, ff: int) -> ExpertMix:
-    """Routes every row of ``h`` by its fp32 ``logits`` (``n`` scores, the first ``n_experts`` of them experts with weights, the
-    others identity experts) and runs the gated SiLU experts as two grouped products.  ``w_gu [experts * 2 ff, W]`` (gate and up
-    interleaved), ``w_down [experts * W, >= ff]``; ``counters [experts + 1]`` int32 are zero between calls."""
+            w_gu: torch.Tensor, w_down: torch.Tensor, n: int, n_experts: int, top: int, ff: int, *, sigmoid: bool = False,
+            scale_input: bool = False, epi: int = gemm.EPI_SWIGLU, limit: float = 0.0) -> ExpertMix:
+    """Routes every row of ``h`` by its fp32 ``logits`` (``n`` scores -- their softmax, or with ``sigmoid`` each one's sigmoid --, the
+    first ``n_experts`` of them experts with weights, the others identity experts) and runs the experts, GLU layers with the activation
+    ``epi``, as two grouped products.  ``w_gu [experts * 2 ff, W]`` (gate and up interleaved), ``w_down [experts * W, >= ff]``;
+    ``counters [experts + 1]`` int32 are zero between calls.  ``scale_input``: a token's weight multiplies the expert's input instead
+    of its output (no identity experts)."""
     T, W = h.shape
     dev, E, P = h.device, n_experts, T * top
     I, ldf = 2 * ff, w_down.shape[1]
@@ -425,25 +452,29 @@ def experts(b: StepBatch, h: torch.Tensor, logits: torch.Tensor, correction: Opt
     weights, ident = torch.empty((T, top), **f32), torch.empty(T, **f32)
     _call("apb_moe_serve_route", _lib.ptr(logits), logits.stride(0), _lib.ptr(correction), _lib.ptr(b.kv_slot), T, n, E, top,
           _lib.ptr(expert), _lib.ptr(rank), _lib.ptr(weights), _lib.ptr(ident), _lib.ptr(counters), _lib.ptr(first), _lib.ptr(tiles1),
-          _lib.ptr(tiles2), _lib.ptr(n_tiles), I, W, tile, dtype_code(h.dtype))
+          _lib.ptr(tiles2), _lib.ptr(n_tiles), I, W, tile, int(sigmoid), dtype_code(h.dtype))
     xs = torch.empty((P, W), device=dev, dtype=h.dtype)
-    _call("apb_moe_serve_gather", _lib.ptr(h), T, W * h.element_size(), _lib.ptr(expert), _lib.ptr(rank), _lib.ptr(first), top,
-          _lib.ptr(slots), _lib.ptr(xs))
+    if scale_input:
+        _call("apb_moe_serve_gather_scaled", _lib.ptr(h), T, W, _lib.ptr(expert), _lib.ptr(rank), _lib.ptr(first), _lib.ptr(weights), top,
+              _lib.ptr(slots), _lib.ptr(xs), dtype_code(h.dtype))
+    else:
+        _call("apb_moe_serve_gather", _lib.ptr(h), T, W * h.element_size(), _lib.ptr(expert), _lib.ptr(rank), _lib.ptr(first), top,
+              _lib.ptr(slots), _lib.ptr(xs))
     act = (torch.zeros if ldf != ff else torch.empty)((P, ldf), device=dev, dtype=h.dtype)
     out = torch.empty((P, W), device=dev, dtype=h.dtype)
     n1, n2 = _lib.ptr(n_tiles), _lib.ptr(n_tiles[1:])
     if simt:
         dt = dtype_code(h.dtype)
-        _call("apb_gemm_simt_grouped", _lib.ptr(xs), _lib.ptr(w_gu), None, P, I, W, W, w_gu.stride(0), 0, gemm.EPI_SWIGLU, _lib.ptr(act),
-              ldf, _lib.ptr(tiles1), max1, n1, dt)
+        _call("apb_gemm_simt_grouped", _lib.ptr(xs), _lib.ptr(w_gu), None, P, I, W, W, w_gu.stride(0), 0, epi, _lib.ptr(act),
+              ldf, float(limit), _lib.ptr(tiles1), max1, n1, dt)
         _call("apb_gemm_simt_grouped", _lib.ptr(act), _lib.ptr(w_down), _lib.ptr(out), P, W, ff, ldf, w_down.stride(0), W, gemm.EPI_BF16,
-              None, 0, _lib.ptr(tiles2), max2, n2, dt)
+              None, 0, 0.0, _lib.ptr(tiles2), max2, n2, dt)
     else:
-        _call("apb_gemm_bf16_grouped_dev", _lib.ptr(xs), _lib.ptr(w_gu), None, P, I, W, W, w_gu.stride(0), 0, gemm.EPI_SWIGLU, 1.0,
-              _lib.ptr(act), ldf, _lib.ptr(tiles1), max1, n1, w_gu.shape[0])
+        _call("apb_gemm_bf16_grouped_glu", _lib.ptr(xs), _lib.ptr(w_gu), P, I, W, W, w_gu.stride(0), epi, float(limit), _lib.ptr(act), ldf,
+              _lib.ptr(tiles1), max1, n1, w_gu.shape[0])
         _call("apb_gemm_bf16_grouped_dev", _lib.ptr(act), _lib.ptr(w_down), _lib.ptr(out), P, W, ff, ldf, w_down.stride(0), W,
               gemm.EPI_BF16, 1.0, None, 0, _lib.ptr(tiles2), max2, n2, w_down.shape[0])
-    return ExpertMix(out, slots, weights, ident, h)
+    return ExpertMix(out, slots, None, None, h) if scale_input else ExpertMix(out, slots, weights, ident, h)
 
 
 # --------------------------------------------------------------------------------------------- sequence mixers
@@ -923,3 +954,110 @@ def gated_group_norm(y: torch.Tensor, z: torch.Tensor, gain: torch.Tensor, parts
     ``y`` fp32, ``z`` a column slice in the activation type."""
     _call("apb_ssm_out", _lib.ptr(y), _lib.ptr(z), z.stride(0), _lib.ptr(gain), _lib.ptr(out), out.stride(0), y.shape[0],
           y.shape[1], parts, float(eps), dtype_code(out.dtype))
+
+
+# --------------------------------------------------------------------------------------------- matrix states per head
+RULES = {"memory": 0, "delta": 1, "time_mix": 2}
+
+
+@dataclass(frozen=True)
+class RecurrentSpec:
+    """A mixer with an fp32 state ``[dim, vdim]`` per head (``csrc/recurrent.cuh`` has the recurrences): ``rule`` "memory" (matrix
+    memory with exponential gates capped at ``cap``), "delta" (gated delta rule behind a short convolution) or "time_mix" (decay per
+    key channel, bonus for the current token).  The head's output is normed, multiplied by a gain (``shared_gain``: one of ``vdim``
+    for all heads) and by the silu (else the sigmoid) of the gate columns."""
+    rule: str
+    heads: int
+    key_heads: int
+    dim: int
+    vdim: int
+    eps: float
+    cap: float = 0.0
+    silu: bool = True
+    shared_gain: bool = False
+
+    @property
+    def channels(self) -> int:
+        return 2 * self.key_heads * self.dim + self.heads * self.vdim
+
+
+@dataclass
+class RecurrentInputs:
+    """Projections and weights of a recurrent mixer.  ``p [rows, ...]`` activations; ``q``, ``k``, ``v``, ``g`` (gate), ``a``, ``b`` (gates of
+    the recurrence, one column per head) are offsets in elements from a row's first.  "memory": ``a``, ``b`` input and forget gate,
+    ``w0``, ``w1`` their biases; "delta": ``a`` the decay, ``b`` the step size, ``w0`` the log decay rates, ``w1`` the decay bias, ``conv
+    [taps, channels]`` over q, k, v side by side; "time_mix": ``z`` the fp32 decay projection, ``w0`` its bias, ``w1`` the bonus."""
+    p: torch.Tensor
+    q: int
+    k: int
+    v: int
+    g: int
+    w0: torch.Tensor
+    w1: torch.Tensor
+    gain: torch.Tensor
+    a: int = 0
+    b: int = 0
+    z: Optional[torch.Tensor] = None
+    conv: Optional[torch.Tensor] = None
+
+
+class _RecurrentParams(ctypes.Structure):           # csrc/recurrent.cuh
+    _p, _l, _i, _f = ctypes.c_void_p, ctypes.c_longlong, ctypes.c_int, ctypes.c_float
+    _fields_ = [("start", _p), ("len", _p), ("slot", _p), ("pos0", _p), ("p", _p), ("ld", _l), ("q_off", _l), ("k_off", _l), ("v_off", _l),
+                ("a_off", _l), ("b_off", _l), ("w0", _p), ("w1", _p), ("z", _p), ("ldz", _l), ("cap", _f), ("conv_w", _p), ("taps", _i),
+                ("hist", _p), ("parity", _p), ("xc", _p), ("ldx", _l), ("state", _p), ("aux", _p), ("H", _i), ("KH", _i), ("D", _i),
+                ("E", _i), ("y", _p), ("gain", _p), ("gain_step", _i), ("g_off", _l), ("silu", _i), ("out", _p), ("ldo", _l), ("eps", _f)]
+
+
+def recurrent(b: StepBatch, s: RecurrentSpec, x: RecurrentInputs, state: torch.Tensor, out: torch.Tensor, *,
+              aux: Optional[torch.Tensor] = None, hist: Optional[torch.Tensor] = None, parity: Optional[torch.Tensor] = None) -> None:
+    """Advances ``state [slots, H, D, E]`` (fp32) by the batch's tokens; ``out [rows, H * E]`` (column slice).  ``aux [slots, H, D + 1]``
+    ("memory": normaliser and running maximum), ``hist [slots, 2, taps - 1, channels]`` ("delta": convolution history), fp32."""
+    H, D, E = s.heads, s.dim, s.vdim
+    rule, dt, p = RULES[s.rule], dtype_code(x.p.dtype), x.p
+    y = torch.empty((b.rows, H * E), device=p.device, dtype=torch.float32) if b.longer else None
+    taps = 0 if x.conv is None else x.conv.shape[0]
+    xc, ldx = None, (s.channels + 7) // 8 * 8
+    if s.rule == "delta" and b.longer:
+        xc = torch.empty((b.rows, ldx), device=p.device, dtype=p.dtype)
+        tiles = b.table(("rows", SSM_ROWS), lambda: row_tiles(b.host, SSM_ROWS))
+        _call("apb_short_conv", _lib.ptr(p), p.stride(0), x.q, _lib.ptr(x.conv), None, taps, _lib.ptr(hist), _lib.ptr(parity), _lib.ptr(xc),
+              ldx, s.channels, *b.entry_ptrs(), _lib.ptr(tiles), tiles.shape[0], dt)
+    params = _RecurrentParams(
+        *b.entry_ptrs(), _lib.ptr(p), p.stride(0), x.q, x.k, x.v, x.a, x.b, _lib.ptr(x.w0), _lib.ptr(x.w1), _lib.ptr(x.z),
+        0 if x.z is None else x.z.stride(0), s.cap, _lib.ptr(x.conv), taps, _lib.ptr(hist), _lib.ptr(parity), _lib.ptr(xc), ldx, _lib.ptr(state),
+        _lib.ptr(aux), H, s.key_heads, D, E, _lib.ptr(y), _lib.ptr(x.gain), 0 if s.shared_gain else E, x.g, int(s.silu), _lib.ptr(out),
+        out.stride(0), s.eps)
+    ref = ctypes.byref(params)
+    _call("apb_recurrent", rule, ref, _lib.ptr(b.row_entry), b.n_entries, b.rows, int(b.one_token), int(b.longer), int(b.longer), dt)
+
+
+def token_shift(b: StepBatch, h: torch.Tensor, mu: torch.Tensor, hist: torch.Tensor, parity: torch.Tensor, w: torch.Tensor, step: int,
+                cols: Sequence[int]) -> torch.Tensor:
+    """``h [rows, W]`` blended with the row of the token before, ``h + (h' - h) mu[s]`` for every ``mu [n, W]``, and the products of the
+    blends with their weights: rows ``s * step`` and following of ``w``, ``cols[s]`` of them.  ``hist [slots, 2, 1, W]`` fp32 carries the
+    last row.  Returns ``[n, rows, N]`` with ``N >= max(cols)``; columns from ``cols[s]`` on are undefined."""
+    T, W = h.shape
+    n, N = len(cols), (max(cols) + 7) // 8 * 8
+    dev, dt = h.device, dtype_code(h.dtype)
+    mixed = torch.empty((n, T, W), device=dev, dtype=h.dtype)
+    out = torch.empty((n, T, N), device=dev, dtype=h.dtype)
+    simt = _simt(h, w, out[0]) or bool(step % 8)
+    tile = 64 if simt else 128
+    most = sum(-(-T // tile) * -(-c // tile) for c in cols)
+    tiles = torch.empty(4 * most + 4, device=dev, dtype=torch.int32)
+    count = tiles[4 * most:]
+    _call("apb_token_shift", _lib.ptr(h), _lib.ptr(mu), _lib.ptr(hist), _lib.ptr(parity), _lib.ptr(mixed), _lib.ptr(b.row_entry),
+          *b.entry_ptrs(), T, W, n, _lib.ptr(tiles), _lib.ptr(count), tile, step, (ctypes.c_int * n)(*cols), dt)
+    if simt:
+        _call("apb_gemm_simt_grouped", _lib.ptr(mixed), _lib.ptr(w), _lib.ptr(out), n * T, N, W, W, w.stride(0), N, gemm.EPI_BF16, None, 0, 0.0,
+              _lib.ptr(tiles), most, _lib.ptr(count), dt)
+    else:
+        _call("apb_gemm_bf16_grouped_dev", _lib.ptr(mixed), _lib.ptr(w), _lib.ptr(out), n * T, N, W, W, w.stride(0), N, gemm.EPI_BF16, 1.0, None,
+              0, _lib.ptr(tiles), most, _lib.ptr(count), w.shape[0])
+    return out
+
+
+def tanh_rows(x: torch.Tensor) -> None:
+    """``x [rows, n]`` (column slice) <- tanh(x), rounded to the activation type."""
+    _call("apb_tanh_rows", _lib.ptr(x), x.stride(0), x.shape[0], x.shape[1], dtype_code(x.dtype))
