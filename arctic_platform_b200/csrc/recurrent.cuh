@@ -55,6 +55,10 @@ inline bool recurrent_params_ok(int rule, const RecurrentParams& a) {
                                : rule == kRuleTimeMix && a.z);
 }
 
+// Chunked kernels sum log2 decays and exponentiate differences of the sums.  A token's decay counts at most this much there: 2^-64
+// leaves nothing of a state either, and the sums of a chunk stay small enough for fp32 differences.
+constexpr float kMaxLogDecay = 64.f;
+
 __device__ __forceinline__ float rec_softplus(float v) { return v > 20.f ? v : log1pf(expf(v)); }
 __device__ __forceinline__ float rec_gate(float z, int silu) {
   const float s = 1.f / (1.f + expf(-z));

@@ -16,6 +16,7 @@
 #include "common.cuh"
 #include "host_utils.cuh"
 #include "retention.cuh"
+#include "warp_mma.cuh"
 
 namespace apb {
 
@@ -31,35 +32,6 @@ struct RetentionSegments {
                           // state or zero), scratch index for its own contribution (-1: none), 1 = last of its entry
   float* carry;           // [scratch states][H][D][E]
 };
-
-// 16 bytes, or zeros when `bytes` is 0
-__device__ __forceinline__ void rm_cp_async16(uint32_t dst, const void* src, int bytes) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ void rm_ldsm4(const __nv_bfloat16* a, uint32_t (&r)[4]) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(a)));
-}
-__device__ __forceinline__ void rm_ldsm4_t(const __nv_bfloat16* a, uint32_t (&r)[4]) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(a)));
-}
-__device__ __forceinline__ void rm_ldsm2(const __nv_bfloat16* a, uint32_t (&r)[2]) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0, %1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(smem_u32(a)));
-}
-__device__ __forceinline__ void rm_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
-      "{%0, %1, %2, %3};"
-      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-// x = hi + lo with both parts bf16; two neighbouring elements packed per word
-__device__ __forceinline__ void rm_split2(float x, float y, uint32_t& hi, uint32_t& lo) {
-  hi = pack_bf16x2(x, y);
-  const float2 h = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&hi));
-  lo = pack_bf16x2(x - h.x, y - h.y);
-}
 
 // qk [rows][H][4][dp]: hi and lo of the rotated q, hi and lo of the rotated and scaled k; dp = D rounded up to 16, the
 // padding zero.  Rows of one-token entries are skipped.  One warp per (row, head).
@@ -80,7 +52,7 @@ retention_split_kernel(const RetentionParams p, const int* __restrict__ row_entr
   __nv_bfloat16* out = qk + gw * 4 * dp;
   auto put = [&](int part, int d, float x, float y) {
     uint32_t hi, lo;
-    rm_split2(x, y, hi, lo);
+    wm_split2(x, y, hi, lo);
     *reinterpret_cast<uint32_t*>(out + part * dp + d) = hi;
     *reinterpret_cast<uint32_t*>(out + (part + 1) * dp + d) = lo;
   };
@@ -156,14 +128,14 @@ retention_mma_kernel(const RetentionParams p, const RetentionSegments sg, const 
     for (int i = threadIdx.x; i < kRmC * 2 * pc; i += kRmThreads) {
       const int r = i / (2 * pc), c = i % (2 * pc), ok = t0 + r < n_tok;
       const __nv_bfloat16* src = qk + ((static_cast<long long>(start + (ok ? t0 + r : 0)) * p.H + h) * 4 + part) * dp + c * 8;
-      rm_cp_async16(smem_u32(dst + (c / pc) * (kRmC * ds) + r * ds + (c % pc) * 8), src, ok ? 16 : 0);
+      wm_cp_async16(smem_u32(dst + (c / pc) * (kRmC * ds) + r * ds + (c % pc) * 8), src, ok ? 16 : 0);
     }
   };
   auto fetch_kv = [&](int t0, int buf) {
     fetch_part(t0, 2, K2 + buf * 2 * kRmC * ds);
     const int r = threadIdx.x >> 3, c = threadIdx.x & 7, ok = t0 + r < n_tok && c * 8 < be;
     const __nv_bfloat16* src = pb + static_cast<long long>(start + (ok ? t0 + r : 0)) * p.ld + p.v_col + h * E + e0 + (ok ? c * 8 : 0);
-    rm_cp_async16(smem_u32(V2 + buf * kRmC * kRmVS + r * kRmVS + c * 8), src, ok ? 16 : 0);
+    wm_cp_async16(smem_u32(V2 + buf * kRmC * kRmVS + r * kRmVS + c * 8), src, ok ? 16 : 0);
   };
   static_assert(kRmThreads == kRmC * kRmBE / 8, "one 16-byte chunk of the values per thread");
   if (!state_only) fetch_part(0, 0, Qh);
@@ -187,7 +159,7 @@ retention_mma_kernel(const RetentionParams p, const RetentionSegments sg, const 
 #pragma unroll
         for (int hh = 0; hh < 2; ++hh) {
           uint32_t hi, lo;
-          rm_split2(s[nt][2 * hh], s[nt][2 * hh + 1], hi, lo);
+          wm_split2(s[nt][2 * hh], s[nt][2 * hh + 1], hi, lo);
           const int o = (sr + 8 * hh) * kRmVS + nt * 8 + quad_col;
           *reinterpret_cast<uint32_t*>(Sh + o) = hi;
           *reinterpret_cast<uint32_t*>(Sl + o) = lo;
@@ -221,7 +193,7 @@ retention_mma_kernel(const RetentionParams p, const RetentionSegments sg, const 
       const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(V + o));
       const float g = r < n ? pw[n - 1 - r] : 0.f;
       uint32_t wh, wl;
-      rm_split2(f.x * g, f.y * g, wh, wl);
+      wm_split2(f.x * g, f.y * g, wh, wl);
       *reinterpret_cast<uint32_t*>(Wh + o) = wh;
       *reinterpret_cast<uint32_t*>(Wl + o) = wl;
     }
@@ -238,27 +210,27 @@ retention_mma_kernel(const RetentionParams p, const RetentionSegments sg, const 
       for (int ks = 0; ks < d16; ++ks) {
         uint32_t qh[4], ql[4];
         const int ao = (r0 + rowin + (mat & 1) * 8) * ds + ks * 16 + (mat >> 1) * 8;
-        rm_ldsm4(Qh + ao, qh);
-        rm_ldsm4(Ql + ao, ql);
+        wm_ldsm4(Qh + ao, qh);
+        wm_ldsm4(Ql + ao, ql);
         if (live) {
           uint32_t kh[2], kl[2];
           const int bo = (k0 + rowin) * ds + ks * 16 + (mat & 1) * 8;
-          rm_ldsm2(Kh + bo, kh);
-          rm_ldsm2(Kl + bo, kl);
-          rm_mma(a, ql, kh[0], kh[1]);
-          rm_mma(a, qh, kl[0], kl[1]);
-          rm_mma(a, qh, kh[0], kh[1]);
+          wm_ldsm2(Kh + bo, kh);
+          wm_ldsm2(Kl + bo, kl);
+          wm_mma(a, ql, kh[0], kh[1]);
+          wm_mma(a, qh, kl[0], kl[1]);
+          wm_mma(a, qh, kh[0], kh[1]);
         }
         if (have_state) {                          // q S of the carried state
           uint32_t sh[4], sl[4];
           const int so = (ks * 16 + rowin + 8 * (mat & 1)) * kRmVS + c0 + (mat >> 1) * 8;
-          rm_ldsm4_t(Sh + so, sh);
-          rm_ldsm4_t(Sl + so, sl);
+          wm_ldsm4_t(Sh + so, sh);
+          wm_ldsm4_t(Sl + so, sl);
 #pragma unroll
           for (int nt = 0; nt < 2; ++nt) {
-            rm_mma(o[nt], ql, sh[2 * nt], sh[2 * nt + 1]);
-            rm_mma(o[nt], qh, sl[2 * nt], sl[2 * nt + 1]);
-            rm_mma(o[nt], qh, sh[2 * nt], sh[2 * nt + 1]);
+            wm_mma(o[nt], ql, sh[2 * nt], sh[2 * nt + 1]);
+            wm_mma(o[nt], qh, sl[2 * nt], sl[2 * nt + 1]);
+            wm_mma(o[nt], qh, sh[2 * nt], sh[2 * nt + 1]);
           }
         }
       }
@@ -266,7 +238,7 @@ retention_mma_kernel(const RetentionParams p, const RetentionSegments sg, const 
       for (int hh = 0; hh < 2; ++hh) {
         const int i = r0 + quad_row + 8 * hh, j = k0 + quad_col;
         uint32_t hi, lo;
-        rm_split2(j <= i ? a[2 * hh] * pw[i - j] : 0.f, j + 1 <= i ? a[2 * hh + 1] * pw[i - j - 1] : 0.f, hi, lo);
+        wm_split2(j <= i ? a[2 * hh] * pw[i - j] : 0.f, j + 1 <= i ? a[2 * hh + 1] * pw[i - j - 1] : 0.f, hi, lo);
         *reinterpret_cast<uint32_t*>(Ah + i * kRmAS + j) = hi;
         *reinterpret_cast<uint32_t*>(Al + i * kRmAS + j) = lo;
         const float g = pw[i + 1];
@@ -284,13 +256,13 @@ retention_mma_kernel(const RetentionParams p, const RetentionSegments sg, const 
       for (int ks = 0; ks < (r0 + 16) / 16; ++ks) {
         uint32_t ah[4], al[4], v[4];
         const int ao = (r0 + rowin + (mat & 1) * 8) * kRmAS + ks * 16 + (mat >> 1) * 8;
-        rm_ldsm4(Ah + ao, ah);
-        rm_ldsm4(Al + ao, al);
-        rm_ldsm4_t(V + (ks * 16 + rowin + 8 * (mat & 1)) * kRmVS + c0 + (mat >> 1) * 8, v);
+        wm_ldsm4(Ah + ao, ah);
+        wm_ldsm4(Al + ao, al);
+        wm_ldsm4_t(V + (ks * 16 + rowin + 8 * (mat & 1)) * kRmVS + c0 + (mat >> 1) * 8, v);
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt) {
-          rm_mma(o[nt], al, v[2 * nt], v[2 * nt + 1]);
-          rm_mma(o[nt], ah, v[2 * nt], v[2 * nt + 1]);
+          wm_mma(o[nt], al, v[2 * nt], v[2 * nt + 1]);
+          wm_mma(o[nt], ah, v[2 * nt], v[2 * nt + 1]);
         }
       }
 #pragma unroll
@@ -317,19 +289,19 @@ retention_mma_kernel(const RetentionParams p, const RetentionSegments sg, const 
       for (int ks = 0; ks < kRmC / 16; ++ks) {
         uint32_t kh[4], kl[4];
         const int ao = (ks * 16 + rowin + (mat >> 1) * 8) * ds + warp * 16 + (mat & 1) * 8;
-        rm_ldsm4_t(Kh + ao, kh);
-        rm_ldsm4_t(Kl + ao, kl);
+        wm_ldsm4_t(Kh + ao, kh);
+        wm_ldsm4_t(Kl + ao, kl);
 #pragma unroll
         for (int n2 = 0; n2 < 4; ++n2) {
           uint32_t wh[4], wl[4];
           const int bo = (ks * 16 + rowin + 8 * (mat & 1)) * kRmVS + n2 * 16 + (mat >> 1) * 8;
-          rm_ldsm4_t(Wh + bo, wh);
-          rm_ldsm4_t(Wl + bo, wl);
+          wm_ldsm4_t(Wh + bo, wh);
+          wm_ldsm4_t(Wl + bo, wl);
 #pragma unroll
           for (int k = 0; k < 2; ++k) {
-            rm_mma(s[2 * n2 + k], kl, wh[2 * k], wh[2 * k + 1]);
-            rm_mma(s[2 * n2 + k], kh, wl[2 * k], wl[2 * k + 1]);
-            rm_mma(s[2 * n2 + k], kh, wh[2 * k], wh[2 * k + 1]);
+            wm_mma(s[2 * n2 + k], kl, wh[2 * k], wh[2 * k + 1]);
+            wm_mma(s[2 * n2 + k], kh, wl[2 * k], wl[2 * k + 1]);
+            wm_mma(s[2 * n2 + k], kh, wh[2 * k], wh[2 * k + 1]);
           }
         }
       }

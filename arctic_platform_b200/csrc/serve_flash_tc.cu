@@ -1,5 +1,5 @@
-// Causal softmax attention on tcgen05 tensor cores for long portions of prompts: one map, optional sliding window, sinks and
-// output gates (see SoftmaxSpec), no bound on the scores.
+// Causal softmax attention on tcgen05 tensor cores for long portions of prompts: one map, optional sliding window, sinks, output
+// gates and score cap (see SoftmaxSpec), no bound on the scores needed.
 //
 // A CTA = two tiles of 128 query rows that share their keys: two query heads of one KV head on the same rows, or two
 // consecutive row tiles of one head.  352 threads: warp 0 TMA producer, warps 2-5 and 6-9 the weight groups and warps 1 and 10 the MMA
@@ -11,7 +11,7 @@
 //
 // K and V travel in chunks of 64 columns x 128 keys through one ring.  The weights are taken relative to a reference that
 // follows the running maximum only when it falls behind by more than 2^8: the products of all key blocks accumulate in tensor
-// memory and are rescaled there on those rare occasions.
+// memory and are rescaled there on those rare occasions.  Under a score cap up to 64 the reference is fixed.
 #include "common.cuh"
 #include "host_utils.cuh"
 #include "serve_softmax.cuh"
@@ -72,6 +72,75 @@ __device__ __forceinline__ uint64_t flash_weights(uint32_t t_s, uint64_t scale2,
   return xtc_add2(sum[0], sum[1]);
 }
 
+// The same for capped scores, 2^(gain tanh(zs score) + off): the series of tanh_series with the scales folded into its coefficients,
+// or the exponential form for a warp that holds a larger score.
+struct CapSeries {
+  float zs, gain, small;       // small: largest squared score of the series
+  uint64_t c[5];
+};
+__device__ __forceinline__ CapSeries cap_series(const SoftmaxSpec& sp) {
+  CapSeries k;
+  k.zs = sp.scale / sp.cap;
+  k.gain = sp.cap * 1.4426950408889634f;
+  k.small = (kSmallTanh / k.zs) * (kSmallTanh / k.zs);
+  const float z2 = k.zs * k.zs, t[5] = {1.f, -1.f / 3.f, 2.f / 15.f, -17.f / 315.f, 62.f / 2835.f};
+  float f = k.gain * k.zs;
+#pragma unroll
+  for (int i = 0; i < 5; ++i, f *= z2) k.c[i] = xtc_pair(f * t[i], f * t[i]);
+  return k;
+}
+template <bool WHOLE>
+__device__ __forceinline__ uint64_t flash_capped_weights(uint32_t t_s, const CapSeries& k, float off, int limit, int skip, float& top,
+                                                         uint32_t (&pk)[4][16]) {
+  const uint64_t off2 = xtc_pair(off, off);
+  uint64_t sum[2] = {xtc_pair(0.f, 0.f), xtc_pair(0.f, 0.f)};
+  float t0 = -INFINITY, t1 = -INFINITY;
+  uint32_t stage[2][32];
+  tmem_ld_32x32(t_s, stage[0]);
+#pragma unroll
+  for (int c = 0; c < 4; ++c) {
+    uint32_t(&r)[32] = stage[c & 1];
+    xtc_wait_load(r);
+    if (c < 3) tmem_ld_32x32(t_s + (c + 1) * 32, stage[(c + 1) & 1]);
+    uint64_t v[16];
+    float large = 0.f;
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+      const uint64_t x = xtc_pair(__uint_as_float(r[2 * i]), __uint_as_float(r[2 * i + 1])), a = xtc_mul2(x, x);
+      const float2 f = xtc_unpair(a);
+      large = fmaxf(fmaxf(large, f.x), f.y);
+      uint64_t y = xtc_fma2(a, k.c[4], k.c[3]);
+      y = xtc_fma2(a, y, k.c[2]);
+      y = xtc_fma2(a, y, k.c[1]);
+      y = xtc_fma2(a, y, k.c[0]);
+      v[i] = xtc_fma2(x, y, off2);
+    }
+    if (!__all_sync(0xffffffffu, large <= k.small)) {
+#pragma unroll
+      for (int i = 0; i < 16; ++i)
+        v[i] = xtc_pair(fmaf(tanh_any(__uint_as_float(r[2 * i]) * k.zs), k.gain, off),
+                        fmaf(tanh_any(__uint_as_float(r[2 * i + 1]) * k.zs), k.gain, off));
+    }
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+      float2 f = xtc_unpair(v[i]);
+      if (!WHOLE) {
+        const int a = c * 32 + 2 * i;
+        if (a >= limit || a < skip) f.x = -INFINITY;
+        if (a + 1 >= limit || a + 1 < skip) f.y = -INFINITY;
+      }
+      t0 = fmaxf(t0, f.x);
+      t1 = fmaxf(t1, f.y);
+      const float w0 = xtc_ex2(f.x), w1 = xtc_ex2(f.y);
+      sum[i & 1] = xtc_add2(sum[i & 1], xtc_pair(w0, w1));
+      pk[c][i] = pack_bf16x2(w0, w1);
+    }
+  }
+  top = fmaxf(t0, t1);
+  return xtc_add2(sum[0], sum[1]);
+}
+
+template <bool CAP>
 __global__ void __launch_bounds__(kFlThreads, 1)
 flash_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_k,
                 const __grid_constant__ CUtensorMap tma_k2, const __grid_constant__ CUtensorMap tma_v, const FlashParams p) {
@@ -260,7 +329,10 @@ flash_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
     const float scale = p.sp.scale * 1.4426950408889634f;
     const uint64_t scale2 = xtc_pair(scale, scale);
     const int pos = pos0 + min(row, valid - 1);
-    float ref = -INFINITY;                             // reference of the weights (log2)
+    CapSeries cs = {};
+    if (CAP) cs = cap_series(p.sp);
+    const bool fixed = CAP && fixed_reference(p.sp.cap);
+    float ref = fixed ? score_reference(p.sp.cap) * 1.4426950408889634f : -INFINITY;      // reference of the weights (log2)
     uint64_t sum2 = xtc_pair(0.f, 0.f);
     bool ok = true;
     for (int j = 0; j < nb; ++j) {
@@ -277,8 +349,15 @@ flash_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
       for (int pass = 0; pass < 2; ++pass) {           // a second time if the reference had to move
         const float off = ref == -INFINITY ? 0.f : -ref;
         float top;                                     // largest score relative to the reference
-        const uint64_t block2 = whole ? flash_weights<true>(t_s, scale2, off, limit, skip, top, pk)
-                                      : flash_weights<false>(t_s, scale2, off, limit, skip, top, pk);
+        uint64_t block2;
+        if constexpr (CAP)
+          block2 = whole ? flash_capped_weights<true>(t_s, cs, off, limit, skip, top, pk) : flash_capped_weights<false>(t_s, cs, off, limit, skip, top, pk);
+        else
+          block2 = whole ? flash_weights<true>(t_s, scale2, off, limit, skip, top, pk) : flash_weights<false>(t_s, scale2, off, limit, skip, top, pk);
+        if (fixed) {
+          sum2 = xtc_add2(sum2, block2);
+          break;
+        }
         const bool behind = top > kFlLag || (ref == -INFINITY && top > -INFINITY);
         if (pass == 1 || !__any_sync(0xffffffffu, behind)) {
           sum2 = xtc_add2(sum2, block2);
@@ -365,11 +444,11 @@ extern "C" {
 // q: [rows, H * (D + R)] columns of a row-major buffer (row stride ldq); out [rows, H * E] (row stride ldo), 16-byte aligned rows.
 // With a page table: k [pages, G, 16, D], v [pages, G, 16, E], key_rows = pages * G * 16, R = 0.  Without: k [key_rows, G * D]
 // (row stride ldk), k2 [key_rows, R] (contiguous, R > 0), v [key_rows, G * E] (ldv).  D and R multiples of 16, at most 4 chunks of
-// 64 columns together, E a multiple of 8 up to 128; gate (if any): rows of 16-byte aligned columns.
+// 64 columns together, E a multiple of 8 up to 128; cap > 0: capped scores; gate (if any): rows of 16-byte aligned columns.
 int apb_flash_tc(const void* q, long long ldq, int rows, const int* work, int n_work, const int* page_table, int max_pages,
                  const void* k, long long ldk, const void* k2, const void* v, long long ldv, long long key_rows, void* out,
-                 long long ldo, int H, int G, int D, int R, int E, float scale, int window, const float* sink, const void* gate,
-                 long long ldg, int gate_cols, cudaStream_t stream) {
+                 long long ldo, int H, int G, int D, int R, int E, float scale, float cap, int window, const float* sink,
+                 const void* gate, long long ldg, int gate_cols, cudaStream_t stream) {
   using namespace apb;
   if (n_work <= 0) return 0;
   const int kch = (D + 63) / 64 + (R + 63) / 64;
@@ -391,10 +470,13 @@ int apb_flash_tc(const void* q, long long ldq, int rows, const int* work, int n_
   rc = make_tmap_2d(&tv, v, 2, key_rows, static_cast<uint64_t>(heads) * E, ldv, 64, box);
   if (rc) return 4000 + rc;
   const FlashParams p{work, page_table, max_pages, static_cast<__nv_bfloat16*>(out), ldo, G, D, R, E,
-                      SoftmaxSpec{scale, 0.f, 0, 1, nullptr, 1.f, 0.f, window, sink, gate, ldg, gate_cols}, status_device_ptr()};
-  const cudaError_t e = cudaFuncSetAttribute(flash_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kFlSmem);
-  if (e != cudaSuccess) return static_cast<int>(e);
-  flash_tc_kernel<<<n_work, kFlThreads, kFlSmem, stream>>>(tq, tk, tk2, tv, p);
-  return static_cast<int>(cudaGetLastError());
+                      SoftmaxSpec{scale, cap, 0, 1, nullptr, 1.f, 0.f, window, sink, gate, ldg, gate_cols}, status_device_ptr()};
+  auto run = [&](auto fn) -> int {
+    const cudaError_t e = cudaFuncSetAttribute(fn, cudaFuncAttributeMaxDynamicSharedMemorySize, kFlSmem);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    fn<<<n_work, kFlThreads, kFlSmem, stream>>>(tq, tk, tk2, tv, p);
+    return static_cast<int>(cudaGetLastError());
+  };
+  return cap > 0.f ? run(flash_tc_kernel<true>) : run(flash_tc_kernel<false>);
 }
 }

@@ -15,6 +15,7 @@
 #include "common.cuh"
 #include "host_utils.cuh"
 #include "ssm.cuh"
+#include "warp_mma.cuh"
 
 namespace apb {
 
@@ -31,35 +32,6 @@ struct SsmSegments {
   float* carry;           // [scratch states][H][N][E]
   float* decay;           // [n][H] log2 decay over the whole segment
 };
-
-// 16 bytes, or zeros when `bytes` is 0
-__device__ __forceinline__ void ssm_cp_async16(uint32_t dst, const void* src, int bytes) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ void ssm_ldsm4(const __nv_bfloat16* a, uint32_t (&r)[4]) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(a)));
-}
-__device__ __forceinline__ void ssm_ldsm4_t(const __nv_bfloat16* a, uint32_t (&r)[4]) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(a)));
-}
-__device__ __forceinline__ void ssm_ldsm2(const __nv_bfloat16* a, uint32_t (&r)[2]) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0, %1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(smem_u32(a)));
-}
-__device__ __forceinline__ void ssm_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
-      "{%0, %1, %2, %3};"
-      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-// x = hi + lo with both parts bf16; two neighbouring elements packed per word
-__device__ __forceinline__ void ssm_split2(float x, float y, uint32_t& hi, uint32_t& lo) {
-  hi = pack_bf16x2(x, y);
-  const float2 h = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&hi));
-  lo = pack_bf16x2(x - h.x, y - h.y);
-}
 
 __host__ __device__ inline int ssm_smem_bytes(int N) {
   const int np = (N + 15) / 16 * 16, ns = np + 8;
@@ -103,13 +75,13 @@ ssm_mma_kernel(const SsmParams p, const SsmSegments sg, int state_only) {
 #pragma unroll
     for (int i = threadIdx.x; i < kSmC * pc; i += kSmThreads) {
       const int r = i / pc, c = i % pc, ok = t0 + r < n_tok && c * 8 < N;
-      ssm_cp_async16(smem_u32(dst + r * ns + c * 8), xb + (start + (ok ? t0 + r : 0)) * p.ldx + col + (ok ? c * 8 : 0), ok ? 16 : 0);
+      wm_cp_async16(smem_u32(dst + r * ns + c * 8), xb + (start + (ok ? t0 + r : 0)) * p.ldx + col + (ok ? c * 8 : 0), ok ? 16 : 0);
     }
   };
   auto fetch_bx = [&](int t0, int buf) {
     fetch_rows(t0, b_col, B2 + buf * kSmC * ns);
     const int r = threadIdx.x >> 3, c = threadIdx.x & 7, ok = t0 + r < n_tok && c * 8 < be;
-    ssm_cp_async16(smem_u32(V2 + buf * kSmC * kSmVS + r * kSmVS + c * 8),
+    wm_cp_async16(smem_u32(V2 + buf * kSmC * kSmVS + r * kSmVS + c * 8),
                    xb + (start + (ok ? t0 + r : 0)) * p.ldx + x_col + (ok ? c * 8 : 0), ok ? 16 : 0);
   };
   static_assert(kSmThreads == kSmC * kSmBE / 8 && kSmC == 32, "one 16-byte piece of x per thread, one token per lane");
@@ -146,7 +118,7 @@ ssm_mma_kernel(const SsmParams p, const SsmSegments sg, int state_only) {
 #pragma unroll
         for (int hh = 0; hh < 2; ++hh) {
           uint32_t hi, lo;
-          ssm_split2(s[nt][2 * hh], s[nt][2 * hh + 1], hi, lo);
+          wm_split2(s[nt][2 * hh], s[nt][2 * hh + 1], hi, lo);
           const int o = (sr + 8 * hh) * kSmVS + nt * 8 + quad_col;
           *reinterpret_cast<uint32_t*>(Sh + o) = hi;
           *reinterpret_cast<uint32_t*>(Sl + o) = lo;
@@ -187,7 +159,7 @@ ssm_mma_kernel(const SsmParams p, const SsmSegments sg, int state_only) {
       const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(V + o));
       const float wt = exp2f(l_end - L[r]) * dt[r];
       uint32_t wh, wl;
-      ssm_split2(f.x * wt, f.y * wt, wh, wl);
+      wm_split2(f.x * wt, f.y * wt, wh, wl);
       *reinterpret_cast<uint32_t*>(Wh + o) = wh;
       *reinterpret_cast<uint32_t*>(Wl + o) = wl;
     }
@@ -203,21 +175,21 @@ ssm_mma_kernel(const SsmParams p, const SsmSegments sg, int state_only) {
 #pragma unroll 4
       for (int ks = 0; ks < n16; ++ks) {
         uint32_t q[4];
-        ssm_ldsm4(Cs + (r0 + rowin + (mat & 1) * 8) * ns + ks * 16 + (mat >> 1) * 8, q);
+        wm_ldsm4(Cs + (r0 + rowin + (mat & 1) * 8) * ns + ks * 16 + (mat >> 1) * 8, q);
         if (live) {
           uint32_t k[2];
-          ssm_ldsm2(B + (k0 + rowin) * ns + ks * 16 + (mat & 1) * 8, k);
-          ssm_mma(a, q, k[0], k[1]);
+          wm_ldsm2(B + (k0 + rowin) * ns + ks * 16 + (mat & 1) * 8, k);
+          wm_mma(a, q, k[0], k[1]);
         }
         if (have_state) {                          // C S of the carried state
           uint32_t sh[4], sl[4];
           const int so = (ks * 16 + rowin + 8 * (mat & 1)) * kSmVS + c0 + (mat >> 1) * 8;
-          ssm_ldsm4_t(Sh + so, sh);
-          ssm_ldsm4_t(Sl + so, sl);
+          wm_ldsm4_t(Sh + so, sh);
+          wm_ldsm4_t(Sl + so, sl);
 #pragma unroll
           for (int nt = 0; nt < 2; ++nt) {
-            ssm_mma(o[nt], q, sl[2 * nt], sl[2 * nt + 1]);
-            ssm_mma(o[nt], q, sh[2 * nt], sh[2 * nt + 1]);
+            wm_mma(o[nt], q, sl[2 * nt], sl[2 * nt + 1]);
+            wm_mma(o[nt], q, sh[2 * nt], sh[2 * nt + 1]);
           }
         }
       }
@@ -226,7 +198,7 @@ ssm_mma_kernel(const SsmParams p, const SsmSegments sg, int state_only) {
         const int i = r0 + quad_row + 8 * hh, j = k0 + quad_col;
         const float li = L[i];
         uint32_t hi, lo;
-        ssm_split2(j <= i ? a[2 * hh] * exp2f(li - L[j]) * dt[j] : 0.f,
+        wm_split2(j <= i ? a[2 * hh] * exp2f(li - L[j]) * dt[j] : 0.f,
                    j + 1 <= i ? a[2 * hh + 1] * exp2f(li - L[j + 1]) * dt[j + 1] : 0.f, hi, lo);
         *reinterpret_cast<uint32_t*>(Ah + i * kSmAS + j) = hi;
         *reinterpret_cast<uint32_t*>(Al + i * kSmAS + j) = lo;
@@ -245,13 +217,13 @@ ssm_mma_kernel(const SsmParams p, const SsmSegments sg, int state_only) {
       for (int ks = 0; ks < (r0 + 16) / 16; ++ks) {
         uint32_t ah[4], al[4], v[4];
         const int ao = (r0 + rowin + (mat & 1) * 8) * kSmAS + ks * 16 + (mat >> 1) * 8;
-        ssm_ldsm4(Ah + ao, ah);
-        ssm_ldsm4(Al + ao, al);
-        ssm_ldsm4_t(V + (ks * 16 + rowin + 8 * (mat & 1)) * kSmVS + c0 + (mat >> 1) * 8, v);
+        wm_ldsm4(Ah + ao, ah);
+        wm_ldsm4(Al + ao, al);
+        wm_ldsm4_t(V + (ks * 16 + rowin + 8 * (mat & 1)) * kSmVS + c0 + (mat >> 1) * 8, v);
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt) {
-          ssm_mma(o[nt], al, v[2 * nt], v[2 * nt + 1]);
-          ssm_mma(o[nt], ah, v[2 * nt], v[2 * nt + 1]);
+          wm_mma(o[nt], al, v[2 * nt], v[2 * nt + 1]);
+          wm_mma(o[nt], ah, v[2 * nt], v[2 * nt + 1]);
         }
       }
 #pragma unroll
@@ -280,17 +252,17 @@ ssm_mma_kernel(const SsmParams p, const SsmSegments sg, int state_only) {
 #pragma unroll
       for (int ks = 0; ks < kSmC / 16; ++ks) {
         uint32_t k[4];
-        ssm_ldsm4_t(B + (ks * 16 + rowin + (mat >> 1) * 8) * ns + warp * 16 + (mat & 1) * 8, k);
+        wm_ldsm4_t(B + (ks * 16 + rowin + (mat >> 1) * 8) * ns + warp * 16 + (mat & 1) * 8, k);
 #pragma unroll
         for (int n2 = 0; n2 < 4; ++n2) {
           uint32_t wh[4], wl[4];
           const int bo = (ks * 16 + rowin + 8 * (mat & 1)) * kSmVS + n2 * 16 + (mat >> 1) * 8;
-          ssm_ldsm4_t(Wh + bo, wh);
-          ssm_ldsm4_t(Wl + bo, wl);
+          wm_ldsm4_t(Wh + bo, wh);
+          wm_ldsm4_t(Wl + bo, wl);
 #pragma unroll
           for (int q = 0; q < 2; ++q) {
-            ssm_mma(s[2 * n2 + q], k, wl[2 * q], wl[2 * q + 1]);
-            ssm_mma(s[2 * n2 + q], k, wh[2 * q], wh[2 * q + 1]);
+            wm_mma(s[2 * n2 + q], k, wl[2 * q], wl[2 * q + 1]);
+            wm_mma(s[2 * n2 + q], k, wh[2 * q], wh[2 * q + 1]);
           }
         }
       }

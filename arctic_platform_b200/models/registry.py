@@ -26,7 +26,8 @@ register_architecture("Rigulorn", "arctic_platform_b200.models.rigulorn", "Rigul
 register_architecture("Titatar", "arctic_platform_b200.models.titatar", "TitatarConfig", "TitatarLM",
                       ("serve_residual", "serve_latent", "serve_moe", "serve_softmax", "serve_softmax_wide", "serve_flash_tc"))
 register_architecture("Meronex", "arctic_platform_b200.models.meronex", "MeronexConfig", "MeronexLM",
-                      ("serve_residual", "serve_moe", "serve_softmax", "serve_flash_tc", "ssm", "recurrent"))
+                      ("serve_residual", "serve_moe", "serve_softmax", "serve_flash_tc", "ssm", "recurrent", "memory_mma", "delta_mma",
+                       "time_mix_mma"))
 
 
 def kernel_sources(architecture: str) -> Tuple[str, ...]:

@@ -42,6 +42,9 @@ def _fn(name: str):
             "apb_residual_step": [vp] * 7 + [i, f] + [vp] * 5 + [i, i, i, f, f, i, i, vp, vp, vp, ll, i, vp, f, i, i, vp],
             "apb_half_rope_cache": [vp, ll, i, i, i] + [vp] * 8 + [i, vp, vp] + [i] * 5 + [f, i, vp],
             "apb_recurrent": [i, vp, vp] + [i] * 6 + [vp],
+            "apb_memory_mma": [vp, i, i, vp, vp, vp, i, vp, vp, vp, vp, i, vp],
+            "apb_delta_mma": [vp, vp, i, vp, i, vp, vp, vp],
+            "apb_time_mix_mma": [vp, vp, i, vp, vp, vp, i, vp],
             "apb_short_conv": [vp, ll, i, vp, vp, i, vp, vp, vp, ll, i] + [vp] * 5 + [i, i, vp],
             "apb_token_shift": [vp] * 10 + [i, i, i, vp, vp, i, i, vp, i, vp],
             "apb_tanh_rows": [vp, ll, i, i, i, vp],
@@ -57,7 +60,7 @@ def _fn(name: str):
             "apb_gemm_bf16_grouped_dev": [vp, vp, vp, i, i, i, ll, ll, ll, i, f, vp, ll, vp, i, vp, ll, vp],
             "apb_gemm_bf16_heads": [vp, vp, vp, i, i, i, i, ll, ll, ll, i, i, i, vp, ll, vp],
             "apb_softmax_attn_wide": [vp, ll] + [vp] * 4 + [i, vp, i, vp, vp, ll, vp] + [i] * 7 + [f, i, vp, vp, ll, i, vp],
-            "apb_flash_tc": [vp, ll, i, vp, i, vp, i, vp, ll, vp, vp, ll, ll, vp, ll] + [i] * 5 + [f, i, vp, vp, ll, i, vp],
+            "apb_flash_tc": [vp, ll, i, vp, i, vp, i, vp, ll, vp, vp, ll, ll, vp, ll] + [i] * 5 + [f, f, i, vp, vp, ll, i, vp],
             "apb_softmax_attn_tc": [vp, ll, i, vp, i, vp, i, vp, vp, i, vp, ll, i, i, i, i, f, f, vp, f, f, vp],
             "apb_ssm": [vp, ll, i, i, vp, vp, i] + [vp] * 6 + [ll] + [vp] * 7 + [i, vp] + [i] * 8 + [vp],
             "apb_ssm_mma": [vp, ll] + [vp] * 9 + [i, vp, vp, vp] + [i] * 5 + [vp],
@@ -672,7 +675,7 @@ def softmax_attention(b: StepBatch, q: torch.Tensor, heads: int, kcache: torch.T
               b.page_table.stride(0), _lib.ptr(kcache), _lib.ptr(vcache), _lib.ptr(out), out.stride(0), b.rows, heads, G, D, E,
               *tail, dtype_code(q.dtype))
         return
-    plain = spec.maps == 1 and not spec.cap and not spec.chunk
+    plain = spec.maps == 1 and not spec.chunk
     tc = spec.maps == 2 and D % 16 == 0 and D <= 64 and E <= 128 and 0 < spec.cap <= MAX_FIXED_CAP
     flash = plain and vcache is not None and flash_fits(D, 0, E) and not out.data_ptr() & 15
     lens = np.ones(1, dtype=np.int64) if b.host is None else b.host[:, 1]
@@ -700,7 +703,7 @@ def softmax_attention(b: StepBatch, q: torch.Tensor, heads: int, kcache: torch.T
         work = b.table(("flash", heads, G, spec.window), lambda: flash_tiles(b.host, heads, G, limit + 1, spec.window))
         _call("apb_flash_tc", _lib.ptr(q), q.stride(0), b.rows, _lib.ptr(work), work.shape[0], _lib.ptr(b.page_table),
               b.page_table.stride(0), _lib.ptr(kcache), D, None, _lib.ptr(vcache), E, kcache.shape[0] * G * PAGE, _lib.ptr(out),
-              out.stride(0), heads, G, D, 0, E, float(spec.scale), *tail[7:])
+              out.stride(0), heads, G, D, 0, E, float(spec.scale), float(spec.cap), *tail[7:])
     else:
         work = b.table(("softmax", heads, G, spec.chunk), lambda: chunk_tiles(b.host, heads, G, limit + 1, spec.chunk))
         _call("apb_softmax_attn_tc", _lib.ptr(q), q.stride(0), b.rows, _lib.ptr(work), work.shape[0], _lib.ptr(b.page_table),
@@ -825,7 +828,7 @@ def latent_attention(b: StepBatch, q: torch.Tensor, s: LatentSpec, cache: torch.
         kv = linear(latents, w_expand[:, :C])
         v = kv[:, v_col:]
         _call("apb_flash_tc", _lib.ptr(q), q.stride(0), b.rows, _lib.ptr(work), work.shape[0], None, 0, _lib.ptr(kv), kv.stride(0),
-              _lib.ptr(rotated), _lib.ptr(v), kv.stride(0), keys, _lib.ptr(out), out.stride(0), H, H, D, R, E, float(s.scale), 0,
+              _lib.ptr(rotated), _lib.ptr(v), kv.stride(0), keys, _lib.ptr(out), out.stride(0), H, H, D, R, E, float(s.scale), 0.0, 0,
               _lib.ptr(sink), _lib.ptr(gate), 0 if gate is None else gate.stride(0), E)
 
 
@@ -864,6 +867,16 @@ def segment_plan(host: np.ndarray, slices: int, slots: int) -> Dict[str, object]
             "chains": np.array(chains, dtype=np.int32).reshape(-1, 4)}
 
 
+def segments(b: StepBatch, slices: int):
+    """``(plan, seg, chains)`` of :func:`segment_plan` for two blocks per SM, the tables on the device (``chains`` None: no entry has
+    several segments)."""
+    key = ("segments", slices)
+    if key not in b.host_tables:
+        b.host_tables[key] = segment_plan(b.host, slices, 2 * _sm_count(b.tokens.device))
+    plan = b.host_tables[key]
+    return plan, b.table(key + ("seg",), lambda: plan["seg"]), b.table(key + ("chains",), lambda: plan["chains"]) if len(plan["chains"]) else None
+
+
 def retention(b: StepBatch, p: torch.Tensor, cols: Tuple[int, int, int, int], rope: Tuple[torch.Tensor, torch.Tensor],
               rot_dims: int, log2_decay: torch.Tensor, state: torch.Tensor, out: torch.Tensor, eps: float,
               k_scale: float, out_scale: float = 1.0) -> None:
@@ -880,12 +893,7 @@ def retention(b: StepBatch, p: torch.Tensor, cols: Tuple[int, int, int, int], ro
               int(b.one_token), int(b.longer and not mma), dtype_code(p.dtype))
     if mma:
         slices = H * ((E + 63) // 64)
-        key = ("retention", slices)
-        if key not in b.host_tables:
-            b.host_tables[key] = segment_plan(b.host, slices, 2 * _sm_count(p.device))
-        plan = b.host_tables[key]
-        seg = b.table(key + ("seg",), lambda: plan["seg"])
-        chains = b.table(key + ("chains",), lambda: plan["chains"]) if len(plan["chains"]) else None
+        plan, seg, chains = segments(b, slices)
         qk = torch.empty((b.rows, H, 4, (D + 15) // 16 * 16), device=p.device, dtype=torch.bfloat16)
         carry = torch.empty((plan["states"], H, D, E), device=p.device, dtype=torch.float32) if plan["states"] else None
         _call("apb_retention_mma", _lib.ptr(p), p.stride(0), *cols[:3], _lib.ptr(rope[0]), _lib.ptr(rope[1]), rot_dims,
@@ -934,12 +942,7 @@ def state_space(b: StepBatch, p: torch.Tensor, xbc_col: int, dt_col: int, w: Ssm
           tiles.shape[0] if b.longer else 0, H, E, groups, N, int(b.one_token), int(b.longer and not mma), dtype_code(p.dtype))
     if mma:
         slices = H * ((E + 63) // 64)
-        key = ("segments", slices)
-        if key not in b.host_tables:
-            b.host_tables[key] = segment_plan(b.host, slices, 2 * _sm_count(p.device))
-        plan = b.host_tables[key]
-        seg = b.table(key + ("seg",), lambda: plan["seg"])
-        chains = b.table(key + ("chains",), lambda: plan["chains"]) if len(plan["chains"]) else None
+        plan, seg, chains = segments(b, slices)
         f32 = dict(device=p.device, dtype=torch.float32)
         carry = torch.empty((plan["states"], H, N, E), **f32) if plan["states"] else None
         decay = torch.empty((len(plan["seg"]), H), **f32) if plan["states"] else None
@@ -957,6 +960,20 @@ def gated_group_norm(y: torch.Tensor, z: torch.Tensor, gain: torch.Tensor, parts
 
 
 # --------------------------------------------------------------------------------------------- matrix states per head
+CHUNK = 32              # tokens per chunk of the tensor-core kernels
+MAX_MMA_STATE = 128     # rows of a state that they hold in registers
+
+
+def first_tiles(host: np.ndarray, rows: int) -> np.ndarray:
+    """``[m, 2]`` int32 (entry, index of its first block in :func:`row_tiles`) of the entries longer than one row."""
+    out, at = [], 0
+    for en, n in enumerate(host[:, 1].tolist()):
+        if n > 1:
+            out.append((en, at))
+            at += -(-n // rows)
+    return np.array(out, dtype=np.int32)
+
+
 RULES = {"memory": 0, "delta": 1, "time_mix": 2}
 
 
@@ -1029,7 +1046,34 @@ def recurrent(b: StepBatch, s: RecurrentSpec, x: RecurrentInputs, state: torch.T
         _lib.ptr(aux), H, s.key_heads, D, E, _lib.ptr(y), _lib.ptr(x.gain), 0 if s.shared_gain else E, x.g, int(s.silu), _lib.ptr(out),
         out.stride(0), s.eps)
     ref = ctypes.byref(params)
-    _call("apb_recurrent", rule, ref, _lib.ptr(b.row_entry), b.n_entries, b.rows, int(b.one_token), int(b.longer), int(b.longer), dt)
+    aligned = not (D % 8 or E % 8 or p.stride(0) % 8 or p.data_ptr() & 15 or (x.q | x.k | x.v) % 8 or (x.z is not None and x.z.stride(0) % 4))
+    mma = b.longer and p.dtype == torch.bfloat16 and aligned and D <= MAX_MMA_STATE
+    if b.one_token or (b.longer and not mma):
+        _call("apb_recurrent", rule, ref, _lib.ptr(b.row_entry), b.n_entries, b.rows, int(b.one_token), int(b.longer and not mma), 0, dt)
+    if not b.longer:
+        return
+    if mma:
+        f32 = dict(device=p.device, dtype=torch.float32)
+        if s.rule == "delta":
+            tiles = b.table(("rows", CHUNK), lambda: row_tiles(b.host, CHUNK))
+            heads = b.table(("chunks", CHUNK), lambda: first_tiles(b.host, CHUNK))
+            square = torch.empty((tiles.shape[0], H, 4, CHUNK, CHUNK), device=p.device, dtype=torch.bfloat16)
+            scalars = torch.empty((tiles.shape[0], H, 4 * CHUNK + 4), **f32)
+            _call("apb_delta_mma", ref, _lib.ptr(tiles), tiles.shape[0], _lib.ptr(heads), heads.shape[0], _lib.ptr(square), _lib.ptr(scalars))
+        else:
+            plan, seg, chains = segments(b, H * ((E + 63) // 64))
+            n_seg, parts = len(plan["seg"]), plan["states"]
+            carry = torch.empty((parts, H, D, E), **f32) if parts else None
+            if s.rule == "memory":
+                gates, aux0 = torch.empty((b.rows, H, 2), **f32), torch.empty((b.n_entries, H, D + 1), **f32)
+                carry_aux = torch.empty((parts, H, D + 1), **f32) if parts else None
+                totals = torch.empty((n_seg, H, 2), **f32) if parts else None
+                _call("apb_memory_mma", ref, b.rows, b.n_entries, _lib.ptr(gates), _lib.ptr(aux0), _lib.ptr(seg), n_seg, _lib.ptr(carry),
+                      _lib.ptr(carry_aux), _lib.ptr(totals), _lib.ptr(chains), len(plan["chains"]))
+            else:
+                decay = torch.empty((n_seg, H, D), **f32) if parts else None
+                _call("apb_time_mix_mma", ref, _lib.ptr(seg), n_seg, _lib.ptr(carry), _lib.ptr(decay), _lib.ptr(chains), len(plan["chains"]))
+    _call("apb_recurrent", rule, ref, _lib.ptr(b.row_entry), b.n_entries, b.rows, 0, 0, 1, dt)
 
 
 def token_shift(b: StepBatch, h: torch.Tensor, mu: torch.Tensor, hist: torch.Tensor, parity: torch.Tensor, w: torch.Tensor, step: int,
