@@ -147,7 +147,7 @@ __device__ __forceinline__ void rec_store(float* p, const float4& v) {
 
 // AHEAD: state rows per thread that are on their way while the token's parts are computed (and stay in registers).
 template <int RULE, typename T, int VEC, int AHEAD>
-__global__ void __launch_bounds__(kRecThreads)
+__global__ void __launch_bounds__(kRecThreads, AHEAD > 8 ? 2 : AHEAD > 4 ? 3 : 4)
 recurrent_decode_kernel(const RecurrentParams p) {
   pdl_entry();
   extern __shared__ __align__(16) float rec_smem[];
@@ -530,8 +530,9 @@ static int recurrent_run(const RecurrentParams& a, const int* row_entry, int n_e
       const int rc = rec_smem_limit(fn, smem);
       return rc ? rc : static_cast<int>(launch_kernel(fn, dim3(n_entries, a.H), dim3(kRecThreads), smem, s, a));
     };
-    constexpr int kAhead = RULE == kRuleDelta ? 16 : 8;
-    const int rc = v4 ? run(recurrent_decode_kernel<RULE, T, 4, kAhead>) : run(recurrent_decode_kernel<RULE, T, 1, kAhead>);
+    const int each = (a.D + ny - 1) / ny;      // state rows per thread
+    const int rc = !v4 ? run(recurrent_decode_kernel<RULE, T, 1, 8>) : each <= 4 ? run(recurrent_decode_kernel<RULE, T, 4, 4>)
+                   : each <= 8 || RULE != kRuleDelta ? run(recurrent_decode_kernel<RULE, T, 4, 8>) : run(recurrent_decode_kernel<RULE, T, 4, 16>);
     if (rc) return rc;
   }
   if (scan) {

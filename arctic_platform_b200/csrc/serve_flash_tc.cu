@@ -72,55 +72,58 @@ __device__ __forceinline__ uint64_t flash_weights(uint32_t t_s, uint64_t scale2,
   return xtc_add2(sum[0], sum[1]);
 }
 
-// The same for capped scores, 2^(gain tanh(zs score) + off): the series of tanh_series with the scales folded into its coefficients,
-// or the exponential form for a warp that holds a larger score.
+// The same for capped scores, 2^(gain tanh(z) + off): the series of tanh_series with the scales folded into its coefficients, or the
+// exponential form for a warp that holds a larger score (an exponent needs absolute accuracy only).
 struct CapSeries {
-  float zs, gain, small;       // small: largest squared score of the series
+  float gain, e2, small;       // e2: log2 e^(2 z) of a score; small: largest squared score of the series
   uint64_t c[5];
 };
 __device__ __forceinline__ CapSeries cap_series(const SoftmaxSpec& sp) {
   CapSeries k;
-  k.zs = sp.scale / sp.cap;
+  const float zs = sp.scale / sp.cap, z2 = zs * zs;
   k.gain = sp.cap * 1.4426950408889634f;
-  k.small = (kSmallTanh / k.zs) * (kSmallTanh / k.zs);
-  const float z2 = k.zs * k.zs, t[5] = {1.f, -1.f / 3.f, 2.f / 15.f, -17.f / 315.f, 62.f / 2835.f};
-  float f = k.gain * k.zs;
+  k.e2 = 2.f * 1.4426950408889634f * zs;
+  k.small = (kSmallTanh / zs) * (kSmallTanh / zs);
+  const float t[5] = {1.f, -1.f / 3.f, 2.f / 15.f, -17.f / 315.f, 62.f / 2835.f};
+  float f = k.gain * zs;
 #pragma unroll
   for (int i = 0; i < 5; ++i, f *= z2) k.c[i] = xtc_pair(f * t[i], f * t[i]);
   return k;
 }
+// 32 of a row's scores r as exponents v, pairs of neighbouring keys.
+__device__ __forceinline__ void capped_exponents(const uint32_t (&r)[32], const CapSeries& k, float off, uint64_t (&v)[16]) {
+  const uint64_t off2 = xtc_pair(off, off);
+  float large = 0.f;
+#pragma unroll
+  for (int i = 0; i < 16; ++i) {
+    const uint64_t x = xtc_pair(__uint_as_float(r[2 * i]), __uint_as_float(r[2 * i + 1])), a = xtc_mul2(x, x);
+    const float2 f = xtc_unpair(a);
+    large = fmaxf(fmaxf(large, f.x), f.y);
+    uint64_t y = xtc_fma2(a, k.c[4], k.c[3]);
+    y = xtc_fma2(a, y, k.c[2]);
+    y = xtc_fma2(a, y, k.c[1]);
+    y = xtc_fma2(a, y, k.c[0]);
+    v[i] = xtc_fma2(x, y, off2);
+  }
+  if (!__all_sync(0xffffffffu, large <= k.small)) {
+#pragma unroll
+    for (int i = 0; i < 16; ++i)                       // gain tanh(z) = gain - 2 gain / (1 + e^(2 z))
+      v[i] = xtc_pair((k.gain + off) - __fdividef(2.f * k.gain, 1.f + xtc_ex2(__uint_as_float(r[2 * i]) * k.e2)),
+                      (k.gain + off) - __fdividef(2.f * k.gain, 1.f + xtc_ex2(__uint_as_float(r[2 * i + 1]) * k.e2)));
+  }
+}
 template <bool WHOLE>
 __device__ __forceinline__ uint64_t flash_capped_weights(uint32_t t_s, const CapSeries& k, float off, int limit, int skip, float& top,
                                                          uint32_t (&pk)[4][16]) {
-  const uint64_t off2 = xtc_pair(off, off);
-  uint64_t sum[2] = {xtc_pair(0.f, 0.f), xtc_pair(0.f, 0.f)};
-  float t0 = -INFINITY, t1 = -INFINITY;
-  uint32_t stage[2][32];
-  tmem_ld_32x32(t_s, stage[0]);
+  uint64_t sum = xtc_pair(0.f, 0.f);
+  float t0 = -INFINITY;
 #pragma unroll
   for (int c = 0; c < 4; ++c) {
-    uint32_t(&r)[32] = stage[c & 1];
-    xtc_wait_load(r);
-    if (c < 3) tmem_ld_32x32(t_s + (c + 1) * 32, stage[(c + 1) & 1]);
+    uint32_t r[32];
     uint64_t v[16];
-    float large = 0.f;
-#pragma unroll
-    for (int i = 0; i < 16; ++i) {
-      const uint64_t x = xtc_pair(__uint_as_float(r[2 * i]), __uint_as_float(r[2 * i + 1])), a = xtc_mul2(x, x);
-      const float2 f = xtc_unpair(a);
-      large = fmaxf(fmaxf(large, f.x), f.y);
-      uint64_t y = xtc_fma2(a, k.c[4], k.c[3]);
-      y = xtc_fma2(a, y, k.c[2]);
-      y = xtc_fma2(a, y, k.c[1]);
-      y = xtc_fma2(a, y, k.c[0]);
-      v[i] = xtc_fma2(x, y, off2);
-    }
-    if (!__all_sync(0xffffffffu, large <= k.small)) {
-#pragma unroll
-      for (int i = 0; i < 16; ++i)
-        v[i] = xtc_pair(fmaf(tanh_any(__uint_as_float(r[2 * i]) * k.zs), k.gain, off),
-                        fmaf(tanh_any(__uint_as_float(r[2 * i + 1]) * k.zs), k.gain, off));
-    }
+    tmem_ld_32x32(t_s + c * 32, r);
+    xtc_wait_load(r);
+    capped_exponents(r, k, off, v);
 #pragma unroll
     for (int i = 0; i < 16; ++i) {
       float2 f = xtc_unpair(v[i]);
@@ -129,18 +132,50 @@ __device__ __forceinline__ uint64_t flash_capped_weights(uint32_t t_s, const Cap
         if (a >= limit || a < skip) f.x = -INFINITY;
         if (a + 1 >= limit || a + 1 < skip) f.y = -INFINITY;
       }
-      t0 = fmaxf(t0, f.x);
-      t1 = fmaxf(t1, f.y);
+      t0 = fmaxf(t0, fmaxf(f.x, f.y));
       const float w0 = xtc_ex2(f.x), w1 = xtc_ex2(f.y);
-      sum[i & 1] = xtc_add2(sum[i & 1], xtc_pair(w0, w1));
+      sum = xtc_add2(sum, xtc_pair(w0, w1));
       pk[c][i] = pack_bf16x2(w0, w1);
     }
   }
-  top = fmaxf(t0, t1);
+  top = t0;
+  return sum;
+}
+// With a fixed reference nothing is looked at twice: the weights replace the scores run by run (weights c lie over scores c / 2, which
+// have been read).
+template <bool WHOLE>
+__device__ __forceinline__ uint64_t flash_fixed_weights(uint32_t t_s, const CapSeries& k, float off, int limit, int skip) {
+  uint64_t sum[2] = {xtc_pair(0.f, 0.f), xtc_pair(0.f, 0.f)};
+  uint32_t stage[2][32];
+  tmem_ld_32x32(t_s, stage[0]);
+#pragma unroll
+  for (int c = 0; c < 4; ++c) {
+    uint32_t(&r)[32] = stage[c & 1];
+    xtc_wait_load(r);
+    if (c < 3) tmem_ld_32x32(t_s + (c + 1) * 32, stage[(c + 1) & 1]);
+    uint64_t v[16];
+    capped_exponents(r, k, off, v);
+    uint32_t pk[16];
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+      const float2 f = xtc_unpair(v[i]);
+      float w0 = xtc_ex2(f.x), w1 = xtc_ex2(f.y);
+      if (!WHOLE) {
+        const int a = c * 32 + 2 * i;
+        if (a >= limit || a < skip) w0 = 0.f;
+        if (a + 1 >= limit || a + 1 < skip) w1 = 0.f;
+      }
+      sum[i & 1] = xtc_add2(sum[i & 1], xtc_pair(w0, w1));
+      pk[i] = pack_bf16x2(w0, w1);
+    }
+    tmem_st_32x16(t_s + c * 16, pk);
+  }
   return xtc_add2(sum[0], sum[1]);
 }
 
-template <bool CAP>
+enum FlashCap : int { kFlashUncapped = 0, kFlashCapped = 1, kFlashFixed = 2 };
+
+template <int CAP>
 __global__ void __launch_bounds__(kFlThreads, 1)
 flash_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_k,
                 const __grid_constant__ CUtensorMap tma_k2, const __grid_constant__ CUtensorMap tma_v, const FlashParams p) {
@@ -330,9 +365,8 @@ flash_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
     const uint64_t scale2 = xtc_pair(scale, scale);
     const int pos = pos0 + min(row, valid - 1);
     CapSeries cs = {};
-    if (CAP) cs = cap_series(p.sp);
-    const bool fixed = CAP && fixed_reference(p.sp.cap);
-    float ref = fixed ? score_reference(p.sp.cap) * 1.4426950408889634f : -INFINITY;      // reference of the weights (log2)
+    if (CAP != kFlashUncapped) cs = cap_series(p.sp);
+    float ref = CAP == kFlashFixed ? score_reference(p.sp.cap) * 1.4426950408889634f : -INFINITY;      // reference of the weights (log2)
     uint64_t sum2 = xtc_pair(0.f, 0.f);
     bool ok = true;
     for (int j = 0; j < nb; ++j) {
@@ -345,19 +379,22 @@ flash_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant
       const int limit = pos + 1 - base;                                  // visible keys: [skip, limit) of the block
       const int skip = window > 0 ? pos + 1 - window - base : 0;
       const bool whole = pos0 + 1 - base >= kFlKeys && (window <= 0 || pos0 + valid - window - base <= 0);   // all 128 for every row
+      if constexpr (CAP == kFlashFixed) {
+        sum2 = xtc_add2(sum2, whole ? flash_fixed_weights<true>(t_s, cs, -ref, limit, skip) : flash_fixed_weights<false>(t_s, cs, -ref, limit, skip));
+        tmem_st_wait();
+        tc_fence_before();
+        mbar_arrive(&p_full[g]);
+        continue;
+      }
       uint32_t pk[4][16];
       for (int pass = 0; pass < 2; ++pass) {           // a second time if the reference had to move
         const float off = ref == -INFINITY ? 0.f : -ref;
         float top;                                     // largest score relative to the reference
         uint64_t block2;
-        if constexpr (CAP)
+        if constexpr (CAP != kFlashUncapped)
           block2 = whole ? flash_capped_weights<true>(t_s, cs, off, limit, skip, top, pk) : flash_capped_weights<false>(t_s, cs, off, limit, skip, top, pk);
         else
           block2 = whole ? flash_weights<true>(t_s, scale2, off, limit, skip, top, pk) : flash_weights<false>(t_s, scale2, off, limit, skip, top, pk);
-        if (fixed) {
-          sum2 = xtc_add2(sum2, block2);
-          break;
-        }
         const bool behind = top > kFlLag || (ref == -INFINITY && top > -INFINITY);
         if (pass == 1 || !__any_sync(0xffffffffu, behind)) {
           sum2 = xtc_add2(sum2, block2);
@@ -477,6 +514,6 @@ int apb_flash_tc(const void* q, long long ldq, int rows, const int* work, int n_
     fn<<<n_work, kFlThreads, kFlSmem, stream>>>(tq, tk, tk2, tv, p);
     return static_cast<int>(cudaGetLastError());
   };
-  return cap > 0.f ? run(flash_tc_kernel<true>) : run(flash_tc_kernel<false>);
+  return fixed_reference(cap) ? run(flash_tc_kernel<kFlashFixed>) : cap > 0.f ? run(flash_tc_kernel<kFlashCapped>) : run(flash_tc_kernel<kFlashUncapped>);
 }
 }

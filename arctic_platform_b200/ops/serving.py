@@ -1076,6 +1076,9 @@ def recurrent(b: StepBatch, s: RecurrentSpec, x: RecurrentInputs, state: torch.T
     _call("apb_recurrent", rule, ref, _lib.ptr(b.row_entry), b.n_entries, b.rows, 0, 0, 1, dt)
 
 
+MANY_ROWS = 1024
+
+
 def token_shift(b: StepBatch, h: torch.Tensor, mu: torch.Tensor, hist: torch.Tensor, parity: torch.Tensor, w: torch.Tensor, step: int,
                 cols: Sequence[int]) -> torch.Tensor:
     """``h [rows, W]`` blended with the row of the token before, ``h + (h' - h) mu[s]`` for every ``mu [n, W]``, and the products of the
@@ -1087,12 +1090,17 @@ def token_shift(b: StepBatch, h: torch.Tensor, mu: torch.Tensor, hist: torch.Ten
     mixed = torch.empty((n, T, W), device=dev, dtype=h.dtype)
     out = torch.empty((n, T, N), device=dev, dtype=h.dtype)
     simt = _simt(h, w, out[0]) or bool(step % 8)
+    ptrs = (_lib.ptr(h), _lib.ptr(mu), _lib.ptr(hist), _lib.ptr(parity), _lib.ptr(mixed), _lib.ptr(b.row_entry), *b.entry_ptrs(), T, W, n)
+    if not simt and T >= MANY_ROWS:          # each product fills the GPU
+        _call("apb_token_shift", *ptrs, None, None, 1, step, None, dt)
+        for i, c in enumerate(cols):
+            linear(mixed[i], w[i * step:i * step + (c + 7) // 8 * 8], out[i][:, :(c + 7) // 8 * 8])
+        return out
     tile = 64 if simt else 128
     most = sum(-(-T // tile) * -(-c // tile) for c in cols)
     tiles = torch.empty(4 * most + 4, device=dev, dtype=torch.int32)
     count = tiles[4 * most:]
-    _call("apb_token_shift", _lib.ptr(h), _lib.ptr(mu), _lib.ptr(hist), _lib.ptr(parity), _lib.ptr(mixed), _lib.ptr(b.row_entry),
-          *b.entry_ptrs(), T, W, n, _lib.ptr(tiles), _lib.ptr(count), tile, step, (ctypes.c_int * n)(*cols), dt)
+    _call("apb_token_shift", *ptrs, _lib.ptr(tiles), _lib.ptr(count), tile, step, (ctypes.c_int * n)(*cols), dt)
     if simt:
         _call("apb_gemm_simt_grouped", _lib.ptr(mixed), _lib.ptr(w), _lib.ptr(out), n * T, N, W, W, w.stride(0), N, gemm.EPI_BF16, None, 0, 0.0,
               _lib.ptr(tiles), most, _lib.ptr(count), dt)

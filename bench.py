@@ -48,7 +48,8 @@ def parse_args():
     ap.add_argument("--workload", default="grpo", choices=["grpo", "serving"],
                     help="grpo: the benchmark step (default); serving: prefill / decode speed and per-kernel roofline "
                          "fractions of the stateful architectures beside the closest older model (benchmarks/bench_serving.py)")
-    ap.add_argument("--serving-models", default="reninex-2048,reninex-4096,rigulorn-2048,rigulorn-4096,titatar-2048,titatar-4096")
+    ap.add_argument("--serving-models", default="reninex-2048,reninex-4096,rigulorn-2048,rigulorn-4096,titatar-2048,titatar-4096,"
+                                                  "meronex-2048,meronex-4096")
     ap.add_argument("--model", default="qwen3-4b")
     ap.add_argument("--prompts-per-gpu", type=int, default=8)
     ap.add_argument("--samples", type=int, default=16)

@@ -10,12 +10,13 @@ For every model (random weights, synthetic prompts) two parts are measured on on
   width, heads and feed-forward (for retention the gated delta rule of the hybrid family at the same heads and sizes); for
   Rigulorn a Reninex layer whose K/V rows, state and feed-forward have the same size; for Titatar the dense decoder's layer
   with the heads of its windowed attention, and the decoder family's mixture of experts with as many experts and (on average)
-  as many routed rows.  ``floor_ms`` is the slower of
+  as many routed rows; for Meronex the steps of a Titatar layer with its attention heads and its experts, for the recurrent mixers
+  Rigulorn's state space with as many heads and states of the same size.  ``floor_ms`` is the slower of
   algorithmic bytes over the measured copy bandwidth and FLOPs over the measured bf16 GEMM peak, ``frac`` = floor / time.
   CUDA events around every launch, L2 overwritten before it, median over the iterations.
 * engine: prefill and decode tokens/s through ``generate`` of the model, of the dense decoder with as many layers as the
-  model has layer runs (for Titatar: with a mixture of experts of the same size in every layer) and, for Rigulorn, of the
-  Reninex preset of the same width.
+  model has layer runs (for Titatar and Meronex: with a mixture of experts of the same size in every layer) and, for Rigulorn
+  and Meronex, of the Reninex or Titatar preset of the same width.
 
 Prints one JSON line per measurement.
 """
@@ -90,7 +91,8 @@ def phase_batch(phase):
 
 def stateful_ops(cfg, phase):
     """``(name, fn, bytes, flops)`` of the steps of the model's layers on the phase's batch."""
-    return {"Reninex": reninex_ops, "Rigulorn": rigulorn_ops, "Titatar": titatar_ops}[cfg.architecture](cfg, phase)
+    return {"Reninex": reninex_ops, "Rigulorn": rigulorn_ops, "Titatar": titatar_ops,
+            "Meronex": meronex_ops}[cfg.architecture](cfg, phase)
 
 
 def reninex_ops(cfg, phase):
@@ -279,6 +281,143 @@ def titatar_ops(cfg, phase):
     ]
 
 
+def meronex_ops(cfg, phase):
+    import dataclasses
+    import math
+    from arctic_platform_b200.engine.stateful_sampler import StateCache
+    from arctic_platform_b200.models.meronex import MeronexLM
+    from arctic_platform_b200.ops import gemm as gemm_ops, serving
+    one = dataclasses.replace(cfg, layers=tuple(next(s for s in cfg.layers if s.type == t) for t in ("mlstm", "delta", "parallel")),
+                              vocab_size=1024)
+    model = MeronexLM(one, "cuda", torch.bfloat16).init_weights(0)
+    model.prepare_serving(SEQ + 8)
+    b, n, n_pages, keys = phase_batch(phase)
+    cache = StateCache(model.cache_layout(), n_pages, n, "cuda", torch.bfloat16)
+    for t in cache._paged():
+        t.normal_()
+    T, W, G = b.rows, cfg.hidden_size, cfg.norm_groups
+    mem, dlt, par = (blk.mixer for blk in model.blocks)
+    moe, M = model.blocks[0].mlp, one.layers[0].mlp
+    x = torch.randn(T, W, device="cuda")
+    serving.embed(b, model.embed, None, None, cache.prev, torch.empty_like(x))
+    clear = serving.accumulates(T, W, x.device)
+    y, y2, h = torch.zeros(T, W, device="cuda"), torch.zeros(T, W, device="cuda"), _bf(T, W)
+    pm, pd, pp = (serving.linear(h, m.w_in) for m in (mem, dlt, par))
+    om, od, ol, orr = (_bf(T, m) for m in (mem.n_out, dlt.n_out, par.n_left, par.n_right))
+    L, R, K = par.m.left, par.m.right, par.rank
+    c, rope = par.in_cols, model._rope[L.rot]
+    spin = pp.clone()                                    # rotated in place again and again; attention reads queries rotated once
+    serving.half_rope_cache(b, pp, (c["q"][0], c["k"][0], c["v"][0]), rope, L.rot.dims, L.heads, cache.k[2], cache.v[2], 1e-6)
+    cols = [par.n_right] * 4 + [K]
+    s = serving.token_shift(b, h, par.mu, cache.conv[2], cache.parity, par.w_shift, par.step, cols)
+    low = s[4][:, :K]
+    z = serving.linear(low, par.w_rank[:, :K], out_dtype=torch.float32)
+    zz = serving.linear(h, moe.w_z, out_dtype=torch.float32)
+    gate_col = moe.z_cols["rg"][0]
+
+    def experts():
+        return serving.experts(b, h, zz, None, moe.counters, moe.w_gu, moe.w_down, M.experts, M.experts, M.top, M.ff, sigmoid=True,
+                               scale_input=True, epi=gemm_ops.EPI_CLAMP_GLU, limit=M.limit)
+
+    def decay():
+        serving.tanh_rows(low)
+        serving.linear(low, par.w_rank[:, :K], z)
+
+    mix = experts()
+    pairs = T * M.top
+    touched = M.experts * (1 - math.exp(-pairs / M.experts))
+    ctx = T if phase == "prefill" else keys
+    kv_row = L.kv_heads * (L.dim + L.vdim) * 2
+    norms, bias = model.blocks[2], model.blocks[0]
+    passes = 2 if phase == "decode" else 1
+    state = lambda H, D, E: n * H * D * E * 4 * passes
+    chunked = lambda H, D, E, f: T * H * (2 * 64 * (D + E) / 2 + f * D * E)
+    gemm = lambda N, K: (2 * (T * K + N * K + T * N), 2 * T * N * K)
+    out = lambda K: (2 * (T * K + K * W) + (8 if clear else 4) * T * W, 2 * T * W * K)
+    res = T * W * (8 + 2 + (4 if clear else 0))
+    how = dict(eps=1e-6, offset=0.0, groups=G, mult=0.7, clear=clear)
+    d = mem.m
+    q = dlt.m
+    Hr, Dr = R.heads, R.dim
+    return [
+        ("gated residual update + norm", lambda: serving.residual_step(x, y, None, norms.norm1, gate=pm[:, mem.in_cols["rg"][0]:],
+                                                                      gate_bias=bias.gate_bias1, **how), res + 6 * T * W, 0),
+        ("gated residual update + expert sum + norm", lambda: serving.residual_step(x, None, None, norms.norm1, mix=mix, gate=zz[:, gate_col:],
+                                                                                   gate_bias=bias.gate_bias2, **how),
+         T * W * (8 + 2 + 4) + 2 * pairs * W, 0),
+        ("gated residual update + two sides + norm", lambda: serving.residual_step(x, y, par.left_out, norms.norm2, y2=y2, post2=par.right_out,
+                                                                                  gate=pp[:, c["rg"][0]:], gate_bias=norms.gate_bias1, **how),
+         res + 6 * T * W + (8 if clear else 4) * T * W, 0),
+        ("memory input projections (GEMM)", lambda: serving.linear(h, mem.w_in, pm), *gemm(pm.shape[1], W)),
+        ("matrix memory", lambda: serving.recurrent(b, mem.spec, mem.inputs(pm), cache.state[0], om, aux=cache.aux[0]),
+         2 * T * (2 * d.heads * d.dim + 3 * mem.n_out + 2 * d.heads) + state(d.heads, d.dim, d.vdim), chunked(d.heads, d.dim, d.vdim, 4)),
+        ("memory output projection (GEMM)", lambda: serving.project(om, mem.w_out, y), *out(mem.n_out)),
+        ("delta input projections (GEMM)", lambda: serving.linear(h, dlt.w_in, pd), *gemm(pd.shape[1], W)),
+        ("convolution + delta rule", lambda: serving.recurrent(b, dlt.spec, dlt.inputs(pd), cache.state[1], od, hist=cache.conv[1],
+                                                               parity=cache.parity),
+         2 * T * (2 * q.kv_heads * q.dim + 3 * dlt.n_out + 2 * q.heads) + state(q.heads, q.dim, q.vdim), chunked(q.heads, q.dim, q.vdim, 6)),
+        ("delta output projection (GEMM)", lambda: serving.project(od, dlt.w_out, y), *out(dlt.n_out)),
+        ("parallel input projections (GEMM)", lambda: serving.linear(h, par.w_in, pp), *gemm(pp.shape[1], W)),
+        ("rotation + value norm + cache write", lambda: serving.half_rope_cache(b, spin, (c["q"][0], c["k"][0], c["v"][0]), rope, L.rot.dims,
+                                                                               L.heads, cache.k[2], cache.v[2], 1e-6),
+         2 * T * (2 * L.heads * L.dim) + 2 * T * kv_row, 0),
+        ("capped attention", lambda: serving.softmax_attention(b, pp, L.heads, cache.k[2], cache.v[2], par.softmax, None, ol),
+         ctx * kv_row + 2 * T * L.heads * (L.dim + L.vdim), 2 * keys * L.heads * (L.dim + L.vdim)),
+        ("attention output projection (GEMM)", lambda: serving.project(ol, par.w_left, y), *out(par.n_left)),
+        ("token shift + its products (GEMM)", lambda: serving.token_shift(b, h, par.mu, cache.conv[2], cache.parity, par.w_shift, par.step, cols),
+         2 * (T * W + sum(cols) * W + T * sum(cols)), 2 * T * W * sum(cols)),
+        ("decay projection (GEMM)", decay, 2 * (2 * T * K + par.n_right * K) + 4 * T * par.n_right, 2 * T * K * par.n_right),
+        ("time mixing", lambda: serving.recurrent(b, par.spec, par.inputs(s, z), cache.state[2], orr),
+         2 * T * 5 * par.n_right + 4 * T * par.n_right + state(Hr, Dr, Dr), chunked(Hr, Dr, Dr, 4)),
+        ("time mixing output projection (GEMM)", lambda: serving.project(orr, par.w_right, y2), *out(par.n_right)),
+        ("router + gate (GEMM)", lambda: serving.linear(h, moe.w_z, zz), 2 * T * W + 2 * zz.shape[1] * W + 4 * T * zz.shape[1],
+         2 * T * W * zz.shape[1]),
+        ("routed experts", experts, touched * 6 * W * M.ff + 2 * T * W + 2 * pairs * W, 6 * pairs * W * M.ff),
+    ]
+
+
+# step of a Meronex layer -> (model, the like step of its layer)
+MERONEX_LIKE = {
+    "gated residual update + norm": ("titatar", "residual update + norms"),
+    "gated residual update + expert sum + norm": ("titatar", "residual update + expert sum + norms"),
+    "gated residual update + two sides + norm": ("titatar", "residual update + norms"),
+    "memory input projections (GEMM)": ("titatar", "windowed input projections (GEMM)"), "matrix memory": ("memory", "recurrent mixer"),
+    "memory output projection (GEMM)": ("titatar", "windowed output projection (GEMM)"),
+    "delta input projections (GEMM)": ("titatar", "windowed input projections (GEMM)"), "convolution + delta rule": ("delta", "recurrent mixer"),
+    "delta output projection (GEMM)": ("titatar", "windowed output projection (GEMM)"),
+    "parallel input projections (GEMM)": ("titatar", "windowed input projections (GEMM)"),
+    "rotation + value norm + cache write": ("titatar", "q/k norm + rotation + cache write"), "capped attention": ("titatar", "windowed attention"),
+    "attention output projection (GEMM)": ("titatar", "windowed output projection (GEMM)"),
+    "token shift + its products (GEMM)": ("titatar", "windowed input projections (GEMM)"),
+    "decay projection (GEMM)": ("titatar", "router (GEMM)"), "time mixing": ("time_mix", "recurrent mixer"),
+    "time mixing output projection (GEMM)": ("titatar", "windowed output projection (GEMM)"),
+    "router + gate (GEMM)": ("titatar", "router (GEMM)"), "routed experts": ("titatar", "routed experts"),
+}
+
+
+def meronex_like(cfg, phase):
+    """Steps of a Titatar layer with the attention heads (no window) and the experts of the Meronex model, and of Rigulorn's state
+    space with the heads and state sizes of its recurrent mixers: ``model -> {name: (fn, bytes, flops)}``."""
+    import dataclasses
+    from arctic_platform_b200.models import rigulorn, titatar
+    mem, dlt, par = (next(s for s in cfg.layers if s.type == t) for t in ("mlstm", "delta", "parallel"))
+    L, M = par.mixer.left, mem.mlp
+    t = titatar.PRESETS["titatar-2048"]
+    latent = next(s for s in t.layers if s.latent)
+    window = titatar.WindowAttnSpec(L.heads, L.kv_heads, L.dim, L.vdim, L.scale, 0, L.rot)
+    layers = (dataclasses.replace(latent, mlp=titatar.MoeSpec(M.experts, 0, M.top, M.ff)), titatar.LayerSpec(window, 2 * cfg.hidden_size))
+    ops = {"titatar": titatar_ops(dataclasses.replace(t, hidden_size=cfg.hidden_size, layers=layers, loop=None), phase)}
+    r = rigulorn.PRESETS["rigulorn-2048"]
+    attn = next(s for s in r.layers if s.attention and s.ff)
+    sizes = {"memory": (mem.mixer.heads, mem.mixer.vdim, mem.mixer.dim, mem.mixer.heads),
+             "delta": (dlt.mixer.heads, dlt.mixer.vdim, dlt.mixer.dim, dlt.mixer.kv_heads),
+             "time_mix": (par.mixer.right.heads, par.mixer.right.dim, par.mixer.right.dim, par.mixer.right.heads)}
+    for name, (heads, vdim, dim, groups) in sizes.items():
+        ssm = rigulorn.LayerSpec(rigulorn.Mamba2Spec(heads, vdim, dim, groups, 4, heads), attn.ff, attn.limit)
+        ops[name] = rigulorn_ops(dataclasses.replace(r, hidden_size=cfg.hidden_size, layers=(attn, ssm)), phase)
+    return {k: {n: rest for n, *rest in v} for k, v in ops.items()}
+
+
 # step of a Titatar layer -> the like step of the dense decoder's layer (experts: of its mixture)
 TITATAR_LIKE = {
     "residual update + norms": "norm + 2 input convolutions", "residual update + expert sum + norms": "norm + 2 input convolutions",
@@ -309,6 +448,16 @@ def moe_config(cfg):
     return dataclasses.replace(dense_config(titatar_like(cfg)), num_layers=len(cfg.layer_runs()), num_experts=m.experts,
                                num_experts_per_tok=round(m.top * m.experts / m.scores), moe_intermediate_size=m.ff,
                                name=f"moe-{cfg.hidden_size}")
+
+
+def meronex_moe_config(cfg):
+    """The decoder family's mixture-of-experts model with the attention heads and experts of a Meronex model, one layer per layer."""
+    from arctic_platform_b200.models.config import DecoderConfig
+    L = next(s for s in cfg.layers if s.type == "parallel").mixer.left
+    M = next(s.mlp for s in cfg.layers if s.mlp is not None)
+    return DecoderConfig(vocab_size=cfg.vocab_size, hidden_size=cfg.hidden_size, intermediate_size=M.ff, num_layers=cfg.num_layers,
+                         num_heads=L.heads, num_kv_heads=L.kv_heads, head_dim=L.dim, tie_word_embeddings=False, num_experts=M.experts,
+                         num_experts_per_tok=M.top, moe_intermediate_size=M.ff, name=f"moe-{cfg.hidden_size}")
 
 
 def moe_ops(cfg, phase):
@@ -357,6 +506,9 @@ def reninex_like(cfg):
 
 def like_ops(cfg, phase):
     """Steps of the closest older model, keyed by the names of ``stateful_ops``: ``name -> (fn, bytes, flops)``."""
+    if cfg.architecture == "Meronex":
+        ops = meronex_like(cfg, phase)
+        return {mine: ops[model][theirs] for mine, (model, theirs) in MERONEX_LIKE.items()}
     if cfg.architecture == "Titatar":
         ops = {**dense_ops(titatar_like(cfg), phase), **moe_ops(cfg, phase)}
         return {mine: ops[theirs] for mine, theirs in TITATAR_LIKE.items()}
@@ -510,9 +662,13 @@ def bench_engine(name, cfg, seqs, new_tokens):
     from arctic_platform_b200.models.config import resolve_config
     prompts = [np.random.default_rng(i).integers(1, cfg.vocab_size, SEQ).tolist() for i in range(seqs)]
     limits = dict(kv_cache_tokens=seqs * (SEQ + new_tokens + 32), max_batch=seqs, max_seq_len=SEQ + new_tokens + 16)
-    models = [cfg, moe_config(cfg) if cfg.architecture == "Titatar" else dense_config(cfg)]
-    if cfg.architecture == "Rigulorn" and f"reninex-{cfg.hidden_size}" in registry.presets():
-        models.append(resolve_config(f"reninex-{cfg.hidden_size}"))
+    older = {"Rigulorn": f"reninex-{cfg.hidden_size}", "Meronex": f"titatar-{cfg.hidden_size}"}.get(cfg.architecture)
+    if cfg.architecture == "Meronex":
+        models = [cfg, meronex_moe_config(cfg)]
+    else:
+        models = [cfg, moe_config(cfg) if cfg.architecture == "Titatar" else dense_config(cfg)]
+    if older in registry.presets():
+        models.append(resolve_config(older))
     for m in models:
         model = registry.new_model(m, "cuda", torch.bfloat16).init_weights(0)
         if registry.is_stateful(m):
@@ -560,7 +716,8 @@ def main(models, kernels_only=False, only=None, iters=20, seqs=64, new_tokens=12
 
 if __name__ == "__main__":
     ap = argparse.ArgumentParser()
-    ap.add_argument("--models", default="reninex-2048,reninex-4096,rigulorn-2048,rigulorn-4096,titatar-2048,titatar-4096")
+    ap.add_argument("--models", default="reninex-2048,reninex-4096,rigulorn-2048,rigulorn-4096,titatar-2048,titatar-4096,"
+                                         "meronex-2048,meronex-4096")
     ap.add_argument("--kernels-only", action="store_true")
     ap.add_argument("--only", choices=["prefill", "decode", "none"], help="which kernels are timed")
     ap.add_argument("--step", help="only the steps whose name contains this")

@@ -7,9 +7,9 @@ with the package.  ``forward(cfg, tensors, tokens)`` takes the parsed config.jso
 
 ``faults`` (a set of names) plants a deliberate mistake, so that a test can show that its inputs would reveal one:
 norms ``one_group``, ``one_plus``; sublayers ``no_gate``, ``gate_without_bias``, ``gate_of_residual``, ``no_mult``; matrix memory
-``no_input_cap``, ``no_forget_cap``, ``max_from_minus_infinity``, ``no_floor`` (the denominator without its lower bound),
-``signed_denominator``, ``silu_out`` (silu in place of the sigmoid), ``unscaled_q``; delta rule ``read_before_write``,
-``decay_after_write``, ``no_unit``, ``no_conv_state`` (the convolution starts anew every 5 tokens), ``reversed_taps``,
+``no_input_cap``, ``no_forget_cap``, ``no_floor`` (the denominator without its lower bound), ``signed_denominator``, ``silu_out``
+(silu in place of the sigmoid), ``unscaled_q``; delta rule ``read_before_write``, ``decay_after_write``, ``no_unit``,
+``no_conv_state`` (the convolution starts anew every 5 tokens), ``reversed_taps``,
 ``spread_heads`` (query head h reads h mod kv_heads), ``no_dt_bias``; attention ``neighbour_pairs``, ``no_yarn``, ``no_yarn_gain``,
 ``no_softcap``, ``cap_before_scale``, ``raw_values``, ``values_rotated``; time mixing ``shift_two``, ``no_shift_state`` (no previous
 token every 5 tokens), ``no_bonus``, ``read_after_write``, ``scalar_decay``, ``linear_rank`` (no tanh); side by side ``sum_of_sides``,
@@ -57,7 +57,7 @@ def matrix_memory(q, k, v, log_i, log_f, faults=()):
     """``q, k [T, H, D]`` (q scaled), ``v [T, H, E]``, log gates ``[T, H]`` -> ``[T, H, E]``."""
     T, H, D = q.shape
     S, n = q.new_zeros(H, D, v.shape[2]), q.new_zeros(H, D)
-    m = q.new_full((H,), -math.inf) if "max_from_minus_infinity" in faults else q.new_zeros(H)
+    m = q.new_zeros(H)
     out = []
     for t in range(T):
         new = torch.maximum(log_f[t] + m, log_i[t])
