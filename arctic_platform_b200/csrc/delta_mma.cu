@@ -112,7 +112,7 @@ delta_chunk_kernel(const RecurrentParams p, const DeltaChunks dc) {
       float a[2];
 #pragma unroll
       for (int x = 0; x < 2; ++x) {
-        const float f = j + x <= i ? exp2f(s_l[i] - s_l[j + x]) * s_k[j + x] : 0.f;
+        const float f = j + x <= i ? wm_ex2(s_l[i] - s_l[j + x]) * s_k[j + x] : 0.f;
         a[x] = qk[nt][2 * hh + x] * f * s_q[i];
         s_mat[i][j + x] = j + x < i ? kk[nt][2 * hh + x] * f * s_k[i] * s_beta[i] : 0.f;
       }
@@ -133,12 +133,12 @@ delta_chunk_kernel(const RecurrentParams p, const DeltaChunks dc) {
     }
   } else if (warp == 1) {
     float* sc = dc.scalars + (static_cast<long long>(tile) * p.H + h) * kDlScalars;
-    const float l = s_l[lane], end = s_l[kDlC - 1], e = exp2f(l);
+    const float l = s_l[lane], end = s_l[kDlC - 1], e = wm_ex2(l);
     sc[lane] = s_beta[lane];
     sc[kDlC + lane] = s_beta[lane] * e * s_k[lane];
     sc[2 * kDlC + lane] = e * s_q[lane];
-    sc[3 * kDlC + lane] = lane < n ? exp2f(end - l) * s_k[lane] : 0.f;
-    if (lane == 0) sc[4 * kDlC] = exp2f(end);
+    sc[3 * kDlC + lane] = lane < n ? wm_ex2(end - l) * s_k[lane] : 0.f;
+    if (lane == 0) sc[4 * kDlC] = wm_ex2(end);
   }
 }
 

@@ -42,7 +42,8 @@ memory_gates_kernel(const RecurrentParams p, float2* __restrict__ gates, long lo
     if (j < n_entries * per && p.e.pos0[j / per] > 0) aux0[j] = p.aux[p.e.slot[j / per] * per + j % per];
     return;
   }
-  const float2 g = memory_gates<__nv_bfloat16>(p, i / p.H, static_cast<int>(i % p.H));
+  const unsigned j = static_cast<unsigned>(i), H = p.H;
+  const float2 g = memory_gates<__nv_bfloat16>(p, j / H, static_cast<int>(j % H));
   gates[i] = make_float2(g.x * kLog2e, g.y * kLog2e);
 }
 
@@ -133,7 +134,7 @@ memory_mma_kernel(const RecurrentParams p, const MemoryScan ms, int state_only) 
     M = fmaxf(M, m_run);
     s_g[buf][lane] = G;
     s_m[buf][lane] = M;
-    s_floor[buf][lane] = exp2f(-(F + M));
+    s_floor[buf][lane] = wm_ex2(-(F + M));
     if (lane == 0) s_m0[buf] = m_run;
     f_run += __shfl_sync(0xffffffffu, F, 31);
     m_run = __shfl_sync(0xffffffffu, F + M, 31);
@@ -161,11 +162,11 @@ memory_mma_kernel(const RecurrentParams p, const MemoryScan ms, int state_only) 
       fetch_kv(t0 + kMmC, buf ^ 1);
       if (warp == 7) gates_of(t0 + kMmC, buf ^ 1);
     }
-    if (threadIdx.x < kMmC) s_w[threadIdx.x] = exp2f(G[threadIdx.x] - m_end);
+    if (threadIdx.x < kMmC) s_w[threadIdx.x] = wm_ex2(G[threadIdx.x] - m_end);
     for (int i = threadIdx.x; i < kMmC * (kMmBE / 2); i += kMmThreads) {
       const int r = i / (kMmBE / 2), o = r * kMmVS + (i % (kMmBE / 2)) * 2;
       const float2 f = wm_pair(V + o);
-      const float wt = exp2f(G[r] - m_end);
+      const float wt = wm_ex2(G[r] - m_end);
       wm_store_split2(Wh + o, Wl + o, f.x * wt, f.y * wt);
     }
     const int r0 = (warp & 1) * 16, c0 = (warp >> 1) * 16;     // this warp's tile of the output
@@ -202,14 +203,14 @@ memory_mma_kernel(const RecurrentParams p, const MemoryScan ms, int state_only) 
       for (int hh = 0; hh < 2; ++hh) {
         const int i = r0 + quad_row + 8 * hh, j = k0 + quad_col;
         const float mi = M[i];
-        const float x = j <= i ? a[2 * hh] * q_scale * exp2f(G[j] - mi) : 0.f;
-        const float y = j + 1 <= i ? a[2 * hh + 1] * q_scale * exp2f(G[j + 1] - mi) : 0.f;
+        const float x = j <= i ? a[2 * hh] * q_scale * wm_ex2(G[j] - mi) : 0.f;
+        const float y = j + 1 <= i ? a[2 * hh + 1] * q_scale * wm_ex2(G[j + 1] - mi) : 0.f;
         wm_store_split2(Ah + i * kMmAS + j, Al + i * kMmAS + j, x, y);
         float sum = x + y;
         sum += __shfl_xor_sync(0xffffffffu, sum, 1);
         sum += __shfl_xor_sync(0xffffffffu, sum, 2);
         if ((lane & 3) == 0) s_rows[warp >> 1][i] = sum;
-        const float f = q_scale * exp2f(m0 - mi);
+        const float f = q_scale * wm_ex2(m0 - mi);
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt) {
           o[nt][2 * hh] *= f;
@@ -233,7 +234,7 @@ memory_mma_kernel(const RecurrentParams p, const MemoryScan ms, int state_only) 
     __syncthreads();                               // scores and weights visible; nobody reads q, n or the state operand any more
     if (more && !state_only) fetch_rows(t0 + kMmC, p.q_off + static_cast<long long>(kh) * D, Qs);
     asm volatile("cp.async.commit_group;" ::: "memory");
-    const float dn = exp2f(m0 - m_end);
+    const float dn = wm_ex2(m0 - m_end);
     if (!state_only) {
       for (int ks = 0; ks < (r0 + 16) / 16; ++ks) {
         uint32_t ah[4], al[4], v[4];
@@ -251,7 +252,7 @@ memory_mma_kernel(const RecurrentParams p, const MemoryScan ms, int state_only) 
       for (int hh = 0; hh < 2; ++hh) {
         const int i = r0 + quad_row + 8 * hh;
         if (i < n) {
-          const float den = s_rows[0][i] + s_rows[1][i] + s_rows[2][i] + s_rows[3][i] + q_scale * exp2f(m0 - M[i]) * s_qn[i];
+          const float den = s_rows[0][i] + s_rows[1][i] + s_rows[2][i] + s_rows[3][i] + q_scale * wm_ex2(m0 - M[i]) * s_qn[i];
           const float f = 1.f / (fmaxf(fabsf(den), s_floor[buf][i]) + 1e-6f);
           float* dst = p.y + (start + t0 + i) * p.H * E + static_cast<long long>(h) * E + e0;
 #pragma unroll
@@ -336,7 +337,7 @@ memory_carry_kernel(const RecurrentParams p, const MemoryScan ms, const int* __r
   for (int k = 0; k + 1 < n_seg; ++k) {
     const float2 t = ms.totals[static_cast<long long>(first + k) * p.H + h];
     const float top = fmaxf(t.x + m, t.y);
-    s = is_m ? top : s * exp2f(t.x + m - top) + x[(k + 1) * stride] * exp2f(t.y - top);
+    s = is_m ? top : s * wm_ex2(t.x + m - top) + x[(k + 1) * stride] * wm_ex2(t.y - top);
     x[(k + 1) * stride] = s;
     m = top;
   }
@@ -354,7 +355,7 @@ int apb_memory_mma(const RecurrentParams* params, int rows, int n_entries, void*
                    void* totals, const int* chains, int n_chains, cudaStream_t s) {
   if (n_seg <= 0) return 0;
   const RecurrentParams& a = *params;
-  if (!recurrent_params_ok(kRuleMemory, a) || (a.D % 8) || (a.E % 8) || a.D > kMmMaxD || !a.y || !gates || !aux0 || !seg ||
+  if (!recurrent_params_ok(kRuleMemory, a) || (a.D % 8) || (a.E % 8) || a.D > kMmMaxD || static_cast<long long>(rows) * a.H > 0x7fffffffLL || !a.y || !gates || !aux0 || !seg ||
       ((a.ld | a.q_off | a.k_off | a.v_off) & 7) || (reinterpret_cast<uintptr_t>(a.p) & 15) ||
       (n_chains > 0 && (!carry || !carry_aux || !totals || !chains)))
     return kBadArgument;

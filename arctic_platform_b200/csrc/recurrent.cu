@@ -374,12 +374,12 @@ template <typename T, int V>
 __global__ void __launch_bounds__(256)
 head_norm_gate_kernel(const RecurrentParams p, const int* __restrict__ row_entry, int rows) {
   pdl_entry();
-  const long long gw = (blockIdx.x * 256LL + threadIdx.x) >> 5;
-  if (gw >= static_cast<long long>(rows) * p.H) return;
-  const int lane = threadIdx.x & 31, h = static_cast<int>(gw % p.H), E = p.E;
-  const long long row = gw / p.H;
+  const unsigned gw = blockIdx.x * 8u + (threadIdx.x >> 5), H = p.H;       // rows * heads fits: the entry point checks
+  if (gw >= rows * H) return;
+  const int lane = threadIdx.x & 31, h = static_cast<int>(gw % H), E = p.E;
+  const long long row = gw / H;
   if (row_entry && p.e.len[row_entry[row]] <= 1) return;
-  const float* y = p.y + gw * E;
+  const float* y = p.y + static_cast<long long>(gw) * E;
   const T* z = static_cast<const T*>(p.p) + row * p.ld + p.g_off + h * E;
   const T* gain = static_cast<const T*>(p.gain) + static_cast<long long>(h) * p.gain_step;
   T* out = static_cast<T*>(p.out) + row * p.ldo + h * E;
@@ -507,9 +507,9 @@ template <typename T>
 __global__ void __launch_bounds__(256)
 tanh_rows_kernel(T* __restrict__ x, long long ld, int rows, int n) {
   pdl_entry();
-  const long long i = blockIdx.x * 256LL + threadIdx.x;
-  if (i >= static_cast<long long>(rows) * n) return;
-  T* v = x + i / n * ld + i % n;
+  const unsigned i = blockIdx.x * 256u + threadIdx.x, w = n;
+  if (i >= rows * w) return;
+  T* v = x + static_cast<long long>(i / w) * ld + i % w;
   *v = from_f32<T>(tanhf(to_f32(*v)));
 }
 
@@ -568,7 +568,7 @@ int apb_recurrent(int rule, const RecurrentParams* params, const int* row_entry,
                   int finish, int dtype, cudaStream_t s) {
   if (n_entries <= 0 || rows <= 0) return 0;
   const RecurrentParams& a = *params;
-  if (!recurrent_params_ok(rule, a) || ((scan || finish) && !a.y) || (rule == kRuleDelta && scan && !a.xc)) return kBadArgument;
+  if (!recurrent_params_ok(rule, a) || ((scan || finish) && !a.y) || static_cast<long long>(rows) * a.H > 0x7fffffffLL || (rule == kRuleDelta && scan && !a.xc)) return kBadArgument;
   APB_SERVE_DTYPE(dtype, if (rule == kRuleMemory) return recurrent_run<kRuleMemory, T>(a, row_entry, n_entries, rows, decode, scan, finish, s);
                   if (rule == kRuleDelta) return recurrent_run<kRuleDelta, T>(a, row_entry, n_entries, rows, decode, scan, finish, s);
                   if (rule == kRuleTimeMix) return recurrent_run<kRuleTimeMix, T>(a, row_entry, n_entries, rows, decode, scan, finish, s));
@@ -598,6 +598,7 @@ int apb_token_shift(const void* h, const void* mu, float* hist, const int* parit
 // x [rows, n] columns (row stride ld) <- tanh(x)
 int apb_tanh_rows(void* x, long long ld, int rows, int n, int dtype, cudaStream_t s) {
   if (rows <= 0 || n <= 0) return 0;
+  if (static_cast<long long>(rows) * n > 0x7fffffffLL) return kBadArgument;
   const dim3 grid(static_cast<unsigned>((static_cast<long long>(rows) * n + 255) / 256));
   APB_SERVE_DTYPE(dtype, return static_cast<int>(launch_kernel(tanh_rows_kernel<T>, grid, dim3(256), 0, s, static_cast<T*>(x), ld, rows, n)));
 }

@@ -548,9 +548,9 @@ half_rope_cache_kernel(T* __restrict__ p, long long ld, int q_col, int k_col, in
                        const float* __restrict__ sin_t, int rot, T* __restrict__ kcache, T* __restrict__ vcache, int rows, int H,
                        int G, int D, int E, float v_eps) {
   pdl_entry();
-  const int lane = threadIdx.x & 31, heads = H + 2 * G;
-  const long long gw = (blockIdx.x * 256LL + threadIdx.x) >> 5;
-  if (gw >= static_cast<long long>(rows) * heads) return;
+  const int lane = threadIdx.x & 31;
+  const unsigned heads = H + 2 * G, gw = blockIdx.x * 8u + (threadIdx.x >> 5);       // rows * heads fits: the entry point checks
+  if (gw >= rows * heads) return;
   const int row = static_cast<int>(gw / heads), hh = static_cast<int>(gw % heads);
   const int en = row_entry ? row_entry[row] : row;
   const int at = row - e.start[en];
@@ -756,9 +756,10 @@ int apb_half_rope_cache(void* p, long long ld, int q_col, int k_col, int v_col, 
       !vcache)
     return kBadArgument;
   const ServeEntries e{e_start, e_len, e_slot, e_pos0};
-  const bool vec = dtype == 0 && !((D | E | q_col | k_col | v_col) & 1) && !(rot & 3) && !(ld & 1) &&
-                   !((reinterpret_cast<uintptr_t>(p) | reinterpret_cast<uintptr_t>(kcache) | reinterpret_cast<uintptr_t>(vcache)) & 3);
+  const uintptr_t at = reinterpret_cast<uintptr_t>(p) | reinterpret_cast<uintptr_t>(kcache) | reinterpret_cast<uintptr_t>(vcache);
+  const bool vec = dtype == 0 && !((D | E | q_col | k_col | v_col) & 1) && !(rot & 3) && !(ld & 1) && !(at & 3);
   const long long warps = static_cast<long long>(rows) * (H + 2 * G);
+  if (warps > 0x7fffffffLL) return kBadArgument;
   const dim3 grid(static_cast<unsigned>((warps + 7) / 8));
 #define APB_HALF_ROPE(TT, VV)                                                                                             \
   return static_cast<int>(launch_kernel(half_rope_cache_kernel<TT, VV>, grid, dim3(256), 0, s, static_cast<TT*>(p), ld,   \

@@ -114,7 +114,10 @@ __device__ __forceinline__ Run<V> gate_run(const ResidualParams& p, int row, int
   Run<V> z = p.gate_f32 ? load_run<V>(static_cast<const float*>(p.gate) + o) : load_run<V>(static_cast<const T*>(p.gate) + o);
   const Run<V> b = load_run<V>(static_cast<const T*>(p.gate_bias) + c);
 #pragma unroll
-  for (int i = 0; i < V; ++i) z.v[i] = 1.f / (1.f + expf(-(z.v[i] + b.v[i])));
+  for (int i = 0; i < V; ++i) {
+    const float x = -(z.v[i] + b.v[i]);
+    z.v[i] = sizeof(T) == 2 ? __fdividef(1.f, 1.f + __expf(x)) : 1.f / (1.f + expf(x));
+  }
   return z;
 }
 

@@ -23,6 +23,7 @@ constexpr int kTmBE = 64;
 constexpr int kTmVS = kTmBE + 8;
 constexpr int kTmAS = kTmC + 8;
 constexpr int kTmMaxD = 128;
+constexpr int kTmPairs = kTmHalf * (kTmHalf + 1) / 2;
 
 struct TimeMixScan {
   ScanSegments sg;
@@ -41,6 +42,7 @@ __global__ void __launch_bounds__(kTmThreads, NP == 128 || NP == 0 ? 1 : 2)
 time_mix_mma_kernel(const RecurrentParams p, const TimeMixScan ts, int state_only) {
   pdl_entry();
   extern __shared__ __align__(128) uint8_t tm_smem[];
+  __shared__ uint8_t s_pair[kTmPairs];           // (i, j <= i) of a half, i in the upper four bits
   const ScanSegments& sg = ts.sg;
   const int* w = sg.seg + blockIdx.x * 6;
   const int en = w[0], t_begin = w[1], n_tok = w[2], carry_in = w[3], carry_out = w[4], is_last = w[5];
@@ -99,6 +101,8 @@ time_mix_mma_kernel(const RecurrentParams p, const TimeMixScan ts, int state_onl
     bonus[i] = i < D ? __bfloat162float(static_cast<const __nv_bfloat16*>(p.w1)[h * D + i]) : 0.f;
     w0[i] = i < D ? __bfloat162float(static_cast<const __nv_bfloat16*>(p.w0)[h * D + i]) : 0.f;
   }
+  if (threadIdx.x < kTmHalf)
+    for (int j = 0; j <= threadIdx.x; ++j) s_pair[threadIdx.x * (threadIdx.x + 1) / 2 + j] = threadIdx.x << 4 | j;
   for (int i = threadIdx.x; i < kTmC * kTmAS; i += kTmThreads) Ah[i] = Al[i] = __float2bfloat16(0.f);      // above the diagonal for good
   const float* s_in = nullptr;
   if (!state_only) {
@@ -130,7 +134,7 @@ time_mix_mma_kernel(const RecurrentParams p, const TimeMixScan ts, int state_onl
     if (ch < np) {
       float sum = 0.f;
       for (int i = run * run_len; i < (run + 1) * run_len; ++i) {
-        if (i < n) sum -= fminf(exp2f((L[i * ls + ch] + w0[ch]) * 1.4426950408889634f) * 1.4426950408889634f, kMaxLogDecay);
+        if (i < n) sum -= fminf(wm_ex2((L[i * ls + ch] + w0[ch]) * 1.4426950408889634f) * 1.4426950408889634f, kMaxLogDecay);
         L[i * ls + ch] = sum;
       }
       part[run * np + ch] = sum;
@@ -150,26 +154,22 @@ time_mix_mma_kernel(const RecurrentParams p, const TimeMixScan ts, int state_onl
       const int r = i / (np >> 1), c = (i % (np >> 1)) * 2, o = r * ns + c;
       const float2 li = *reinterpret_cast<const float2*>(L + r * ls + c), ln = *reinterpret_cast<const float2*>(L + (kTmC - 1) * ls + c);
       const float2 k = wm_pair(K + o);
-      wm_store_split2(Kh + o, Kl + o, k.x * exp2f(ln.x - li.x), k.y * exp2f(ln.y - li.y));
+      wm_store_split2(Kh + o, Kl + o, k.x * wm_ex2(ln.x - li.x), k.y * wm_ex2(ln.y - li.y));
       if (state_only) continue;
       const float2 lp = r ? *reinterpret_cast<const float2*>(L + (r - 1) * ls + c) : make_float2(0.f, 0.f);
       const float2 lm = *reinterpret_cast<const float2*>(L + (kTmHalf - 1) * ls + c);
       const float2 q = wm_pair(R + o);
-      wm_store_split2(Rh + o, Rl + o, q.x * exp2f(lp.x), q.y * exp2f(lp.y));
+      wm_store_split2(Rh + o, Rl + o, q.x * wm_ex2(lp.x), q.y * wm_ex2(lp.y));
       if (r >= kTmHalf)
-        wm_store_split2(Xh + o - kTmHalf * ns, Xl + o - kTmHalf * ns, q.x * exp2f(lp.x - lm.x), q.y * exp2f(lp.y - lm.y));
+        wm_store_split2(Xh + o - kTmHalf * ns, Xl + o - kTmHalf * ns, q.x * wm_ex2(lp.x - lm.x), q.y * wm_ex2(lp.y - lm.y));
       else
-        wm_store_split2(Yh + o, Yl + o, k.x * exp2f(lm.x - li.x), k.y * exp2f(lm.y - li.y));
+        wm_store_split2(Yh + o, Yl + o, k.x * wm_ex2(lm.x - li.x), k.y * wm_ex2(lm.y - li.y));
     }
-    // ---- A inside the halves: 2 x 136 pairs (i, j <= i), four lanes each
+    // ---- A inside the halves: 2 x kTmPairs pairs (i, j <= i), four lanes each
     if (!state_only)
-      for (int task = warp * 8 + (lane >> 2); task < 2 * 136; task += 64) {        // 272 = 4 * 64 + 16: whole warps stay together
-        const int half = task >= 136, x = half ? task - 136 : task;
-        int i = static_cast<int>((sqrtf(8.f * x + 1.f) - 1.f) * 0.5f);
-        while (i * (i + 1) / 2 > x) --i;
-        while ((i + 1) * (i + 2) / 2 <= x) ++i;
-        const int j = half * kTmHalf + x - i * (i + 1) / 2;
-        i += half * kTmHalf;
+      for (int task = warp * 8 + (lane >> 2); task < 2 * kTmPairs; task += 64) {        // 272 = 4 * 64 + 16: whole warps stay together
+        const int half = task >= kTmPairs, pair = s_pair[half ? task - kTmPairs : task];
+        const int i = half * kTmHalf + (pair >> 4), j = half * kTmHalf + (pair & 15);
         float sum = 0.f;
         for (int d = (lane & 3) * 4; d < np; d += 16) {
           const uint2 qr = *reinterpret_cast<const uint2*>(R + i * ns + d), kr = *reinterpret_cast<const uint2*>(K + j * ns + d);
@@ -180,7 +180,7 @@ time_mix_mma_kernel(const RecurrentParams p, const TimeMixScan ts, int state_onl
             f = *reinterpret_cast<const float4*>(bonus + d);
           } else {
             const float4 a = *reinterpret_cast<const float4*>(L + (i - 1) * ls + d), b = *reinterpret_cast<const float4*>(L + j * ls + d);
-            f = make_float4(exp2f(a.x - b.x), exp2f(a.y - b.y), exp2f(a.z - b.z), exp2f(a.w - b.w));
+            f = make_float4(wm_ex2(a.x - b.x), wm_ex2(a.y - b.y), wm_ex2(a.z - b.z), wm_ex2(a.w - b.w));
           }
           sum += q0.x * k0.x * f.x + q0.y * k0.y * f.y + q1.x * k1.x * f.z + q1.y * k1.y * f.w;
         }
@@ -268,7 +268,7 @@ time_mix_mma_kernel(const RecurrentParams p, const TimeMixScan ts, int state_onl
     // ---- S = diag(e^(L_n)) S + K^T V
     if (warp < n16) {
       const float* ln = L + (kTmC - 1) * ls + warp * 16 + quad_row;
-      st.scale(exp2f(ln[0]), exp2f(ln[8]));
+      st.scale(wm_ex2(ln[0]), wm_ex2(ln[8]));
 #pragma unroll
       for (int ks = 0; ks < kTmC / 16; ++ks) {
         uint32_t kh4[4], kl4[4];
@@ -311,7 +311,7 @@ time_mix_carry_kernel(const RecurrentParams p, const TimeMixScan ts, const int* 
   float s = p.e.pos0[en] > 0 ? p.state[static_cast<long long>(p.e.slot[en]) * stride + static_cast<long long>(h) * size + i] : 0.f;
   x[0] = s;
   for (int k = 0; k + 1 < n_seg; ++k) {
-    s = s * exp2f(ts.decay[(static_cast<long long>(first + k) * p.H + h) * p.D + i / p.E]) + x[(k + 1) * stride];
+    s = s * wm_ex2(ts.decay[(static_cast<long long>(first + k) * p.H + h) * p.D + i / p.E]) + x[(k + 1) * stride];
     x[(k + 1) * stride] = s;
   }
 }

@@ -39,6 +39,12 @@ __device__ __forceinline__ void wm_store_split2(__nv_bfloat16* hi, __nv_bfloat16
   *reinterpret_cast<uint32_t*>(hi) = h;
   *reinterpret_cast<uint32_t*>(lo) = l;
 }
+// 2^x, results below the normal range are zero
+__device__ __forceinline__ float wm_ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 __device__ __forceinline__ float2 wm_pair(const __nv_bfloat16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
 
 // Segments of the entries of a batch, for recurrences whose segments can be chained (serving.segment_plan).
