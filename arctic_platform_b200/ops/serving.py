@@ -44,7 +44,7 @@ def _fn(name: str):
             "apb_recurrent": [i, vp, vp] + [i] * 6 + [vp],
             "apb_memory_mma": [vp, i, i, vp, vp, vp, i, vp, vp, vp, vp, i, vp],
             "apb_delta_mma": [vp, vp, i, vp, i, vp, vp, vp],
-            "apb_time_mix_mma": [vp, vp, i, vp, vp, vp, i, vp],
+            "apb_time_mix_mma": [vp, vp, i, vp, vp, i, vp, vp, vp, vp, i, vp],
             "apb_short_conv": [vp, ll, i, vp, vp, i, vp, vp, vp, ll, i] + [vp] * 5 + [i, i, vp],
             "apb_token_shift": [vp] * 10 + [i, i, i, vp, vp, i, i, vp, i, vp],
             "apb_tanh_rows": [vp, ll, i, i, i, vp],
@@ -974,6 +974,12 @@ def first_tiles(host: np.ndarray, rows: int) -> np.ndarray:
     return np.array(out, dtype=np.int32)
 
 
+def segment_chunks(host: np.ndarray, seg: np.ndarray) -> np.ndarray:
+    """Index of the first chunk (in :func:`row_tiles`) of every segment of a :func:`segment_plan`."""
+    first = dict(first_tiles(host, CHUNK).tolist())
+    return np.array([first[en] + t // CHUNK for en, t in seg[:, :2].tolist()], dtype=np.int32)
+
+
 RULES = {"memory": 0, "delta": 1, "time_mix": 2}
 
 
@@ -1072,7 +1078,11 @@ def recurrent(b: StepBatch, s: RecurrentSpec, x: RecurrentInputs, state: torch.T
                       _lib.ptr(carry_aux), _lib.ptr(totals), _lib.ptr(chains), len(plan["chains"]))
             else:
                 decay = torch.empty((n_seg, H, D), **f32) if parts else None
-                _call("apb_time_mix_mma", ref, _lib.ptr(seg), n_seg, _lib.ptr(carry), _lib.ptr(decay), _lib.ptr(chains), len(plan["chains"]))
+                tiles = b.table(("rows", CHUNK), lambda: row_tiles(b.host, CHUNK))
+                at = b.table(("segment chunks", H * ((E + 63) // 64)), lambda: segment_chunks(b.host, plan["seg"]))
+                square = torch.empty((tiles.shape[0], H, 2, CHUNK, CHUNK), device=p.device, dtype=torch.bfloat16)
+                _call("apb_time_mix_mma", ref, _lib.ptr(tiles), tiles.shape[0], _lib.ptr(seg), _lib.ptr(at), n_seg, _lib.ptr(square),
+                      _lib.ptr(carry), _lib.ptr(decay), _lib.ptr(chains), len(plan["chains"]))
     _call("apb_recurrent", rule, ref, _lib.ptr(b.row_entry), b.n_entries, b.rows, 0, 0, 1, dt)
 
 

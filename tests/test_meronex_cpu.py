@@ -229,9 +229,15 @@ def test_recurrences_against_their_closed_forms():
 
 
 def test_chunks_of_long_entries():
-    from arctic_platform_b200.ops.serving import first_tiles, row_tiles
+    from arctic_platform_b200.ops.serving import first_tiles, row_tiles, segment_chunks, segment_plan
     host = np.array([[0, 1, 0, 5], [1, 40, 1, 0], [41, 2, 2, 9], [43, 1, 3, 7], [44, 96, 4, 0]])
     tiles, heads = row_tiles(host, 32), first_tiles(host, 32)
     assert tiles.tolist() == [[1, 0], [1, 32], [2, 0], [4, 0], [4, 32], [4, 64]]
     assert heads.tolist() == [[1, 0], [2, 2], [4, 3]]
     assert all(tiles[at].tolist() == [en, 0] for en, at in heads.tolist())
+    host = np.array([[0, 2000, 0, 0], [2000, 1, 1, 4], [2001, 700, 2, 16]])
+    plan, tiles = segment_plan(host, 1, 296), row_tiles(host, 32)
+    at = segment_chunks(host, plan["seg"])
+    assert len(at) == len(plan["seg"]) > 2
+    for (en, t, *_), i in zip(plan["seg"].tolist(), at.tolist()):
+        assert tiles[i].tolist() == [en, t]
