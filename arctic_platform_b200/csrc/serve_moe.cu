@@ -61,7 +61,10 @@ moe_serve_route_kernel(const MoeRouteParams p) {
     }
     if (p.sigmoid) {
 #pragma unroll
-      for (int j = 0; j < kMoePerLane; ++j) sc[j] = 1.f / (1.f + expf(-sc[j]));
+      for (int j = 0; j < kMoePerLane; ++j) {
+        pick[j] = sc[j];                             // without a correction the logits order the scores, also where those round to 1
+        sc[j] = 1.f / (1.f + expf(-sc[j]));
+      }
     } else {
       mx = warp_max(mx);
       float sum = 0.f;
@@ -77,7 +80,10 @@ moe_serve_route_kernel(const MoeRouteParams p) {
 #pragma unroll
     for (int j = 0; j < kMoePerLane; ++j) {
       const int e = lane + 32 * j;
-      pick[j] = e < p.N ? sc[j] + (p.correction ? to_f32(static_cast<const T*>(p.correction)[e]) : 0.f) : -INFINITY;
+      if (e >= p.N)
+        pick[j] = -INFINITY;
+      else if (p.correction || !p.sigmoid)
+        pick[j] = sc[j] + (p.correction ? to_f32(static_cast<const T*>(p.correction)[e]) : 0.f);
     }
     for (int r = 0; r < p.top; ++r) {
       float best = -INFINITY, w = 0.f;

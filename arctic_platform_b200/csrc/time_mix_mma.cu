@@ -128,8 +128,7 @@ time_mix_chunk_kernel(const RecurrentParams p, const TimeMixScan ts) {
     const int i = half * kTmHalf + (pair >> 4), j = half * kTmHalf + (pair & 15);
     float sum = 0.f;
     for (int d = (lane & 3) * 4; d < np; d += 16) {
-      const float2 q0 = wm_pair(R + i * ns + d), q1 = wm_pair(R + i * ns + d + 2);
-      const float2 k0 = wm_pair(K + j * ns + d), k1 = wm_pair(K + j * ns + d + 2);
+      const float4 q = wm_quad(R + i * ns + d), k = wm_quad(K + j * ns + d);
       float4 f;
       if (i == j) {
         f = *reinterpret_cast<const float4*>(bonus + d);
@@ -137,7 +136,7 @@ time_mix_chunk_kernel(const RecurrentParams p, const TimeMixScan ts) {
         const float4 a = *reinterpret_cast<const float4*>(L + (i - 1) * ls + d), b = *reinterpret_cast<const float4*>(L + j * ls + d);
         f = make_float4(wm_ex2(a.x - b.x), wm_ex2(a.y - b.y), wm_ex2(a.z - b.z), wm_ex2(a.w - b.w));
       }
-      sum += q0.x * k0.x * f.x + q0.y * k0.y * f.y + q1.x * k1.x * f.z + q1.y * k1.y * f.w;
+      sum += q.x * k.x * f.x + q.y * k.y * f.y + q.z * k.z * f.z + q.w * k.w * f.w;
     }
     const unsigned mask = __activemask();
     sum += __shfl_xor_sync(mask, sum, 1);

@@ -46,6 +46,11 @@ __device__ __forceinline__ float wm_ex2(float x) {
   return y;
 }
 __device__ __forceinline__ float2 wm_pair(const __nv_bfloat16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
+__device__ __forceinline__ float4 wm_quad(const __nv_bfloat16* p) {       // 8-byte aligned
+  const uint2 r = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
 
 // Segments of the entries of a batch, for recurrences whose segments can be chained (serving.segment_plan).
 struct ScanSegments {

@@ -103,6 +103,7 @@ class StatefulSampler(SamplerEngine):
         self._open: Dict[int, _Open] = {}
         self._dropped: List[tuple] = []
         super().__init__(cfg, device, model=model, cascade=False, **kw)
+        self._places = [p.data_ptr() for p in self.model.parameters()]
 
     # ------------------------------------------------------------------ memory
     def _alloc_cache(self) -> None:
@@ -110,6 +111,14 @@ class StatefulSampler(SamplerEngine):
         self.cache = StateCache(self.model.cache_layout(), self.num_pages, self.max_batch, self.device, self.model.dtype)
         from ..utils import memory_budget
         memory_budget.set_kv_resident(self.device, self.kv_bytes())
+
+    def weights_updated(self) -> None:
+        """A checkpoint may bring tensors of another size than the model was made with; captured steps hold the old addresses."""
+        super().weights_updated()
+        places = [p.data_ptr() for p in self.model.parameters()]
+        if places != self._places:
+            self._graphs.clear()
+        self._places = places
 
     def _alloc_layer_buffers(self) -> None:
         self.d_slots = torch.full((self.max_batch,), -1, device=self.device, dtype=torch.int32)

@@ -57,7 +57,7 @@ CONFIGS = {
                           moe(mlstm(heads=2, dim=136, vdim=64), ff=64), moe(parallel(heads=2, kv=1, dim=64, vdim=96, rot=64, r_heads=1, r_dim=128))],
                          width=256, vocab=456, groups=8),
     # many positions: keys far back beside states that last
-    "long-range": config([moe(mlstm(heads=2, dim=64, vdim=64)), moe(parallel(heads=4, kv=1, dim=48, vdim=80, r_heads=2, r_dim=64)),
+    "long-range": config([moe(mlstm(heads=2, dim=64, vdim=64)), moe(parallel(heads=4, kv=1, dim=48, vdim=88, r_heads=2, r_dim=64)),
                           moe(delta(heads=2, kv=2, dim=64, vdim=96))], width=160, vocab=320, groups=5),
 }
 

@@ -192,6 +192,18 @@ def test_greedy_generation(dtype, tol, graph):
         assert again["token_ids"] == outs[0]["token_ids"][:first + 1] and again["finish_reason"] == "stop"
 
 
+def test_a_checkpoint_with_another_rank_replaces_captured_steps():
+    cfg = H.CONFIGS["mixed-layers"]
+    w, other = H.weights(cfg, 5), H.weights(cfg, 6, rank=40)
+    eng = H.engine(cfg, w, torch.float32, slots=4, max_seq_len=128)
+    p, sp = H.tokens(cfg, 20, 1), {"temperature": 0.0, "max_tokens": 8, "ignore_eos": True}
+    _follow(cfg, w, p, eng.generate([p], sp)[0], 1e-3)
+    for n, t in other.items():
+        eng.model.load_named_tensor(n, t)
+    eng.weights_updated()
+    _follow(cfg, other, p, eng.generate([p], sp)[0], 1e-3)
+
+
 def test_sampling_is_seeded_filtered_and_reports_log_probs():
     cfg = H.CONFIGS["mixed-layers"]
     w = H.weights(cfg, 6)
