@@ -90,20 +90,21 @@ __device__ __forceinline__ float sumsq(const Run<V>& a) {
   return s;
 }
 
-// Sum over the block of two values per thread.
+// Sums over the block of one or two values per thread.
+template <bool TWO>
 __device__ __forceinline__ float2 block_sum_residual(float a, float b, float (*red)[kResThreads / 32]) {
   a = warp_sum(a);
-  b = warp_sum(b);
+  if (TWO) b = warp_sum(b);
   if ((threadIdx.x & 31) == 0) {
     red[0][threadIdx.x >> 5] = a;
-    red[1][threadIdx.x >> 5] = b;
+    if (TWO) red[1][threadIdx.x >> 5] = b;
   }
   __syncthreads();
   a = b = 0.f;
 #pragma unroll
   for (int i = 0; i < kResThreads / 32; ++i) {
     a += red[0][i];
-    b += red[1][i];
+    if (TWO) b += red[1][i];
   }
   return make_float2(a, b);
 }
@@ -121,8 +122,9 @@ __device__ __forceinline__ Run<V> gate_run(const ResidualParams& p, int row, int
   return z;
 }
 
-// One block per row; every thread keeps its own columns in shared memory between the passes.
-template <typename T, int V>
+// One block per row; every thread keeps its own columns in shared memory between the passes.  SIDES: there is a y2; GATED: a gate or
+// a multiplier; GROUPED: several groups.
+template <typename T, int V, bool SIDES, bool GATED, bool GROUPED>
 __global__ void __launch_bounds__(kResThreads)
 residual_step_kernel(const ResidualParams p) {
   pdl_entry();
@@ -131,7 +133,7 @@ residual_step_kernel(const ResidualParams p) {
   const int row = blockIdx.x, W = p.W;
   float* x = p.x + static_cast<long long>(row) * W;
   float* y = p.y ? p.y + static_cast<long long>(row) * W : nullptr;
-  float* y2 = p.y2 ? p.y2 + static_cast<long long>(row) * W : nullptr;
+  float* y2 = SIDES ? p.y2 + static_cast<long long>(row) * W : nullptr;
   float* buf2 = buf + W;
   const bool has_y = y || p.ex.eo;
   float2 ry = make_float2(1.f, 1.f);
@@ -147,7 +149,7 @@ residual_step_kernel(const ResidualParams p) {
         v = load_run<V>(y + c);
         if (p.clear_y) store_run<V>(y + c, Run<V>{});
       }
-      if (y2) {
+      if constexpr (SIDES) {
         const Run<V> v2 = load_run<V>(y2 + c);
         if (p.clear_y) store_run<V>(y2 + c, Run<V>{});
         store_run<V>(buf2 + c, v2);
@@ -164,8 +166,8 @@ residual_step_kernel(const ResidualParams p) {
       ss += sumsq<V>(v);
     }
     if (p.post) {
-      const float2 s = block_sum_residual(ss, ss2, red);
-      ry = make_float2(1.f / sqrtf(s.x / W + p.eps), 1.f / sqrtf(s.y / W + p.eps));
+      const float2 s = block_sum_residual<SIDES>(ss, ss2, red);
+      ry = make_float2(1.f / sqrtf(s.x / W + p.eps), SIDES ? 1.f / sqrtf(s.y / W + p.eps) : 0.f);
     }
   }
   const T* e = nullptr;
@@ -184,31 +186,31 @@ residual_step_kernel(const ResidualParams p) {
 #pragma unroll
         for (int i = 0; i < V; ++i) u.v[i] *= ry.x * (p.offset + g.v[i]);
       }
-      if (y2) {
+      if constexpr (SIDES) {
         const Run<V> u2 = load_run<V>(buf2 + c), g = load_run<V>(static_cast<const T*>(p.post2) + c);
 #pragma unroll
         for (int i = 0; i < V; ++i) u.v[i] += u2.v[i] * ry.y * (p.offset + g.v[i]);
       }
-      if (p.gate) {
+      if (GATED && p.gate) {
         const Run<V> g = gate_run<T, V>(p, row, c);
 #pragma unroll
         for (int i = 0; i < V; ++i) u.v[i] *= g.v[i];
       }
-      axpy<V>(v, p.mult, u);
+      axpy<V>(v, GATED ? p.mult : 1.f, u);
     }
     if (e) axpy<V>(v, p.embed_scale, load_run<V>(e + c));
     if (p.write_x && (has_y || e)) store_run<V>(x + c, v);
     if (p.pre) {
       store_run<V>(buf + c, v);
-      ss += sumsq<V>(v);
+      if (!GROUPED) ss += sumsq<V>(v);
     } else {
       store_run<V>(static_cast<float*>(p.h) + static_cast<long long>(row) * W + c, v);
     }
   }
   if (!p.pre) return;
   T* h = static_cast<T*>(p.h) + static_cast<long long>(row) * W;
-  if (p.groups == 1) {
-    const float r = 1.f / sqrtf(block_sum_residual(ss, 0.f, red2).x / W + p.eps);
+  if constexpr (!GROUPED) {
+    const float r = 1.f / sqrtf(block_sum_residual<false>(ss, 0.f, red2).x / W + p.eps);
 #pragma unroll 2
     for (int c = threadIdx.x * V; c < W; c += kResThreads * V) {
       Run<V> v = load_run<V>(buf + c);
@@ -219,7 +221,7 @@ residual_step_kernel(const ResidualParams p) {
     }
     return;
   }
-  float* sums = buf + (p.y2 ? 2 * W : W);
+  float* sums = buf + (SIDES ? 2 * W : W);
   const int size = W / p.groups, parts = group_parts(p.groups);
   __syncthreads();
   group_sums(p.groups, size, sums, [&](int c) { return buf[c]; });
@@ -263,6 +265,15 @@ int apb_residual_step(float* x, float* y, const void* post, const void* pre, voi
     return static_cast<int>(launch_kernel(fn, dim3(rows), dim3(kResThreads), smem, s, p));
   };
   const bool vec = (W & 3) == 0 && (!gate || (!(ld_gate & 3) && !(reinterpret_cast<uintptr_t>(gate) & 15)));
-  APB_SERVE_DTYPE(dtype, if (vec) return run(residual_step_kernel<T, 4>); return run(residual_step_kernel<T, 1>));
+  const bool grouped = groups > 1 && pre;
+#define APB_RESIDUAL(V)                                                                                          \
+  do {                                                                                                           \
+    if (y2) return grouped ? run(residual_step_kernel<T, V, true, true, true>) : run(residual_step_kernel<T, V, true, true, false>);    \
+    if (scaled) return grouped ? run(residual_step_kernel<T, V, false, true, true>) : run(residual_step_kernel<T, V, false, true, false>); \
+    return grouped ? run(residual_step_kernel<T, V, false, false, true>) : run(residual_step_kernel<T, V, false, false, false>);       \
+  } while (0)
+  const bool scaled = gate || mult != 1.f;
+  APB_SERVE_DTYPE(dtype, if (vec) APB_RESIDUAL(4); APB_RESIDUAL(1));
+#undef APB_RESIDUAL
 }
 }
